@@ -1,7 +1,7 @@
 """The cache manager: device arenas plus the host bookkeeping (C++, csrc/host).
 
 What a model needs comes from its parts: a schedule entry asks for paged keys/values
-(all positions, or a window of them) or for a fixed-size state slot.  Entries with the
+(all positions, a window of them, or the stretch a position sees) or for a fixed-size state slot.  Entries with the
 same paged need form a GROUP that shares one page pool and one block table per request
 (the reference installs one table on every full-attention layer,
 imparo-model/src/kv.rs:1353; groups by state kind, imparo-kv/src/state.rs:16-21).
@@ -42,6 +42,7 @@ class PagedKVView:
     n_pages: int
     window: Optional[int]
     writes: bool               # False: this entry reads a cache another entry writes
+    chunk: Optional[int] = None
 
 
 @dataclass
@@ -90,7 +91,8 @@ class CacheManager:
         arr = lambda xs: (ctypes.c_int * max(1, ng))(*xs) if ng else (ctypes.c_int * 1)()
         self._h = _lib.host()
         self._cm = self._h.imparo_cm_create(ng, arr([self.page_size] * ng), arr(self.num_pages),
-                                            arr([k.window or 0 for k in self.group_keys]), self.num_slots)
+                                            arr([k.window or 0 for k in self.group_keys]),
+                                            arr([k.chunk or 0 for k in self.group_keys]), self.num_slots)
         if not self._cm:
             raise CacheError("cache manager: bad sizes")
         # device arenas
@@ -254,7 +256,8 @@ class CacheManager:
                 g, idx = self._paged_of_entry[src]
                 k_view = self.k_arena[g][idx]
                 out.append(PagedKVView(k=k_view, v=k_view if self.v_arena[g] is None else self.v_arena[g][idx], group=g, page_size=self.page_size,
-                                       n_pages=self.num_pages[g] + 1, window=spec.window, writes=owner is None))
+                                       n_pages=self.num_pages[g] + 1, window=spec.window,
+                                       writes=owner is None, chunk=spec.chunk))
             else:
                 if owner is not None:
                     raise CacheError("a fixed-size state cannot be read through cache_from")

@@ -13,8 +13,9 @@ CacheManager::CacheManager(const std::vector<GroupSpec>& groups, int n_slots)
 }
 
 int CacheManager::first_block_needed(const GroupSpec& g, int next_pos) const {
-    if (g.window <= 0) return 0;
-    const int lo = std::max(0, next_pos + 1 - g.window);
+    int lo = 0;
+    if (g.window > 0) lo = std::max(0, next_pos + 1 - g.window);
+    if (g.chunk > 0) lo = std::max(lo, next_pos / g.chunk * g.chunk);
     return lo / g.page_size;
 }
 

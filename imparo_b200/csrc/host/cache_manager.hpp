@@ -10,7 +10,7 @@
 // a request takes pages as it grows, not up front (imparo-server/src/sched.rs:671-696);
 // recurrent state lives in a per-conversation slot that starts from zero
 // (imparo-model/src/lib.rs:1951-1972).  What differs: pages go back to the free set the
-// moment a request ends or a window has passed them (there is no prefix store).
+// moment a request ends or a window (or the stretch it sees) has passed them (there is no prefix store).
 #pragma once
 #include <cstdint>
 #include <map>
@@ -24,6 +24,7 @@ struct GroupSpec {
     int page_size;
     int n_pages;
     int window;   // 0: keep every position
+    int chunk;    // > 0: positions see only their own stretch of this many (counted from position 0); earlier ones are not kept
 };
 
 class CacheManager {

@@ -11,11 +11,11 @@ using imparo::Scheduler;
 
 extern "C" {
 
-void* imparo_cm_create(int n_groups, const int* page_size, const int* n_pages, const int* window, int n_slots) {
+void* imparo_cm_create(int n_groups, const int* page_size, const int* n_pages, const int* window, const int* chunk, int n_slots) {
     std::vector<GroupSpec> groups;
     for (int g = 0; g < n_groups; ++g) {
-        if (page_size[g] < 1 || n_pages[g] < 0 || window[g] < 0) return nullptr;
-        groups.push_back({page_size[g], n_pages[g], window[g]});
+        if (page_size[g] < 1 || n_pages[g] < 0 || window[g] < 0 || chunk[g] < 0) return nullptr;
+        groups.push_back({page_size[g], n_pages[g], window[g], chunk[g]});
     }
     if (n_slots < 0) return nullptr;
     return new CacheManager(groups, n_slots);

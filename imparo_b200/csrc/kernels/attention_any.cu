@@ -12,6 +12,8 @@
 //      With a sink the running max starts at 0 and the running sum at 1: the extra term is a key
 //      of score 0 seen before all others; with sink values (one number per head) the extra term is exp(value) instead of 1:
 //      the running max starts at the head's value.  With a soft cap c the scaled score becomes c * tanh(score / c).
+//      Chunked masks (a position sees only its own stretch of `chunk` positions).  With score_bias (a number per head) there
+//      is no softmax: a visible key weighs sigmoid(score + bias) and the weights are not normalised.
 //      Heads up to 640 wide (a cache of latent vectors that every head reads is one wide key/value head).
 //  (3) qkv_prepare_store: the same rows as a 32-bit product, for variants that work on whole heads in 32-bit before
 //      anything is rounded: biases added, half-split rotation, then q and k divided by their own root mean square
@@ -19,6 +21,9 @@
 //      same rows (v = (1 - lambda) v + lambda v_other, lambda a device scalar) and optionally saved for that use.
 //      v_from_k: the row has no value columns; a value head is the key head of the same number as it stands before the
 //      rotation (keys that are their own values).
+//  (4) qkv_norm_rotate_store: rows as in (1); every query and key head is divided by its own root mean square and multiplied
+//      by a weight (one for the queries, one for the keys, each shared by the heads), then half-split rotation; a block per
+//      token (or per stretch of its heads) that computes the position's sines and cosines once.
 #include "common.cuh"
 
 namespace imparo {
@@ -245,13 +250,95 @@ qkv_prepare_store_kernel(const float* __restrict__ qkv, size_t in_width, const f
     }
 }
 
+// A block owns one token's heads [blockIdx.y * heads_per_block, + heads_per_block) of the row [q heads | k heads | v heads].
+// A lane moves pairs of neighbouring elements where PAIRS (sizes and strides even, pointers aligned), else single ones.
+template <typename T, bool PAIRS>
+__global__ void __launch_bounds__(ANY_WARPS * 32)
+qkv_norm_rotate_store_kernel(const T* __restrict__ qkv, size_t in_width, const int* __restrict__ positions,
+                             const int* __restrict__ item_of_token, const float* __restrict__ q_w, const float* __restrict__ k_w,
+                             float eps, const float* __restrict__ inv_freq, int n_rot, T* __restrict__ q_out,
+                             T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ table, int max_blocks,
+                             int page_size, int n_pages, int nh, int nkv, int hd, int vd, int heads_per_block, int* status) {
+    using P = typename Pair<T>::type;
+    __shared__ float sn_s[ANY_MAX_HEAD / 2], cs_s[ANY_MAX_HEAD / 2];
+    __shared__ float head[ANY_WARPS][ANY_MAX_HEAD];
+    pdl_trigger();
+    const int t = blockIdx.x;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int total = nh + 2 * nkv;
+    const int h_first = blockIdx.y * heads_per_block, h_end = min(total, h_first + heads_per_block);
+    const int pos = positions[t];
+    const int half = inv_freq ? (n_rot >> 1) : 0;
+    if (h_first < nh + nkv) {
+        for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * inv_freq[i], &sn_s[i], &cs_s[i]);
+    }
+    size_t cache_row = 0;
+    int page = 0;
+    bool mapped = true;
+    if (nkv > 0) {
+        const int blk = pos / page_size;
+        page = blk < max_blocks ? table[(size_t)item_of_token[t] * max_blocks + blk] : -1;
+        mapped = page >= 0 && page < n_pages;
+        if (mapped) cache_row = (size_t)page * page_size + (pos % page_size);
+    }
+    __syncthreads();
+    pdl_wait();
+    if (!mapped && threadIdx.x == 0 && h_end > nh) report(status, IMPARO_ST_PAGE_RANGE, 44, t, page);    // its keys and values are skipped
+    const T* row = qkv + (size_t)t * in_width;
+    float* hv = head[warp];
+    for (int hh = h_first + warp; hh < h_end; hh += ANY_WARPS) {
+        const bool is_q = hh < nh, is_k = !is_q && hh < nh + nkv;
+        const T* src;
+        T* dst;
+        int n;
+        if (is_q) {
+            src = row + (size_t)hh * hd;
+            dst = q_out + ((size_t)t * nh + hh) * hd;
+            n = hd;
+        } else {
+            if (!mapped) continue;
+            const int kvh = is_k ? hh - nh : hh - nh - nkv;
+            n = is_k ? hd : vd;
+            src = row + (size_t)nh * hd + (is_k ? (size_t)kvh * hd : (size_t)nkv * hd + (size_t)kvh * vd);
+            dst = is_k ? k_cache + cache_row * ((size_t)nkv * hd) + (size_t)kvh * hd : v_cache + cache_row * ((size_t)nkv * vd) + (size_t)kvh * vd;
+        }
+        if (!is_q && !is_k) {                                       // a value head: as it is
+            if (PAIRS) for (int i = lane; i < n / 2; i += 32) reinterpret_cast<P*>(dst)[i] = reinterpret_cast<const P*>(src)[i];
+            else for (int d = lane; d < n; d += 32) dst[d] = src[d];
+            continue;
+        }
+        float ss = 0.f;
+        __syncwarp();                                               // the head before has been read
+        if (PAIRS) {
+            for (int i = lane; i < n / 2; i += 32) {
+                const float2 v = pair_f32(reinterpret_cast<const P*>(src)[i]);
+                *reinterpret_cast<float2*>(hv + 2 * i) = v;
+                ss += v.x * v.x + v.y * v.y;
+            }
+        } else {
+            for (int d = lane; d < n; d += 32) { const float v = to_f32(src[d]); hv[d] = v; ss += v * v; }
+        }
+        const float scale = 1.0f / sqrtf(warp_sum(ss) / (float)n + eps);
+        const float* w = is_q ? q_w : k_w;
+        for (int d = lane; d < n; d += 32) hv[d] *= scale * w[d];
+        __syncwarp();
+        auto turned = [&](int d) {
+            if (d >= 2 * half) return hv[d];
+            const int i = d < half ? d : d - half;
+            return d < half ? hv[d] * cs_s[i] - hv[d + half] * sn_s[i] : hv[d] * cs_s[i] + hv[d - half] * sn_s[i];
+        };
+        if (PAIRS) for (int i = lane; i < n / 2; i += 32) reinterpret_cast<P*>(dst)[i] = pair_from<P>(turned(2 * i), turned(2 * i + 1));
+        else for (int d = lane; d < n; d += 32) dst[d] = from_f32<T>(turned(d));
+    }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(ANY_WARPS * 32)
 attention_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                      const int* __restrict__ positions, const int* __restrict__ item_of_token,
                      const int* __restrict__ table, int max_blocks, int page_size, int n_pages,
-                     int window, float scale, int sink, const float* __restrict__ sink_values, float softcap,
-                     T* __restrict__ out, int nh, int nkv, int hd, int vd, int* status) {
+                     int window, int chunk, float scale, int sink, const float* __restrict__ sink_values, float softcap,
+                     const float* __restrict__ score_bias, T* __restrict__ out, int nh, int nkv, int hd, int vd, int* status) {
     __shared__ float qbuf[ANY_WARPS][ANY_ATT_MAX_HEAD];
     pdl_trigger();
     pdl_wait();
@@ -268,7 +355,8 @@ attention_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, con
     for (int d = lane; d < hd; d += 32) qs[d] = to_f32(qrow[d]);
     __syncwarp();
 
-    const int lo = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
+    const int lo = first_key(pos, window, chunk);
+    const float bias = score_bias ? score_bias[h] : 0.f;
     constexpr int PER = ANY_ATT_MAX_HEAD / 32;
     float acc[PER];
 #pragma unroll
@@ -293,14 +381,19 @@ attention_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, con
                 if (softcap > 0.f) s = softcap * tanhf(s / softcap);
             }
         }
-        const float m_new = fmaxf(m, warp_max(s));
-        if (m_new == -INFINITY) continue;
-        const float p = (rowi >= 0) ? expf(s - m_new) : 0.f;
-        const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);
-        l = l * corr + warp_sum(p);
+        float p;
+        if (score_bias) {
+            p = (rowi >= 0) ? 1.0f / (1.0f + expf(-(s + bias))) : 0.f;
+        } else {
+            const float m_new = fmaxf(m, warp_max(s));
+            if (m_new == -INFINITY) continue;
+            p = (rowi >= 0) ? expf(s - m_new) : 0.f;
+            const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);
+            l = l * corr + warp_sum(p);
 #pragma unroll
-        for (int i = 0; i < PER; ++i) acc[i] *= corr;
-        m = m_new;
+            for (int i = 0; i < PER; ++i) acc[i] *= corr;
+            m = m_new;
+        }
         const int cnt = min(32, pos - base + 1);
         for (int jj = 0; jj < cnt; ++jj) {
             const float pj = __shfl_sync(0xffffffffu, p, jj);
@@ -314,7 +407,7 @@ attention_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, con
             }
         }
     }
-    const float inv = l > 0.f ? 1.0f / l : 0.f;
+    const float inv = score_bias ? 1.0f : (l > 0.f ? 1.0f / l : 0.f);
     T* orow = out + ((size_t)t * nh + h) * vd;
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
@@ -371,11 +464,40 @@ extern "C" int imparo_qkv_rotate_store(const void* qkv, int dtype, const int* po
     return 0;
 }
 
+// qkv: rows of row_stride elements [nh*hd | nkv*hd | nkv*vd] in dtype; q_w, k_w float32 [hd]; half-split rotation of the first
+// n_rot dimensions (inv_freq null: none).
+extern "C" int imparo_qkv_norm_rotate_store(const void* qkv, long long row_stride, int dtype, const int* positions,
+                                            const int* item_of_token, const float* q_w, const float* k_w, float eps,
+                                            const float* inv_freq, int n_rot, void* q_out, void* k_cache, void* v_cache,
+                                            const int* table, int max_blocks, int page_size, int n_pages, int n_tok, int nh,
+                                            int nkv, int hd, int vd, int* status, cudaStream_t stream) {
+    if (n_tok <= 0) return 0;
+    if (hd < 1 || hd > ANY_MAX_HEAD || vd < 1 || vd > ANY_MAX_HEAD) return -3;
+    if (n_rot < 0 || n_rot > hd || (n_rot & 1)) return -4;
+    if (row_stride < (long long)(nh + nkv) * hd + (long long)nkv * vd) return -2;
+    const int es = dtype == IMPARO_DT_F32 ? 4 : 2;
+    const bool pairs = hd % 2 == 0 && vd % 2 == 0 && row_stride % 2 == 0 &&
+                       (((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & (uintptr_t)(2 * es - 1)) == 0;
+    const int total = nh + 2 * nkv;
+    const int per = n_tok >= 256 ? total : ANY_WARPS;         // few tokens: a block per four heads
+    dim3 grid(n_tok, (total + per - 1) / per);
+#define IMPARO_QN(T_, P_) launch(qkv_norm_rotate_store_kernel<T_, P_>, grid, dim3(ANY_WARPS * 32), 0, stream, (const T_*)qkv, \
+        (size_t)row_stride, positions, item_of_token, q_w, k_w, eps, inv_freq, n_rot, (T_*)q_out, (T_*)k_cache, (T_*)v_cache, table, \
+        max_blocks, page_size, n_pages, nh, nkv, hd, vd, per, status)
+    if (dtype == IMPARO_DT_F32) { if (pairs) IMPARO_QN(float, true); else IMPARO_QN(float, false); }
+    else if (dtype == IMPARO_DT_BF16) { if (pairs) IMPARO_QN(__nv_bfloat16, true); else IMPARO_QN(__nv_bfloat16, false); }
+    else return -1;
+#undef IMPARO_QN
+    IMPARO_CHECK_LAUNCH();
+    return 0;
+}
+
 extern "C" int imparo_attention_any(const void* q, const void* k_cache, const void* v_cache, int dtype,
                                     const int* positions, const int* item_of_token,
                                     const int* table, int max_blocks, int page_size, int n_pages,
-                                    int window, float scale, int sink, const float* sink_values, float softcap, void* out,
-                                    int n_tok, int nh, int nkv, int hd, int vd, int* status, cudaStream_t stream) {
+                                    int window, int chunk, float scale, int sink, const float* sink_values, float softcap,
+                                    const float* score_bias, void* out, int n_tok, int nh, int nkv, int hd, int vd, int* status,
+                                    cudaStream_t stream) {
     if (n_tok <= 0) return 0;
     if (hd < 1 || hd > ANY_ATT_MAX_HEAD || vd < 1 || vd > ANY_ATT_MAX_HEAD) return -3;
     if (nkv <= 0 || nh % nkv != 0) return -5;
@@ -383,12 +505,12 @@ extern "C" int imparo_attention_any(const void* q, const void* k_cache, const vo
     if (dtype == IMPARO_DT_F32)
         launch(attention_any_kernel<float>, grid, dim3(ANY_WARPS * 32), 0, stream,
                (const float*)q, (const float*)k_cache, (const float*)v_cache, positions, item_of_token, table,
-               max_blocks, page_size, n_pages, window, scale, sink, sink_values, softcap, (float*)out, nh, nkv, hd, vd, status);
+               max_blocks, page_size, n_pages, window, chunk, scale, sink, sink_values, softcap, score_bias, (float*)out, nh, nkv, hd, vd, status);
     else if (dtype == IMPARO_DT_BF16)
         launch(attention_any_kernel<__nv_bfloat16>, grid, dim3(ANY_WARPS * 32), 0, stream,
                (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, positions,
-               item_of_token, table, max_blocks, page_size, n_pages, window, scale, sink, sink_values, softcap, (__nv_bfloat16*)out, nh, nkv, hd,
-               vd, status);
+               item_of_token, table, max_blocks, page_size, n_pages, window, chunk, scale, sink, sink_values, softcap, score_bias,
+               (__nv_bfloat16*)out, nh, nkv, hd, vd, status);
     else return -1;
     IMPARO_CHECK_LAUNCH();
     return 0;

@@ -84,6 +84,15 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
     return scratch[32];
 }
 
+// The first key that the query at position pos sees: position 0, or the last `window` positions up to its own (window > 0),
+// or the start of its own stretch of `chunk` positions (chunk > 0; stretches are counted from position 0).  It never
+// falls as pos grows, so the first row of a tile of consecutive positions has the tile's first key.
+__device__ __forceinline__ int first_key(int pos, int window, int chunk) {
+    int lo = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
+    if (chunk > 0) lo = max(lo, pos / chunk * chunk);
+    return lo;
+}
+
 // x / (1 + exp(-x))
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + expf(-x)); }
 // The same for results that are rounded to bfloat16 at once: the exponential and the division by their

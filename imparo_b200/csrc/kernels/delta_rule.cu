@@ -11,7 +11,7 @@
 //      that the CTA copies asynchronously two blocks ahead; the two sums over the key channels are finished by shuffles
 //      among the LPC lanes, the read-out's off the recurrence's chain.  The additions' order depends on the key size only.
 //  (3) head_norm_gate: every head's output divided by its root mean square over vdim, times a weight ([vdim] shared
-//      by the heads, or [heads * vdim] with each head's own), times sigmoid(gate).
+//      by the heads, or [heads * vdim] with each head's own), times sigmoid(gate) or silu(gate).
 #include "common.cuh"
 #include <type_traits>
 
@@ -266,9 +266,9 @@ delta_scan_kernel(const float* __restrict__ qkv, size_t qkv_stride, int q_off, i
 }
 
 // ---- (3) ------------------------------------------------------------------------------------------------------
-template <typename TOut>
+template <typename TOut, typename TGate, bool SILU>
 __global__ void __launch_bounds__(128)
-head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, float eps, const float* __restrict__ gate,
+head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, float eps, const TGate* __restrict__ gate,
                       size_t gate_stride, TOut* __restrict__ out, int heads, int vdim, int w_head_stride) {
     pdl_trigger();
     pdl_wait();
@@ -276,15 +276,17 @@ head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, 
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
     for (int h = blockIdx.y * nw + warp; h < heads; h += gridDim.y * nw) {
         const float* orow = o + ((size_t)t * heads + h) * vdim;
-        const float* grow = gate + (size_t)t * gate_stride + (size_t)h * vdim;
+        const TGate* grow = gate + (size_t)t * gate_stride + (size_t)h * vdim;
         float ss = 0.f;
         for (int p = lane; p < vdim; p += 32) ss += orow[p] * orow[p];
         ss = warp_sum(ss);
         const float scale = 1.0f / sqrtf(ss / (float)vdim + eps);
         TOut* dst = out + ((size_t)t * heads + h) * vdim;
         const float* wh = w + (size_t)h * w_head_stride;
-        for (int p = lane; p < vdim; p += 32)
-            dst[p] = from_f32<TOut>(orow[p] * scale * wh[p] * (1.0f / (1.0f + expf(-grow[p]))));
+        for (int p = lane; p < vdim; p += 32) {
+            const float z = to_f32(grow[p]);
+            dst[p] = from_f32<TOut>(orow[p] * scale * wh[p] * (SILU ? silu(z) : 1.0f / (1.0f + expf(-z))));
+        }
     }
 }
 
@@ -343,19 +345,24 @@ extern "C" int imparo_delta_scan(const float* qkv, long long qkv_stride, int q_o
     return 0;
 }
 
-// o: float32 [n_tok, heads * vdim]; w: float32 [vdim] (w_head_stride 0) or [heads * vdim] (w_head_stride vdim); gate: float32
-// rows of gate_stride floats (heads * vdim used).
-extern "C" int imparo_head_norm_gate(const float* o, const float* w, float eps, const float* gate, long long gate_stride,
-                                     void* out, int out_dtype, int n_tok, int heads, int vdim, int w_head_stride,
-                                     cudaStream_t stream) {
+// o: float32 [n_tok, heads * vdim]; w: float32 [vdim] (w_head_stride 0) or [heads * vdim] (w_head_stride vdim); gate: rows of
+// gate_stride elements of gate_dtype (heads * vdim used), its sigmoid or (gate_silu) its silu.
+extern "C" int imparo_head_norm_gate(const float* o, const float* w, float eps, const void* gate, int gate_dtype, int gate_silu,
+                                     long long gate_stride, void* out, int out_dtype, int n_tok, int heads, int vdim,
+                                     int w_head_stride, cudaStream_t stream) {
     if (n_tok <= 0) return 0;
     const dim3 grid(n_tok, (heads + 15) / 16 > 0 ? (heads + 15) / 16 : 1);
-    if (out_dtype == IMPARO_DT_F32)
-        launch(head_norm_gate_kernel<float>, grid, dim3(128), 0, stream, o, w, eps, gate, (size_t)gate_stride, (float*)out, heads, vdim, w_head_stride);
-    else if (out_dtype == IMPARO_DT_BF16)
-        launch(head_norm_gate_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, o, w, eps, gate, (size_t)gate_stride,
-               (__nv_bfloat16*)out, heads, vdim, w_head_stride);
+#define IMPARO_HN3(T_, G_, S_) launch(head_norm_gate_kernel<T_, G_, S_>, grid, dim3(128), 0, stream, o, w, eps, (const G_*)gate, \
+        (size_t)gate_stride, (T_*)out, heads, vdim, w_head_stride)
+#define IMPARO_HN2(T_, G_) do { if (gate_silu) IMPARO_HN3(T_, G_, true); else IMPARO_HN3(T_, G_, false); } while (0)
+#define IMPARO_HN(T_) do { if (gate_dtype == IMPARO_DT_F32) IMPARO_HN2(T_, float); else if (gate_dtype == IMPARO_DT_BF16) \
+        IMPARO_HN2(T_, __nv_bfloat16); else return -1; } while (0)
+    if (out_dtype == IMPARO_DT_F32) IMPARO_HN(float);
+    else if (out_dtype == IMPARO_DT_BF16) IMPARO_HN(__nv_bfloat16);
     else return -1;
+#undef IMPARO_HN
+#undef IMPARO_HN2
+#undef IMPARO_HN3
     IMPARO_CHECK_LAUNCH();
     return 0;
 }

@@ -78,6 +78,8 @@ class LaunchState:
         self.pending = {}            # data_ptr -> (scratch, n_splits, rows, width)
         self.pending_mean = {}       # data_ptr -> arguments of a norm_mean_add the next reader of the stream carries out
         self.pending_mix = {}        # data_ptr -> arguments of a streams_mix_add the next reader of the stream carries out
+        self.pending_gnorm = {}      # data_ptr -> arguments of a group_norm_add the next reader of the stream carries out
+        self.unfinished = {}         # data_ptr of an output buffer whose reader finishes it -> [partials or None, bias or None]
         self.partials = {}           # device index -> scratch of products into the stream
         self.consumer_parts = {}     # device index -> scratch of products a consumer kernel folds
         self.tc_scratch = {}         # device index -> (floats, counters) of the cluster-folded products
@@ -172,6 +174,8 @@ def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, stat
     _S.pending.pop(out.data_ptr(), None)       # the stream starts afresh: partials of an unfinished step are void
     _S.pending_mean.pop(out.data_ptr(), None)
     _S.pending_mix.pop(out.data_ptr(), None)
+    _S.pending_gnorm.pop(out.data_ptr(), None)
+    _S.unfinished.clear()
     n, width = out.shape
     _need(ids.dtype == torch.int32 and ids.numel() >= n, "ids must be int32, one per output row")
     _need(out.dtype == torch.float32 and table.shape[1] == width, "embedding output is float32 [tokens, width]")
@@ -246,11 +250,97 @@ def settle(stream: torch.Tensor) -> None:
     px = _S.pending_mix.pop(stream.data_ptr(), None)
     if px is not None:
         streams_mix_add(stream, *px)
+    pg = _S.pending_gnorm.pop(stream.data_ptr(), None)
+    if pg is not None:
+        _group_norm_add(stream, pg)
+    u = _S.unfinished.get(stream.data_ptr())
+    if u is not None and (u[0] is not None or u[1] is not None):
+        _finish(stream)
     p = _S.pending.pop(stream.data_ptr(), None)
     if p is not None:
         scratch, S, T, N = p
         _check(_lib.kernels().imparo_add_partials_rmsnorm(_ptr(stream), _ptr(scratch), S, T * N, None, 0.0, None, 0, T, N,
                                                           _stream()), "add_partials")
+
+
+# ---- output buffers that their reader finishes ---------------------------------------------------
+# A sublayer that writes its output into a float32 buffer of its own (not into the stream) ends with a product and perhaps a
+# bias.  When the buffer's reader promises to finish it (group_norm_add does), the product may leave its split partials and the
+# bias is only noted: the reader sums and adds while it reads.
+
+def allow_unfinished(out: torch.Tensor) -> None:
+    if defer_adds():
+        _S.unfinished[out.data_ptr()] = [None, None]
+
+
+def disallow_unfinished(out: torch.Tensor) -> None:
+    """No more may be left unfinished; what has been left stays for the reader."""
+    u = _S.unfinished.get(out.data_ptr())
+    if u is not None and u[0] is None and u[1] is None:
+        _S.unfinished.pop(out.data_ptr())
+
+
+def _take_unfinished(out: torch.Tensor):
+    """(tensor with the parts, parts, stride, bias or None) of an output buffer; the caller finishes it."""
+    u = _S.unfinished.pop(out.data_ptr(), None)
+    if u is None:
+        return out, 1, out.numel(), None
+    if u[0] is None:
+        return out, 1, out.numel(), u[1]
+    buf, splits = u[0]
+    return buf, splits, out.numel(), u[1]
+
+
+def _finish(out: torch.Tensor) -> None:
+    src, parts, stride, bias = _take_unfinished(out)
+    if src is not out:
+        _check(_lib.kernels().imparo_fold_partials(_ptr(src), parts, stride, _ptr(out), _code(out), stride, _stream()), "fold_partials")
+    if bias is not None:
+        _check(_lib.kernels().imparo_add_bias(_ptr(out), _code(out), _ptr(bias), out.shape[0], out.shape[1], _stream()), "add_bias")
+
+
+def group_rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, groups: int, out: torch.Tensor,
+                  rows: Optional[torch.Tensor] = None) -> None:
+    """out[r] = x[rows[r]] (or x[r]) cut into `groups` equal stretches, each divided by its own root mean square, times w.
+    A group_norm_add left pending on x is carried out by the same kernel when the norm reads every row in place."""
+    _cuda(x, w, out, rows)
+    n, width = out.shape
+    _need(x.dtype == torch.float32 and w.dtype == torch.float32, "group_rmsnorm reads a float32 stream and float32 weights")
+    _need(x.shape[1] == width and w.numel() == width and width % groups == 0, "group_rmsnorm: widths and groups")
+    pg = _S.pending_gnorm.get(x.data_ptr())
+    if pg is not None and rows is None and x.shape[0] == n and pg[3] == groups and x.data_ptr() not in _S.pending:
+        _S.pending_gnorm.pop(x.data_ptr())
+        _group_norm_add(x, pg, w, eps, out)
+        return
+    settle(x)
+    if rows is None:
+        _need(x.shape[0] >= n, "group_rmsnorm: fewer input rows than output rows")
+    else:
+        _need(rows.dtype == torch.int32 and rows.numel() >= n, "group_rmsnorm: rows must be int32, one per output row")
+    _check(_lib.kernels().imparo_group_rmsnorm(_ptr(x), _ptr(rows), _ptr(w), float(eps), _ptr(out), _code(out), n, width, int(groups),
+                                               _stream()), "group_rmsnorm")
+
+
+def group_norm_add(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: float, groups: int, defer: bool = False) -> None:
+    """x += y cut into `groups` stretches, each divided by its own root mean square, times w; x, y float32 [rows, width].  y may
+    be an unfinished output buffer (allow_unfinished): its partials are summed and its bias added on the way.  defer: the add is
+    left to the next reader of x (group_rmsnorm does it in its own pass, settle() alone); y must stay as it is until then."""
+    _cuda(x, y, w)
+    _need(x.dtype == torch.float32 and y.dtype == torch.float32 and y.shape == x.shape, "group_norm_add: float32 [rows, width]")
+    _need(w.dtype == torch.float32 and w.numel() == x.shape[1] and x.shape[1] % groups == 0, "group_norm_add: weight float32 [width], groups")
+    settle(x)
+    args = (_take_unfinished(y), w, float(eps), int(groups))
+    if defer and defer_adds():
+        _S.pending_gnorm[x.data_ptr()] = args
+        return
+    _group_norm_add(x, args)
+
+
+def _group_norm_add(x, args, nw=None, neps=0.0, out=None) -> None:
+    (src, parts, stride, bias), w, eps, groups = args
+    _check(_lib.kernels().imparo_group_norm_add(_ptr(x), _ptr(src), parts, stride, _ptr(bias), _ptr(w), eps, _ptr(nw), float(neps),
+                                                _ptr(out), _code(out) if out is not None else F32, x.shape[0], x.shape[1], groups,
+                                                _stream()), "group_norm_add")
 
 
 def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor,
@@ -318,9 +408,13 @@ def gated_act(gu: torch.Tensor, out: torch.Tensor, kind: str = "silu", limit: fl
 
 def add_bias(out: torch.Tensor, bias: torch.Tensor) -> None:
     _cuda(out, bias)
-    settle(out)
     n, width = out.shape
     _need(bias.dtype == torch.float32 and bias.numel() == width, "bias must be float32 [width]")
+    u = _S.unfinished.get(out.data_ptr())
+    if u is not None and u[1] is None:
+        u[1] = bias                                               # the buffer's reader adds it
+        return
+    settle(out)
     _check(_lib.kernels().imparo_add_bias(_ptr(out), _code(out), _ptr(bias), n, width, _stream()), "add_bias")
 
 
@@ -552,6 +646,19 @@ def linear(x, w: torch.Tensor, out: torch.Tensor, accumulate: bool = False,
         _need(not accumulate or out.dtype == torch.float32, "linear: accumulate needs a float32 output")
         if gemm_backend() == "tcgen05" and tc_usable(x, w):
             epi = EPI_ADD_F32 if accumulate else (EPI_STORE_F32 if out.dtype == torch.float32 else EPI_STORE_BF16)
+            u = _S.unfinished.get(out.data_ptr()) if not accumulate else None
+            if u is not None and out.dtype == torch.float32:
+                nt, splits, floats, _ = _tc_plan(M, N, K, EPI_PARTIAL)
+                if splits > 1:
+                    key = torch.device(x.device).index or 0
+                    buf = _S.partials.get(key)
+                    if buf is None or buf.numel() < floats:
+                        _need(not torch.cuda.is_current_stream_capturing(), "partials scratch would grow during graph capture")
+                        _S.generation += 0 if buf is None else 1
+                        buf = _S.partials[key] = torch.empty(_grown(floats, buf), dtype=torch.float32, device=x.device)
+                    gemm_tc(x, w, out, EPI_PARTIAL, status, scratch=buf)
+                    u[0] = (buf, splits)
+                    return
             if accumulate and out.data_ptr() in _S.deferrable and out.is_contiguous():
                 settle(out)                                       # one set of partials at a time
                 nt, splits, floats, _ = _tc_plan(M, N, K, EPI_PARTIAL)
@@ -1087,11 +1194,26 @@ def sample_rows(logits, temperature, uniform, out) -> None:
 ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2}
 
 
-def activation(x: torch.Tensor, out: torch.Tensor, kind: str) -> None:
+def linear_act(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, kind: str, bias: Optional[torch.Tensor] = None,
+               status: Optional[torch.Tensor] = None) -> None:
+    """out = act(x w^T + bias) (bias float32 [features] or None)."""
+    linear(x, w, out, status=status)
+    activation(out, out, kind, bias=bias)
+
+
+def activation(x: torch.Tensor, out: torch.Tensor, kind: str, bias: Optional[torch.Tensor] = None) -> None:
     """out = act(x) elementwise (relu2: relu(x)^2, gelu_tanh, silu); out may be x.  x may be a [rows, width] stretch of
-    wider rows (a column range of a product that several consumers share); out is then dense [rows, width]."""
+    wider rows (a column range of a product that several consumers share); out is then dense [rows, width].  bias: float32
+    [width], added to every row of x first."""
     _need(kind in ACTIVATIONS, f"activation: unknown kind '{kind}' (known: {', '.join(sorted(ACTIVATIONS))})")
     _need(x.shape == out.shape and x.dtype == out.dtype, "activation: out must match x")
+    if bias is not None:
+        _cuda(out, bias)
+        _need(x.is_cuda and x.dim() == 2 and x.stride(1) == 1, "activation: rows of x must be dense CUDA memory")
+        _need(bias.dtype == torch.float32 and bias.numel() == x.shape[1], "activation: bias float32 [width]")
+        _check(_lib.kernels().imparo_bias_act_rows(_ptr(x), x.stride(0), _ptr(bias), _ptr(out), _code(x), x.shape[0], x.shape[1],
+                                                   ACTIVATIONS[kind], _stream()), "activation")
+        return
     if x.dim() == 2 and not x.is_contiguous():
         _need(x.is_cuda and out.is_cuda and out.is_contiguous() and x.stride(1) == 1, "activation: rows of x must be dense")
         _check(_lib.kernels().imparo_act_rows_strided(_ptr(x), x.stride(0), _ptr(out), _code(x), x.shape[0], x.shape[1],
@@ -1211,13 +1333,44 @@ def qkv_rotate_store(qkv, positions, item_of_token, inv_freq, n_rot, interleaved
         page_size, n_pages, T, nh, nkv, hd, vd, qkv.stride(0), _ptr(status), _stream()), "qkv_rotate_store")
 
 
+def qkv_norm_rotate_store(qkv, positions, item_of_token, q_w, k_w, eps, inv_freq, n_rot, q_out, k_cache, v_cache, table, page_size,
+                          n_pages, nh, nkv, hd, vd, status) -> None:
+    """qkv [T, nh*hd + nkv*hd + nkv*vd] (rows dense, any row stride): every query and key head divided by its own root mean square
+    times a weight (q_w, k_w float32 [hd]), then half-split rotation of the first n_rot dimensions; q -> q_out [T, nh*hd], keys
+    and plain values into their pages (K rows nkv*hd wide, V rows nkv*vd wide)."""
+    _need(qkv.is_cuda and qkv.stride(1) == 1, "qkv_norm_rotate_store: rows of qkv must be dense CUDA memory")
+    _cuda(positions, item_of_token, q_w, k_w, inv_freq, q_out, k_cache, v_cache, table, status)
+    T = q_out.shape[0]
+    _need(tuple(qkv.shape) == (T, nh * hd + nkv * (hd + vd)) and q_out.shape[1] == nh * hd and qkv.dtype == q_out.dtype,
+          "qkv_norm_rotate_store: widths")
+    _need(all(w.dtype == torch.float32 and w.numel() == hd for w in (q_w, k_w)), "qkv_norm_rotate_store: norm weights float32 [head]")
+    _need(positions.dtype == torch.int32 and item_of_token.dtype == torch.int32 and positions.numel() >= T
+          and item_of_token.numel() >= T, "positions / item_of_token must be int32 per token")
+    if nkv:
+        _need(k_cache.dtype == qkv.dtype and v_cache.dtype == qkv.dtype, "cache dtype must match activations")
+        _need(k_cache.numel() >= n_pages * page_size * nkv * hd and v_cache.numel() >= n_pages * page_size * nkv * vd,
+              "cache arena smaller than n_pages")
+        _need(table.dtype == torch.int32 and table.dim() == 2, "block table must be int32 [items, blocks]")
+    if inv_freq is not None:
+        _need(inv_freq.dtype == torch.float32 and inv_freq.numel() >= n_rot // 2, "inv_freq must be float32 [n_rot/2]")
+    _check(_lib.kernels().imparo_qkv_norm_rotate_store(
+        _ptr(qkv), qkv.stride(0), _code(q_out), _ptr(positions), _ptr(item_of_token), _ptr(q_w), _ptr(k_w), float(eps), _ptr(inv_freq),
+        int(n_rot), _ptr(q_out), _ptr(k_cache), _ptr(v_cache), _ptr(table), table.shape[1], page_size, n_pages, T, nh, nkv, hd, vd,
+        _ptr(status), _stream()), "qkv_norm_rotate_store")
+
+
 def attention_any(q, k_cache, v_cache, positions, item_of_token, table, page_size, n_pages, window, scale, sink,
-                  out, nh, nkv, hd, vd, status, softcap: float = 0.0, sink_values: Optional[torch.Tensor] = None) -> None:
+                  out, nh, nkv, hd, vd, status, softcap: float = 0.0, sink_values: Optional[torch.Tensor] = None,
+                  chunk: Optional[int] = None, score_bias: Optional[torch.Tensor] = None) -> None:
     """General attention: any head size hd and value size vd up to 640, optional window, optional sink (one more
     term in the softmax's denominator that has no value: of score 0, or with sink_values, float32 [nh], of the head's
     own number, exp(value)), optional soft cap c > 0 on the scaled scores (c * tanh(score / c)).  out [T, nh*vd].
-    k_cache and v_cache may be the same tensor (keys that are their own values)."""
-    _cuda(q, k_cache, v_cache, positions, item_of_token, table, out, status, sink_values)
+    k_cache and v_cache may be the same tensor (keys that are their own values).  chunk c: a position sees only keys of its own
+    stretch of c positions (stretches counted from position 0).  score_bias (float32 [nh]): no softmax, a visible key weighs
+    sigmoid(score + bias of the head), weights are not normalised."""
+    _cuda(q, k_cache, v_cache, positions, item_of_token, table, out, status, sink_values, score_bias)
+    _need(score_bias is None or (score_bias.dtype == torch.float32 and score_bias.numel() == nh and not sink and sink_values is None),
+          "attention_any: score bias float32 [heads], without a sink")
     _need(sink_values is None or (sink_values.dtype == torch.float32 and sink_values.numel() == nh), "attention_any: sink values float32 [heads]")
     T = q.shape[0]
     _need(q.shape == (T, nh * hd) and out.shape == (T, nh * vd) and out.dtype == q.dtype, "attention_any: q/out shapes")
@@ -1227,8 +1380,8 @@ def attention_any(q, k_cache, v_cache, positions, item_of_token, table, page_siz
     _need(table.dtype == torch.int32 and table.dim() == 2, "block table must be int32 [items, blocks]")
     _check(_lib.kernels().imparo_attention_any(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _code(q), _ptr(positions), _ptr(item_of_token), _ptr(table),
-        table.shape[1], page_size, n_pages, int(window or 0), float(scale), int(bool(sink) or sink_values is not None),
-        _ptr(sink_values), float(softcap or 0.0), _ptr(out), T, nh, nkv, hd, vd, _ptr(status), _stream()), "attention_any")
+        table.shape[1], page_size, n_pages, int(window or 0), int(chunk or 0), float(scale), int(bool(sink) or sink_values is not None),
+        _ptr(sink_values), float(softcap or 0.0), _ptr(score_bias), _ptr(out), T, nh, nkv, hd, vd, _ptr(status), _stream()), "attention_any")
 
 
 def qkv_prepare_store(qkv, bias, positions, item_of_token, inv_freq, n_rot, unit_eps, v_other, v_lambda, v_save, q_out,
@@ -1532,8 +1685,9 @@ def embed_copies(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, stat
         _need(pos_table.dtype == table.dtype and pos_table.is_contiguous() and pos_table.shape[1] == table.shape[1],
               "position table: the embedding table's dtype and width")
         _need(positions.dtype == torch.int32 and positions.numel() >= out.shape[0], "positions must be int32, one per output row")
-    for d in (_S.pending, _S.pending_mean, _S.pending_mix):      # the stream starts afresh
+    for d in (_S.pending, _S.pending_mean, _S.pending_mix, _S.pending_gnorm):      # the stream starts afresh
         d.pop(out.data_ptr(), None)
+    _S.unfinished.clear()
     n = out.shape[0]
     width = table.shape[1]
     _need(ids.dtype == torch.int32 and ids.numel() >= n, "ids must be int32, one per output row")
@@ -1663,19 +1817,54 @@ def delta_scan(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, g: torch.T
                                             dim, vdim, _ptr(status), _stream()), "delta_scan")
 
 
-def head_norm_gate(o: torch.Tensor, w: torch.Tensor, eps: float, gate: torch.Tensor, out: torch.Tensor, heads: int, vdim: int) -> None:
-    """out[t, h] = o[t, h] / rms(o[t, h]) * w * sigmoid(gate[t, h]) per head.  o float32 [T, heads * vdim]; w float32 [vdim]
-    (one weight shared by the heads) or [heads * vdim] (each head's own); gate float32 rows (dense, any row stride)."""
+def head_norm_gate(o: torch.Tensor, w: torch.Tensor, eps: float, gate: torch.Tensor, out: torch.Tensor, heads: int, vdim: int,
+                   act: str = "sigmoid") -> None:
+    """out[t, h] = o[t, h] / rms(o[t, h]) * w * sigmoid(gate[t, h]) per head (act "silu": times silu(gate[t, h])).  o float32
+    [T, heads * vdim]; w float32 [vdim] (one weight shared by the heads) or [heads * vdim] (each head's own); gate float32 or
+    bfloat16 rows (dense, any row stride)."""
+    _need(act in ("sigmoid", "silu"), "head_norm_gate: act is 'sigmoid' or 'silu'")
     _cuda(o, w, out)
     _need(gate.is_cuda, "kernels run on CUDA tensors only (there is no CPU path)")
     T = o.shape[0]
     _need(o.dtype == torch.float32 and o.is_contiguous() and tuple(o.shape) == (T, heads * vdim), "head_norm_gate: o float32 [T, heads * vdim]")
     _need(w.dtype == torch.float32 and w.numel() in (vdim, heads * vdim), "head_norm_gate: weight float32 [vdim] or [heads * vdim]")
-    _need(gate.dtype == torch.float32 and gate.stride(1) == 1 and tuple(gate.shape) == (T, heads * vdim), "head_norm_gate: gate float32")
+    _need(gate.stride(1) == 1 and tuple(gate.shape) == (T, heads * vdim), "head_norm_gate: gate [T, heads * vdim]")
     _need(out.is_contiguous() and tuple(out.shape) == (T, heads * vdim), "head_norm_gate: out [T, heads * vdim]")
-    _check(_lib.kernels().imparo_head_norm_gate(_ptr(o), _ptr(w), float(eps), _ptr(gate), gate.stride(0), _ptr(out), _code(out), T,
-                                                heads, vdim, vdim if w.numel() == heads * vdim and heads > 1 else 0, _stream()),
+    _check(_lib.kernels().imparo_head_norm_gate(_ptr(o), _ptr(w), float(eps), _ptr(gate), _code(gate), int(act == "silu"),
+                                                gate.stride(0), _ptr(out), _code(out), T, heads, vdim, vdim if w.numel() == heads * vdim and heads > 1 else 0, _stream()),
            "head_norm_gate")
+
+
+# ---- gated linear attention with a decay per key channel (csrc/kernels/gla.cu) ----------------------------------
+def gla_decay(low: torch.Tensor, w2: torch.Tensor, bias: torch.Tensor, tau: float, out: torch.Tensor) -> None:
+    """out float32 [T, channels] = log sigmoid(w2 low + bias) / tau: the logarithms of the decays.  low [T, rank] (rows dense, any
+    row stride), w2 [channels, rank] of the same dtype, bias float32 [channels]."""
+    _need(low.is_cuda and low.stride(1) == 1, "gla_decay: rows of low must be dense CUDA memory")
+    _cuda(w2, bias, out)
+    T, rank = low.shape
+    _need(tuple(w2.shape) == (out.shape[1], rank) and w2.dtype == low.dtype, "gla_decay: w2 [channels, rank] of low's dtype")
+    _need(bias.dtype == torch.float32 and bias.numel() == out.shape[1] and out.dtype == torch.float32 and out.shape[0] == T,
+          "gla_decay: bias float32 [channels], out float32 [T, channels]")
+    _check(_lib.kernels().imparo_gla_decay(_ptr(low), low.stride(0), _code(low), _ptr(w2), _ptr(bias), float(tau), _ptr(out), T,
+                                           out.shape[1], rank, _stream()), "gla_decay")
+
+
+def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g: torch.Tensor, q_scale: float, state: torch.Tensor,
+             item_row_start, item_slot, n_items: int, out: torch.Tensor, heads: int, dim: int, vdim: int, status: torch.Tensor) -> None:
+    """Per request and head, rows in order, from and into state[slot] (float32 [slots, heads, dim, vdim]): S = diag(exp(g)) S +
+    k v^T, out = S^T (q_scale q).  proj: rows (dense, any row stride) with q, k (heads * dim) and v (heads * vdim) at the given
+    columns; g float32 [T, heads * dim]; out float32 [T, heads * vdim]."""
+    _need(proj.is_cuda and proj.stride(1) == 1, "gla_scan: rows of proj must be dense CUDA memory")
+    _cuda(g, state, item_row_start, item_slot, out, status)
+    T = proj.shape[0]
+    _need(g.dtype == torch.float32 and tuple(g.shape) == (T, heads * dim), "gla_scan: g float32 [T, heads * dim]")
+    _need(state.dtype == torch.float32 and tuple(state.shape[1:]) == (heads, dim, vdim), "gla_scan: state float32 [slots, heads, dim, vdim]")
+    _need(out.dtype == torch.float32 and tuple(out.shape) == (T, heads * vdim), "gla_scan: out float32 [T, heads * vdim]")
+    _need(max(q_off, k_off) + heads * dim <= proj.shape[1] and v_off + heads * vdim <= proj.shape[1], "gla_scan: columns")
+    _need(item_row_start.numel() >= n_items + 1 and item_slot.numel() >= n_items, "gla_scan: item arrays")
+    _check(_lib.kernels().imparo_gla_recurrent(_ptr(proj), proj.stride(0), _code(proj), int(q_off), int(k_off), int(v_off), _ptr(g),
+                                               float(q_scale), _ptr(state), _ptr(item_row_start), _ptr(item_slot), state.shape[0],
+                                               n_items, _ptr(out), heads, dim, vdim, _ptr(status), _stream()), "gla_recurrent")
 
 
 # ---- a matrix memory with exponential gates (csrc/kernels/mlstm.cu) ---------------------------------------------

@@ -4,3 +4,4 @@ from . import vipotar  # noqa: F401
 from . import negotar  # noqa: F401
 from . import keralix  # noqa: F401
 from . import zepesun  # noqa: F401
+from . import modinex  # noqa: F401

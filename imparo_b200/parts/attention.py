@@ -34,11 +34,14 @@ class AttentionMixer(Part):
     projection; a key head as it stands before the rotation is also the value head, so the value size is the head size),
     gate (bool: the heads' outputs, side by side, are multiplied element by element with sigmoid(W_g h), W_g the tensor
     "g" [n_heads * v_head_dim, hidden], before the output projection; with the 32-bit head preparation only), o_bias
-    "required" (an output bias the file must carry, with the 32-bit head preparation).
+    "required" (an output bias the file must carry, with the 32-bit head preparation), chunk (c: a position sees only its own
+    stretch of c positions, stretches counted from position 0; the cache gives earlier stretches back), weights ("softmax", or
+    "sigmoid": a visible key weighs sigmoid(score + b_h) with b the tensor "score_bias" [n_heads], and the weights are not
+    normalised over the keys).
 
     Shapes and variants the specialised kernels do not take (a value size of its own, a sink, a rotation of interleaved
-    pairs or with a magnitude, a head size that is no multiple of 16) run on the general pair of kernels
-    (ops.qkv_rotate_store, ops.attention_any).
+    pairs or with a magnitude, a head size that is no multiple of 16, chunks, sigmoid weights) run on the general kernels
+    (ops.qkv_rotate_store, or ops.qkv_norm_rotate_store where heads are normed; ops.attention_any).
 
     forward(..., accumulate=False) overwrites `residual` (then any float32 [tokens, hidden] buffer) instead of adding
     into it: a mixer that runs beside others hands its output to whoever combines them."""
@@ -48,7 +51,8 @@ class AttentionMixer(Part):
     NAMES = {"q": "self_attn.q_proj.weight", "k": "self_attn.k_proj.weight", "v": "self_attn.v_proj.weight",
              "o": "self_attn.out_proj.weight", "q_norm": "self_attn.q_layernorm.weight",
              "k_norm": "self_attn.k_layernorm.weight", "q_bias": "self_attn.q_proj.bias", "k_bias": "self_attn.k_proj.bias",
-             "v_bias": "self_attn.v_proj.bias", "o_bias": "self_attn.out_proj.bias", "g": "self_attn.gate.weight"}
+             "v_bias": "self_attn.v_proj.bias", "o_bias": "self_attn.out_proj.bias", "g": "self_attn.gate.weight",
+             "score_bias": "self_attn.score_bias"}
 
     def __init__(self, params, prefix, rt):
         super().__init__(params, prefix, rt)
@@ -82,6 +86,12 @@ class AttentionMixer(Part):
         self.v_from_k = bool(p.get("v_from_k", False))
         self.gate = bool(p.get("gate", False))
         self.o_bias_required = p.get("o_bias") == "required"
+        self.chunk = int(p["chunk"]) if p.get("chunk") else None
+        if p.get("weights", "softmax") not in ("softmax", "sigmoid"):
+            raise ValueError(f"attention: weights must be 'softmax' or 'sigmoid', found {p['weights']!r}")
+        self.sigmoid = p.get("weights") == "sigmoid"
+        if self.sigmoid and self.sink:
+            raise ValueError("attention: a sink belongs to a softmax; sigmoid weights have none")
         if self.v_from_k and (self.vd != self.hd or self.v_share is not None):
             raise ValueError("attention: keys that are their own values need value size = head size and no shared values")
         if self.qk_conv is not None and not 1 <= int(self.qk_conv["taps"]) <= 17:
@@ -90,15 +100,18 @@ class AttentionMixer(Part):
         self.prepared = (self.unit_norm or self.v_share is not None or self.bias_required or self.qk_conv is not None
                          or self.v_from_k or self.gate or self.o_bias_required)
         self.general = (self.sink or self.vd != self.hd or self.hd % 16 != 0 or self.position.interleaved
-                        or self.position.magnitude != 1.0 or self.prepared or self.softcap > 0.0)
+                        or self.position.magnitude != 1.0 or self.prepared or self.softcap > 0.0
+                        or self.chunk is not None or self.sigmoid)
         if self.prepared and (self.qk_norm or self.position.interleaved or self.position.magnitude != 1.0):
             raise ValueError("attention: the 32-bit head preparation (unit_norm, v_share, required biases) takes a half-split "
                              "rotation and no weighted q/k norms")
-        if self.general and not self.prepared and (self.qk_norm or self.bias):
-            raise ValueError("attention: per-head q/k norms and biases are not available together with a sink, a value size "
-                             "of its own, an interleaved or scaled rotation, or a head size that is no multiple of 16")
+        if self.general and not self.prepared and self.bias:
+            raise ValueError("attention: optional biases are not available together with a sink, a value size of its own, an "
+                             "interleaved or scaled rotation, chunks, sigmoid weights, or a head size that is no multiple of 16")
+        if self.general and self.qk_norm and (self.position.interleaved or self.position.magnitude != 1.0):
+            raise ValueError("attention: per-head q/k norms are not available together with an interleaved or scaled rotation")
         self.v_lambda = None
-        self.w_qkv = self.w_o = self.q_norm = self.k_norm = self.b_qkv = self.b_o = None
+        self.w_qkv = self.w_o = self.q_norm = self.k_norm = self.b_qkv = self.b_o = self.score_bias = None
 
     def weight_specs(self):
         n, H, hd, vd = self.names, self.hidden, self.hd, self.vd
@@ -125,6 +138,8 @@ class AttentionMixer(Part):
                       WeightSpec(n["o_bias"], ((H,),), role="vector", init=("bias",), optional=True)]
         if self.v_share is not None:
             specs.append(WeightSpec(self.prefix + self.v_share["lambda"], ((),), role="vector", init=("uniform", 0.2, 0.8)))
+        if self.sigmoid:
+            specs.append(WeightSpec(n["score_bias"], ((self.nh,),), role="vector", init=("uniform", -4.0, -1.0)))
         if self.gate:
             specs.append(WeightSpec(n["g"], ((self.nh * vd, H),)))
         if self.o_bias_required:
@@ -154,10 +169,12 @@ class AttentionMixer(Part):
             self.b_o = tensors.get(n["o_bias"])
         if self.o_bias_required:
             self.b_o = tensors[n["o_bias"]]
+        if self.sigmoid:
+            self.score_bias = tensors[n["score_bias"]]
         self.position.bind(tensors)
 
     def cache_specs(self):
-        paged = PagedKV(self.nkv, self.hd, self.window, None if self.vd == self.hd else self.vd)
+        paged = PagedKV(self.nkv, self.hd, self.window, None if self.vd == self.hd else self.vd, chunk=self.chunk)
         if self.qk_conv is not None:
             return (paged, SlotState((max(int(self.qk_conv["taps"]) - 1, 1), (self.nh + self.nkv) * self.hd)))
         return (paged,)
@@ -246,11 +263,16 @@ class AttentionMixer(Part):
             else:
                 qkv = rt.workspace.get("attn_qkv", (T, width), rt.act_dtype, first="tokens")
                 ops.linear(x, self.w_qkv[:width], qkv, status=rt.status)
-            ops.qkv_rotate_store(qkv, batch.positions, batch.item_of_token, inv_freq, n_rot, self.position.interleaved,
-                                 self.position.magnitude, q, kv.k, kv.v, table, kv.page_size, kv.n_pages, nh, nkv, hd, vd, rt.status)
+            if self.qk_norm:
+                ops.qkv_norm_rotate_store(qkv, batch.positions, batch.item_of_token, self.q_norm, self.k_norm, self.eps, inv_freq,
+                                          n_rot, q, kv.k, kv.v, table, kv.page_size, kv.n_pages, nh, nkv, hd, vd, rt.status)
+            else:
+                ops.qkv_rotate_store(qkv, batch.positions, batch.item_of_token, inv_freq, n_rot, self.position.interleaved,
+                                     self.position.magnitude, q, kv.k, kv.v, table, kv.page_size, kv.n_pages, nh, nkv, hd, vd, rt.status)
         out = rt.workspace.get("attn_out", (T, nh * vd), rt.act_dtype, first="tokens")
         done = False
-        if rt.act_dtype == torch.bfloat16 and hd == vd and hd in (64, 128) and nh // self.nkv <= 8 and T <= 65535:
+        if (rt.act_dtype == torch.bfloat16 and hd == vd and hd in (64, 128) and nh // self.nkv <= 8 and T <= 65535
+                and not self.sigmoid and self.chunk is None):
             # the tensor-core kernels take these sizes (the sink as a flag): prompt portions on the tcgen05 kernel, rows
             # of one token (and portions too short for a tile, or pages it does not take) on the split-key kernel
             n1 = getattr(batch, "n_single", 0)
@@ -278,7 +300,8 @@ class AttentionMixer(Part):
                                                  chunk, n_splits, nh, self.nkv, hd, rt.status, sink=self.sink, softcap=self.softcap)
         if not done:
             ops.attention_any(q, kv.k, kv.v, batch.positions, batch.item_of_token, table, kv.page_size, kv.n_pages, self.window,
-                              self.scale, self.sink, out, nh, self.nkv, hd, vd, rt.status, softcap=self.softcap)
+                              self.scale, self.sink, out, nh, self.nkv, hd, vd, rt.status, softcap=self.softcap, chunk=self.chunk,
+                              score_bias=self.score_bias)
         if self.prepared and self.gate:
             ops.sigmoid_gate(out, gate)
         ops.linear(out, self.w_o, residual, accumulate=accumulate, status=rt.status)

@@ -400,3 +400,98 @@ class HyperConnectionBlock(Block):
         if probe:
             probe("stream_out", x)
         return None
+
+
+class SandwichResidualBlock(Block):
+    """A norm before and a norm after each sublayer:  x += norm1b(mixer(norm1(x)));  x += norm2b(feed_forward(norm2(x))).
+
+    params: layer (LayerSpec): mixer_norm and feed_forward_norm are the norms before ("rmsnorm" parts with `groups`, 1 for the
+    plain norm); layer.params: "mixer_out_norm" and, where the layer has a feed-forward, "feed_forward_out_norm" (PartSpecs of
+    the same kind; their weight and eps are what the add applies, their groups those of the norms before).
+
+    Sublayers write their output into a float32 buffer (forward(..., accumulate=False)); a sublayer whose last product leaves
+    split partials, and whose output bias comes after it, may leave both unfinished there (ops.allow_unfinished).  The normed add
+    is left to the next reader of the stream: the next sublayer's norm (of this block or of the one after it) finishes the
+    output, norms it, adds it and norms the updated rows in one pass.  As the model's last block the feed-forward runs on the
+    wanted rows only."""
+
+    def __init__(self, params, prefix, rt):
+        super().__init__(params, prefix, rt)
+        spec = params["layer"]
+        self.mixer_norm = make_part("norm", spec.mixer_norm, prefix, rt)
+        self.mixer = make_part("mixer", spec.mixer, prefix, rt)
+        self.mixer_out = make_part("norm", spec.params["mixer_out_norm"], prefix, rt)
+        self.ff = self.ff_norm = self.ff_out = None
+        if spec.feed_forward is not None:
+            self.ff_norm = make_part("norm", spec.feed_forward_norm, prefix, rt)
+            self.ff = make_part("feed_forward", spec.feed_forward, prefix, rt)
+            self.ff_out = make_part("norm", spec.params["feed_forward_out_norm"], prefix, rt)
+        self.parts = tuple(p for p in (self.mixer_norm, self.mixer, self.mixer_out, self.ff_norm, self.ff, self.ff_out) if p is not None)
+        for p in (self.mixer_norm, self.mixer_out, self.ff_norm, self.ff_out):
+            if p is not None and not getattr(p, "groups", 0):
+                raise ValueError("sandwich block: its norms are given with groups (1 for the plain norm)")
+        self.graph_safe = all(p.graph_safe for p in self.parts)
+        self.picks_rows = True
+
+    def weight_specs(self):
+        return [w for p in self.parts for w in p.weight_specs()]
+
+    def bind(self, tensors):
+        for p in self.parts:
+            p.bind(tensors)
+
+    def cache_specs(self):
+        return self.mixer.cache_specs()
+
+    @staticmethod
+    def _into(part, y, call) -> None:
+        from ..kernels import ops
+        if part.adds_with_linear:
+            ops.allow_unfinished(y)
+            try:
+                call()
+            finally:
+                ops.disallow_unfinished(y)
+        else:
+            call()
+
+    def forward(self, x, batch, caches, only_rows=None):
+        import torch
+        from ..kernels import ops
+        probe = self.rt.probe if self.rt.probe_now else None
+        ws = self.rt.workspace
+        if probe:
+            ops.settle(x)
+            probe("stream_in", x)
+        h = self.mixer_norm.forward(x, tag="normed_mixer")           # (carries out the add the sublayer before left pending)
+        if probe:
+            probe("mixer_norm", h)
+        y = ws.get("sublayer_out", tuple(x.shape), torch.float32, first="tokens")
+        self._into(self.mixer, y, lambda: self.mixer.forward(h, batch, caches, y, accumulate=False))
+        ops.group_norm_add(x, y, self.mixer_out.weight, self.mixer_out.eps, self.mixer_out.groups, defer=not probe)
+        if probe:
+            probe("stream_mixer", x)
+        if only_rows is not None:
+            rows, n = only_rows
+            if n == 0:
+                ops.settle(x)
+                return None
+            xs = ws.get("stream_picked", (n, x.shape[1]), x.dtype, first="rows")
+            ops.gather_rows(x, rows, xs)
+            if self.ff is not None:
+                hs = self.ff_norm.forward(xs, tag="normed_ff_picked")
+                ys = ws.get("sublayer_out_picked", (n, x.shape[1]), torch.float32, first="rows")
+                self._into(self.ff, ys, lambda: self.ff.forward(hs, batch, ys, accumulate=False))
+                ops.group_norm_add(xs, ys, self.ff_out.weight, self.ff_out.eps, self.ff_out.groups, defer=not probe)
+            if probe:
+                probe("stream_out", xs)
+            return xs
+        if self.ff is not None:
+            h = self.ff_norm.forward(x, tag="normed_ff")
+            if probe:
+                probe("ff_norm", h)
+            self._into(self.ff, y, lambda: self.ff.forward(h, batch, y, accumulate=False))
+            ops.group_norm_add(x, y, self.ff_out.weight, self.ff_out.eps, self.ff_out.groups, defer=not probe)
+        if probe:
+            probe("stream_out", x)
+        return None

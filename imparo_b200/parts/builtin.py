@@ -1,10 +1,12 @@
 """Registers the built-in parts."""
 from .attention import AttentionMixer
 from .base import register_part
-from .block import HyperConnectionBlock, OutputNormResidualBlock, ParallelResidualBlock, PreNormResidualBlock
+from .block import (HyperConnectionBlock, OutputNormResidualBlock, ParallelResidualBlock, PreNormResidualBlock,
+                    SandwichResidualBlock)
 from .delta_rule import GatedDeltaRule
 from .embedding import LinearHead, TokenEmbedding
 from .feedforward import DenseFeedForward, SwiGLU
+from .gated_linear_attention import GatedLinearAttention
 from .latent_attention import LatentAttention
 from .linear_attention import DecayLinearAttention
 from .mamba2 import Mamba2Mixer
@@ -38,3 +40,5 @@ register_part("block", "hyper_connections", HyperConnectionBlock, replace=True)
 register_part("mixer", "latent_attention", LatentAttention, replace=True)
 register_part("mixer", "gated_delta_rule", GatedDeltaRule, replace=True)
 register_part("mixer", "matrix_memory", MatrixMemory, replace=True)
+register_part("block", "sandwich_residual", SandwichResidualBlock, replace=True)
+register_part("mixer", "gated_linear_attention", GatedLinearAttention, replace=True)

@@ -67,13 +67,15 @@ class SwiGLU(Part):
 
 class DenseFeedForward(Part):
     """down(act(up(x))) with one activation on its own: params hidden, ff, act ("relu2": relu(z)^2, "gelu_tanh",
-    "silu"), names (optional).
+    "silu"), names (optional), bias (bool, default False: True declares a bias for each of the two products, names "up_bias" and
+    "down_bias"; 32-bit, added before the activation / after the down product).
 
-    forward(x, batch, residual, scale=1.0) adds scale * output into the stream; forward_into(x, out) writes the
+    forward(x, batch, residual, scale=1.0, accumulate=True) adds scale * output into the stream; forward_into(x, out) writes the
     output into a float32 buffer instead (for an arrangement that adds several sublayers in one pass)."""
     takes_scale = True
+    adds_with_linear = True
 
-    NAMES = {"up": "up", "down": "down"}
+    NAMES = {"up": "up", "down": "down", "up_bias": "up.b", "down_bias": "down.b"}
 
     def __init__(self, params, prefix, rt):
         super().__init__(params, prefix, rt)
@@ -83,15 +85,22 @@ class DenseFeedForward(Part):
         if self.act not in ops.ACTIVATIONS:
             raise ValueError(f"feed-forward: unknown activation '{self.act}'; known: {', '.join(sorted(ops.ACTIVATIONS))}")
         self.names = {k: prefix + v for k, v in {**self.NAMES, **params.get("names", {})}.items()}
-        self.w_up = self.w_down = None
+        self.bias = bool(params.get("bias", False))
+        self.w_up = self.w_down = self.b_up = self.b_down = None
 
     def weight_specs(self):
         n, H, F = self.names, self.hidden, self.ff
-        return [WeightSpec(n["up"], ((F, H),)), WeightSpec(n["down"], ((H, F),))]
+        specs = [WeightSpec(n["up"], ((F, H),)), WeightSpec(n["down"], ((H, F),))]
+        if self.bias:
+            specs += [WeightSpec(n["up_bias"], ((F,),), role="vector", init=("bias",)),
+                      WeightSpec(n["down_bias"], ((H,),), role="vector", init=("bias",))]
+        return specs
 
     def bind(self, tensors):
         self.w_up = tensors[self.names["up"]]
         self.w_down = tensors[self.names["down"]]
+        if self.bias:
+            self.b_up, self.b_down = tensors[self.names["up_bias"]], tensors[self.names["down_bias"]]
 
     def input_rows(self) -> int:
         return self.ff
@@ -106,19 +115,25 @@ class DenseFeedForward(Part):
         rt, T = self.rt, x.shape[0]
         h = rt.workspace.get("ffn_h", (T, self.ff), rt.act_dtype, first="tokens")
         if projected is not None:
-            ops.activation(projected, h, self.act)          # from the shared product's columns into a dense tensor
+            ops.activation(projected, h, self.act, bias=self.b_up)          # from the shared product's columns into a dense tensor
         else:
-            ops.linear(x, self.w_up, h, status=rt.status)
-            ops.activation(h, h, self.act)
+            ops.linear_act(x, self.w_up, h, self.act, bias=self.b_up, status=rt.status)
         ops.linear(h, self.w_down, out, status=rt.status)
+        if self.b_down is not None:
+            ops.add_bias(out, self.b_down)
 
-    def forward(self, x, batch, residual, scale: float = 1.0):
+    def forward(self, x, batch, residual, scale: float = 1.0, accumulate: bool = True):
+        if not accumulate:
+            if scale != 1.0:
+                raise ValueError("dense feed-forward: an output that is written, not added, is not scaled")
+            return self.forward_into(x, residual)
         if scale == 1.0:
             rt, T = self.rt, x.shape[0]
             h = rt.workspace.get("ffn_h", (T, self.ff), rt.act_dtype, first="tokens")
-            ops.linear(x, self.w_up, h, status=rt.status)
-            ops.activation(h, h, self.act)
+            ops.linear_act(x, self.w_up, h, self.act, bias=self.b_up, status=rt.status)
             ops.linear(h, self.w_down, residual, accumulate=True, status=rt.status)
+            if self.b_down is not None:
+                ops.add_bias(residual, self.b_down)
             return
         out = self.rt.workspace.get("ffn_out", (x.shape[0], self.hidden), torch.float32, first="tokens")
         self.forward_into(x, out)

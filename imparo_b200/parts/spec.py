@@ -84,13 +84,15 @@ class PagedKV:
     """Keys and values that grow with the sequence, kept in pages.
 
     window=None keeps every position; window=w keeps the last w positions a query
-    can still see, and pages wholly behind that are given back.
+    can still see, and pages wholly behind that are given back; chunk=c cuts the sequence at the multiples
+    of c, a position sees only its own stretch, and the pages of earlier stretches are given back.
     (imparo-kv/src/state.rs:16-21 StateKind::{Full, Window})"""
     n_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     v_head_dim: Optional[int] = None        # None: values are as wide as keys
     values_are_keys: bool = False           # True: one row per position serves as key and as value (no value arena)
+    chunk: Optional[int] = None             # stretches of this many positions, counted from position 0
 
     @property
     def width(self) -> int:
