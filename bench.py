@@ -22,7 +22,7 @@ continuous batching; LFM2-350M sizes with 32,768-token prompts in bfloat16 and 3
 print one JSON line each; --workload sizes runs the headline's model at further prompt lengths
 and decode contexts; --workload vipotar / negotar run the Vipotar / Negotar design at two sizes that resemble a real model's layers beside
 LFM2 at equal width, depth, heads and feed-forward size (prefill of one prompt, decode at batch 8), --workload keralix the
-Keralix design beside Vipotar likewise, --workload zepesun the Zepesun design beside Negotar; the default is the headline above.
+Keralix design beside Vipotar likewise, --workload zepesun the Zepesun design beside Negotar, --workload modinex the Modinex design beside Vipotar; the default is the headline above.
 """
 import argparse
 import json
@@ -644,6 +644,95 @@ def workload_zepesun(args):
     return 0
 
 
+def modinex_config(width, layers, heads, kv_heads, head, vdim, chunk, lin_heads, lin_dim, lin_vdim, ff, vocab, positions):
+    """A Modinex config.json of the given sizes: gated linear attention without a feed-forward and attention with one in turn
+    (`layers` of each), half of each head rotated, norms in four groups, decays of about 0.9 to 1 per step."""
+    rec = {"type": "gla", "mixer": {"heads": lin_heads, "dim": lin_dim, "vdim": lin_vdim, "tau": 16.0, "rank": 16}, "mlp": None}
+    att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": head, "vdim": vdim, "scale": head ** -0.5,
+                                          "mask": {"size": chunk}, "rot": {"dims": head // 2, "base": 500000.0}},
+           "mlp": {"kind": "dense", "ff": ff}}
+    return {"architecture": "Modinex", "vocab": vocab, "width": width, "max_positions": positions, "norm": {"eps": 1e-6, "groups": 4},
+            "layers": [rec, att] * layers}
+
+
+def workload_modinex(args):
+    """Modinex at three sizes beside Vipotar (a grouped-query attention, a linear attention with decay and a dense feed-forward
+    per layer: the closest design the engine serves) at equal width, heads, mask size, recurrent state, feed-forward size and
+    number of each (a Vipotar layer holds what a pair of Modinex layers holds): prefill of one prompt of 512 and 2,048 tokens,
+    decode steps of 8 requests with 2,048 positions each.  Rooflines: prefill against the measured bfloat16 peak with the flops
+    the design needs (products over all tokens, attention over what a position sees, the recurrence's 4 * heads * dim * vdim per
+    token); decode against the measured copy bandwidth with the bytes a step must move (every matrix once, the keys and values the
+    rows see (of a stretch: those since its start), the states read and written)."""
+    import numpy as np
+    import torch
+    from imparo_b200.engine import Engine
+    rng = np.random.default_rng(0)
+    pk = peaks()
+    sizes = {"width1024": dict(width=1024, layers=8, heads=16, kv_heads=4, head=64, window=512, lin_heads=8, lin_dim=64, lin_vdim=128,
+                               ff=4096, vocab=32768),
+             "width2048": dict(width=2048, layers=8, heads=32, kv_heads=8, head=64, window=1024, lin_heads=16, lin_dim=128, lin_vdim=128,
+                               ff=8192, vocab=65536),
+             "width2048_head128": dict(width=2048, layers=8, heads=16, kv_heads=4, head=128, window=1024, lin_heads=16, lin_dim=64,
+                                       lin_vdim=128, ff=8192, vocab=65536)}
+    out = {"metric": "Modinex beside Vipotar at equal sizes: prefill of one prompt, decode at batch 8 with 2,048 positions",
+           "unit": "tokens/s", "dtype": "bf16", "data": "synthetic (random weights, uniform-random token ids)", "sizes": {}}
+    with ClockSampler() as clocks:
+        for name, z in sizes.items():
+            row = {}
+            W, L, F, V, C = z["width"], z["layers"], z["ff"], z["vocab"], z["window"]
+            qkv = (z["heads"] + 2 * z["kv_heads"]) * z["head"] * W + W * z["heads"] * z["head"]
+            lin = (2 * z["lin_heads"] * z["lin_dim"] + 2 * z["lin_heads"] * z["lin_vdim"]) * W + W * z["lin_heads"] * z["lin_vdim"]
+            state = L * z["lin_heads"] * z["lin_dim"] * z["lin_vdim"] * 4
+            kv_tok = L * 2 * z["kv_heads"] * z["head"] * 2
+            for model in ("modinex", "vipotar"):
+                matrix = L * (qkv + lin + 2 * W * F)
+                if model == "modinex":
+                    sizes_of = {k: v for k, v in z.items() if k != "window"}
+                    cfg = modinex_config(vdim=z["head"], chunk=C, positions=CTX, **sizes_of)
+                    matrix += L * (16 * W + z["lin_heads"] * z["lin_dim"] * 16)
+
+                    def keys(T):
+                        return sum(t % C + 1 for t in range(T))
+
+                    def step_keys(ctx):
+                        return ctx % C
+                else:
+                    cfg = vipotar_config(**z)
+
+                    def keys(T):
+                        return sum(min(t + 1, C) for t in range(T))
+
+                    def step_keys(ctx):
+                        return min(ctx, C)
+
+                def flops(T):
+                    return (2.0 * T * matrix + 2.0 * V * W + L * 4.0 * z["heads"] * z["head"] * keys(T)
+                            + L * 4.0 * z["lin_heads"] * z["lin_dim"] * z["lin_vdim"] * T)
+
+                def step_bytes(batch, ctx):
+                    return (matrix + V * W) * 2 + batch * (2 * state + step_keys(ctx) * kv_tok)
+                engine = Engine(config=cfg, seed=0, dtype="bfloat16", ctx=CTX, parallel=8, page_size=PAGE, max_step_tokens=PROMPT,
+                                random_init={"norm_jitter": 0.0})
+                r = {"params": matrix + 2 * V * W, "prefill": {}}
+                for T in (512, 2048):
+                    ms = measure_prefill(engine, reps=5, warmup=3, rng=rng, prompt=T)
+                    r["prefill"][str(T)] = {"value": round(T * 1000.0 / ms, 1), "ms": round(ms, 3),
+                                            "frac": round(flops(T) / (ms * 1e-3) / (pk["bf16_tflops_burst"] * 1e12), 4)}
+                ms, launches, library, ctx = measure_decode(engine, 8, max(20, args.steps // 4), max(args.warmup, 3), rng, prompt=PROMPT)
+                nbytes = step_bytes(8, ctx)
+                r["decode_b8"] = {"value": round(8 * 1000.0 / ms, 1), "ms_per_step": round(ms, 4), "own_kernels_per_step": round(launches, 1),
+                                  "library_gemms_per_step": round(library, 1), "bytes_per_step": int(nbytes),
+                                  "frac": round(nbytes / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)}
+                row[model] = r
+                del engine
+                torch.cuda.empty_cache()
+            out["sizes"][name] = dict(row, config=z)
+    out["peaks"] = pk["source"]
+    out["clocks"] = clocks.summary()
+    print(json.dumps(out))
+    return 0
+
+
 def _preset(name):
     with open(os.path.join(ROOT, "imparo_b200", "config", "presets", name + ".json")) as f:
         return json.load(f)
@@ -862,7 +951,7 @@ def main():
     ap.add_argument("--skip-points", action="store_true", help="skip the batch-1 and batch-64 points")
     ap.add_argument("--only-decode", action="store_true", help="time the decode steps only (for profiler captures)")
     ap.add_argument("--only-prefill", action="store_true", help="time the 2,048-token prompt only (for profiler captures)")
-    ap.add_argument("--workload", default="headline", choices=["headline", "continuous", "long", "sizes", "vipotar", "negotar", "keralix", "zepesun"],
+    ap.add_argument("--workload", default="headline", choices=["headline", "continuous", "long", "sizes", "vipotar", "negotar", "keralix", "zepesun", "modinex"],
                     help="headline (default): the one JSON line described at the top of this file.  continuous: LFM2-700M sizes, requests with prompts "
                          "of 64 to 4,096 tokens through 32 slots in 512-token portions beside decode rows, temperature 0.7, 128 new "
                          "tokens each.  long: LFM2-350M sizes, 4 prompts of 32,768 tokens and 512 greedy tokens each, bfloat16 and 32-bit.  "
@@ -896,6 +985,8 @@ def main():
         return workload_keralix(args)
     if args.workload == "zepesun":
         return workload_zepesun(args)
+    if args.workload == "modinex":
+        return workload_modinex(args)
     cfg = dict(LFM2_1_2B)
     if args.layers is not None and args.layers < cfg["num_hidden_layers"]:
         cfg["layer_types"] = cfg["layer_types"][:args.layers]

@@ -625,6 +625,17 @@ def linear_gated(x, w_gu: torch.Tensor, out: torch.Tensor, kind: str, limit: flo
     gated_act(tmp, out, kind, limit, bias)
 
 
+def _partials_scratch(device, floats: int) -> torch.Tensor:
+    """Scratch for the split partials of a product whose reader folds them (one set at a time), at least `floats` long."""
+    key = torch.device(device).index or 0
+    buf = _S.partials.get(key)
+    if buf is None or buf.numel() < floats:
+        _need(not torch.cuda.is_current_stream_capturing(), "partials scratch would grow during graph capture")
+        _S.generation += 0 if buf is None else 1              # a buffer that did not exist is in no captured graph
+        buf = _S.partials[key] = torch.empty(_grown(floats, buf), dtype=torch.float32, device=device)
+    return buf
+
+
 def linear(x, w: torch.Tensor, out: torch.Tensor, accumulate: bool = False,
            status: Optional[torch.Tensor] = None) -> None:
     """out[M,N] (+)= x[M,K] @ w[N,K]^T.  float32 x/w -> the FFMA kernel (true 32-bit);
@@ -650,12 +661,7 @@ def linear(x, w: torch.Tensor, out: torch.Tensor, accumulate: bool = False,
             if u is not None and out.dtype == torch.float32:
                 nt, splits, floats, _ = _tc_plan(M, N, K, EPI_PARTIAL)
                 if splits > 1:
-                    key = torch.device(x.device).index or 0
-                    buf = _S.partials.get(key)
-                    if buf is None or buf.numel() < floats:
-                        _need(not torch.cuda.is_current_stream_capturing(), "partials scratch would grow during graph capture")
-                        _S.generation += 0 if buf is None else 1
-                        buf = _S.partials[key] = torch.empty(_grown(floats, buf), dtype=torch.float32, device=x.device)
+                    buf = _partials_scratch(x.device, floats)
                     gemm_tc(x, w, out, EPI_PARTIAL, status, scratch=buf)
                     u[0] = (buf, splits)
                     return
@@ -663,12 +669,7 @@ def linear(x, w: torch.Tensor, out: torch.Tensor, accumulate: bool = False,
                 settle(out)                                       # one set of partials at a time
                 nt, splits, floats, _ = _tc_plan(M, N, K, EPI_PARTIAL)
                 if splits > 1:
-                    key = torch.device(x.device).index or 0
-                    buf = _S.partials.get(key)
-                    if buf is None or buf.numel() < floats:
-                        _need(not torch.cuda.is_current_stream_capturing(), "partials scratch would grow during graph capture")
-                        _S.generation += 0 if buf is None else 1      # a buffer that did not exist is in no captured graph
-                        buf = _S.partials[key] = torch.empty(_grown(floats, buf), dtype=torch.float32, device=x.device)
+                    buf = _partials_scratch(x.device, floats)
                     gemm_tc(x, w, out, EPI_PARTIAL, status, scratch=buf)
                     _S.pending[out.data_ptr()] = (buf, splits, M, N)
                     return
@@ -763,13 +764,7 @@ def _into_stream(out: torch.Tensor, M: int, N: int, K: int):
         settle(out)                                           # one set of partials at a time
         nt, splits, floats, _ = _tc_plan(M, N, K, EPI_PARTIAL)
         if splits > 1:
-            key = torch.device(out.device).index or 0
-            buf = _S.partials.get(key)
-            if buf is None or buf.numel() < floats:
-                _need(not torch.cuda.is_current_stream_capturing(), "partials scratch would grow during graph capture")
-                _S.generation += 0 if buf is None else 1
-                buf = _S.partials[key] = torch.empty(_grown(floats, buf), dtype=torch.float32, device=out.device)
-            return EPI_PARTIAL, buf, splits
+            return EPI_PARTIAL, _partials_scratch(out.device, floats), splits
     settle(out)
     return EPI_ADD_F32, None, 1
 
@@ -786,20 +781,31 @@ def _after_stream_product(out, epi, buf, splits, M, N) -> None:
         _S.pending[out.data_ptr()] = (buf, splits, M, N)
 
 
-def linear_of_attention_partials(part_acc, part_ml, n_tok, nh, hd, n_splits, w_out, out, status) -> bool:
-    """out += combine(partials) w_out^T: the ordered combine of the split-key attention's partial results (as
+def linear_of_attention_partials(part_acc, part_ml, n_tok, nh, hd, n_splits, w_out, out, status, accumulate: bool = True) -> bool:
+    """out += combine(partials) w_out^T (accumulate False: out, which must be an unfinished buffer, receives the product): the ordered combine of the split-key attention's partial results (as
     paged_attention_split(out=None) leaves them) computed inside the output product.  Returns False, having launched
     nothing, when the kernel does not take the case; the caller then combines with attention_split_combine."""
     if not (_produced_usable(n_tok, w_out, out) and w_out.shape[1] == nh * hd and hd % 8 == 0 and n_splits <= 64):
         return False
     _cuda(part_acc, part_ml, w_out, out, status)
     N, K = w_out.shape
-    epi, buf, splits = _into_stream(out, n_tok, N, K)
+    u = None
+    if accumulate:
+        epi, buf, splits = _into_stream(out, n_tok, N, K)
+    else:
+        u = _S.unfinished.get(out.data_ptr())
+        epi, splits = EPI_PARTIAL, _tc_plan(n_tok, N, K, EPI_PARTIAL)[1]
+        if u is None or splits < 2:
+            return False
+        buf = _partials_scratch(out.device, _tc_plan(n_tok, N, K, EPI_PARTIAL)[2])
     rc = _lib.kernels().imparo_gemm_tc_combine(_ptr(part_acc), _ptr(part_ml), nh, hd, n_splits, _ptr(w_out), _ptr(out),
                                                out.stride(0), n_tok, N, K, epi, _ptr(buf), _ptr(status), _stream())
     if rc == -25:
         return False
     _check(rc, "gemm_tc_combine")
+    if u is not None:
+        u[0] = (buf, splits)
+        return True
     _after_stream_product(out, epi, buf, splits, n_tok, N)
     return True
 
@@ -1106,6 +1112,68 @@ def attention_prefill(q, k_cache, v_cache, item_row_start, item_start_pos, n_ite
     if only_tc:
         return False
     _check(_lib.kernels().imparo_attention_prefill(*args), "attention_prefill")
+    return True
+
+
+# ---- attention with sigmoid weights (csrc/kernels/attention_sigmoid.cu) -----------------------------------------
+def _sigmoid_takes(q, k_cache, v_cache, nh, nkv, hd, vd) -> bool:
+    return (q.dtype == torch.bfloat16 and k_cache.dtype == q.dtype and v_cache.dtype == q.dtype and hd % 16 == 0 and vd % 16 == 0
+            and 16 <= hd <= 128 and 16 <= vd <= 128 and nkv >= 1 and nh % nkv == 0)
+
+
+def attention_sigmoid_prefill(q, k_cache, v_cache, item_row_start, item_start_pos, n_items, table, page_size, n_pages, window, chunk,
+                              scale, score_bias, out, nh, nkv, hd, vd, status) -> bool:
+    """Prompt portions on the tcgen05 kernel: out = sum over visible keys of sigmoid(scale q.k + score_bias[head]) v.  window /
+    chunk: as in attention_any.  bfloat16, key and value size multiples of 16 up to 128, at most 128 query heads per kv head,
+    pages of 16 to 128 positions; returns False, having launched nothing, for other shapes."""
+    if not _sigmoid_takes(q, k_cache, v_cache, nh, nkv, hd, vd) or nh // nkv > 128 or page_size not in (16, 32, 64, 128):
+        return False
+    if _S.switches.attn_prefill == "mma":
+        return False
+    _cuda(q, k_cache, v_cache, item_row_start, item_start_pos, table, score_bias, out, status)
+    T = q.shape[0]
+    _need(q.shape == (T, nh * hd) and out.shape == (T, nh * vd) and out.dtype == q.dtype, "attention_sigmoid_prefill: q/out shapes")
+    _need(k_cache.numel() >= n_pages * page_size * nkv * hd and v_cache.numel() >= n_pages * page_size * nkv * vd,
+          "cache arena smaller than n_pages")
+    _need(table.dtype == torch.int32 and table.dim() == 2 and table.shape[0] >= n_items, "block table must be int32 [items, blocks]")
+    _need(item_row_start.numel() >= n_items + 1 and item_start_pos.numel() >= n_items, "attention_sigmoid_prefill: item arrays")
+    _need(score_bias.dtype == torch.float32 and score_bias.numel() == nh, "attention_sigmoid_prefill: score bias float32 [heads]")
+    rc = _lib.kernels().imparo_attention_sigmoid_prefill(
+        _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(item_row_start), _ptr(item_start_pos), n_items, _ptr(table), table.shape[1], page_size,
+        n_pages, int(window or 0), int(chunk or 0), float(scale), _ptr(score_bias), _ptr(out), T, nh, nkv, hd, vd, _ptr(status), _stream())
+    if rc == -8:
+        return False
+    _check(rc, "attention_sigmoid_prefill")
+    return True
+
+
+def attention_sigmoid_split(q, k_cache, v_cache, positions, item_of_token, table, page_size, n_pages, window, chunk, scale, score_bias,
+                            out, part_acc, part_ml, range_, n_splits, nh, nkv, hd, vd, status, fresh: int = 0) -> bool:
+    """Single query tokens on tensor cores, a CTA per (range of `range_` keys counted from the query's first key, kv head, token),
+    then the ordered combine into out (out None: the partials stay for linear_of_attention_partials).  At most 8 query heads per
+    kv head; sizes, masks and fresh as in attention_sigmoid_prefill / paged_attention_split.  Returns False for other shapes."""
+    if not _sigmoid_takes(q, k_cache, v_cache, nh, nkv, hd, vd) or nh // nkv > 8:
+        return False
+    _cuda(q, k_cache, v_cache, positions, item_of_token, table, score_bias, out, part_acc, part_ml, status)
+    T = q.shape[0]
+    _need(q.shape == (T, nh * hd) and (out is None or (out.shape == (T, nh * vd) and out.dtype == q.dtype)), "attention_sigmoid_split: q/out shapes")
+    _need(k_cache.numel() >= n_pages * page_size * nkv * hd and v_cache.numel() >= n_pages * page_size * nkv * vd,
+          "cache arena smaller than n_pages")
+    _need(table.dtype == torch.int32 and table.dim() == 2, "block table must be int32 [items, blocks]")
+    _need(score_bias.dtype == torch.float32 and score_bias.numel() == nh, "attention_sigmoid_split: score bias float32 [heads]")
+    _need(part_acc.dtype == torch.float32 and part_acc.numel() >= T * nh * n_splits * vd
+          and part_ml.dtype == torch.float32 and part_ml.numel() >= T * nh * n_splits * 2, "split scratch too small")
+    span = min([table.shape[1] * page_size] + [int(x) for x in (window, chunk) if x])
+    _need(T <= 65535 and 1 <= n_splits <= MAX_SPLITS and range_ * n_splits >= span, "attention_sigmoid_split: ranges must cover what a query sees")
+    rc = _lib.kernels().imparo_attention_sigmoid_split(
+        _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(positions), _ptr(item_of_token), _ptr(table), table.shape[1], page_size, n_pages,
+        int(window or 0), int(chunk or 0), float(scale), _ptr(score_bias), _ptr(part_acc), _ptr(part_ml), T, nh, nkv, hd, vd, int(range_),
+        int(n_splits), int(fresh), _ptr(status), _stream())
+    if rc == -8:
+        return False
+    _check(rc, "attention_sigmoid_split")
+    if out is not None:
+        attention_split_combine(part_acc, part_ml, out, T * nh, vd, n_splits)
     return True
 
 
@@ -1865,6 +1933,77 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g: torch.Te
     _check(_lib.kernels().imparo_gla_recurrent(_ptr(proj), proj.stride(0), _code(proj), int(q_off), int(k_off), int(v_off), _ptr(g),
                                                float(q_scale), _ptr(state), _ptr(item_row_start), _ptr(item_slot), state.shape[0],
                                                n_items, _ptr(out), heads, dim, vdim, _ptr(status), _stream()), "gla_recurrent")
+
+
+def gla_step(proj: torch.Tensor, offsets, rank: int, w2: torch.Tensor, bias: torch.Tensor, tau: float, w_norm: torch.Tensor, eps: float,
+             q_scale: float, state: torch.Tensor, item_row_start, item_slot, n_items: int, out: torch.Tensor, heads: int, dim: int,
+             vdim: int, status: torch.Tensor) -> bool:
+    """gla_decay, gla_scan and head_norm_gate (silu) in one kernel for a step in which every request brings one row.  offsets: the
+    columns of q, k, v, the gate and the decay's inner rows in proj.  Returns False, having launched nothing, for head sizes it
+    does not take."""
+    if (vdim + (8 if dim > 128 else 16 if dim > 64 else 32) - 1) // (8 if dim > 128 else 16 if dim > 64 else 32) > 16:
+        return False
+    _need(proj.is_cuda and proj.stride(1) == 1, "gla_step: rows of proj must be dense CUDA memory")
+    _cuda(w2, bias, w_norm, state, item_row_start, item_slot, out, status)
+    T = proj.shape[0]
+    q_off, k_off, v_off, g_off, l_off = (int(x) for x in offsets)
+    _need(T == n_items and item_row_start.numel() >= n_items + 1 and item_slot.numel() >= n_items, "gla_step: one row per request")
+    _need(tuple(w2.shape) == (heads * dim, rank) and w2.dtype == proj.dtype and bias.dtype == torch.float32 and bias.numel() == heads * dim,
+          "gla_step: w2 [heads * dim, rank] of proj's dtype, bias float32 [heads * dim]")
+    _need(w_norm.dtype == torch.float32 and w_norm.numel() == vdim, "gla_step: norm weight float32 [vdim]")
+    _need(state.dtype == torch.float32 and tuple(state.shape[1:]) == (heads, dim, vdim), "gla_step: state float32 [slots, heads, dim, vdim]")
+    _need(out.dtype == proj.dtype and tuple(out.shape) == (T, heads * vdim), "gla_step: out [T, heads * vdim] of proj's dtype")
+    _need(max(q_off, k_off) + heads * dim <= proj.shape[1] and max(v_off, g_off) + heads * vdim <= proj.shape[1]
+          and l_off + rank <= proj.shape[1], "gla_step: columns")
+    rc = _lib.kernels().imparo_gla_step(_ptr(proj), proj.stride(0), _code(proj), q_off, k_off, v_off, g_off, l_off, _ptr(w2), _ptr(bias),
+                                        float(tau), int(rank), _ptr(w_norm), float(eps), float(q_scale), _ptr(state), _ptr(item_row_start),
+                                        _ptr(item_slot), state.shape[0], n_items, _ptr(out), heads, dim, vdim, _ptr(status), _stream())
+    if rc == -8:
+        return False
+    _check(rc, "gla_step")
+    return True
+
+
+GLA_CHUNK = 64             # rows per chunk of gla_chunked
+GLA_CHUNK_COLUMNS = 128    # up to this value size gla_chunked also norms and gates
+
+
+def gla_chunked_takes(proj: torch.Tensor, offsets, dim: int, vdim: int) -> bool:
+    """Whether gla_chunked takes these sizes: bfloat16, key size a multiple of 16 up to 128, value size a multiple of 16, aligned
+    columns."""
+    q_off, k_off, v_off, g_off = (int(x) for x in offsets[:4])
+    return (proj.dtype == torch.bfloat16 and dim % 16 == 0 and 16 <= dim <= 128 and vdim % 16 == 0 and proj.stride(0) % 8 == 0
+            and v_off % 8 == 0 and q_off % 2 == 0 and k_off % 2 == 0 and g_off % 2 == 0 and proj.data_ptr() % 16 == 0)
+
+
+def gla_chunked(proj: torch.Tensor, offsets, g: torch.Tensor, q_scale: float, w_norm: torch.Tensor, eps: float, state: torch.Tensor,
+                item_row_start, item_slot, n_items: int, chunk_state: torch.Tensor, chunk_decay: torch.Tensor, o: Optional[torch.Tensor],
+                y: torch.Tensor, heads: int, dim: int, vdim: int, status: torch.Tensor) -> bool:
+    """gla_scan for batches with long portions, in chunks of GLA_CHUNK rows side by side on tensor cores (gla_chunked_takes).
+    chunk_state / chunk_decay: float32 scratch for (T // GLA_CHUNK + n_items) * heads * dim * vdim (* dim) values.  vdim up to
+    GLA_CHUNK_COLUMNS: y [T, heads * vdim] receives the outputs normed per head, times w_norm, times silu of the gate's columns
+    (True); else o (float32) the plain outputs (False)."""
+    _need(gla_chunked_takes(proj, offsets, dim, vdim), "gla_chunked: sizes")
+    _cuda(g, w_norm, state, item_row_start, item_slot, chunk_state, chunk_decay, o, y, status)
+    T = proj.shape[0]
+    q_off, k_off, v_off, g_off = (int(x) for x in offsets[:4])
+    chunks = T // GLA_CHUNK + n_items
+    normed = vdim <= GLA_CHUNK_COLUMNS
+    _need(g.dtype == torch.float32 and tuple(g.shape) == (T, heads * dim), "gla_chunked: g float32 [T, heads * dim]")
+    _need(chunk_state.dtype == torch.float32 and chunk_state.numel() >= chunks * heads * dim * vdim and chunk_decay.dtype == torch.float32
+          and chunk_decay.numel() >= chunks * heads * dim, "gla_chunked: scratch too small")
+    _need(state.dtype == torch.float32 and tuple(state.shape[1:]) == (heads, dim, vdim), "gla_chunked: state float32 [slots, heads, dim, vdim]")
+    _need(w_norm.dtype == torch.float32 and w_norm.numel() == vdim, "gla_chunked: norm weight float32 [vdim]")
+    _need(y.dtype == torch.bfloat16 and tuple(y.shape) == (T, heads * vdim), "gla_chunked: y bfloat16 [T, heads * vdim]")
+    _need(normed or (o is not None and o.dtype == torch.float32 and tuple(o.shape) == (T, heads * vdim)), "gla_chunked: o float32 [T, heads * vdim]")
+    _need(max(q_off, k_off) + heads * dim <= proj.shape[1] and max(v_off, g_off) + heads * vdim <= proj.shape[1], "gla_chunked: columns")
+    _need(item_row_start.numel() >= n_items + 1 and item_slot.numel() >= n_items, "gla_chunked: item arrays")
+    _check(_lib.kernels().imparo_gla_chunked(_ptr(proj), proj.stride(0), q_off, k_off, v_off, g_off, _ptr(g), float(q_scale), _ptr(w_norm),
+                                             float(eps), _ptr(state), _ptr(item_row_start), _ptr(item_slot), state.shape[0], n_items, T,
+                                             _ptr(chunk_state), _ptr(chunk_decay), _ptr(o), _ptr(y), heads, dim, vdim, _ptr(status),
+                                             _stream()), "gla_chunked")
+    COUNTS["own"] += 2
+    return normed
 
 
 # ---- a matrix memory with exponential gates (csrc/kernels/mlstm.cu) ---------------------------------------------

@@ -271,6 +271,10 @@ class AttentionMixer(Part):
                                      self.position.magnitude, q, kv.k, kv.v, table, kv.page_size, kv.n_pages, nh, nkv, hd, vd, rt.status)
         out = rt.workspace.get("attn_out", (T, nh * vd), rt.act_dtype, first="tokens")
         done = False
+        if self.sigmoid and rt.act_dtype == torch.bfloat16 and T <= 65535:
+            done = self._attend_sigmoid(q, batch, kv, table, out, residual, accumulate)
+            if done == "product":
+                return
         if (rt.act_dtype == torch.bfloat16 and hd == vd and hd in (64, 128) and nh // self.nkv <= 8 and T <= 65535
                 and not self.sigmoid and self.chunk is None):
             # the tensor-core kernels take these sizes (the sink as a flag): prompt portions on the tcgen05 kernel, rows
@@ -307,6 +311,41 @@ class AttentionMixer(Part):
         ops.linear(out, self.w_o, residual, accumulate=accumulate, status=rt.status)
         if self.prepared and self.b_o is not None:
             ops.add_bias(residual, self.b_o)
+
+    def _attend_sigmoid(self, q, batch, kv, table, out, residual, accumulate):
+        """Sigmoid weights on the tensor-core kernels: prompt portions on the tcgen05 kernel, rows of one token (and portions too
+        short for a tile, or pages it does not take) on the split-key kernel.  False: they do not take these sizes; "product": the
+        output product is made too (decode rows, the partial sums added inside it)."""
+        rt, T = self.rt, q.shape[0]
+        nh, hd, vd = self.nh, self.hd, self.vd
+        n1 = getattr(batch, "n_single", 0)
+        n = T                                # rows left to the split-key kernel: the first n
+        if batch.max_tokens_per_item >= 8:
+            first = n1 if 0 < n1 < batch.n_items else 0
+            if ops.attention_sigmoid_prefill(q, kv.k, kv.v, batch.item_row_start[first:], batch.item_start_pos[first:],
+                                             batch.n_items - first, table[first:], kv.page_size, kv.n_pages, self.window, self.chunk,
+                                             self.scale, self.score_bias, out, nh, self.nkv, hd, vd, rt.status):
+                n = first
+        if n == 0:
+            return True
+        spans = [table.shape[1] * kv.page_size] + [x for x in (self.window, self.chunk) if x]
+        range_, n_splits = ops.split_plan(n, self.nkv, min(spans))
+        rows = max(rt.workspace.most.get("rows", 0), n)
+        room = rows * nh * n_splits if len(spans) > 1 else self._partials_room(spans[0])
+        part_acc = rt.workspace.get("attn_part_acc", (n * nh * n_splits * vd,), torch.float32, reserve=room * vd)
+        part_ml = rt.workspace.get("attn_part_ml", (n * nh * n_splits * 2,), torch.float32, reserve=room * 2)
+        in_product = batch.decode_only and n == T and n_splits <= 64 and ops.fuse_producers() and self.b_o is None and not self.gate
+        if not ops.attention_sigmoid_split(q[:n], kv.k, kv.v, batch.positions[:n], batch.item_of_token[:n], table, kv.page_size,
+                                           kv.n_pages, self.window, self.chunk, self.scale, self.score_bias,
+                                           None if in_product else out[:n], part_acc, part_ml, range_, n_splits, nh, self.nkv, hd, vd,
+                                           rt.status, fresh=batch.max_tokens_per_item):
+            return False
+        if in_product:
+            if ops.linear_of_attention_partials(part_acc, part_ml, T, nh, vd, n_splits, self.w_o, residual, rt.status,
+                                                accumulate=accumulate):
+                return "product"
+            ops.attention_split_combine(part_acc, part_ml, out, T * nh, vd, n_splits)
+        return True
 
     def forward(self, x, batch, caches, residual, accumulate=True, projected=None):
         kv = caches[0]

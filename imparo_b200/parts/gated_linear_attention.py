@@ -21,6 +21,7 @@ class GatedLinearAttention(Part):
 
     forward(..., accumulate=False) overwrites `residual` (then any float32 [tokens, hidden] buffer)."""
     adds_with_linear = True
+    CHUNK_FROM = 128          # portions from this many tokens on (rounded up to a power of two) run in chunks
 
     NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o", "norm": "norm", "a1": "a1", "a2": "a2", "a2_bias": "a2.b"}
 
@@ -65,7 +66,7 @@ class GatedLinearAttention(Part):
         self.w_in = torch.zeros(((at + 7) // 8 * 8, first.shape[1]), dtype=first.dtype, device=first.device)
         for a, w in parts:
             self.w_in[a:a + w.shape[0]] = w
-        self.q_at, self.k_at, self.v_at, self.g_at, self.a_at = (a for a, _ in parts)
+        self.columns = tuple(a for a, _ in parts)
         self.w_a2, self.b_a2 = tensors[n["a2"]], tensors[n["a2_bias"]]
         self.w_o = tensors[n["o"]]
         self.w_norm = tensors[n["norm"]]
@@ -80,12 +81,28 @@ class GatedLinearAttention(Part):
         H, D, V = self.heads, self.dim, self.vdim
         proj = ws.get("gla_in", (T, self.w_in.shape[0]), rt.act_dtype, first="tokens")
         ops.linear(x, self.w_in, proj, status=rt.status)
-        low, gate = proj[:, self.a_at:self.a_at + self.rank], proj[:, self.g_at:self.g_at + self.vv]
+        q_at, k_at, v_at, g_at, a_at = self.columns
+        q_scale = float(D) ** -0.5
         y = ws.get("gla_y", (T, self.vv), rt.act_dtype, first="tokens")
-        g = ws.get("gla_decay", (T, self.qk), torch.float32, first="tokens")
-        ops.gla_decay(low, self.w_a2, self.b_a2, self.tau, g)
-        o = ws.get("gla_o", (T, self.vv), torch.float32, first="tokens")
-        ops.gla_scan(proj, self.q_at, self.k_at, self.v_at, g, float(D) ** -0.5, st.state, batch.item_row_start, batch.item_slot,
-                     batch.n_items, o, H, D, V, rt.status)
-        ops.head_norm_gate(o, self.w_norm, self.eps, gate, y, H, V, act="silu")
+        # one row per request: decay, recurrence, norm and gate are one kernel
+        done = batch.decode_only and ops.gla_step(proj, self.columns, self.rank, self.w_a2, self.b_a2, self.tau, self.w_norm, self.eps,
+                                                  q_scale, st.state, batch.item_row_start, batch.item_slot, batch.n_items, y, H, D, V,
+                                                  rt.status)
+        if not done:
+            g = ws.get("gla_decay", (T, self.qk), torch.float32, first="tokens")
+            ops.gla_decay(proj[:, a_at:a_at + self.rank], self.w_a2, self.b_a2, self.tau, g)
+            in_chunks = batch.max_tokens_per_item >= self.CHUNK_FROM and ops.gla_chunked_takes(proj, self.columns, D, V)
+            o = None
+            if not in_chunks or V > ops.GLA_CHUNK_COLUMNS:
+                o = ws.get("gla_o", (T, self.vv), torch.float32, first="tokens")
+            if in_chunks:
+                chunks = T // ops.GLA_CHUNK + batch.n_items
+                done = ops.gla_chunked(proj, self.columns, g, q_scale, self.w_norm, self.eps, st.state, batch.item_row_start,
+                                       batch.item_slot, batch.n_items, ws.get("gla_chunk_state", (chunks * H * D * V,), torch.float32),
+                                       ws.get("gla_chunk_decay", (chunks * H * D,), torch.float32), o, y, H, D, V, rt.status)
+            else:
+                ops.gla_scan(proj, q_at, k_at, v_at, g, q_scale, st.state, batch.item_row_start, batch.item_slot, batch.n_items, o, H, D,
+                             V, rt.status)
+            if not done:
+                ops.head_norm_gate(o, self.w_norm, self.eps, proj[:, g_at:g_at + self.vv], y, H, V, act="silu")
         ops.linear(y, self.w_o, residual, accumulate=accumulate, status=rt.status)
