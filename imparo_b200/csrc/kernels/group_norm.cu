@@ -9,9 +9,10 @@
 //      updated row: the norm after one sublayer, its add into the 32-bit stream and the norm before the next sublayer.
 //      y may still be the split partials of the product that makes it (summed in split order) and may lack its bias.
 //
-// A block per row.  A group belongs to a team of `wpg` warps (one warp per group when there are at least as many groups as
-// warps); the sum over a group is a fixed tree over the team's lanes, so a row's result depends on the row alone.  All
-// arithmetic is 32-bit.
+// Few rows: a block per row.  A group belongs to a team of `wpg` warps (one warp per group when there are at least as many groups as
+// warps); the sum over a group is a fixed tree over the team's lanes, so a row's result depends on the row alone.
+// Many rows (a prompt portion) with groups of up to 1,024 elements: a warp per (row, group) that keeps the group in registers;
+// every load of the group is in flight at once and there is no barrier.  All arithmetic is 32-bit.
 #include "common.cuh"
 
 namespace imparo {
@@ -24,7 +25,7 @@ template <typename TOut, int V> struct Vec;
 template <typename TOut> struct Vec<TOut, 1> {
     float v[1];
     __device__ __forceinline__ void load(const float* p) { v[0] = *p; }
-    __device__ __forceinline__ void add(const float* p) { v[0] += __ldcg(p); }
+    __device__ __forceinline__ void load_cg(const float* p) { v[0] = __ldcg(p); }
     __device__ __forceinline__ void store(float* p) const { *p = v[0]; }
     static __device__ __forceinline__ void put(TOut* p, const float (&o)[1]) { *p = from_f32<TOut>(o[0]); }
 };
@@ -34,9 +35,9 @@ template <typename TOut> struct Vec<TOut, 4> {
         const float4 q = *reinterpret_cast<const float4*>(p);
         v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
     }
-    __device__ __forceinline__ void add(const float* p) {
+    __device__ __forceinline__ void load_cg(const float* p) {
         const float4 q = __ldcg(reinterpret_cast<const float4*>(p));
-        v[0] += q.x; v[1] += q.y; v[2] += q.z; v[3] += q.w;
+        v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
     }
     __device__ __forceinline__ void store(float* p) const { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
     static __device__ __forceinline__ void put(TOut* p, const float (&o)[4]) {
@@ -144,7 +145,18 @@ __global__ void group_norm_add_kernel(float* __restrict__ x, const float* __rest
 #pragma unroll
                 for (int e = 0; e < V; ++e) t.v[e] = 0.f;
             }
-            for (int s = 0; s < parts; ++s) t.add(y + (size_t)s * part_stride + row + i);
+            for (int s0 = 0; s0 < parts; s0 += 8) {            // eight partials' loads in flight, added in order
+                W p[8];
+#pragma unroll
+                for (int u = 0; u < 8; ++u) if (s0 + u < parts) p[u].load_cg(y + (size_t)(s0 + u) * part_stride + row + i);
+#pragma unroll
+                for (int u = 0; u < 8; ++u) {
+                    if (s0 + u < parts) {
+#pragma unroll
+                        for (int e = 0; e < V; ++e) t.v[e] += p[u].v[e];
+                    }
+                }
+            }
             return t;
         };
         W v[REGS], xv[REGS];
@@ -211,6 +223,99 @@ __global__ void group_norm_add_kernel(float* __restrict__ x, const float* __rest
     }
 }
 
+// ---- many rows: a warp per (row, group), NV float4 per lane (groups of up to 128 * NV elements, multiples of 4) ---------------
+constexpr int ROW_WARPS = 4, MANY_ROWS = 256;
+
+template <typename TOut, int NV>
+__global__ void __launch_bounds__(ROW_WARPS * 32)
+group_rmsnorm_rows_kernel(const float* __restrict__ x, const int* __restrict__ rows, const float* __restrict__ w, float eps,
+                          TOut* __restrict__ out, int n_rows, int width, int groups) {
+    pdl_trigger();
+    const int lane = threadIdx.x & 31;
+    const long long task = (long long)blockIdx.x * ROW_WARPS + (threadIdx.x >> 5);
+    const int r = (int)(task / groups), g = (int)(task - (long long)r * groups), gw = width / groups, n4 = gw / 4;
+    const float4* wg = reinterpret_cast<const float4*>(w + (size_t)g * gw);
+    float4 ww[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) if (lane + 32 * i < n4) ww[i] = __ldg(wg + lane + 32 * i);
+    pdl_wait();
+    if (r >= n_rows) return;
+    const float4* xr = reinterpret_cast<const float4*>(x + (size_t)(rows ? rows[r] : r) * width + (size_t)g * gw);
+    float4 v[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) v[i] = lane + 32 * i < n4 ? xr[lane + 32 * i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    const float scale = 1.0f / sqrtf(warp_sum(ss) / (float)gw + eps);
+    TOut* o = out + (size_t)r * width + (size_t)g * gw;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        if (lane + 32 * i < n4) {
+            const float y[4] = {v[i].x * scale * ww[i].x, v[i].y * scale * ww[i].y, v[i].z * scale * ww[i].z, v[i].w * scale * ww[i].w};
+            Vec<TOut, 4>::put(o + 4 * (lane + 32 * i), y);
+        }
+    }
+}
+
+template <typename TOut, int NV>
+__global__ void __launch_bounds__(ROW_WARPS * 32)
+group_norm_add_rows_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ ybias,
+                           const float* __restrict__ wb, float eps_b, const float* __restrict__ wn, float eps_n,
+                           TOut* __restrict__ out, int n_rows, int width, int groups) {
+    pdl_trigger();
+    const int lane = threadIdx.x & 31;
+    const long long task = (long long)blockIdx.x * ROW_WARPS + (threadIdx.x >> 5);
+    const int r = (int)(task / groups), g = (int)(task - (long long)r * groups), gw = width / groups, n4 = gw / 4;
+    const size_t col = (size_t)g * gw;
+    pdl_wait();
+    if (r >= n_rows) return;
+    const size_t row = (size_t)r * width + col;
+    const float4* yr = reinterpret_cast<const float4*>(y + row);
+    float4* xr = reinterpret_cast<float4*>(x + row);
+    float4 v[NV], xv[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) v[i] = lane + 32 * i < n4 ? yr[lane + 32 * i] : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) xv[i] = lane + 32 * i < n4 ? xr[lane + 32 * i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    if (ybias) {
+        const float4* b = reinterpret_cast<const float4*>(ybias + col);
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            if (lane + 32 * i < n4) {
+                const float4 t = __ldg(b + lane + 32 * i);
+                v[i].x += t.x; v[i].y += t.y; v[i].z += t.z; v[i].w += t.w;
+            }
+        }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    const float scale = 1.0f / sqrtf(warp_sum(ss) / (float)gw + eps_b);
+    float ss2 = 0.f;
+    const float4* b4 = reinterpret_cast<const float4*>(wb + col);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        if (lane + 32 * i < n4) {
+            const float4 t = __ldg(b4 + lane + 32 * i);
+            xv[i].x += v[i].x * scale * t.x; xv[i].y += v[i].y * scale * t.y; xv[i].z += v[i].z * scale * t.z; xv[i].w += v[i].w * scale * t.w;
+            xr[lane + 32 * i] = xv[i];
+            ss2 += xv[i].x * xv[i].x + xv[i].y * xv[i].y + xv[i].z * xv[i].z + xv[i].w * xv[i].w;
+        }
+    }
+    if (out == nullptr) return;
+    const float nscale = 1.0f / sqrtf(warp_sum(ss2) / (float)gw + eps_n);
+    const float4* n4w = reinterpret_cast<const float4*>(wn + col);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        if (lane + 32 * i < n4) {
+            const float4 t = __ldg(n4w + lane + 32 * i);
+            const float o[4] = {xv[i].x * nscale * t.x, xv[i].y * nscale * t.y, xv[i].z * nscale * t.z, xv[i].w * nscale * t.w};
+            Vec<TOut, 4>::put(out + row + 4 * (lane + 32 * i), o);
+        }
+    }
+}
+
 // warps of a block and warps per group: as many warps as keep a thread at REGS vectors of its group or fewer, up to 8
 static void plan(int width, int groups, int v, int* warps, int* wpg) {
     int nw = (width + 32 * v * 2 - 1) / (32 * v * 2);         // about two vectors per thread
@@ -231,6 +336,19 @@ extern "C" int imparo_group_rmsnorm(const float* x, const int* rows, const float
     if (n_rows <= 0) return 0;
     if (groups < 1 || width < 1 || width % groups != 0) return -2;
     const bool vec = (width / groups) % 4 == 0 && (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) == 0;
+    if (vec && n_rows >= gn::MANY_ROWS && width / groups <= 1024) {
+        const dim3 grid((unsigned)(((long long)n_rows * groups + gn::ROW_WARPS - 1) / gn::ROW_WARPS)), block(gn::ROW_WARPS * 32);
+        const int nv = (width / groups + 127) / 128;
+#define IMPARO_GR(T_, N_) launch(gn::group_rmsnorm_rows_kernel<T_, N_>, grid, block, 0, stream, x, rows, w, eps, (T_*)out, n_rows, width, groups)
+#define IMPARO_GRN(T_) do { if (nv <= 1) IMPARO_GR(T_, 1); else if (nv <= 2) IMPARO_GR(T_, 2); else if (nv <= 4) IMPARO_GR(T_, 4); else IMPARO_GR(T_, 8); } while (0)
+        if (out_dtype == IMPARO_DT_F32) IMPARO_GRN(float);
+        else if (out_dtype == IMPARO_DT_BF16) IMPARO_GRN(__nv_bfloat16);
+        else return -1;
+#undef IMPARO_GRN
+#undef IMPARO_GR
+        IMPARO_CHECK_LAUNCH();
+        return 0;
+    }
     int nw, wpg;
     gn::plan(width, groups, vec ? 4 : 1, &nw, &wpg);
 #define IMPARO_GN(T_, V_) launch(gn::group_rmsnorm_kernel<T_, V_>, dim3(n_rows), dim3(32 * nw), 0, stream, x, rows, w, eps, (T_*)out, \
@@ -254,6 +372,20 @@ extern "C" int imparo_group_norm_add(float* x, const float* y, int parts, long l
     if (out != nullptr && wn == nullptr) return -2;
     const uintptr_t all = (uintptr_t)x | (uintptr_t)y | (uintptr_t)ybias | (uintptr_t)wb | (uintptr_t)wn | (uintptr_t)out;
     const bool vec = (width / groups) % 4 == 0 && (all & 15) == 0 && (parts == 1 || part_stride % 4 == 0);
+    if (vec && parts == 1 && n_rows >= gn::MANY_ROWS && width / groups <= 1024) {
+        const dim3 grid((unsigned)(((long long)n_rows * groups + gn::ROW_WARPS - 1) / gn::ROW_WARPS)), block(gn::ROW_WARPS * 32);
+        const int nv = (width / groups + 127) / 128;
+#define IMPARO_GR(T_, N_) launch(gn::group_norm_add_rows_kernel<T_, N_>, grid, block, 0, stream, x, y, ybias, wb, eps_b, wn, eps_n, (T_*)out, \
+        n_rows, width, groups)
+#define IMPARO_GRN(T_) do { if (nv <= 1) IMPARO_GR(T_, 1); else if (nv <= 2) IMPARO_GR(T_, 2); else if (nv <= 4) IMPARO_GR(T_, 4); else IMPARO_GR(T_, 8); } while (0)
+        if (out == nullptr || out_dtype == IMPARO_DT_F32) IMPARO_GRN(float);
+        else if (out_dtype == IMPARO_DT_BF16) IMPARO_GRN(__nv_bfloat16);
+        else return -1;
+#undef IMPARO_GRN
+#undef IMPARO_GR
+        IMPARO_CHECK_LAUNCH();
+        return 0;
+    }
     int nw, wpg;
     gn::plan(width, groups, vec ? 4 : 1, &nw, &wpg);
 #define IMPARO_GN(T_, V_) launch(gn::group_norm_add_kernel<T_, V_>, dim3(n_rows), dim3(32 * nw), 0, stream, x, y, parts, \
