@@ -332,6 +332,88 @@ qkv_norm_rotate_store_kernel(const T* __restrict__ qkv, size_t in_width, const i
     }
 }
 
+// The same 16 bytes at a time (bfloat16): a head lies on LPH lanes, eight elements each, so a warp works on 32 / LPH heads at
+// once; weights, sines and cosines of a lane's elements stay in registers for all of the block's heads, a rotation partner comes by
+// shuffle.  hd = 8 * LPH, half of the rotated dimensions a multiple of 8, value sizes and strides multiples of 8, aligned pointers.
+template <int LPH>
+__global__ void __launch_bounds__(ANY_WARPS * 32)
+qkv_norm_rotate_store_vec_kernel(const __nv_bfloat16* __restrict__ qkv, size_t in_width, const int* __restrict__ positions,
+                                 const int* __restrict__ item_of_token, const float* __restrict__ q_w, const float* __restrict__ k_w,
+                                 float eps, const float* __restrict__ inv_freq, int n_rot, __nv_bfloat16* __restrict__ q_out,
+                                 __nv_bfloat16* __restrict__ k_cache, __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ table,
+                                 int max_blocks, int page_size, int n_pages, int nh, int nkv, int vd, int heads_per_block, int* status) {
+    constexpr int hd = 8 * LPH, HPW = 32 / LPH;
+    __shared__ float sn_s[ANY_MAX_HEAD / 2], cs_s[ANY_MAX_HEAD / 2];
+    pdl_trigger();
+    const int t = blockIdx.x;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, sub = lane % LPH;
+    const int h_first = blockIdx.y * heads_per_block, h_end = min(nh + nkv, h_first + heads_per_block);
+    const int pos = positions[t];
+    const int half = inv_freq ? (n_rot >> 1) : 0, hl = half / 8;         // hl: lanes between an element's and its partner's
+    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * inv_freq[i], &sn_s[i], &cs_s[i]);
+    const int blk = pos / page_size;
+    const int page = blk < max_blocks ? table[(size_t)item_of_token[t] * max_blocks + blk] : -1;
+    const bool mapped = page >= 0 && page < n_pages;
+    const size_t cache_row = mapped ? (size_t)page * page_size + (pos % page_size) : 0;
+    float qw[8], kw[8], cs[8], sn[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) { qw[e] = q_w[sub * 8 + e]; kw[e] = k_w[sub * 8 + e]; cs[e] = 1.f; sn[e] = 0.f; }
+    __syncthreads();
+    int from = lane;
+    if (sub < 2 * hl) {
+        const bool low = sub < hl;
+        from = low ? lane + hl : lane - hl;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+            const int f = (low ? sub : sub - hl) * 8 + e;
+            cs[e] = cs_s[f];
+            sn[e] = low ? -sn_s[f] : sn_s[f];
+        }
+    }
+    pdl_wait();
+    if (!mapped && threadIdx.x == 0 && blockIdx.y == 0) report(status, IMPARO_ST_PAGE_RANGE, 45, t, page);      // its keys and values are skipped
+    const __nv_bfloat16* row = qkv + (size_t)t * in_width;
+    if (mapped) {                                               // the values, as they are
+        const uint4* src = reinterpret_cast<const uint4*>(row + (size_t)(nh + nkv) * hd);
+        uint4* dst = reinterpret_cast<uint4*>(v_cache + cache_row * ((size_t)nkv * vd));
+        for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < nkv * vd / 8; i += gridDim.y * blockDim.x) dst[i] = src[i];
+    }
+    for (int h0 = h_first + warp * HPW; h0 < h_end; h0 += ANY_WARPS * HPW) {
+        const int hh = h0 + lane / LPH;                         // query heads, then key heads
+        const bool live = hh < h_end, is_q = hh < nh;
+        uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+        if (live) raw = *reinterpret_cast<const uint4*>(row + (size_t)hh * hd + sub * 8);
+        const __nv_bfloat162* in = reinterpret_cast<const __nv_bfloat162*>(&raw);
+        float v[8], ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float2 f = __bfloat1622float2(in[e]);
+            v[2 * e] = f.x; v[2 * e + 1] = f.y;
+            ss += f.x * f.x + f.y * f.y;
+        }
+#pragma unroll
+        for (int s = LPH / 2; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+        const float scale = 1.0f / sqrtf(ss / (float)hd + eps);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] *= scale * (is_q ? qw[e] : kw[e]);
+        if (hl > 0) {
+            float o[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) o[e] = __shfl_sync(0xffffffffu, v[e], from);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = v[e] * cs[e] + o[e] * sn[e];
+        }
+        if (live && (is_q || mapped)) {
+            __nv_bfloat16* dst = is_q ? q_out + ((size_t)t * nh + hh) * hd : k_cache + cache_row * ((size_t)nkv * hd) + (size_t)(hh - nh) * hd;
+            uint4 res;
+            __nv_bfloat162* r = reinterpret_cast<__nv_bfloat162*>(&res);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) r[e] = __floats2bfloat162_rn(v[2 * e], v[2 * e + 1]);
+            *reinterpret_cast<uint4*>(dst + sub * 8) = res;
+        }
+    }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(ANY_WARPS * 32)
 attention_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
@@ -481,6 +563,19 @@ extern "C" int imparo_qkv_norm_rotate_store(const void* qkv, long long row_strid
     const int total = nh + 2 * nkv;
     const int per = n_tok >= 256 ? total : ANY_WARPS;         // few tokens: a block per four heads
     dim3 grid(n_tok, (total + per - 1) / per);
+    const bool vec = dtype == IMPARO_DT_BF16 && hd >= 8 && (hd & (hd - 1)) == 0 && n_rot % 16 == 0 && vd % 8 == 0 && row_stride % 8 == 0 &&
+                     nkv > 0 && (((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) == 0;
+    if (vec) {
+        const int hpw = 32 / (hd / 8), heads = nh + nkv, hpb = n_tok >= 256 ? heads : ANY_WARPS * hpw;
+        dim3 vgrid(n_tok, (heads + hpb - 1) / hpb);
+#define IMPARO_QV(L_) case 8 * L_: launch(qkv_norm_rotate_store_vec_kernel<L_>, vgrid, dim3(ANY_WARPS * 32), 0, stream, \
+        (const __nv_bfloat16*)qkv, (size_t)row_stride, positions, item_of_token, q_w, k_w, eps, inv_freq, n_rot, (__nv_bfloat16*)q_out, \
+        (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, table, max_blocks, page_size, n_pages, nh, nkv, vd, hpb, status); break
+        switch (hd) { IMPARO_QV(1); IMPARO_QV(2); IMPARO_QV(4); IMPARO_QV(8); IMPARO_QV(16); IMPARO_QV(32); }
+#undef IMPARO_QV
+        IMPARO_CHECK_LAUNCH();
+        return 0;
+    }
 #define IMPARO_QN(T_, P_) launch(qkv_norm_rotate_store_kernel<T_, P_>, grid, dim3(ANY_WARPS * 32), 0, stream, (const T_*)qkv, \
         (size_t)row_stride, positions, item_of_token, q_w, k_w, eps, inv_freq, n_rot, (T_*)q_out, (T_*)k_cache, (T_*)v_cache, table, \
         max_blocks, page_size, n_pages, nh, nkv, hd, vd, per, status)
