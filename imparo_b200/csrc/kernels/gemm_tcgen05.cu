@@ -64,7 +64,15 @@ struct Params {
     int act;
     float limit;
     const float* bias;
+    int plain;                   // STORE_BF16: 1 + a plain_act_bf16 kind applied to the product plus bias ([N], or null); 0: none
 };
+
+// what a plain store writes: the product, or one activation of it
+template <int EPI>
+__device__ __forceinline__ float finished(const Params& p, int n, float v) {
+    if (EPI == STORE_BF16 && p.plain) v = plain_act_bf16(p.plain - 1, v + (p.bias ? p.bias[n] : 0.f));
+    return v;
+}
 
 __device__ __forceinline__ uint4 pack8(const float* v) {
     __nv_bfloat162 h0 = __floats2bfloat162_rn(v[0], v[1]), h1 = __floats2bfloat162_rn(v[2], v[3]);
@@ -409,7 +417,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ C
 #pragma unroll
                             for (int j = 0; j < 16; ++j) {
                                 const int t = t0 + c + j;
-                                if (t < p.T) store_out<EPI>(p.out, (size_t)t * p.ldo + n, v[j]);
+                                if (t < p.T) store_out<EPI>(p.out, (size_t)t * p.ldo + n, finished<EPI>(p, n, v[j]));
                             }
                         }
                     }
@@ -458,7 +466,7 @@ done:
 #pragma unroll
                     for (int u = 0; u < 8; ++u) if (s0 + u < p.splits) acc += v[u];
                 }
-                if (n < p.N) store_out<EPI>(p.out, (size_t)t * p.ldo + n, acc);
+                if (n < p.N) store_out<EPI>(p.out, (size_t)t * p.ldo + n, finished<EPI>(p, n, acc));
             }
         }
         // nobody leaves while its shared memory may still be read
@@ -652,7 +660,7 @@ static int partials_map(float* scratch, int T, int N, int splits, int nt, Params
 // scratch / counters: from imparo_gemm_tc_plan; counters must be zero (they are left zero).
 static int gemm_tc_impl(const void* x, int ldx, int x_rows_alloc, const void* w, void* out, int ldo,
                         int T, int N, int K, int epilogue, float* scratch, int* counters, int* status,
-                        int act, float limit, const float* bias, cudaStream_t stream) {
+                        int act, float limit, const float* bias, cudaStream_t stream, int plain = 0) {
     if (T <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 != 0 || ldx % 8 != 0) return -23;                   // TMA: 16-byte rows
     if (((uintptr_t)x | (uintptr_t)w) & 15) return -23;
@@ -669,6 +677,7 @@ static int gemm_tc_impl(const void* x, int ldx, int x_rows_alloc, const void* w,
     p.out = out; p.scratch = scratch; p.counters = counters; p.status = status;
     p.T = T; p.N = N; p.K = K; p.ldo = ldo; p.splits = splits; p.kblocks = (K + BK - 1) / BK;
     p.act = act; p.limit = limit; p.bias = bias;
+    p.plain = plain;
     const int row_tiles = epilogue == SWIGLU_BF16 ? (N + 63) / 64 : (N + BM - 1) / BM;
     dim3 grid(row_tiles, (T + nt - 1) / nt, splits);
     if (grid.y > 65535) return -2;
@@ -703,6 +712,13 @@ extern "C" int imparo_gemm_tc_gated(const void* x, int ldx, int x_rows_alloc, co
     return gemm_tc_impl(x, ldx, x_rows_alloc, w, out, ldo, T, N, K, SWIGLU_BF16, scratch, counters, status, act, limit, bias, stream);
 }
 
+// The bfloat16 store (epilogue 0) with one activation on its own (kind: plain_act_bf16's): out [T, N] = act(x w^T + bias), bias
+// float32 [N] or null.
+extern "C" int imparo_gemm_tc_act(const void* x, int ldx, int x_rows_alloc, const void* w, void* out, int ldo, int T, int N, int K,
+                                  int kind, const float* bias, float* scratch, int* counters, int* status, cudaStream_t stream) {
+    if (kind < 0 || kind > 2) return -22;
+    return gemm_tc_impl(x, ldx, x_rows_alloc, w, out, ldo, T, N, K, STORE_BF16, scratch, counters, status, 0, 0.f, bias, stream, kind + 1);
+}
 
 // ---- a product whose token operand the kernel makes itself: the attention's output product ----------------
 // It takes out (32-bit stream, [T, N]) and either adds into it (epilogue 2) or leaves split partials in

@@ -68,6 +68,10 @@ __global__ void act_rows_strided_kernel(const T* __restrict__ x, size_t x_stride
     }
 }
 
+template <typename T> __device__ __forceinline__ float act_apply_to(float z, int kind) {
+    return sizeof(T) == 2 ? plain_act_bf16(kind, z) : act_apply(z, kind);
+}
+
 // out[r, :] = act(x[r, :] + bias) for dense or strided rows of x; VEC as above (the bias too is read 16 bytes at a time)
 template <typename T, bool VEC>
 __global__ void bias_act_rows_kernel(const T* x, size_t x_stride, const float* __restrict__ bias, T* out, int n_rows, int width, int kind) {
@@ -82,11 +86,19 @@ __global__ void bias_act_rows_kernel(const T* x, size_t x_stride, const float* _
         if (VEC) {
             uint4 raw = *reinterpret_cast<const uint4*>(x + r * x_stride + c);
             T* e = reinterpret_cast<T*>(&raw);
+            float b[N];
+            if (VEC) {                                        // (N is a multiple of 4 here)
 #pragma unroll
-            for (int u = 0; u < N; ++u) e[u] = from_f32<T>(act_apply(to_f32(e[u]) + __ldg(bias + c + u), kind));
+                for (int u = 0; u + 3 < N; u += 4) {
+                    const float4 q = __ldg(reinterpret_cast<const float4*>(bias + c + u));
+                    b[u] = q.x; b[u + 1] = q.y; b[u + 2] = q.z; b[u + 3] = q.w;
+                }
+            }
+#pragma unroll
+            for (int u = 0; u < N; ++u) e[u] = from_f32<T>(act_apply_to<T>(to_f32(e[u]) + b[u], kind));
             *reinterpret_cast<uint4*>(out + r * width + c) = raw;
         } else {
-            out[r * width + c] = from_f32<T>(act_apply(to_f32(x[r * x_stride + c]) + bias[c], kind));
+            out[r * width + c] = from_f32<T>(act_apply_to<T>(to_f32(x[r * x_stride + c]) + bias[c], kind));
         }
     }
 }
@@ -436,7 +448,7 @@ extern "C" int imparo_bias_act_rows(const void* x, long long x_stride, const flo
     if (kind < 0 || kind > 2) return -22;
     if (x_stride < width) return -2;
     const int es = dtype == IMPARO_DT_F32 ? 4 : 2, nvec = 16 / es;
-    const bool vec = width % nvec == 0 && x_stride % nvec == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0;
+    const bool vec = width % nvec == 0 && x_stride % nvec == 0 && (((uintptr_t)x | (uintptr_t)out | (uintptr_t)bias) & 15) == 0;
     const size_t total = (size_t)n_rows * (vec ? width / nvec : width);
 #define IMPARO_ACT(T_, V_) launch(bias_act_rows_kernel<T_, V_>, dim3(flat_grid(total)), dim3(256), 0, stream, (const T_*)x, \
         (size_t)x_stride, bias, (T_*)out, n_rows, width, kind)

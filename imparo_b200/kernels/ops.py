@@ -492,8 +492,10 @@ def tc_usable(x: torch.Tensor, w: torch.Tensor, any_size: bool = False) -> bool:
 
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, status: Optional[torch.Tensor] = None,
-            scratch: Optional[torch.Tensor] = None, act: str = "silu", limit: float = 0.0, bias: Optional[torch.Tensor] = None) -> None:
-    """The hand-written tensor-core product (csrc/kernels/gemm_tcgen05.cu).
+            scratch: Optional[torch.Tensor] = None, act: str = "silu", limit: float = 0.0, bias: Optional[torch.Tensor] = None,
+            plain: Optional[str] = None) -> None:
+    """The hand-written tensor-core product (csrc/kernels/gemm_tcgen05.cu).  plain: with EPI_STORE_BF16, one of ACTIVATIONS applied
+    to the product plus bias (float32 [N] or None).
     epilogue: EPI_STORE_BF16 | EPI_STORE_F32 | EPI_ADD_F32 (out += x w^T) | EPI_SWIGLU
     (w = [gate rows; up rows] of shape [2F, K], out = act(x gate^T + b_g, x up^T + b_u), [T, F]; act one of gated_act's kinds,
     "silu" by default; bias float32 [2F] or None)."""
@@ -520,6 +522,14 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, 
             status = _S.status_fallback[key] = new_status(x.device)
     rows_alloc = (x.untyped_storage().nbytes() // x.element_size() - x.storage_offset()) // x.stride(0) if x.stride(0) else T
     rows_alloc = max(T, min(rows_alloc, 1 << 30))
+    if plain is not None:
+        if bias is not None:
+            _cuda(bias)
+        _need(epilogue == EPI_STORE_BF16 and (bias is None or (bias.dtype == torch.float32 and bias.numel() == N)), "gemm_tc: plain activation")
+        _check(_lib.kernels().imparo_gemm_tc_act(_ptr(x), x.stride(0), rows_alloc, _ptr(w), _ptr(out), out.stride(0), T, N, K,
+                                                 ACTIVATIONS[plain], _ptr(bias), _ptr(scratch), _ptr(cnt), _ptr(status), _stream()),
+               "gemm_tc_act")
+        return
     if epilogue == EPI_SWIGLU and (act != "silu" or bias is not None):
         if bias is not None:
             _cuda(bias)
@@ -1264,7 +1274,13 @@ ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2}
 
 def linear_act(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, kind: str, bias: Optional[torch.Tensor] = None,
                status: Optional[torch.Tensor] = None) -> None:
-    """out = act(x w^T + bias) (bias float32 [features] or None)."""
+    """out = act(x w^T + bias) (bias float32 [features] or None).  Few bfloat16 tokens: one launch of the weight-streaming
+    tensor-core product, bias and activation in its epilogue.  Otherwise: the product, then the activation kernel."""
+    _need(kind in ACTIVATIONS, f"linear_act: unknown activation '{kind}' (known: {', '.join(sorted(ACTIVATIONS))})")
+    if (x.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and out.is_contiguous() and gemm_backend() == "tcgen05"
+            and tc_usable(x, w)):
+        gemm_tc(x, w, out, EPI_STORE_BF16, status, plain=kind, bias=bias)
+        return
     linear(x, w, out, status=status)
     activation(out, out, kind, bias=bias)
 
