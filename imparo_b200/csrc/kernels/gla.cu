@@ -35,6 +35,8 @@ namespace imparo {
 namespace gla {
 
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+// by the approximate exponential and logarithm: within 2e-7 of the above (a decay is the exponential of this over tau)
+__device__ __forceinline__ float log_sigmoid_fast(float z) { return fminf(z, 0.f) - __logf(1.0f + __expf(-fabsf(z))); }
 
 // ---- (1) ------------------------------------------------------------------------------------------------------
 constexpr int DECAY_ROWS = 8;
@@ -260,7 +262,11 @@ struct Chunks {
     const bf16* proj;
     size_t stride;
     int q_off, k_off, v_off, g_off;
-    const float* g;             // log decays [tokens, heads * dim]
+    float* g;                   // log decays [tokens, heads * dim]: read, or (DECAY) made and written by chunk_local
+    int l_off, rank;            // DECAY: the decay's inner columns, w2 [heads * dim, rank], bias [heads * dim], tau
+    const bf16* w2;
+    const float* bias;
+    float tau;
     float q_scale;
     const int* item_row_start;
     int n_items;
@@ -285,28 +291,27 @@ __device__ __forceinline__ bool find_chunk(const int* __restrict__ item_row_star
     return false;
 }
 
-// Running sums of the chunk's log decays.  Channel pairs are shared out over dim / 2 threads, the chunk's rows over `segs`
-// segments of `per` rows; a thread walks its rows twice: once for the segment's total (here), once in the caller, starting from
-// the sum of the segments before it (start), with the chunk's total at hand (total).
+// A thread's share of the chunk's log decays.  Channel pairs are shared out over dim / 2 threads, the chunk's rows over `segs`
+// segments of `per` <= PER rows, which the thread keeps in registers (x; rows the chunk does not have are 0).
+constexpr int PER = 16;
 struct Walk {
-    int pair, seg, segs, per, r0, r1;      // r0, r1: the thread's rows inside the chunk; pair < 0: the thread has none
-    float2 start, total;
+    int pair, seg, segs, per, r0;       // r0: the segment's first row; pair < 0: the thread has none
+    float2 x[PER], start, total;        // start: the sum of the segments before; total: the chunk's
 };
-__device__ __forceinline__ Walk walk_begin(const float* __restrict__ g, size_t g_stride, int n, int dim, float* seg_sum /* [segs][dim] */) {
-    Walk w;
+__device__ __forceinline__ void walk_share(Walk& w, int dim) {
     const int pairs = dim / 2;
     w.segs = min(C, CT / pairs);
     w.per = (C + w.segs - 1) / w.segs;
     w.seg = threadIdx.x / pairs;
     w.pair = w.seg < w.segs ? (int)threadIdx.x % pairs : -1;
-    w.r0 = min(n, w.seg * w.per);
-    w.r1 = min(n, w.r0 + w.per);
-    float2 s = make_float2(0.f, 0.f);
+    w.r0 = w.seg * w.per;
+}
+// x -> start and total; all threads of the CTA call it
+__device__ __forceinline__ void walk_sums(Walk& w, int dim, float* seg_sum /* [segs][dim] */) {
     if (w.pair >= 0) {
-        for (int r = w.r0; r < w.r1; ++r) {
-            const float2 x = *reinterpret_cast<const float2*>(g + (size_t)r * g_stride + 2 * w.pair);
-            s.x += x.x; s.y += x.y;
-        }
+        float2 s = make_float2(0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < PER; ++i) { s.x += w.x[i].x; s.y += w.x[i].y; }
         *reinterpret_cast<float2*>(seg_sum + (size_t)w.seg * dim + 2 * w.pair) = s;
     }
     __syncthreads();
@@ -318,7 +323,6 @@ __device__ __forceinline__ Walk walk_begin(const float* __restrict__ g, size_t g
             w.total.x += x.x; w.total.y += x.y;
         }
     }
-    return w;
 }
 
 // rows [0, n) of the CTA's value columns -> v_s [C][ldv], the rest zero
@@ -332,40 +336,106 @@ __device__ __forceinline__ void stage_values(const bf16* __restrict__ src, size_
     }
 }
 
-__global__ void __launch_bounds__(CT)
+// DECAY: the log decays are made here from the inner columns (rank <= MAX_RANK) and left in a.g for chunk_out.
+constexpr int MAX_RANK = 32;
+
+template <bool DECAY>
+__global__ void __launch_bounds__(CT, 3)
 chunk_local_kernel(const Chunks a) {
     extern __shared__ __align__(16) unsigned char gla_smem[];
     pdl_trigger();
     const int g = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * CCOLS;
     int r_begin, r_end;
     const bool found = find_chunk(a.item_row_start, a.n_items, g, r_begin, r_end);
-    pdl_wait();
-    if (!found) return;
-    const int n = r_end - r_begin, dim = a.dim, vcols = min(CCOLS, a.vdim - v0);
+    const int dim = a.dim, vcols = min(CCOLS, a.vdim - v0);
     const int ldk = dim + PAD, ldv = vcols + PAD;
     bf16* k_hi = reinterpret_cast<bf16*>(gla_smem);
     bf16* k_lo = k_hi + C * ldk;
     bf16* v_s = k_lo + C * ldk;
     float* seg_sum = reinterpret_cast<float*>(v_s + C * ldv);
+    float* w2_s = seg_sum + (size_t)min(C, 2 * CT / dim) * dim;          // [rank][dim]
+    Walk w;
+    walk_share(w, dim);
+    const int per4 = (w.per + 3) & ~3, ldl = w.segs * per4;               // a segment's rows start on 16 bytes
+    float* low_s = w2_s + (size_t)a.rank * dim;                           // [rank][segs][per4], at most 2 * C per inner channel
+    float2 bias2 = make_float2(0.f, 0.f);
+    if (DECAY) {
+        const bf16* src = a.w2 + (size_t)h * dim * a.rank;
+        for (int e = threadIdx.x; e < dim * a.rank; e += CT) w2_s[(e % a.rank) * dim + e / a.rank] = to_f32(src[e]);
+        if (w.pair >= 0) bias2 = make_float2(a.bias[h * dim + 2 * w.pair], a.bias[h * dim + 2 * w.pair + 1]);
+    }
+    pdl_wait();
+    if (!found) return;
+    const int n = r_end - r_begin;
     stage_values(a.proj + (size_t)r_begin * a.stride + a.v_off + (size_t)h * a.vdim + v0, a.stride, n, vcols, v_s, ldv);
     const size_t gs = (size_t)a.heads * dim;
-    const float* gp = a.g + (size_t)r_begin * gs + (size_t)h * dim;
-    const Walk w = walk_begin(gp, gs, n, dim, seg_sum);
+    float* gp = a.g + (size_t)r_begin * gs + (size_t)h * dim + 2 * w.pair;
+    if (DECAY) {
+        for (int e = threadIdx.x; e < C * a.rank; e += CT) {
+            const int r = e / a.rank, k = e - r * a.rank;
+            low_s[k * ldl + r / w.per * per4 + r % w.per] = r < n ? to_f32(a.proj[(size_t)(r_begin + r) * a.stride + a.l_off + k]) : 0.f;
+        }
+        __syncthreads();
+        if (w.pair >= 0) {
+            const float inv_tau = 1.0f / a.tau;
+#pragma unroll
+            for (int i = 0; i < PER; ++i) w.x[i] = bias2;
+            for (int k = 0; k < a.rank; ++k) {
+                const float2 c = *reinterpret_cast<const float2*>(w2_s + (size_t)k * dim + 2 * w.pair);
+                const float* l = low_s + k * ldl + w.seg * per4;
+#pragma unroll
+                for (int i = 0; i < PER; i += 4) {
+                    if (i < per4) {                            // (places past the segment's rows hold anything; their sums are dropped)
+                        const float4 x = *reinterpret_cast<const float4*>(l + i);
+                        w.x[i].x += c.x * x.x; w.x[i].y += c.y * x.x;
+                        w.x[i + 1].x += c.x * x.y; w.x[i + 1].y += c.y * x.y;
+                        w.x[i + 2].x += c.x * x.z; w.x[i + 2].y += c.y * x.z;
+                        w.x[i + 3].x += c.x * x.w; w.x[i + 3].y += c.y * x.w;
+                    }
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < PER; ++i) {
+                const int r = w.r0 + i;
+                if (i < w.per && r < n) {
+                    w.x[i] = make_float2(log_sigmoid_fast(w.x[i].x) * inv_tau, log_sigmoid_fast(w.x[i].y) * inv_tau);
+                    *reinterpret_cast<float2*>(gp + (size_t)r * gs) = w.x[i];
+                } else {
+                    w.x[i] = make_float2(0.f, 0.f);
+                }
+            }
+        }
+    } else if (w.pair >= 0) {
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int r = w.r0 + i;
+            w.x[i] = (i < w.per && r < n) ? *reinterpret_cast<const float2*>(gp + (size_t)r * gs) : make_float2(0.f, 0.f);
+        }
+    }
+    __nv_bfloat162 kr[PER];
     if (w.pair >= 0) {
         const bf16* kp = a.proj + (size_t)r_begin * a.stride + a.k_off + (size_t)h * dim + 2 * w.pair;
-        float2 G = w.start;
-        for (int r = w.r0; r < w.r1; ++r) {
-            const float2 x = *reinterpret_cast<const float2*>(gp + (size_t)r * gs + 2 * w.pair);
-            G.x += x.x; G.y += x.y;
-            const float2 k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(kp + (size_t)r * a.stride));
-            uint32_t hi, lo;
-            split2(k.x * __expf(w.total.x - G.x), k.y * __expf(w.total.y - G.y), hi, lo);
-            *reinterpret_cast<uint32_t*>(k_hi + (size_t)r * ldk + 2 * w.pair) = hi;
-            *reinterpret_cast<uint32_t*>(k_lo + (size_t)r * ldk + 2 * w.pair) = lo;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int r = w.r0 + i;
+            kr[i] = __floats2bfloat162_rn(0.f, 0.f);
+            if (i < w.per && r < n) kr[i] = *reinterpret_cast<const __nv_bfloat162*>(kp + (size_t)r * a.stride);
         }
-        for (int r = max(w.r1, w.seg * w.per); r < min(C, (w.seg + 1) * w.per); ++r) {         // rows the chunk does not have
-            *reinterpret_cast<uint32_t*>(k_hi + (size_t)r * ldk + 2 * w.pair) = 0u;
-            *reinterpret_cast<uint32_t*>(k_lo + (size_t)r * ldk + 2 * w.pair) = 0u;
+    }
+    walk_sums(w, dim, seg_sum);
+    if (w.pair >= 0) {
+        float2 G = w.start;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int r = w.r0 + i;
+            if (i < w.per && r < C) {                         // (rows the chunk does not have: keys of zero)
+                G.x += w.x[i].x; G.y += w.x[i].y;
+                const float2 k = __bfloat1622float2(kr[i]);
+                uint32_t hi, lo;
+                split2(k.x * __expf(w.total.x - G.x), k.y * __expf(w.total.y - G.y), hi, lo);
+                *reinterpret_cast<uint32_t*>(k_hi + (size_t)r * ldk + 2 * w.pair) = hi;
+                *reinterpret_cast<uint32_t*>(k_lo + (size_t)r * ldk + 2 * w.pair) = lo;
+            }
         }
         if (w.seg == 0 && blockIdx.z == 0)
             *reinterpret_cast<float2*>(a.decay + ((size_t)g * a.heads + h) * dim + 2 * w.pair) = make_float2(__expf(w.total.x), __expf(w.total.y));
@@ -475,33 +545,55 @@ chunk_out_kernel(const Chunks a, const float* __restrict__ w_norm, float eps, fl
     const float* S0 = a.state + (((size_t)g * a.heads + h) * dim) * a.vdim + v0 + n0;
     stage_values(a.proj + (size_t)r_begin * a.stride + a.v_off + (size_t)h * a.vdim + v0, a.stride, n, vcols, v_s, ldv);
     const size_t gs = (size_t)a.heads * dim;
-    const float* gp = a.g + (size_t)r_begin * gs + (size_t)h * dim;
-    const Walk w = walk_begin(gp, gs, n, dim, seg_sum);
+    Walk w;
+    walk_share(w, dim);
+    __nv_bfloat162 qr[PER], kr[PER];
+    if (w.pair >= 0) {                                        // everything the thread needs of its rows, requested at once
+        const bf16* row = a.proj + (size_t)r_begin * a.stride + (size_t)h * dim + 2 * w.pair;
+        const float* gp = a.g + (size_t)r_begin * gs + (size_t)h * dim + 2 * w.pair;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int r = w.r0 + i;
+            w.x[i] = make_float2(0.f, 0.f);
+            qr[i] = kr[i] = __floats2bfloat162_rn(0.f, 0.f);
+            if (i < w.per && r < n) {
+                w.x[i] = *reinterpret_cast<const float2*>(gp + (size_t)r * gs);
+                qr[i] = *reinterpret_cast<const __nv_bfloat162*>(row + (size_t)r * a.stride + a.q_off);
+                kr[i] = *reinterpret_cast<const __nv_bfloat162*>(row + (size_t)r * a.stride + a.k_off);
+            }
+        }
+    }
+    float s_next[8];                                          // the starting state's entries of the next 16 channels
+    auto load_state = [&](int kk) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e)
+            s_next[e] = __ldcg(S0 + (size_t)(kk * 16 + ((e >> 1) & 1) * 8 + 2 * tg + (e & 1)) * a.vdim + (e >> 2) * 8 + gq);
+    };
+    if (busy) load_state(0);
+    walk_sums(w, dim, seg_sum);
     float* G_s = reinterpret_cast<float*>(k_hi);              // the slow form keeps the running sums here instead
     const int slow = __syncthreads_or(w.pair >= 0 && (w.total.x < -FAST_DECAY || w.total.y < -FAST_DECAY));
     if (w.pair >= 0) {
-        const bf16* row = a.proj + (size_t)r_begin * a.stride + (size_t)h * dim + 2 * w.pair;
         float2 G = w.start;
-        for (int r = w.seg * w.per; r < min(C, (w.seg + 1) * w.per); ++r) {
-            uint32_t qh = 0u, ql = 0u, kh = 0u, kl = 0u;
-            if (r < n) {
-                const float2 x = *reinterpret_cast<const float2*>(gp + (size_t)r * gs + 2 * w.pair);
-                G.x += x.x; G.y += x.y;
-                const float2 q = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(row + (size_t)r * a.stride + a.q_off));
-                split2(q.x * a.q_scale * __expf(G.x), q.y * a.q_scale * __expf(G.y), qh, ql);
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int r = w.r0 + i;
+            if (i < w.per && r < C) {                         // (rows the chunk does not have: queries and keys of zero)
+                G.x += w.x[i].x; G.y += w.x[i].y;
+                const float2 q = __bfloat1622float2(qr[i]);
+                uint32_t hi, lo;
+                const size_t at = (size_t)r * ldq + 2 * w.pair;
+                split2(q.x * a.q_scale * __expf(G.x), q.y * a.q_scale * __expf(G.y), hi, lo);
+                *reinterpret_cast<uint32_t*>(q_hi + at) = hi;
+                *reinterpret_cast<uint32_t*>(q_lo + at) = lo;
                 if (slow) {
                     *reinterpret_cast<float2*>(G_s + (size_t)r * dim + 2 * w.pair) = G;
                 } else {
-                    const float2 k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(row + (size_t)r * a.stride + a.k_off));
-                    split2(k.x * __expf(-G.x), k.y * __expf(-G.y), kh, kl);
+                    const float2 k = __bfloat1622float2(kr[i]);
+                    split2(k.x * __expf(-G.x), k.y * __expf(-G.y), hi, lo);
+                    *reinterpret_cast<uint32_t*>(k_hi + at) = hi;
+                    *reinterpret_cast<uint32_t*>(k_lo + at) = lo;
                 }
-            }
-            const size_t at = (size_t)r * ldq + 2 * w.pair;
-            *reinterpret_cast<uint32_t*>(q_hi + at) = qh;
-            *reinterpret_cast<uint32_t*>(q_lo + at) = ql;
-            if (!slow) {
-                *reinterpret_cast<uint32_t*>(k_hi + at) = kh;
-                *reinterpret_cast<uint32_t*>(k_lo + at) = kl;
             }
         }
     }
@@ -591,12 +683,8 @@ chunk_out_kernel(const Chunks a, const float* __restrict__ w_norm, float eps, fl
         for (int kk = 0; kk < dim / 16; ++kk) {               // the state the chunk starts from
             uint32_t bh[4], bl[4];
 #pragma unroll
-            for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-                for (int kh = 0; kh < 2; ++kh) {
-                    const float* p = S0 + (size_t)(kk * 16 + kh * 8 + 2 * tg) * a.vdim + nt * 8 + gq;
-                    split2(__ldcg(p), __ldcg(p + a.vdim), bh[nt * 2 + kh], bl[nt * 2 + kh]);
-                }
+            for (int e = 0; e < 4; ++e) split2(s_next[2 * e], s_next[2 * e + 1], bh[e], bl[e]);
+            if (kk + 1 < dim / 16) load_state(kk + 1);
 #pragma unroll
             for (int it = 0; it < 4; ++it) {
                 uint32_t ah[4], al[4];
@@ -671,8 +759,8 @@ chunk_out_kernel(const Chunks a, const float* __restrict__ w_norm, float eps, fl
         }
 }
 
-static size_t local_smem(int dim, int vcols) {
-    return (size_t)C * (2 * (dim + PAD) + (vcols + PAD)) * 2 + (size_t)(2 * CT / dim < C ? 2 * CT / dim : C) * dim * 4;
+static size_t local_smem(int dim, int vcols, int rank) {
+    return (size_t)rank * (dim + 2 * C) * 4 + (size_t)C * (2 * (dim + PAD) + (vcols + PAD)) * 2 + (size_t)(2 * CT / dim < C ? 2 * CT / dim : C) * dim * 4;
 }
 static size_t out_smem(int dim, int vcols) {
     const int ldk = dim + PAD > C + PAD ? dim + PAD : C + PAD;
@@ -748,11 +836,12 @@ extern "C" int imparo_gla_step(const void* proj, long long stride, int dtype, in
     return 0;
 }
 
-// bfloat16 batches with long portions; dim and vdim multiples of 16, dim <= 128, 16-byte aligned columns; else -8.  chunk_state
+// bfloat16 batches with long portions.  g float32 [n_tok, heads * dim]: the log decays, read; or, with w2 not null, made from the
+// inner columns at l_off (rank <= 32) as imparo_gla_decay makes them and written.  dim and vdim multiples of 16, dim <= 128, 16-byte aligned columns; else -8.  chunk_state
 // float32 [chunks, heads, dim, vdim] and chunk_decay [chunks, heads, dim] scratch, chunks = n_tok / 64 + n_items (an upper bound).
 // vdim <= 128: y receives the normed, weighted, gated outputs (bfloat16 [n_tok, heads * vdim]); else o (float32) the plain ones.
-extern "C" int imparo_gla_chunked(const void* proj, long long stride, int q_off, int k_off, int v_off, int g_off, const float* g,
-                                  float q_scale, const float* w_norm, float eps, float* slots, const int* item_row_start,
+extern "C" int imparo_gla_chunked(const void* proj, long long stride, int q_off, int k_off, int v_off, int g_off, int l_off, float* g,
+                                  const void* w2, const float* bias, float tau, int rank, float q_scale, const float* w_norm, float eps, float* slots, const int* item_row_start,
                                   const int* item_slot, int n_slots, int n_items, int n_tok, float* chunk_state, float* chunk_decay,
                                   float* o, void* y, int heads, int dim, int vdim, int* status, cudaStream_t stream) {
     if (n_items <= 0 || n_tok <= 0) return 0;
@@ -760,11 +849,14 @@ extern "C" int imparo_gla_chunked(const void* proj, long long stride, int q_off,
     if (dim < 16 || dim > 128 || dim % 16 || vdim < 16 || vdim % 16) return -8;
     if (stride % 8 || v_off % 8 || q_off % 2 || k_off % 2 || g_off % 2 || ((uintptr_t)proj & 15) || ((uintptr_t)g & 7)) return -8;
     if (((uintptr_t)slots | (uintptr_t)chunk_state) & 15) return -8;
+    if (w2 != nullptr && (rank < 1 || rank > gla::MAX_RANK || bias == nullptr || !(tau > 0.f))) return -8;
+    if (w2 == nullptr) rank = 0;
     const bool norm = vdim <= gla::CCOLS;
     if (norm ? y == nullptr : o == nullptr) return -2;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(gla::chunk_local_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)gla::local_smem(128, 128));
+        cudaError_t e = cudaFuncSetAttribute(gla::chunk_local_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)gla::local_smem(128, 128, gla::MAX_RANK));
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(gla::chunk_local_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)gla::local_smem(128, 128, 0));
         if (e == cudaSuccess) e = cudaFuncSetAttribute(gla::chunk_out_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)gla::out_smem(128, 128));
         if (e == cudaSuccess) e = cudaFuncSetAttribute(gla::chunk_out_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)gla::out_smem(128, 128));
         if (e != cudaSuccess) return (int)e;
@@ -772,12 +864,14 @@ extern "C" int imparo_gla_chunked(const void* proj, long long stride, int q_off,
     }
     gla::Chunks a;
     a.proj = (const __nv_bfloat16*)proj; a.stride = (size_t)stride;
-    a.q_off = q_off; a.k_off = k_off; a.v_off = v_off; a.g_off = g_off; a.g = g; a.q_scale = q_scale;
+    a.q_off = q_off; a.k_off = k_off; a.v_off = v_off; a.g_off = g_off; a.g = g;
+    a.l_off = l_off; a.rank = rank; a.w2 = (const __nv_bfloat16*)w2; a.bias = bias; a.tau = tau; a.q_scale = q_scale;
     a.item_row_start = item_row_start; a.n_items = n_items; a.state = chunk_state; a.decay = chunk_decay;
     a.heads = heads; a.dim = dim; a.vdim = vdim;
     const int vcols = vdim < gla::CCOLS ? vdim : gla::CCOLS;
     const dim3 grid(n_tok / gla::C + n_items, heads, (vdim + gla::CCOLS - 1) / gla::CCOLS);
-    launch(gla::chunk_local_kernel, grid, dim3(gla::CT), gla::local_smem(dim, vcols), stream, a);
+    if (w2 != nullptr) launch(gla::chunk_local_kernel<true>, grid, dim3(gla::CT), gla::local_smem(dim, vcols, rank), stream, a);
+    else launch(gla::chunk_local_kernel<false>, grid, dim3(gla::CT), gla::local_smem(dim, vcols, 0), stream, a);
     IMPARO_CHECK_LAUNCH();
     launch(gla::chunk_scan_kernel, dim3(n_items, heads, (dim * vdim / 4 + 255) / 256), dim3(256), 0, stream, a, slots, item_slot, n_slots, status);
     IMPARO_CHECK_LAUNCH();

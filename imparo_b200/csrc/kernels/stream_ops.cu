@@ -83,16 +83,14 @@ __global__ void bias_act_rows_kernel(const T* x, size_t x_stride, const float* _
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
         const size_t r = i / per_row;
         const int c = (int)(i - r * per_row) * N;
-        if (VEC) {
+        if constexpr (VEC) {
             uint4 raw = *reinterpret_cast<const uint4*>(x + r * x_stride + c);
             T* e = reinterpret_cast<T*>(&raw);
             float b[N];
-            if (VEC) {                                        // (N is a multiple of 4 here)
 #pragma unroll
-                for (int u = 0; u + 3 < N; u += 4) {
-                    const float4 q = __ldg(reinterpret_cast<const float4*>(bias + c + u));
-                    b[u] = q.x; b[u + 1] = q.y; b[u + 2] = q.z; b[u + 3] = q.w;
-                }
+            for (int u = 0; u + 3 < N; u += 4) {
+                const float4 q = __ldg(reinterpret_cast<const float4*>(bias + c + u));
+                b[u] = q.x; b[u + 1] = q.y; b[u + 2] = q.z; b[u + 3] = q.w;
             }
 #pragma unroll
             for (int u = 0; u < N; ++u) e[u] = from_f32<T>(act_apply_to<T>(to_f32(e[u]) + b[u], kind));

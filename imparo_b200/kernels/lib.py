@@ -160,7 +160,7 @@ def _declare_kernels(lib):
     _declare(lib, "imparo_group_norm_add", [P, P, I, c_int64, P, P, c_float, P, c_float, P, I, I, I, I, S])
     _declare(lib, "imparo_gla_decay", [P, c_int64, I, P, P, c_float, P, I, I, I, S])
     _declare(lib, "imparo_gla_step", [P, c_int64, I, I, I, I, I, I, P, P, c_float, I, P, c_float, c_float, P, P, P, I, I, P, I, I, I, P, S])
-    _declare(lib, "imparo_gla_chunked", [P, c_int64, I, I, I, I, P, c_float, P, c_float, P, P, P, I, I, I, P, P, P, P, I, I, I, P, S])
+    _declare(lib, "imparo_gla_chunked", [P, c_int64, I, I, I, I, I, P, P, P, c_float, I, c_float, P, c_float, P, P, P, I, I, I, P, P, P, P, I, I, I, P, S])
     _declare(lib, "imparo_gla_recurrent", [P, c_int64, I, I, I, I, P, c_float, P, P, P, I, I, P, I, I, I, P, S])
     _declare(lib, "imparo_latent_norm_store", [P, c_int64, I, I, I, I, P, P, c_float, P, P, P, P, I, P, I, I, I, I, P, S])
     _declare(lib, "imparo_latent_rot_store", [P, c_int64, I, I, I, I, P, c_float, P, I, P, P, P, P, P, I, P, I, I, I, I, P, S])

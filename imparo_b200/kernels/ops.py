@@ -1981,6 +1981,7 @@ def gla_step(proj: torch.Tensor, offsets, rank: int, w2: torch.Tensor, bias: tor
 
 
 GLA_CHUNK = 64             # rows per chunk of gla_chunked
+GLA_CHUNK_RANK = 32        # up to this inner size gla_chunked makes the decays itself
 GLA_CHUNK_COLUMNS = 128    # up to this value size gla_chunked also norms and gates
 
 
@@ -1994,16 +1995,24 @@ def gla_chunked_takes(proj: torch.Tensor, offsets, dim: int, vdim: int) -> bool:
 
 def gla_chunked(proj: torch.Tensor, offsets, g: torch.Tensor, q_scale: float, w_norm: torch.Tensor, eps: float, state: torch.Tensor,
                 item_row_start, item_slot, n_items: int, chunk_state: torch.Tensor, chunk_decay: torch.Tensor, o: Optional[torch.Tensor],
-                y: torch.Tensor, heads: int, dim: int, vdim: int, status: torch.Tensor) -> bool:
+                y: torch.Tensor, heads: int, dim: int, vdim: int, status: torch.Tensor, decay=None) -> bool:
     """gla_scan for batches with long portions, in chunks of GLA_CHUNK rows side by side on tensor cores (gla_chunked_takes).
     chunk_state / chunk_decay: float32 scratch for (T // GLA_CHUNK + n_items) * heads * dim * vdim (* dim) values.  vdim up to
     GLA_CHUNK_COLUMNS: y [T, heads * vdim] receives the outputs normed per head, times w_norm, times silu of the gate's columns
-    (True); else o (float32) the plain outputs (False)."""
+    (True); else o (float32) the plain outputs (False).  decay (w2, bias, tau, rank; offsets then holds the inner columns' place
+    too, rank at most GLA_CHUNK_RANK): g is not read but made by the first launch, as gla_decay makes it."""
     _need(gla_chunked_takes(proj, offsets, dim, vdim), "gla_chunked: sizes")
     _cuda(g, w_norm, state, item_row_start, item_slot, chunk_state, chunk_decay, o, y, status)
     T = proj.shape[0]
     q_off, k_off, v_off, g_off = (int(x) for x in offsets[:4])
     chunks = T // GLA_CHUNK + n_items
+    l_off, w2, bias, tau, rank = 0, None, None, 1.0, 0
+    if decay is not None:
+        w2, bias, tau, rank = decay
+        l_off = int(offsets[4])
+        _cuda(w2, bias)
+        _need(1 <= rank <= GLA_CHUNK_RANK and tuple(w2.shape) == (heads * dim, rank) and w2.dtype == proj.dtype and bias.dtype == torch.float32
+              and bias.numel() == heads * dim and l_off + rank <= proj.shape[1], "gla_chunked: the decay's inner columns, w2 and bias")
     normed = vdim <= GLA_CHUNK_COLUMNS
     _need(g.dtype == torch.float32 and tuple(g.shape) == (T, heads * dim), "gla_chunked: g float32 [T, heads * dim]")
     _need(chunk_state.dtype == torch.float32 and chunk_state.numel() >= chunks * heads * dim * vdim and chunk_decay.dtype == torch.float32
@@ -2014,8 +2023,8 @@ def gla_chunked(proj: torch.Tensor, offsets, g: torch.Tensor, q_scale: float, w_
     _need(normed or (o is not None and o.dtype == torch.float32 and tuple(o.shape) == (T, heads * vdim)), "gla_chunked: o float32 [T, heads * vdim]")
     _need(max(q_off, k_off) + heads * dim <= proj.shape[1] and max(v_off, g_off) + heads * vdim <= proj.shape[1], "gla_chunked: columns")
     _need(item_row_start.numel() >= n_items + 1 and item_slot.numel() >= n_items, "gla_chunked: item arrays")
-    _check(_lib.kernels().imparo_gla_chunked(_ptr(proj), proj.stride(0), q_off, k_off, v_off, g_off, _ptr(g), float(q_scale), _ptr(w_norm),
-                                             float(eps), _ptr(state), _ptr(item_row_start), _ptr(item_slot), state.shape[0], n_items, T,
+    _check(_lib.kernels().imparo_gla_chunked(_ptr(proj), proj.stride(0), q_off, k_off, v_off, g_off, l_off, _ptr(g), _ptr(w2), _ptr(bias),
+                                             float(tau), int(rank), float(q_scale), _ptr(w_norm), float(eps), _ptr(state), _ptr(item_row_start), _ptr(item_slot), state.shape[0], n_items, T,
                                              _ptr(chunk_state), _ptr(chunk_decay), _ptr(o), _ptr(y), heads, dim, vdim, _ptr(status),
                                              _stream()), "gla_chunked")
     COUNTS["own"] += 2

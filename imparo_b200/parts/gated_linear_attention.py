@@ -90,8 +90,12 @@ class GatedLinearAttention(Part):
                                                   rt.status)
         if not done:
             g = ws.get("gla_decay", (T, self.qk), torch.float32, first="tokens")
-            ops.gla_decay(proj[:, a_at:a_at + self.rank], self.w_a2, self.b_a2, self.tau, g)
             in_chunks = batch.max_tokens_per_item >= self.CHUNK_FROM and ops.gla_chunked_takes(proj, self.columns, D, V)
+            decay = None
+            if in_chunks and self.rank <= ops.GLA_CHUNK_RANK:
+                decay = (self.w_a2, self.b_a2, self.tau, self.rank)
+            else:
+                ops.gla_decay(proj[:, a_at:a_at + self.rank], self.w_a2, self.b_a2, self.tau, g)
             o = None
             if not in_chunks or V > ops.GLA_CHUNK_COLUMNS:
                 o = ws.get("gla_o", (T, self.vv), torch.float32, first="tokens")
@@ -99,7 +103,8 @@ class GatedLinearAttention(Part):
                 chunks = T // ops.GLA_CHUNK + batch.n_items
                 done = ops.gla_chunked(proj, self.columns, g, q_scale, self.w_norm, self.eps, st.state, batch.item_row_start,
                                        batch.item_slot, batch.n_items, ws.get("gla_chunk_state", (chunks * H * D * V,), torch.float32),
-                                       ws.get("gla_chunk_decay", (chunks * H * D,), torch.float32), o, y, H, D, V, rt.status)
+                                       ws.get("gla_chunk_decay", (chunks * H * D,), torch.float32), o, y, H, D, V, rt.status,
+                                       decay=decay)
             else:
                 ops.gla_scan(proj, q_at, k_at, v_at, g, q_scale, st.state, batch.item_row_start, batch.item_slot, batch.n_items, o, H, D,
                              V, rt.status)

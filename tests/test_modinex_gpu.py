@@ -245,8 +245,9 @@ def _bf16_round(a):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("width,groups", [(72, 3), (40, 20), (52, 1), (52, 4), (128, 8), (2048, 4), (1024, 1), (4100, 2), (96, 96), (6144, 3)])
-def test_group_norms_and_the_normed_add(width, groups, dtype):
+@pytest.mark.parametrize("T,width,groups", [(7, 72, 3), (7, 40, 20), (7, 52, 1), (7, 52, 4), (7, 128, 8), (7, 2048, 4), (7, 1024, 1), (7, 4100, 2), (7, 96, 96),
+                                            (7, 6144, 3), (300, 2048, 4), (257, 72, 3), (260, 96, 12), (256, 1000, 1), (300, 768, 2), (270, 2100, 2)])
+def test_group_norms_and_the_normed_add(T, width, groups, dtype):
     """The norm in groups (rows in place and picked), the add of a normed output alone and with the next norm in the same
     pass, with a bias and with split partials of the output."""
     import torch
@@ -254,7 +255,6 @@ def test_group_norms_and_the_normed_add(width, groups, dtype):
     tdt = torch.float32 if dtype == "float32" else torch.bfloat16
     tol = 1e-5 if dtype == "float32" else 1e-2
     rng = np.random.default_rng(width + groups)
-    T = 7
     x, y, w, wn, bias = rng.standard_normal((T, width)) * 3, rng.standard_normal((T, width)) * 1e-2, rng.uniform(0.5, 1.5, width), rng.uniform(0.5, 1.5, width), rng.standard_normal(width) * 1e-2
     eps = 1e-5
     out = torch.empty(T, width, dtype=tdt, device="cuda")
@@ -623,6 +623,37 @@ def test_one_row_step_with_decay_norm_and_gate(H, D, V, rank, tau, dtype):
             assert np.abs(y.float().cpu().numpy() - want).max() <= tol
     ops.read_status(status)
     assert float((S1[[0, 1, 3, 4]] - S2[[0, 1, 3, 4]]).abs().max()) <= 1e-4 and float(S1[2].min()) == 3.0
+
+
+@pytest.mark.parametrize("H,D,V,rank,tau", [(2, 64, 64, 16, 16.0), (1, 128, 128, 5, 1.0), (3, 48, 32, 32, 4.0), (2, 16, 144, 1, 2.0), (1, 96, 80, 27, 0.3)])
+def test_chunks_make_their_decays(H, D, V, rank, tau):
+    """The first launch of the chunked form makes the log decays from the inner columns: the same as gla_decay's, and the same
+    outputs and states as with decays given."""
+    import torch
+    from imparo_b200.kernels import ops
+    rng = np.random.default_rng(H + D + V + rank)
+    qk, vv = H * D, H * V
+    l_at = (2 * qk + 2 * vv + 7) // 8 * 8
+    T, starts = 333, np.array([0, 130, 133, 333], dtype=np.int32)
+    proj = _dev(rng.standard_normal((T, (l_at + rank + 7) // 8 * 8)), torch.bfloat16)
+    w2, b = _dev(rng.standard_normal((qk, rank)) / np.sqrt(rank), torch.bfloat16), _f32(rng.uniform(-1.0, 4.0, qk))
+    offs = (0, qk, 2 * qk, 2 * qk + vv, l_at)
+    slots, w = _dev(np.array([2, 0, 1], dtype=np.int32)), _f32(rng.uniform(0.5, 1.5, V))
+    status = ops.new_status("cuda")
+    g1, g2 = torch.empty(T, qk, device="cuda"), torch.full((T, qk), 5.0, device="cuda")
+    ops.gla_decay(proj[:, l_at:l_at + rank], w2, b, tau, g1)
+    n = T // ops.GLA_CHUNK + 3
+    res = []
+    for g, decay in ((g1, None), (g2, (w2, b, tau, rank))):
+        S = torch.ones(3, H, D, V, device="cuda")
+        o, y = torch.zeros(T, vv, device="cuda"), torch.zeros(T, vv, dtype=torch.bfloat16, device="cuda")
+        ops.gla_chunked(proj, offs, g, D ** -0.5, w, 1e-5, S, _dev(starts), slots, 3, torch.empty(n * H * D * V, device="cuda"),
+                        torch.empty(n * H * D, device="cuda"), o, y, H, D, V, status, decay=decay)
+        res.append((S, o if V > 128 else y.float()))
+    ops.read_status(status)
+    assert float((g1 - g2).abs().max()) <= 1e-5 * max(1.0, float(g1.abs().max()))
+    for x, y in zip(*res):
+        assert float((x - y).abs().max()) <= 1e-2 * float(x.abs().max())
 
 
 @pytest.mark.parametrize("T,width,F,kind,biased,dtype", [(300, 128, 256, "gelu_tanh", True, "bfloat16"), (700, 64, 136, "gelu_tanh", True, "bfloat16"),
