@@ -157,6 +157,7 @@ prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
         pdl_wait();                                          // this step's keys were written by the kernel before
         const int pages_per_step = KEYS / a.page_size;
         const int first_blk = lo_min / a.page_size, last_blk = pos_last / a.page_size;
+        int issued = 0;
         for (int i = 0; i < n_steps; ++i) {
             const int s = i % STAGES;
             int ok = 1;
@@ -189,7 +190,11 @@ prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
 #pragma unroll
                 for (int nb = 0; nb < NBV; ++nb) tma_load_2d(vdst + nb * REGION + off, &map_v, &kv_full[s], kvh * a.vd + nb * 64, y);
             }
+            issued = i + 1;
         }
+        // nobody leaves while copies are in flight (they have landed already unless a wait ran out somewhere)
+        if (lane == 0)
+            for (int i = max(0, issued - STAGES); i < issued; ++i) mbar_wait(&kv_full[i % STAGES], (i / STAGES) & 1);
     } else if (warp == 1) {
         if (lane == 0) {
             const uint32_t idesc_s = instr_desc_ab(ROWS, KEYS, false);
@@ -219,16 +224,21 @@ prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
                 umma_commit(o_done);
             };
             bool ok = wait_for(q_ready, 0, 103, 0) && wait_for(&kv_full[0], 0, 104, 0);
-            if (ok) issue_s(0);
+            int s_issued = 0, pv_issued = 0;
+            if (ok) { issue_s(0); s_issued = 1; }
             for (int i = 0; i < n_steps && ok; ++i) {
                 if (i + 1 < n_steps) {
                     ok = wait_for(s_free, i & 1, 105, i) && wait_for(&kv_full[(i + 1) % STAGES], ((i + 1) / STAGES) & 1, 104, i + 1);
                     if (!ok) break;
                     issue_s(i + 1);
+                    s_issued = i + 2;
                 }
                 ok = wait_for(p_ready, i & 1, 106, i);
-                if (ok) issue_pv(i);
+                if (ok) { issue_pv(i); pv_issued = i + 1; }
             }
+            // ... or products that still write tensor memory
+            if (s_issued) mbar_wait(s_ready, (s_issued - 1) & 1);
+            if (pv_issued) mbar_wait(o_done, (pv_issued - 1) & 1);
         }
     } else {
         const int half = (warp - 2) >> 2;                     // keys 0-63 or 64-127 of a step
