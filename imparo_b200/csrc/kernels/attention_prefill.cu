@@ -299,6 +299,10 @@ struct QkvSource {
     float softcap;              // c > 0: the scaled score becomes c * tanh(score / c) (with or without the fields above)
     int kv_groups;              // > 1: that many groups of query heads in a row read the SAME cached head (the launch's
                                 // nkv counts groups; the cache rows hold nkv / kv_groups heads).  Not with the fields above.
+    const float* sinks;         // [nh] or null: one more term exp(sinks[h]) in head h's denominator, without a value; it enters
+                                // the partial result of the chunk that holds the query's own position
+    int v_from_k;               // the product is [q | k]: a key head before the rotation is also the value head, and the
+                                // sums are not rounded before the rotation
 };
 
 template <int HD, bool FROM_QKV>
@@ -413,7 +417,7 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
         // Work items: the group's G query heads; in the CTA whose chunk holds the token's position also the new key
         // (item G) and value (item G + 1).  Warp w takes items w, w + 4, ...; a lane holds the values lane + 32 j.
         const bool owner = pos >= begin && pos < end;
-        const int total_w = (nh + 2 * nkv) * HD;
+        const int total_w = (nh + (src.v_from_k ? 1 : 2) * nkv) * HD;
         __nv_bfloat16* kdst = nullptr;
         __nv_bfloat16* vdst = nullptr;
         if (owner) {
@@ -428,7 +432,7 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
                 vdst = src.v_out + r;
             }
         }
-        const int n_work = G + (owner ? 2 : 0);
+        const int n_work = G + (owner ? (src.v_from_k ? 1 : 2) : 0);
         for (int it = warp; it < n_work; it += 4) {
             const bool is_q = it < G, is_k = it == G;
             const int col0 = is_q ? (h0 + it) * HD : (is_k ? (nh + kvh) * HD : (nh + nkv + kvh) * HD);
@@ -446,8 +450,12 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
 #pragma unroll
                     for (int u = 0; u < 8; ++u) if (s0 + u < src.parts) acc += v[u];
                 }
-                val[j] = __bfloat162float(__float2bfloat16(acc));             // rounded as the stored product would be
+                val[j] = src.v_from_k ? acc : __bfloat162float(__float2bfloat16(acc));      // rounded as the stored product would be
                 ss += val[j] * val[j];
+            }
+            if (is_k && src.v_from_k && vdst) {
+#pragma unroll
+                for (int j = 0; j < PER; ++j) { const int d = lane + 32 * j; vdst[d] = __float2bfloat16(val[j]); }
             }
             if (is_q || is_k) {
                 const float* w = is_q ? src.q_w : src.k_w;
@@ -628,6 +636,13 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
                 L += wl[w * 8 + gg] * f;
             }
         }
+        if (src.sinks != nullptr && pos < end) {                        // the chunk with the query's own position
+            const float sk = src.sinks[h0 + gg] * 1.4426950408889634f;
+            const float M2 = fmaxf(M, sk), f = M == -INFINITY ? 0.f : exp2f(M - M2);
+            acc *= f;
+            L = L * f + exp2f(sk - M2);
+            M = M2;
+        }
         const size_t pb = part_base + (size_t)gg * n_splits;
         part_acc[pb * HD + d] = acc;
         // the combine kernel works in natural-log units
@@ -689,7 +704,8 @@ static int decode_mma_launch(const void* q, const pf::QkvSource* qkv_src, const 
                              const int* table, int max_blocks, int page_size, int n_pages,
                              int window, float scale, void* out, float* part_acc, float* part_ml,
                              int n_tok, int nh, int nkv, int hd, int chunk, int n_splits, int fresh, int overlap_prev,
-                             int* status, cudaStream_t stream, float softcap = 0.f, int kv_groups = 1) {
+                             int* status, cudaStream_t stream, float softcap = 0.f, int kv_groups = 1,
+                             const float* sinks = nullptr) {
     if (n_tok <= 0) return 0;
     if (nkv <= 0 || nh % nkv != 0) return -5;
     if (kv_groups < 1 || nkv % kv_groups != 0 || (kv_groups > 1 && qkv_src != nullptr)) return -5;
@@ -715,6 +731,7 @@ static int decode_mma_launch(const void* q, const pf::QkvSource* qkv_src, const 
     pf::QkvSource none{};
     none.softcap = softcap > 0.f ? softcap : 0.f;
     none.kv_groups = kv_groups;
+    none.sinks = sinks;
     const pf::QkvSource& src = from_qkv ? *qkv_src : none;
 #define IMPARO_DECODE(HD_, F_) launch(pf::attn_decode_mma_kernel<HD_, F_>, grid, dim3(pf::THREADS), smem, stream, \
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, positions, item_of_token, table, \
@@ -738,16 +755,17 @@ extern "C" int imparo_attention_decode_mma(const void* q, const void* k_cache, c
                              status, stream);
 }
 
-// The same with a soft cap c > 0 on the scaled scores: c * tanh(score / c).
+// The same with a soft cap c > 0 on the scaled scores (c * tanh(score / c)) and, with sinks (float32 [nh]), one more term
+// exp(sinks[h]) in head h's denominator, already in the partial results.
 extern "C" int imparo_attention_decode_mma_capped(const void* q, const void* k_cache, const void* v_cache,
                                                   const int* positions, const int* item_of_token,
                                                   const int* table, int max_blocks, int page_size, int n_pages,
                                                   int window, float scale, void* out, float* part_acc, float* part_ml,
                                                   int n_tok, int nh, int nkv, int hd, int chunk, int n_splits, int fresh,
-                                                  int overlap_prev, float softcap, int* status, cudaStream_t stream) {
+                                                  int overlap_prev, float softcap, const float* sinks, int* status, cudaStream_t stream) {
     return decode_mma_launch(q, nullptr, k_cache, v_cache, positions, item_of_token, table, max_blocks, page_size, n_pages, window,
                              scale, out, part_acc, part_ml, n_tok, nh, nkv, hd, chunk, n_splits, fresh, overlap_prev ? 1 : 0,
-                             status, stream, softcap);
+                             status, stream, softcap, 1, sinks);
 }
 
 // The same for query heads in `kv_groups` groups per cached head: nkv counts the groups (nh / nkv <= 8 heads each), the cache
@@ -767,17 +785,21 @@ extern "C" int imparo_attention_decode_mma_grouped(const void* q, const void* k_
 // The same for a step in which every request brings ONE token, straight from the qkv product's split partials
 // (part [parts][n_tok][(nh + 2 nkv) * hd], split s at part + s * part_stride): the queries are made inside the kernel
 // and the new key and value rows are written into their pages by it.  q_w / k_w null: no per-head norm on that side;
-// inv_freq null: no rotation.  n_rot even, at most hd.
+// inv_freq null: no rotation.  n_rot even, at most hd.  v_from_k: the product is [q | k], (nh + nkv) * hd wide, and a key head
+// before the rotation is also the value head.  sinks: float32 [nh] or null, one more term exp(sinks[h]) per denominator.
 extern "C" int imparo_attention_decode_mma_qkv(const float* part, int parts, long long part_stride, const float* q_w,
                                                const float* k_w, const float* inv_freq, int n_rot, float eps,
                                                void* k_cache, void* v_cache, const int* positions, const int* item_of_token,
                                                const int* table, int max_blocks, int page_size, int n_pages, int window,
                                                float scale, void* out, float* part_acc, float* part_ml, int n_tok, int nh,
-                                               int nkv, int hd, int chunk, int n_splits, int* status, cudaStream_t stream) {
+                                               int nkv, int hd, int chunk, int n_splits, int v_from_k, const float* sinks, int* status,
+                                               cudaStream_t stream) {
     if (part == nullptr || parts < 1) return -24;
     if (n_rot < 0 || (n_rot & 1) || n_rot > hd) return -4;
     pf::QkvSource src{part, parts, (size_t)part_stride, q_w, k_w, inv_freq, inv_freq ? n_rot : 0, eps,
                       (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache};
+    src.sinks = sinks;
+    src.v_from_k = v_from_k ? 1 : 0;
     // fresh = 1: a request's only new row is the one this kernel writes; older rows are safe to request early
     return decode_mma_launch(nullptr, &src, k_cache, v_cache, positions, item_of_token, table, max_blocks, page_size, n_pages,
                              window, scale, out, part_acc, part_ml, n_tok, nh, nkv, hd, chunk, n_splits, 1, 0, status, stream);

@@ -131,7 +131,12 @@ __device__ __forceinline__ float gated_act_bf16(int kind, float limit, float g, 
     return silu_bf16(g) * u;
 }
 
-// One activation on its own, for results that are rounded to bfloat16 at once:  0 relu(z)^2,  1 gelu (as above),  2 silu
+// One activation on its own:  0 relu(z)^2,  1 gelu (as above),  2 silu
+__device__ __forceinline__ float plain_act(int kind, float z) {
+    if (kind == 0) { const float r = fmaxf(z, 0.f); return r * r; }
+    return gated_act(kind == 1 ? IMPARO_GATED_GELU_TANH : IMPARO_GATED_SILU, 0.f, z, 1.f);
+}
+// The same for results that are rounded to bfloat16 at once
 __device__ __forceinline__ float plain_act_bf16(int kind, float z) {
     if (kind == 0) { const float r = fmaxf(z, 0.f); return r * r; }
     return gated_act_bf16(kind == 1 ? IMPARO_GATED_GELU_TANH : IMPARO_GATED_SILU, 0.f, z, 1.f);

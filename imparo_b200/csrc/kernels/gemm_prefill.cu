@@ -12,7 +12,7 @@
 //     warps 2-5 read one accumulator out (tcgen05.ld) and run the epilogue, the MMAs of the next
 //     tile already fill the other.
 //   * Epilogues, all on the accumulator in registers, a token row per thread:
-//       store bfloat16 | store float32 | add into float32 (the residual stream) |
+//       store bfloat16, as it is or after one activation | store float32 | add into float32 (the residual stream) |
 //       SwiGLU: the tile's 256 rows of W are 128 gate rows and the 128 up rows of the same
 //       features, h = silu(gate) * up is written as bfloat16 [T, F]
 //       (imparo-cpu/src/ops.rs:73-78; imparo-model/src/lfm2/workflow_cpu.rs:307-313): the
@@ -38,7 +38,7 @@ constexpr uint32_t A_BYTES = TM * BK * 2, B_BYTES = TN * BK * 2, STAGE_BYTES = A
 constexpr uint32_t TMEM_COLS = 2 * TN;
 constexpr size_t SMEM_BYTES = 1024 + (size_t)STAGES * STAGE_BYTES + 256;
 
-enum Epilogue { STORE_BF16 = 0, STORE_F32 = 1, ADD_F32 = 2, SWIGLU_BF16 = 3 };
+enum Epilogue { STORE_BF16 = 0, STORE_F32 = 1, ADD_F32 = 2, SWIGLU_BF16 = 3, ACT_BF16 = 4 };
 
 struct Params {
     void* out;               // [T, ldo]
@@ -52,7 +52,7 @@ struct Params {
     // before its first look at it, and all three skip the same tiles.  null: one matrix for all tiles.
     const int* tile_group;
     int group_rows;
-    // the gated epilogue's activation (gated_act's kinds; 0: silu(gate) * up) and its limit
+    // the gated epilogue's activation (gated_act's kinds; 0: silu(gate) * up) and its limit; ACT_BF16: plain_act_bf16's kind
     int act;
     float limit;
     const float* bias;       // the gated epilogue: [2N] = the gate product's bias, then the up product's; or null
@@ -287,7 +287,11 @@ gemm_prefill_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                         if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(&acc_empty[b])) : "memory");
                     }
                     if (!live) continue;
-                    if (EPI == STORE_BF16) {
+                    if (EPI == ACT_BF16) {
+#pragma unroll
+                        for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(plain_act_bf16(p.act, __uint_as_float(r[j])));
+                    }
+                    if (EPI == STORE_BF16 || EPI == ACT_BF16) {
                         __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)t * p.ldo;
 #pragma unroll
                         for (int j = 0; j < 32; j += 8) {
@@ -383,7 +387,8 @@ using namespace imparo::tcp;
 // x: [T, K] bfloat16 with row stride ldx (elements), inside a buffer of x_rows_alloc rows.
 // w: [N, K] bfloat16 dense (SwiGLU: [2N, K], gate rows then up rows).  out: [T, ldo].
 // epilogue: 0 store bfloat16, 1 store float32, 2 add into float32, 3 gated (bfloat16 [T, N]: act, limit: gated_act's kinds, 0 is
-// SwiGLU; bias: float32 [2N] added to the gate and up products before the activation, or null).
+// SwiGLU; bias: float32 [2N] added to the gate and up products before the activation, or null), 4 one activation, then store
+// bfloat16 (act: plain_act_bf16's kinds).
 // Refused (-23): K or ldx not a multiple of 8, operands not 16-byte aligned, N or ldo not a
 // multiple of 8 (4 for the float32 outputs), out not 16-byte aligned: the caller then takes the
 // library product.
@@ -395,7 +400,7 @@ extern "C" int imparo_gemm_prefill(const void* x, int ldx, int x_rows_alloc, con
     if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) return -23;
     const bool f32_out = epilogue == STORE_F32 || epilogue == ADD_F32;
     if (N % (f32_out ? 4 : 8) != 0 || ldo % (f32_out ? 4 : 8) != 0) return -23;
-    if (epilogue < 0 || epilogue > 3) return -22;
+    if (epilogue < 0 || epilogue > 4) return -22;
     const int w_rows = epilogue == SWIGLU_BF16 ? 2 * N : N;
     CUtensorMap mw, mx;
     int rc = get_map(w, (uint64_t)w_rows, (uint64_t)K, (uint64_t)K, epilogue == SWIGLU_BF16 ? 128u : (uint32_t)TN, &mw);
@@ -414,6 +419,7 @@ extern "C" int imparo_gemm_prefill(const void* x, int ldx, int x_rows_alloc, con
     switch (epilogue) {
         case STORE_BF16: return launch_prefill<STORE_BF16>(mw, mx, p, ctas, stream);
         case STORE_F32: return launch_prefill<STORE_F32>(mw, mx, p, ctas, stream);
+        case ACT_BF16: return launch_prefill<ACT_BF16>(mw, mx, p, ctas, stream);
         case ADD_F32: return launch_prefill<ADD_F32>(mw, mx, p, ctas, stream);
         default: return launch_prefill<SWIGLU_BF16>(mw, mx, p, ctas, stream);
     }
@@ -423,15 +429,15 @@ extern "C" int imparo_gemm_prefill(const void* x, int ldx, int x_rows_alloc, con
 // The same product for rows that are sorted by group: x [rows, K] holds every group's rows from a multiple of 128 on
 // (rows = 128 * m_tiles, padding rows hold anything), w the groups' matrices stacked ([n_groups * N, K]; SwiGLU:
 // [n_groups * 2N, K], each group its gate rows then its up rows), tile_group int32 [m_tiles] on the device (-1: a tile
-// without rows).  epilogue: 0 store bfloat16, 1 store float32, 3 gated (act, limit: gated_act's kinds; 0 is SwiGLU).  Refusals
-// as above.
+// without rows).  epilogue: 0 store bfloat16, 1 store float32, 3 gated (act, limit: gated_act's kinds; 0 is SwiGLU), 4 one
+// activation, then store bfloat16 (act: plain_act_bf16's kinds).  Refusals as above.
 extern "C" int imparo_gemm_prefill_grouped(const void* x, int ldx, const void* w, int n_groups, void* out, int ldo, int m_tiles,
                                            int N, int K, int epilogue, int act, float limit, const int* tile_group, int* status,
                                            cudaStream_t stream) {
     if (m_tiles <= 0 || N <= 0 || n_groups <= 0) return 0;
     if (K <= 0 || K % 8 != 0 || ldx % 8 != 0) return -23;
     if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) return -23;
-    if (epilogue != STORE_BF16 && epilogue != STORE_F32 && epilogue != SWIGLU_BF16) return -22;
+    if (epilogue != STORE_BF16 && epilogue != STORE_F32 && epilogue != SWIGLU_BF16 && epilogue != ACT_BF16) return -22;
     const bool f32_out = epilogue == STORE_F32;
     if (N % (f32_out ? 4 : 8) != 0 || ldo % (f32_out ? 4 : 8) != 0) return -23;
     const int group_rows = epilogue == SWIGLU_BF16 ? 2 * N : N;
@@ -455,6 +461,7 @@ extern "C" int imparo_gemm_prefill_grouped(const void* x, int ldx, const void* w
     switch (epilogue) {
         case STORE_BF16: return launch_prefill<STORE_BF16>(mw, mx, p, ctas, stream);
         case STORE_F32: return launch_prefill<STORE_F32>(mw, mx, p, ctas, stream);
+        case ACT_BF16: return launch_prefill<ACT_BF16>(mw, mx, p, ctas, stream);
         default: return launch_prefill<SWIGLU_BF16>(mw, mx, p, ctas, stream);
     }
 }

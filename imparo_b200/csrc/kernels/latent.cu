@@ -10,9 +10,11 @@
 //      [q: heads x (dim plain | rot rotated) | c_raw: rank | kr: rot]: the page row becomes [rms(c_raw) * w | turn(kr)]
 //      (rank + rot wide; kr is one key part that all heads share); every head's plain query dimensions go to q_plain
 //      [T, heads * dim] and its rotated ones, turned by the position, to the last rot entries of the head's latent-space
-//      query q_lat [T, heads * (rank + rot)] (the first rank entries are U_k^T q_plain, made by heads_linear).  The turn: of the
-//      first n_rot of the rot dimensions, i pairs with i + n_rot/2, angle = position * inv_freq[i] in 32-bit.  Two CTAs per
-//      token: one for the queries, one for the cached row.
+//      query q_lat [T, heads * row_w] (the first rank entries are U_k^T q_plain, made by heads_linear).  The turn: of the
+//      first n_rot of the rot dimensions, i pairs with i + n_rot/2 (or, interleaved, 2i with 2i + 1), angle = position *
+//      inv_freq[i] in 32-bit, sines and cosines times a magnitude.  A row may be wider than rank + rot (row_w): the rest of
+//      cached rows and latent-space queries is zero.  Two CTAs per token: one for the queries, one for the cached row; a layer
+//      that reads rows another layer has cached launches the first alone.
 //  (2) heads_linear: out[t, h, :] = W[h] x[t, h, :] for every head h (W [heads, out, in]), optionally times
 //      sigmoid(gate[t, h, :]) (a 32-bit product's columns).  A warp per output feature of a head and tile of eight rows;
 //      32-bit sums (for steps of few rows: many rows go to the library's batched product).
@@ -58,11 +60,22 @@ latent_norm_store_kernel(const float* __restrict__ proj, size_t stride, int q_of
     for (int i = threadIdx.x; i < n; i += blockDim.x) dst[i] = from_f32<T>(src[i] * scale * w[i]);
 }
 
+// dimension d of a rotated part of which the first n_rot dimensions turn
+__device__ __forceinline__ float turned(const float* __restrict__ v, int d, int n_rot, bool interleaved, const float* cs, const float* sn) {
+    if (d >= n_rot) return v[d];
+    if (interleaved) {
+        const int j = d >> 1;
+        return (d & 1) ? v[d] * cs[j] + v[d - 1] * sn[j] : v[d] * cs[j] - v[d + 1] * sn[j];
+    }
+    const int half = n_rot >> 1;
+    return d < half ? v[d] * cs[d] - v[d + half] * sn[d] : v[d] * cs[d - half] + v[d - half] * sn[d - half];
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128)
-latent_rot_store_kernel(const float* __restrict__ proj, size_t stride, int heads, int dim, int rot, int rank,
-                        const float* __restrict__ wc, float eps, const float* __restrict__ inv_freq, int n_rot,
-                        const int* __restrict__ positions, const int* __restrict__ item_of_token,
+latent_rot_store_kernel(const float* __restrict__ proj, size_t stride, int heads, int dim, int rot, int rank, int row_w,
+                        const float* __restrict__ wc, float eps, const float* __restrict__ inv_freq, int n_rot, int interleaved,
+                        float magnitude, const int* __restrict__ positions, const int* __restrict__ item_of_token,
                         T* __restrict__ q_plain, T* __restrict__ q_lat, T* __restrict__ cache, const int* __restrict__ table,
                         int max_blocks, int page_size, int n_pages, int* status) {
     __shared__ float scratch[33];
@@ -72,10 +85,15 @@ latent_rot_store_kernel(const float* __restrict__ proj, size_t stride, int heads
     const int pos = positions[t];
     const int blk = pos / page_size;
     int page = -1;
-    if (blk < max_blocks) page = table[(size_t)item_of_token[t] * max_blocks + blk];
-    const int q_width = heads * (dim + rot), row_w = rank + rot, half = n_rot / 2;
+    if (blockIdx.y == 1 && blk < max_blocks) page = table[(size_t)item_of_token[t] * max_blocks + blk];
+    const int q_width = heads * (dim + rot), half = n_rot / 2;
     const float fpos = (float)pos;
-    for (int j = threadIdx.x; j < half; j += blockDim.x) sincosf(fpos * inv_freq[j], &sn_s[j], &cs_s[j]);
+    for (int j = threadIdx.x; j < half; j += blockDim.x) {
+        float sn, cs;
+        sincosf(fpos * inv_freq[j], &sn, &cs);
+        sn_s[j] = sn * magnitude;
+        cs_s[j] = cs * magnitude;
+    }
     pdl_wait();
     __syncthreads();
     const float* row = proj + (size_t)t * stride;
@@ -85,15 +103,10 @@ latent_rot_store_kernel(const float* __restrict__ proj, size_t stride, int heads
             const int h = i / dim, d = i % dim;
             q_plain[(size_t)t * heads * dim + i] = from_f32<T>(row[(size_t)h * (dim + rot) + d]);
         }
-        for (int i = threadIdx.x; i < heads * rot; i += blockDim.x) {
-            const int h = i / rot, d = i % rot;
-            const float* qr = row + (size_t)h * (dim + rot) + dim;
-            float v = qr[d];
-            if (d < n_rot) {
-                const int j = d < half ? d : d - half;
-                const float sn = sn_s[j], cs = cs_s[j];
-                v = d < half ? qr[d] * cs - qr[d + half] * sn : qr[d] * cs + qr[d - half] * sn;
-            }
+        const int tail = row_w - rank;
+        for (int i = threadIdx.x; i < heads * tail; i += blockDim.x) {
+            const int h = i / tail, d = i % tail;
+            const float v = d < rot ? turned(row + (size_t)h * (dim + rot) + dim, d, n_rot, interleaved, cs_s, sn_s) : 0.f;
             q_lat[((size_t)t * heads + h) * row_w + rank + d] = from_f32<T>(v);
         }
         return;
@@ -111,15 +124,8 @@ latent_rot_store_kernel(const float* __restrict__ proj, size_t stride, int heads
     const float scale = 1.0f / sqrtf(ss / (float)rank + eps);
     for (int i = threadIdx.x; i < rank; i += blockDim.x) dst[i] = from_f32<T>(c[i] * scale * wc[i]);
     const float* kr = c + rank;
-    for (int d = threadIdx.x; d < rot; d += blockDim.x) {
-        float v = kr[d];
-        if (d < n_rot) {
-            const int j = d < half ? d : d - half;
-            const float sn = sn_s[j], cs = cs_s[j];
-            v = d < half ? kr[d] * cs - kr[d + half] * sn : kr[d] * cs + kr[d - half] * sn;
-        }
-        dst[rank + d] = from_f32<T>(v);
-    }
+    for (int d = threadIdx.x; d < row_w - rank; d += blockDim.x)
+        dst[rank + d] = from_f32<T>(d < rot ? turned(kr, d, n_rot, interleaved, cs_s, sn_s) : 0.f);
 }
 
 constexpr int HL_ROWS = 8;
@@ -216,23 +222,26 @@ extern "C" int imparo_latent_norm_store(const float* proj, long long stride, int
 }
 
 // proj: float32 rows of `stride` floats = [heads * (dim + rot) | rank | rot | ...]; q_plain [n_tok, heads * dim], q_lat
-// [n_tok, heads * (rank + rot)] and cache pages of rank + rot per position, all in dtype; inv_freq float32 [n_rot / 2] (null
-// with n_rot 0).
-extern "C" int imparo_latent_rot_store(const float* proj, long long stride, int heads, int dim, int rot, int rank, const float* wc,
-                                       float eps, const float* inv_freq, int n_rot, const int* positions, const int* item_of_token,
-                                       void* q_plain, void* q_lat, void* cache, int dtype, const int* table, int max_blocks,
-                                       int page_size, int n_pages, int n_tok, int* status, cudaStream_t stream) {
+// [n_tok, heads * row_w] and cache pages of row_w (>= rank + rot) per position, all in dtype; inv_freq float32 [n_rot / 2]
+// (null with n_rot 0).  cache null: only the queries are made (proj rows then need no latent).
+extern "C" int imparo_latent_rot_store(const float* proj, long long stride, int heads, int dim, int rot, int rank, int row_w,
+                                       const float* wc, float eps, const float* inv_freq, int n_rot, int interleaved,
+                                       float magnitude, const int* positions, const int* item_of_token, void* q_plain, void* q_lat,
+                                       void* cache, int dtype, const int* table, int max_blocks, int page_size, int n_pages,
+                                       int n_tok, int* status, cudaStream_t stream) {
     if (n_tok <= 0) return 0;
-    if (heads < 1 || dim < 1 || rot < 0 || rank < 1 || n_rot < 0 || n_rot > rot || n_rot > 512 || n_rot % 2 || (n_rot > 0 && inv_freq == nullptr)
-        || stride < (long long)heads * (dim + rot) + rank + rot) return -2;
+    if (heads < 1 || dim < 1 || rot < 0 || rank < 1 || row_w < rank + rot || n_rot < 0 || n_rot > rot || n_rot > 512 || n_rot % 2
+        || (n_rot > 0 && inv_freq == nullptr) || page_size < 1
+        || stride < (long long)heads * (dim + rot) + (cache != nullptr ? rank + rot : 0)) return -2;
+    const dim3 grid(n_tok, cache != nullptr ? 2 : 1);
     if (dtype == IMPARO_DT_F32)
-        launch(latent_rot_store_kernel<float>, dim3(n_tok, 2), dim3(128), 0, stream, proj, (size_t)stride, heads, dim, rot, rank, wc, eps,
-               inv_freq, n_rot, positions, item_of_token, (float*)q_plain, (float*)q_lat, (float*)cache, table, max_blocks, page_size,
-               n_pages, status);
+        launch(latent_rot_store_kernel<float>, grid, dim3(128), 0, stream, proj, (size_t)stride, heads, dim, rot, rank, row_w, wc, eps,
+               inv_freq, n_rot, interleaved, magnitude, positions, item_of_token, (float*)q_plain, (float*)q_lat, (float*)cache, table,
+               max_blocks, page_size, n_pages, status);
     else if (dtype == IMPARO_DT_BF16)
-        launch(latent_rot_store_kernel<__nv_bfloat16>, dim3(n_tok, 2), dim3(128), 0, stream, proj, (size_t)stride, heads, dim, rot, rank, wc,
-               eps, inv_freq, n_rot, positions, item_of_token, (__nv_bfloat16*)q_plain, (__nv_bfloat16*)q_lat, (__nv_bfloat16*)cache,
-               table, max_blocks, page_size, n_pages, status);
+        launch(latent_rot_store_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, proj, (size_t)stride, heads, dim, rot, rank, row_w, wc,
+               eps, inv_freq, n_rot, interleaved, magnitude, positions, item_of_token, (__nv_bfloat16*)q_plain, (__nv_bfloat16*)q_lat,
+               (__nv_bfloat16*)cache, table, max_blocks, page_size, n_pages, status);
     else return -1;
     IMPARO_CHECK_LAUNCH();
     return 0;

@@ -2,7 +2,9 @@
 //
 //  (1) moe_route: router logits z = W_r h in 32-bit (a warp per expert, four rows per block), then a warp per row picks the
 //      `top` largest (by logit: the scores sigmoid(z) or softmax(z) are monotone in it; ties: the lower expert), optionally
-//      renormalised to sum 1.  Leaves expert ids [rows, top] and weights [rows, top].
+//      renormalised to sum 1.  Leaves expert ids [rows, top] and weights [rows, top].  With a correction per expert the choice
+//      (and the groups' verdict) goes by score + correction, the weights by the score alone; a logit column behind the experts'
+//      may give each row one more number, sigmoid(z) (the factor of an expert that every row uses).
 //  (2) moe_rows_*: each (row, choice) pair on its own: the expert's gate and up rows times the (optionally weighted)
 //      input, silu(gate) * up, then the expert's down rows; the choices of a row are added in order.  Weights are
 //      streamed once per pair: the form for steps of few rows.
@@ -12,8 +14,13 @@
 //      on the device from the counts; CTAs beyond it leave at once, so the launch depends on (rows, top, experts)
 //      only.
 //
-// Expert e's matrices: w_gu[e] = [gate; up] ([2 ff, width]), w_down[e] ([width, ff]).  The weight multiplies the
-// expert's input (weight_input = 1) or its output (0).
+// Expert e's matrices: w_gu[e] = [gate; up] ([2 ff, width]), w_down[e] ([width, ff]); or, without a gate (gated = 0), w_gu[e] = up
+// ([ff, width]) and one activation on its own (plain_act's kinds).  The weight multiplies the expert's input (weight_input = 1)
+// or its output (0).
+//
+// A shared expert without a gate, of any size, may run in the launches of (2): blocks of their own, each for up to eight rows at
+// once, so that its matrices are read once for them.  Its rows' factors and the residual stream come in where the pairs are
+// summed (moe_sum_pairs / moe_tile_sum), which can add into the stream and leave the rounded copy that the next product reads.
 #include "common.cuh"
 #include <mma.h>
 
@@ -131,25 +138,34 @@ moe_logits_kernel(const T* __restrict__ h, const float* __restrict__ w_r, int n_
 // The choice: a warp per row, four rows per block
 // logits: [n_rows, parts * experts]; a logit is the sum of its `parts` entries, experts apart, added in order (parts > 1:
 // the router matrix was cut into bfloat16 pieces whose sum is the 32-bit matrix to its last bit, see imparo_moe_pick)
+// columns >= experts: the logits' columns per part (those beyond the experts' are not candidates); correction: float32
+// [experts] or null; group_pair: a group's score is the sum of its two largest (else its largest); extra_out: float32 [n_rows]
+// or null, sigmoid of column `experts`.
 __global__ void __launch_bounds__(128)
-moe_pick_kernel(const float* __restrict__ logits, int n_rows, int experts, int parts, int top, int softmax_scores, int renormalise,
-                int groups, int keep, float renorm_eps, float weight_scale, int out_stride, int* __restrict__ ids,
-                float* __restrict__ wts) {
-    extern __shared__ __align__(16) float pick_smem[];   // [4][experts] scores, then [4][groups] maxima of the groups
+moe_pick_kernel(const float* __restrict__ logits, int n_rows, int experts, int columns, int parts, int top, int softmax_scores,
+                int renormalise, int groups, int keep, int group_pair, const float* __restrict__ correction, float renorm_eps,
+                float weight_scale, int out_stride, int* __restrict__ ids, float* __restrict__ wts, float* __restrict__ extra_out) {
+    extern __shared__ __align__(16) float pick_smem[];   // [4][experts] scores, then [4][groups] scores of the groups
     pdl_trigger();
     pdl_wait();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int r = blockIdx.x * 4 + warp;
     if (r >= n_rows) return;
     float* s = pick_smem + (size_t)warp * experts;
-    for (int e = lane; e < experts; e += 32) {
-        const float* l = logits + (size_t)r * parts * experts + e;
+    auto logit = [&](int e) {
+        const float* l = logits + (size_t)r * parts * columns + e;
         float v = l[0];
-        for (int k = 1; k < parts; ++k) v += l[(size_t)k * experts];
-        s[e] = v;
+        for (int k = 1; k < parts; ++k) v += l[(size_t)k * columns];
+        return v;
+    };
+    for (int e = lane; e < experts; e += 32) {
+        const float v = logit(e);
+        s[e] = correction ? 1.0f / (1.0f + expf(-v)) + correction[e] : v;
     }
+    if (extra_out && lane == 0) extra_out[r] = 1.0f / (1.0f + expf(-logit(experts)));
     __syncwarp();
-    // The choice goes by the logits: scores are monotone in them, and a sigmoid that has reached 1 in 32-bit would tie.
+    // Without a correction the choice goes by the logits: scores are monotone in them, and a sigmoid that has reached 1 in
+    // 32-bit would tie.
     float m = -INFINITY, l = 1.f;
     if (softmax_scores) {
         for (int e = lane; e < experts; e += 32) m = fmaxf(m, s[e]);
@@ -158,17 +174,22 @@ moe_pick_kernel(const float* __restrict__ logits, int n_rows, int experts, int p
         for (int e = lane; e < experts; e += 32) l += expf(s[e] - m);
         l = warp_sum(l);
     }
-    // Experts in `groups` equal groups of neighbours: a group's score is its largest, and only the `keep` best groups'
-    // experts stay candidates (ties: the lower group).  The others leave the candidates; the softmax above counted them.
+    // Experts in `groups` equal groups of neighbours: a group's score is its largest (or the sum of its two largest), and only
+    // the `keep` best groups' experts stay candidates (ties: the lower group).  The others leave the candidates; the softmax
+    // above counted them.
     if (groups > 1 && keep < groups) {
         const int per = experts / groups;
-        // every group's maximum first (a lane per group), then a lane per group counts the groups that beat its own: a group
+        // every group's score first (a lane per group), then a lane per group counts the groups that beat its own: a group
         // is kept when fewer than `keep` do.  All verdicts are in before any score is masked.
         float* gmax = pick_smem + (size_t)4 * experts + (size_t)warp * groups;
         for (int g = lane; g < groups; g += 32) {
-            float mx = -INFINITY;
-            for (int e = g * per; e < (g + 1) * per; ++e) mx = fmaxf(mx, s[e]);
-            gmax[g] = mx;
+            float mx = -INFINITY, second = -INFINITY;
+            for (int e = g * per; e < (g + 1) * per; ++e) {
+                const float v = s[e];
+                second = fmaxf(second, fminf(mx, v));
+                mx = fmaxf(mx, v);
+            }
+            gmax[g] = group_pair && per > 1 ? mx + second : mx;
         }
         __syncwarp();
         for (int g = lane; g < groups; g += 32) {
@@ -197,7 +218,7 @@ moe_pick_kernel(const float* __restrict__ logits, int n_rows, int experts, int p
             const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
             if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
         }
-        const float score = softmax_scores ? expf(best - m) / l : 1.0f / (1.0f + expf(-best));
+        const float score = softmax_scores ? expf(best - m) / l : 1.0f / (1.0f + expf(-(correction ? logit(arg) : best)));
         if (lane == 0) {
             ids[(size_t)r * out_stride + k] = arg;
             wts[(size_t)r * out_stride + k] = score;
@@ -249,15 +270,107 @@ __device__ __forceinline__ void warp_dot2(const T* __restrict__ w0, const T* __r
     r1 = warp_sum((b[0] + b[1]) + (b[2] + b[3]));
 }
 
-// grid (rows * top, ceil(ff / 32)); 8 warps, each 4 features
+// ---- blocks of the shared expert: up to SHARED_ROWS rows at once ------------------------------------------------------------
+constexpr int SHARED_ROWS = 8;
+
+// acc[j][r] = W row f0 + j . x row r for the four rows of W (those below n_feat) and the block's rows; xs: [rows][n] in shared
+// memory.  A lane takes every 32nd 16 bytes of a row; the sums end with a fixed tree over the warp.
+template <typename T>
+__device__ __forceinline__ void warp_dot_rows(const T* __restrict__ w, int f0, int n_feat, const T* xs, int rows, int n, bool vec,
+                                              int lane, float (&acc)[4][SHARED_ROWS]) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int r = 0; r < SHARED_ROWS; ++r) acc[j][r] = 0.f;
+    if (vec) {
+        constexpr int PER = Vec16<T>::N;
+        const int n4 = n / PER;
+        for (int i = lane; i < n4; i += 32) {
+            uint4 wv[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                wv[j] = f0 + j < n_feat ? reinterpret_cast<const uint4*>(w + (size_t)(f0 + j) * n)[i] : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+            for (int r = 0; r < SHARED_ROWS; ++r) {
+                if (r < rows) {
+                    const uint4 xv = reinterpret_cast<const uint4*>(xs + (size_t)r * n)[i];
+                    float xf[PER];
+#pragma unroll
+                    for (int u = 0; u < PER; ++u) xf[u] = to_f32(reinterpret_cast<const T*>(&xv)[u]);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) acc[j][r] += dot16<T>(wv[j], xf);
+                }
+            }
+        }
+    } else {
+        for (int i = lane; i < n; i += 32)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                if (f0 + j >= n_feat) break;
+                const float wv = to_f32(w[(size_t)(f0 + j) * n + i]);
+#pragma unroll
+                for (int r = 0; r < SHARED_ROWS; ++r) if (r < rows) acc[j][r] += wv * to_f32(xs[(size_t)r * n + i]);
+            }
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int r = 0; r < SHARED_ROWS; ++r) acc[j][r] = warp_sum(acc[j][r]);
+}
+
+// One block of the shared expert: 32 features (8 warps, each 4) of the rows tile * SHARED_ROWS ..; out rows of n_feat entries.
+template <typename T, typename TOut>
+__device__ __forceinline__ void shared_block(const T* __restrict__ x, const T* __restrict__ w, int tile, int block_y, int n_rows, int n,
+                                             int n_feat, int act, void* smem, TOut* __restrict__ out) {
+    if (block_y * 32 >= n_feat) return;
+    T* xs = reinterpret_cast<T*>(smem);
+    const int r0 = tile * SHARED_ROWS, rows = min(SHARED_ROWS, n_rows - r0);
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const bool vec = n % Vec16<T>::N == 0 && (((uintptr_t)w | (uintptr_t)x) & 15) == 0;
+    if (vec) {
+        const uint4* src = reinterpret_cast<const uint4*>(x + (size_t)r0 * n);
+        for (int i = threadIdx.x; i < rows * (n / Vec16<T>::N); i += blockDim.x) reinterpret_cast<uint4*>(xs)[i] = src[i];
+    } else {
+        for (int i = threadIdx.x; i < rows * n; i += blockDim.x) xs[i] = x[(size_t)r0 * n + i];
+    }
+    __syncthreads();
+    const int f0 = block_y * 32 + warp * 4;
+    if (f0 >= n_feat) return;
+    float acc[4][SHARED_ROWS];
+    warp_dot_rows<T>(w, f0, n_feat, xs, rows, n, vec, lane, acc);
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int r = 0; r < SHARED_ROWS; ++r)
+            if (lane == j * SHARED_ROWS + r && r < rows && f0 + j < n_feat)
+                out[(size_t)(r0 + r) * n_feat + f0 + j] = from_f32<TOut>(act >= 0 ? plain_act(act, acc[j][r]) : acc[j][r]);
+}
+
+// What the shared expert adds to a launch of the rows kernels (w null: nothing): the up kernel reads x rows of `n` entries and
+// writes mid rows of `n_feat`, the down kernel the other way round into float32 rows.
+struct SharedRows {
+    const void* w;
+    int n_feat, n;
+    void* out;
+};
+
+// grid (rows * top + shared row tiles, ceil(features / 32)); 8 warps, each 4 features
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_rows_up_kernel(const T* __restrict__ h, const T* __restrict__ w_gu, const int* __restrict__ ids, const float* __restrict__ wts,
-                   int width, int ff, int top, int experts, int weight_input, int act, float limit, T* __restrict__ mid) {
+                   int n_rows, int width, int ff, int top, int experts, int weight_input, int gated, int act, float limit,
+                   T* __restrict__ mid, SharedRows sh) {
     extern __shared__ __align__(16) float up_smem[];
     pdl_trigger();
     pdl_wait();
-    const int pair = blockIdx.x, r = pair / top;
+    // the shared expert's blocks come first: they have the most to do
+    const int shared_tiles = sh.w ? (n_rows + SHARED_ROWS - 1) / SHARED_ROWS : 0;
+    if ((int)blockIdx.x < shared_tiles) {
+        shared_block<T, T>(h, (const T*)sh.w, blockIdx.x, blockIdx.y, n_rows, sh.n, sh.n_feat, act, up_smem, (T*)sh.out);
+        return;
+    }
+    if ((int)blockIdx.y * 32 >= ff) return;
+    const int pair = blockIdx.x - shared_tiles, r = pair / top;
     const int e = ids[pair];
     if (e < 0 || e >= experts) return;
     const float wt = weight_input ? wts[pair] : 1.0f;
@@ -265,8 +378,21 @@ moe_rows_up_kernel(const T* __restrict__ h, const T* __restrict__ w_gu, const in
     for (int i = threadIdx.x; i < width; i += blockDim.x) up_smem[i] = to_f32(from_f32<T>(wt * to_f32(hr[i])));
     __syncthreads();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const T* base = w_gu + (size_t)e * 2 * ff * width;
+    const T* base = w_gu + (size_t)e * (gated ? 2 : 1) * ff * width;
     const bool vec = width % Vec16<T>::N == 0 && ((uintptr_t)w_gu & 15) == 0;
+    if (!gated) {
+        for (int j = 0; j < 4; j += 2) {
+            const int f = blockIdx.y * 32 + warp * 4 + j;
+            if (f >= ff) break;
+            float a0, a1;
+            warp_dot2<T>(base + (size_t)f * width, base + (size_t)min(f + 1, ff - 1) * width, up_smem, width, vec, lane, a0, a1);
+            if (lane == 0) {
+                mid[(size_t)pair * ff + f] = from_f32<T>(plain_act(act, a0));
+                if (f + 1 < ff) mid[(size_t)pair * ff + f + 1] = from_f32<T>(plain_act(act, a1));
+            }
+        }
+        return;
+    }
     for (int j = 0; j < 4; ++j) {
         const int f = blockIdx.y * 32 + warp * 4 + j;
         if (f >= ff) break;
@@ -276,16 +402,21 @@ moe_rows_up_kernel(const T* __restrict__ h, const T* __restrict__ w_gu, const in
     }
 }
 
-// grid (rows, ceil(width / 32)); 8 warps, each 4 outputs; out float32 [rows, width] is overwritten
+// grid (rows + shared row tiles, ceil(width / 32)); 8 warps, each 4 outputs; out float32 [rows, width] is overwritten
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_rows_down_kernel(const T* __restrict__ mid, const T* __restrict__ w_down, const int* __restrict__ ids,
-                     const float* __restrict__ wts, int width, int ff, int top, int experts, int weight_input,
-                     float* __restrict__ out) {
+                     const float* __restrict__ wts, int n_rows, int width, int ff, int top, int experts, int weight_input,
+                     float* __restrict__ out, SharedRows sh, const T* __restrict__ shared_mid) {
     extern __shared__ __align__(16) float down_smem[];
     pdl_trigger();
     pdl_wait();
-    const int r = blockIdx.x;
+    const int shared_tiles = sh.w ? (n_rows + SHARED_ROWS - 1) / SHARED_ROWS : 0;
+    if ((int)blockIdx.x < shared_tiles) {
+        shared_block<T, float>(shared_mid, (const T*)sh.w, blockIdx.x, blockIdx.y, n_rows, sh.n, sh.n_feat, -1, down_smem, (float*)sh.out);
+        return;
+    }
+    const int r = blockIdx.x - shared_tiles;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const bool vec = ff % Vec16<T>::N == 0 && ((uintptr_t)w_down & 15) == 0;
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
@@ -445,7 +576,7 @@ __device__ __forceinline__ void group_tile_product(GroupTile<T>& sm, LoadA load_
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_group_up_kernel(const T* __restrict__ h, const T* __restrict__ w_gu, const int* __restrict__ sorted, const int* __restrict__ plan,
-                    const float* __restrict__ wts, int width, int ff, int top, int weight_input, int act, float limit,
+                    const float* __restrict__ wts, int width, int ff, int top, int weight_input, int gated, int act, float limit,
                     T* __restrict__ mid) {
     __shared__ GroupTile<T> sm;
     __shared__ int pair_of[GM];
@@ -466,8 +597,15 @@ moe_group_up_kernel(const T* __restrict__ h, const T* __restrict__ w_gu, const i
     auto load_a = [&](int m, int k) -> T {
         return from_f32<T>(wt_of[m] * to_f32(h[(size_t)(pair_of[m] / top) * width + k]));
     };
-    const T* base = w_gu + (size_t)e * 2 * ff * width;
+    const T* base = w_gu + (size_t)e * (gated ? 2 : 1) * ff * width;
     group_tile_product<T>(sm, load_a, base, n0, ff, width, rows);
+    if (!gated) {
+        for (int i = threadIdx.x; i < GM * GN; i += 256) {
+            const int m = i / GN, n = i % GN;
+            if (m < rows && n0 + n < ff) mid[(size_t)pair_of[m] * ff + n0 + n] = from_f32<T>(plain_act(act, sm.c[m][n]));
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < GM * GN; i += 256) gate_c[i / GN][i % GN] = sm.c[i / GN][i % GN];
     group_tile_product<T>(sm, load_a, base + (size_t)ff * width, n0, ff, width, rows);
     for (int i = threadIdx.x; i < GM * GN; i += 256) {
@@ -503,17 +641,50 @@ moe_group_down_kernel(const T* __restrict__ mid, const T* __restrict__ w_down, c
     }
 }
 
-// out[r, :] = sum over the row's choices, in order
+// What the sums below may do besides: add extra_w[r] * extra[r, :] (extra float32 [rows, width], extra_w float32 [rows]; null:
+// nothing), add into what `out` holds (accumulate), and leave the result's rows rounded in `copy` (bfloat16 or null).
+struct SumTail {
+    const float* extra;
+    const float* extra_w;
+    int accumulate;
+    __nv_bfloat16* copy;
+};
+
+// out[r, :] = sum over the row's choices, in order; VEC: four columns at a time (width a multiple of 4, 16-byte aligned)
+template <bool VEC>
 __global__ void __launch_bounds__(256)
-moe_sum_pairs_kernel(const float* __restrict__ pair_out, int n_rows, int width, int top, float* __restrict__ out) {
+moe_sum_pairs_kernel(const float* __restrict__ pair_out, int n_rows, int width, int top, float* __restrict__ out, SumTail tail) {
     pdl_trigger();
     pdl_wait();
-    const size_t total = (size_t)n_rows * width;
+    constexpr int N = VEC ? 4 : 1;
+    const size_t total = (size_t)n_rows * width / N;
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
-        const size_t r = i / width, c = i - r * width;
-        float a = 0.f;
-        for (int k = 0; k < top; ++k) a += pair_out[(r * top + k) * width + c];
-        out[i] = a;
+        const size_t r = i * N / width, c = i * N - r * width;
+        float a[N];
+#pragma unroll
+        for (int u = 0; u < N; ++u) a[u] = 0.f;
+        auto add = [&](const float* p, float f) {
+            if constexpr (VEC) {
+                const float4 v = *reinterpret_cast<const float4*>(p);
+                a[0] += f * v.x; a[1] += f * v.y; a[2] += f * v.z; a[3] += f * v.w;
+            } else {
+                a[0] += f * *p;
+            }
+        };
+        for (int k = 0; k < top; ++k) add(pair_out + (r * top + k) * width + c, 1.f);
+        if (tail.extra) add(tail.extra + r * width + c, tail.extra_w[r]);
+        if (tail.accumulate) add(out + r * width + c, 1.f);
+        if constexpr (VEC) {
+            *reinterpret_cast<float4*>(out + r * width + c) = make_float4(a[0], a[1], a[2], a[3]);
+            if (tail.copy) {
+                const __nv_bfloat162 lo = __floats2bfloat162_rn(a[0], a[1]), hi = __floats2bfloat162_rn(a[2], a[3]);
+                *reinterpret_cast<uint2*>(tail.copy + r * width + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo),
+                                                                                  *reinterpret_cast<const uint32_t*>(&hi));
+            }
+        } else {
+            out[r * width + c] = a[0];
+            if (tail.copy) tail.copy[r * width + c] = __float2bfloat16(a[0]);
+        }
     }
 }
 
@@ -600,15 +771,18 @@ moe_tile_gather_kernel(const __nv_bfloat16* __restrict__ h, const int* __restric
 }
 
 // out[r, :] = sum over the row's choices, in order, of out_g[slot_of_pair[r * top + k], :]  (times the weight when it
-// multiplies the output); width a multiple of 4
+// multiplies the output), and what SumTail says; width a multiple of 4
 __global__ void __launch_bounds__(256)
 moe_tile_sum_kernel(const float* __restrict__ out_g, const int* __restrict__ slot_of_pair, const float* __restrict__ wts,
-                    int width, int top, int weight_input, float* __restrict__ out) {
+                    int width, int top, int weight_input, float* __restrict__ out, SumTail tail) {
     pdl_trigger();
     pdl_wait();
     const int r = blockIdx.x;
+    const float ew = tail.extra ? tail.extra_w[r] : 0.f;
     for (int c = threadIdx.x * 4; c < width; c += blockDim.x * 4) {
-        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f), e = a, x = a;
+        if (tail.extra) e = *reinterpret_cast<const float4*>(tail.extra + (size_t)r * width + c);
+        if (tail.accumulate) x = *reinterpret_cast<const float4*>(out + (size_t)r * width + c);
         for (int k = 0; k < top; ++k) {
             const int slot = slot_of_pair[r * top + k];
             if (slot < 0) continue;
@@ -616,7 +790,14 @@ moe_tile_sum_kernel(const float* __restrict__ out_g, const int* __restrict__ slo
             const float4 v = *reinterpret_cast<const float4*>(out_g + (size_t)slot * width + c);
             a.x += wt * v.x; a.y += wt * v.y; a.z += wt * v.z; a.w += wt * v.w;
         }
+        a.x += ew * e.x; a.y += ew * e.y; a.z += ew * e.z; a.w += ew * e.w;
+        if (tail.accumulate) { a.x += x.x; a.y += x.y; a.z += x.z; a.w += x.w; }
         *reinterpret_cast<float4*>(out + (size_t)r * width + c) = a;
+        if (tail.copy) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(a.x, a.y), hi = __floats2bfloat162_rn(a.z, a.w);
+            *reinterpret_cast<uint2*>(tail.copy + (size_t)r * width + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo),
+                                                                                      *reinterpret_cast<const uint32_t*>(&hi));
+        }
     }
 }
 
@@ -624,89 +805,155 @@ moe_tile_sum_kernel(const float* __restrict__ out_g, const int* __restrict__ slo
 
 using namespace imparo;
 
-// logits: float32 scratch [n_rows, experts].  Two launches.
-// The choice's further parameters (both entry points): groups, keep (experts in `groups` equal groups of neighbours, only the
-// `keep` best groups' experts may be chosen; groups <= 1: all), renorm_eps (added to the chosen scores' sum before the
-// division when renormalise is set), weight_scale (a factor on the weights), out_stride (ids and wts have out_stride >= top
-// entries per row: the entries beyond `top` name experts every row uses with weight 1, numbered from `experts` on).
+
+// The choice's parameters (both entry points): groups, keep (experts in `groups` equal groups of neighbours, only the
+// `keep` best groups' experts may be chosen; groups <= 1: all), group_pair (a group's score is the sum of its two largest
+// choice scores, else its largest), correction (float32 [experts] or null: the choice goes by sigmoid(z) + correction, the
+// weights by sigmoid(z); sigmoid scores only), renorm_eps (added to the chosen scores' sum before the division when renormalise
+// is set), weight_scale (a factor on the weights), out_stride (ids and wts have out_stride >= top entries per row: the entries
+// beyond `top` name experts every row uses with weight 1, numbered from `experts` on), extra_out (float32 [n_rows] or null:
+// sigmoid of the logit column behind the experts').
 static inline size_t pick_smem_bytes(int experts, int groups) {
     return (size_t)4 * (experts + (groups > 1 ? groups : 0)) * sizeof(float);
 }
 
-static inline bool pick_args_ok(int experts, int top, int groups, int keep, int out_stride) {
+static inline bool pick_args_ok(int experts, int top, int groups, int keep, int out_stride, int softmax_scores, const float* correction) {
     if (pick_smem_bytes(experts, groups) > 48 * 1024) return false;
     if (top < 1 || top > experts || top > 32 || experts > 2048 || out_stride < top || out_stride > top + 32) return false;
     if (groups > 1 && (experts % groups != 0 || keep < 1 || keep > groups || keep * (experts / groups) < top)) return false;
+    if (softmax_scores && correction != nullptr) return false;
     return true;
 }
 
+// logits: float32 scratch [n_rows, columns], w_r [columns, width] with columns = experts, or experts + 1 with extra_out.  Two
+// launches.
 extern "C" int imparo_moe_route(const void* h, int dtype, const float* w_r, int n_rows, int width, int experts, int top,
-                                int softmax_scores, int renormalise, int groups, int keep, float renorm_eps, float weight_scale,
-                                int out_stride, float* logits, int* ids, float* wts, cudaStream_t stream) {
+                                int softmax_scores, int renormalise, int groups, int keep, int group_pair, const float* correction,
+                                float renorm_eps, float weight_scale, int out_stride, float* logits, int* ids, float* wts,
+                                float* extra_out, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
-    if (!pick_args_ok(experts, top, groups, keep, out_stride) || logits == nullptr) return -2;
+    if (!pick_args_ok(experts, top, groups, keep, out_stride, softmax_scores, correction) || logits == nullptr) return -2;
+    const int columns = experts + (extra_out != nullptr ? 1 : 0);
     int per = 4;
     if ((size_t)4 * width * sizeof(float) > 48 * 1024) per = 1;
     const size_t smem = (size_t)per * width * sizeof(float);
     if (smem > 48 * 1024) return -25;
-    dim3 grid((n_rows + per - 1) / per, (experts + 7) / 8);
+    dim3 grid((n_rows + per - 1) / per, (columns + 7) / 8);
     if (dtype == IMPARO_DT_F32)
-        launch(moe_logits_kernel<float>, grid, dim3(256), smem, stream, (const float*)h, w_r, n_rows, width, experts, per, logits);
+        launch(moe_logits_kernel<float>, grid, dim3(256), smem, stream, (const float*)h, w_r, n_rows, width, columns, per, logits);
     else if (dtype == IMPARO_DT_BF16)
-        launch(moe_logits_kernel<__nv_bfloat16>, grid, dim3(256), smem, stream, (const __nv_bfloat16*)h, w_r, n_rows, width, experts,
+        launch(moe_logits_kernel<__nv_bfloat16>, grid, dim3(256), smem, stream, (const __nv_bfloat16*)h, w_r, n_rows, width, columns,
                per, logits);
     else return -1;
     IMPARO_CHECK_LAUNCH();
     launch(moe_pick_kernel, dim3((n_rows + 3) / 4), dim3(128), pick_smem_bytes(experts, groups), stream, (const float*)logits, n_rows,
-           experts, 1, top, softmax_scores, renormalise, groups, keep, renorm_eps, weight_scale, out_stride, ids, wts);
+           experts, columns, 1, top, softmax_scores, renormalise, groups, keep, group_pair, correction, renorm_eps, weight_scale,
+           out_stride, ids, wts, extra_out);
     IMPARO_CHECK_LAUNCH();
     return 0;
 }
 
-// The choice alone, from logits that a product has made: [n_rows, parts * experts] float32.  With bfloat16 rows h (exact in
-// 32-bit) and the 32-bit router matrix cut into three bfloat16 pieces (w1 = W rounded, w2 = W - w1 rounded, w3 the rest
-// rounded: 8 + 8 + 8 bits of mantissa, their sum is W to its last bit), the
+// The choice alone, from logits that a product has made: [n_rows, parts * columns] float32 (columns: experts, or experts + 1
+// with extra_out).  With bfloat16 rows h (exact in 32-bit) and the 32-bit router matrix cut into three bfloat16 pieces (w1 = W
+// rounded, w2 = W - w1 rounded, w3 the rest rounded: 8 + 8 + 8 bits of mantissa, their sum is W to its last bit), the
 // tensor-core product h [w1; w2; w3]^T has exact products and 32-bit sums: the router's logits in 32-bit, at the product's speed.
 extern "C" int imparo_moe_pick(const float* logits, int n_rows, int experts, int parts, int top, int softmax_scores, int renormalise,
-                               int groups, int keep, float renorm_eps, float weight_scale, int out_stride, int* ids, float* wts,
-                               cudaStream_t stream) {
+                               int groups, int keep, int group_pair, const float* correction, float renorm_eps, float weight_scale,
+                               int out_stride, int* ids, float* wts, float* extra_out, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
-    if (!pick_args_ok(experts, top, groups, keep, out_stride) || parts < 1 || parts > 4) return -2;
+    if (!pick_args_ok(experts, top, groups, keep, out_stride, softmax_scores, correction) || parts < 1 || parts > 4) return -2;
     launch(moe_pick_kernel, dim3((n_rows + 3) / 4), dim3(128), pick_smem_bytes(experts, groups), stream, logits, n_rows, experts,
-           parts, top, softmax_scores, renormalise, groups, keep, renorm_eps, weight_scale, out_stride, ids, wts);
+           experts + (extra_out != nullptr ? 1 : 0), parts, top, softmax_scores, renormalise, groups, keep, group_pair, correction,
+           renorm_eps, weight_scale, out_stride, ids, wts, extra_out);
     IMPARO_CHECK_LAUNCH();
     return 0;
 }
 
-// mid: [n_rows * top, ff] in dtype; out float32 [n_rows, width].  Two launches.
+constexpr size_t ROWS_SMEM_MOST = 160 * 1024;
+
+template <typename K>
+static int rows_smem(K kern, size_t smem, size_t* allowed) {
+    if (smem <= 48 * 1024 || smem <= *allowed) return 0;
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ROWS_SMEM_MOST);
+    if (e != cudaSuccess) return (int)e;
+    *allowed = ROWS_SMEM_MOST;
+    return 0;
+}
+
+template <typename T>
+static int moe_rows_launch(const void* h, const void* w_gu, const void* w_down, const int* ids, const float* wts, int n_rows, int width,
+                           int ff, int top, int experts, int weight_input, int gated, int act, float limit, void* mid, float* out,
+                           const void* s_up, const void* s_down, int s_ff, void* s_mid, float* s_out, cudaStream_t stream) {
+    const bool shared = s_up != nullptr;
+    const int tiles = shared ? (n_rows + SHARED_ROWS - 1) / SHARED_ROWS : 0, rows = n_rows < SHARED_ROWS ? n_rows : SHARED_ROWS;
+    const int most_ff = shared && s_ff > ff ? s_ff : ff;
+    size_t smem1 = (size_t)width * 4, smem2 = (size_t)ff * 4;
+    if (shared) {
+        const size_t a = (size_t)rows * width * sizeof(T), b = (size_t)rows * s_ff * sizeof(T);
+        smem1 = smem1 > a ? smem1 : a;
+        smem2 = smem2 > b ? smem2 : b;
+    }
+    if (smem1 > ROWS_SMEM_MOST || smem2 > ROWS_SMEM_MOST) return -25;
+    static size_t allowed1 = 0, allowed2 = 0;
+    int rc = rows_smem(moe_rows_up_kernel<T>, smem1, &allowed1);
+    if (rc == 0) rc = rows_smem(moe_rows_down_kernel<T>, smem2, &allowed2);
+    if (rc) return rc;
+    SharedRows up = {}, down = {};
+    if (shared) {
+        up = {s_up, s_ff, width, s_mid};
+        down = {s_down, width, s_ff, s_out};
+    }
+    launch(moe_rows_up_kernel<T>, dim3(tiles + n_rows * top, (most_ff + 31) / 32), dim3(256), smem1, stream, (const T*)h, (const T*)w_gu,
+           ids, wts, n_rows, width, ff, top, experts, weight_input, gated, act, limit, (T*)mid, up);
+    IMPARO_CHECK_LAUNCH();
+    launch(moe_rows_down_kernel<T>, dim3(tiles + n_rows, (width + 31) / 32), dim3(256), smem2, stream, (const T*)mid, (const T*)w_down,
+           ids, wts, n_rows, width, ff, top, experts, weight_input, out, down, (const T*)s_mid);
+    IMPARO_CHECK_LAUNCH();
+    return 0;
+}
+
+// gated = 1: w_gu [experts, 2 ff, width], act one of gated_act's kinds (with limit); gated = 0: w_gu [experts, ff, width], act one
+// of plain_act's.  mid: [n_rows * top, ff] in dtype; out float32 [n_rows, width].  With s_up (needs gated = 0): an expert that
+// every row uses, s_up [s_ff, width] and s_down [width, s_ff], runs in the same launches: s_mid [n_rows, s_ff] in dtype, s_out
+// float32 [n_rows, width] receives its output, unweighted.  Two launches.
 extern "C" int imparo_moe_rows(const void* h, const void* w_gu, const void* w_down, int dtype, const int* ids, const float* wts,
-                               int n_rows, int width, int ff, int top, int experts, int weight_input, int act, float limit,
-                               void* mid, float* out, cudaStream_t stream) {
+                               int n_rows, int width, int ff, int top, int experts, int weight_input, int gated, int act, float limit,
+                               void* mid, float* out, const void* s_up, const void* s_down, int s_ff, void* s_mid, float* s_out,
+                               cudaStream_t stream) {
     if (n_rows <= 0) return 0;
-    if ((size_t)width * 4 > 48 * 1024 || (size_t)ff * 4 > 48 * 1024) return -25;
-    dim3 g1(n_rows * top, (ff + 31) / 32), g2(n_rows, (width + 31) / 32);
-    if (dtype == IMPARO_DT_F32) {
-        launch(moe_rows_up_kernel<float>, g1, dim3(256), (size_t)width * 4, stream, (const float*)h, (const float*)w_gu, ids, wts, width,
-               ff, top, experts, weight_input, act, limit, (float*)mid);
-        IMPARO_CHECK_LAUNCH();
-        launch(moe_rows_down_kernel<float>, g2, dim3(256), (size_t)ff * 4, stream, (const float*)mid, (const float*)w_down, ids, wts,
-               width, ff, top, experts, weight_input, out);
-    } else if (dtype == IMPARO_DT_BF16) {
-        launch(moe_rows_up_kernel<__nv_bfloat16>, g1, dim3(256), (size_t)width * 4, stream, (const __nv_bfloat16*)h,
-               (const __nv_bfloat16*)w_gu, ids, wts, width, ff, top, experts, weight_input, act, limit, (__nv_bfloat16*)mid);
-        IMPARO_CHECK_LAUNCH();
-        launch(moe_rows_down_kernel<__nv_bfloat16>, g2, dim3(256), (size_t)ff * 4, stream, (const __nv_bfloat16*)mid,
-               (const __nv_bfloat16*)w_down, ids, wts, width, ff, top, experts, weight_input, out);
-    } else return -1;
+    if (s_up != nullptr && (gated || s_down == nullptr || s_ff < 1 || s_mid == nullptr || s_out == nullptr)) return -2;
+    if (dtype == IMPARO_DT_F32)
+        return moe_rows_launch<float>(h, w_gu, w_down, ids, wts, n_rows, width, ff, top, experts, weight_input, gated, act, limit, mid, out,
+                                      s_up, s_down, s_ff, s_mid, s_out, stream);
+    if (dtype == IMPARO_DT_BF16)
+        return moe_rows_launch<__nv_bfloat16>(h, w_gu, w_down, ids, wts, n_rows, width, ff, top, experts, weight_input, gated, act, limit,
+                                              mid, out, s_up, s_down, s_ff, s_mid, s_out, stream);
+    return -1;
+}
+
+// out[r, :] = (accumulate: its old value +) sum_k pair_out[r * top + k, :] (+ extra_w[r] * extra[r, :]); copy: the result rounded
+// to bfloat16, or null.
+extern "C" int imparo_moe_sum(const float* pair_out, int n_rows, int width, int top, const float* extra, const float* extra_w,
+                              int accumulate, float* out, void* copy, cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    if (top < 0 || (extra != nullptr && extra_w == nullptr)) return -2;
+    const SumTail tail = {extra, extra_w, accumulate, (__nv_bfloat16*)copy};
+    const bool vec = width % 4 == 0 && (((uintptr_t)pair_out | (uintptr_t)extra | (uintptr_t)out | (uintptr_t)copy) & 15) == 0;
+    const size_t total = (size_t)n_rows * width / (vec ? 4 : 1);
+    const dim3 grid((unsigned)((total + 255) / 256 > 4096 ? 4096 : (total + 255) / 256));
+    if (vec) launch(moe_sum_pairs_kernel<true>, grid, dim3(256), 0, stream, pair_out, n_rows, width, top, out, tail);
+    else launch(moe_sum_pairs_kernel<false>, grid, dim3(256), 0, stream, pair_out, n_rows, width, top, out, tail);
     IMPARO_CHECK_LAUNCH();
     return 0;
 }
 
 // scratch_i: int32 [n_pairs + experts + 1 + 1 + 3 * max_tiles], max_tiles = n_pairs / 32 + experts; pair_out float32
-// [n_pairs, width]; mid [n_pairs, ff] in dtype; out float32 [n_rows, width].  Four launches.
+// [n_pairs, width]; mid [n_pairs, ff] in dtype; out float32 [n_rows, width]; gated, act, limit as above; extra, extra_w,
+// accumulate, copy as for imparo_moe_sum.  Four launches.
 extern "C" int imparo_moe_grouped(const void* h, const void* w_gu, const void* w_down, int dtype, const int* ids, const float* wts,
-                                  int n_rows, int width, int ff, int top, int experts, int weight_input, int act, float limit,
-                                  void* mid, float* pair_out, int* scratch_i, float* out, cudaStream_t stream) {
+                                  int n_rows, int width, int ff, int top, int experts, int weight_input, int gated, int act,
+                                  float limit, void* mid, float* pair_out, int* scratch_i, const float* extra, const float* extra_w,
+                                  int accumulate, float* out, void* copy, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
     const int n_pairs = n_rows * top;
     const int max_tiles = n_pairs / GM + experts;
@@ -720,23 +967,19 @@ extern "C" int imparo_moe_grouped(const void* h, const void* w_gu, const void* w
     dim3 g1(max_tiles, (ff + GN - 1) / GN), g2(max_tiles, (width + GN - 1) / GN);
     if (dtype == IMPARO_DT_F32) {
         launch(moe_group_up_kernel<float>, g1, dim3(256), 0, stream, (const float*)h, (const float*)w_gu, (const int*)sorted,
-               (const int*)plan, wts, width, ff, top, weight_input, act, limit, (float*)mid);
+               (const int*)plan, wts, width, ff, top, weight_input, gated, act, limit, (float*)mid);
         IMPARO_CHECK_LAUNCH();
         launch(moe_group_down_kernel<float>, g2, dim3(256), 0, stream, (const float*)mid, (const float*)w_down, (const int*)sorted,
                (const int*)plan, wts, width, ff, weight_input, pair_out);
     } else if (dtype == IMPARO_DT_BF16) {
         launch(moe_group_up_kernel<__nv_bfloat16>, g1, dim3(256), 0, stream, (const __nv_bfloat16*)h, (const __nv_bfloat16*)w_gu,
-               (const int*)sorted, (const int*)plan, wts, width, ff, top, weight_input, act, limit, (__nv_bfloat16*)mid);
+               (const int*)sorted, (const int*)plan, wts, width, ff, top, weight_input, gated, act, limit, (__nv_bfloat16*)mid);
         IMPARO_CHECK_LAUNCH();
         launch(moe_group_down_kernel<__nv_bfloat16>, g2, dim3(256), 0, stream, (const __nv_bfloat16*)mid, (const __nv_bfloat16*)w_down,
                (const int*)sorted, (const int*)plan, wts, width, ff, weight_input, pair_out);
     } else return -1;
     IMPARO_CHECK_LAUNCH();
-    const size_t total = (size_t)n_rows * width;
-    launch(moe_sum_pairs_kernel, dim3((unsigned)((total + 255) / 256 > 4096 ? 4096 : (total + 255) / 256)), dim3(256), 0, stream,
-           (const float*)pair_out, n_rows, width, top, out);
-    IMPARO_CHECK_LAUNCH();
-    return 0;
+    return imparo_moe_sum(pair_out, n_rows, width, top, extra, extra_w, accumulate, out, copy, stream);
 }
 
 extern "C" int imparo_gemm_prefill_grouped(const void* x, int ldx, const void* w, int n_groups, void* out, int ldo, int m_tiles,
@@ -744,14 +987,17 @@ extern "C" int imparo_gemm_prefill_grouped(const void* x, int ldx, const void* w
                                            cudaStream_t stream);
 
 // bfloat16, width and ff multiples of 8, at most 256 experts: rows sorted into tiles of 128 per expert and both products on
-// the tensor-memory kernel (SwiGLU in the first one's epilogue).  m_tiles = n_pairs / 128 + experts; xg bfloat16
+// the tensor-memory kernel (the activation in the first one's epilogue).  m_tiles = n_pairs / 128 + experts; xg bfloat16
 // [m_tiles * 128, width]; mid_g bfloat16 [m_tiles * 128, ff]; out_g float32 [m_tiles * 128, width]; scratch_i int32
-// [n_pairs + m_tiles]; out float32 [n_rows, width].  Five launches.  -25: not a case for this path.
+// [n_pairs + m_tiles]; out float32 [n_rows, width]; gated, act, limit, extra, extra_w, accumulate, copy as above.  Five launches.
+// -25: not a case for this path.
 extern "C" int imparo_moe_tiles(const void* h, const void* w_gu, const void* w_down, const int* ids, const float* wts, int n_rows,
-                                int width, int ff, int top, int experts, int weight_input, int act, float limit, void* xg, void* mid_g,
-                                float* out_g, int* scratch_i, float* out, int* status, cudaStream_t stream) {
+                                int width, int ff, int top, int experts, int weight_input, int gated, int act, float limit, void* xg,
+                                void* mid_g, float* out_g, int* scratch_i, const float* extra, const float* extra_w, int accumulate,
+                                float* out, void* copy, int* status, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
     if (width % 8 != 0 || ff % 8 != 0 || experts > 256) return -25;
+    if (extra != nullptr && extra_w == nullptr) return -2;
     const int n_pairs = n_rows * top;
     const int m_tiles = n_pairs / TILE_ROWS + experts;
     int* slot_of_pair = scratch_i;
@@ -762,12 +1008,14 @@ extern "C" int imparo_moe_tiles(const void* h, const void* w_gu, const void* w_d
     launch(moe_tile_gather_kernel, dim3(n_pairs), dim3(128), 0, stream, (const __nv_bfloat16*)h, (const int*)slot_of_pair, wts, width,
            top, weight_input, (__nv_bfloat16*)xg);
     IMPARO_CHECK_LAUNCH();
-    int rc = imparo_gemm_prefill_grouped(xg, width, w_gu, experts, mid_g, ff, m_tiles, ff, width, 3, act, limit, tile_group, status, stream);
+    int rc = imparo_gemm_prefill_grouped(xg, width, w_gu, experts, mid_g, ff, m_tiles, ff, width, gated ? 3 : 4, act, limit, tile_group,
+                                         status, stream);
     if (rc) return rc;
     rc = imparo_gemm_prefill_grouped(mid_g, ff, w_down, experts, out_g, width, m_tiles, width, ff, 1, 0, 0.f, tile_group, status, stream);
     if (rc) return rc;
+    const SumTail tail = {extra, extra_w, accumulate, (__nv_bfloat16*)copy};
     launch(moe_tile_sum_kernel, dim3(n_rows), dim3(256), 0, stream, (const float*)out_g, (const int*)slot_of_pair, wts, width, top,
-           weight_input, out);
+           weight_input, out, tail);
     IMPARO_CHECK_LAUNCH();
     return 0;
 }

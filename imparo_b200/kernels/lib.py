@@ -93,7 +93,7 @@ def _declare_kernels(lib):
     _declare(lib, "imparo_attention_decode_mma",
              [P, P, P, P, P, P, I, I, I, I, c_float, P, P, P, I, I, I, I, I, I, I, I, P, S])
     _declare(lib, "imparo_attention_decode_mma_capped",
-             [P, P, P, P, P, P, I, I, I, I, c_float, P, P, P, I, I, I, I, I, I, I, I, c_float, P, S])
+             [P, P, P, P, P, P, I, I, I, I, c_float, P, P, P, I, I, I, I, I, I, I, I, c_float, P, P, S])
     _declare(lib, "imparo_attention_decode_mma_grouped",
              [P, P, P, P, P, P, I, I, I, I, c_float, P, P, I, I, I, I, I, I, I, I, c_float, P, S])
     _declare(lib, "imparo_attention_split_combine_sinks", [P, P, P, I, I, I, I, P, I, S])
@@ -102,7 +102,7 @@ def _declare_kernels(lib):
     _declare(lib, "imparo_gemm_bf16_heads", [P, P, P, I, I, I, I, I, I, I, I, S])
     _declare(lib, "imparo_sigmoid_gate", [P, c_int64, P, c_int64, I, I, I, I, S])
     _declare(lib, "imparo_attention_decode_mma_qkv",
-             [P, I, c_int64, P, P, P, I, c_float, P, P, P, P, P, I, I, I, I, c_float, P, P, P, I, I, I, I, I, I, P, S])
+             [P, I, c_int64, P, P, P, I, c_float, P, P, P, P, P, I, I, I, I, c_float, P, P, P, I, I, I, I, I, I, I, P, P, S])
     _declare(lib, "imparo_attention_prefill",
              [P, P, P, P, P, I, P, I, I, I, I, c_float, P, I, I, I, I, P, S])
     _declare(lib, "imparo_attention_prefill_tc",
@@ -137,11 +137,14 @@ def _declare_kernels(lib):
     _declare(lib, "imparo_mamba2_scan", [P, P, P, P, P, P, P, I, I, P, I, I, I, I, P, S])
     _declare(lib, "imparo_mamba2_scan_chunked", [P, P, P, P, P, P, P, I, I, P, I, I, I, I, I, I, P, P, P, P, S])
     _declare(lib, "imparo_gate_group_rmsnorm", [P, P, I, c_int64, P, c_float, P, I, I, I, I, S])
-    _declare(lib, "imparo_moe_route", [P, I, P, I, I, I, I, I, I, I, I, c_float, c_float, I, P, P, P, S])
-    _declare(lib, "imparo_moe_rows", [P, P, P, I, P, P, I, I, I, I, I, I, I, c_float, P, P, S])
-    _declare(lib, "imparo_moe_pick", [P, I, I, I, I, I, I, I, I, c_float, c_float, I, P, P, S])
-    _declare(lib, "imparo_moe_tiles", [P, P, P, P, P, I, I, I, I, I, I, I, c_float, P, P, P, P, P, P, S])
-    _declare(lib, "imparo_moe_grouped", [P, P, P, I, P, P, I, I, I, I, I, I, I, c_float, P, P, P, P, S])
+    _declare(lib, "imparo_moe_route", [P, I, P, I, I, I, I, I, I, I, I, I, P, c_float, c_float, I, P, P, P, P, S])
+    _declare(lib, "imparo_moe_rows", [P, P, P, I, P, P, I, I, I, I, I, I, I, I, c_float, P, P, P, P, I, P, P, S])
+    _declare(lib, "imparo_moe_pick", [P, I, I, I, I, I, I, I, I, I, P, c_float, c_float, I, P, P, P, S])
+    _declare(lib, "imparo_moe_sum", [P, I, I, I, P, P, I, P, P, S])
+    _declare(lib, "imparo_moe_tiles", [P, P, P, P, P, I, I, I, I, I, I, I, I, c_float, P, P, P, P, P, P, I, P, P, P, S])
+    _declare(lib, "imparo_moe_grouped", [P, P, P, I, P, P, I, I, I, I, I, I, I, I, c_float, P, P, P, P, P, I, P, P, S])
+    _declare(lib, "imparo_token_side_gate", [P, P, P, c_int64, I, I, P, P, I, I, I, I, P, P, S])
+    _declare(lib, "imparo_token_side_act", [P, P, c_int64, I, I, P, P, I, I, I, P, P, S])
     _declare(lib, "imparo_linear_attention_recurrent", [P, P, P, c_int64, I, I, P, P, P, P, I, I, P, I, I, I, P, S])
     _declare(lib, "imparo_streams_norm", [P, P, I, P, P, c_float, P, I, I, I, S])
     _declare(lib, "imparo_streams_mix_add", [P, I, P, P, P, P, P, c_float, P, I, I, I, S])
@@ -163,7 +166,7 @@ def _declare_kernels(lib):
     _declare(lib, "imparo_gla_chunked", [P, c_int64, I, I, I, I, I, P, P, P, c_float, I, c_float, P, c_float, P, P, P, I, I, I, P, P, P, P, I, I, I, P, S])
     _declare(lib, "imparo_gla_recurrent", [P, c_int64, I, I, I, I, P, c_float, P, P, P, I, I, P, I, I, I, P, S])
     _declare(lib, "imparo_latent_norm_store", [P, c_int64, I, I, I, I, P, P, c_float, P, P, P, P, I, P, I, I, I, I, P, S])
-    _declare(lib, "imparo_latent_rot_store", [P, c_int64, I, I, I, I, P, c_float, P, I, P, P, P, P, P, I, P, I, I, I, I, P, S])
+    _declare(lib, "imparo_latent_rot_store", [P, c_int64, I, I, I, I, I, P, c_float, P, I, I, c_float, P, P, P, P, P, I, P, I, I, I, I, P, S])
     _declare(lib, "imparo_mlstm_scan", [P, c_int64, I, I, I, I, I, P, P, c_float, c_float, P, P, P, P, P, I, I, I, P, I, I, I, I, P, P, P,
                                         P, S])
     _declare(lib, "imparo_heads_linear", [P, c_int64, P, P, c_int64, P, c_int64, I, I, I, I, I, I, I, I, S])

@@ -360,6 +360,14 @@ def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor,
                                                                x.shape[0], x.shape[1], _stream()), "norm_mean_add_rmsnorm")
             return
         settle(x)
+    pg = _S.pending_gnorm.get(x.data_ptr())
+    if pg is not None:
+        if (rows is None and out.shape == x.shape and pg[3] == 1 and w.numel() == x.shape[1] and w.dtype == torch.float32
+                and x.data_ptr() not in _S.pending):
+            _S.pending_gnorm.pop(x.data_ptr())      # the normed add that was left pending and this norm in one pass
+            _group_norm_add(x, pg, w, eps, out)
+            return
+        settle(x)
     pend = _S.pending.get(x.data_ptr())
     if pend is not None:
         scratch, S, T, N = pend
@@ -433,6 +441,7 @@ def _gemm_lib_ready(device) -> None:
 
 # ---- tcgen05 product ---------------------------------------------------------------------
 EPI_STORE_BF16, EPI_STORE_F32, EPI_ADD_F32, EPI_SWIGLU, EPI_PARTIAL = 0, 1, 2, 3, 4
+EPI_ACT_BF16 = 4            # the persistent product only: one activation, then the bfloat16 store
 _tc_plans = {}
 
 
@@ -568,8 +577,9 @@ def prefill_tc_usable(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swigl
 
 
 def gemm_prefill(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, status: Optional[torch.Tensor] = None,
-                 act: str = "silu", limit: float = 0.0, bias: Optional[torch.Tensor] = None) -> None:
-    """The persistent tensor-core product for many tokens.  epilogue: EPI_STORE_BF16 | EPI_STORE_F32 |
+                 act: str = "silu", limit: float = 0.0, bias: Optional[torch.Tensor] = None, plain: Optional[str] = None) -> None:
+    """The persistent tensor-core product for many tokens.  plain: with EPI_STORE_BF16, one of ACTIVATIONS applied to the product.
+    epilogue: EPI_STORE_BF16 | EPI_STORE_F32 |
     EPI_ADD_F32 (out += x w^T) | EPI_SWIGLU (w = [gate rows; up rows], out = act(x gate^T + b_g, x up^T + b_u) with act one of
     gated_act's kinds, "silu" by default, and bias float32 [2N] or None)."""
     _need(x.is_cuda and w.is_cuda and out.is_cuda, "kernels run on CUDA tensors only (there is no CPU path)")
@@ -591,9 +601,11 @@ def gemm_prefill(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: 
         _cuda(bias)
         _need(epilogue == EPI_SWIGLU and bias.dtype == torch.float32 and bias.numel() == 2 * N and bias.is_contiguous(),
               "gemm_prefill: bias float32 [2N] with the gated epilogue")
+    _need(plain is None or epilogue == EPI_STORE_BF16, "gemm_prefill: a plain activation goes with the bfloat16 store")
+    kind = GATED_ACTIVATIONS[act] if plain is None else ACTIVATIONS[plain]
     _check(_lib.kernels().imparo_gemm_prefill(_ptr(x), x.stride(0), rows_alloc, _ptr(w), _ptr(out), out.stride(0), T, N, K,
-                                              epilogue, GATED_ACTIVATIONS[act], float(limit), _ptr(bias), _ptr(status), _stream()),
-           "gemm_prefill")
+                                              epilogue if plain is None else EPI_ACT_BF16, kind, float(limit), _ptr(bias), _ptr(status),
+                                              _stream()), "gemm_prefill")
 
 
 def linear_swiglu(x, w_gu: torch.Tensor, out: torch.Tensor, status: Optional[torch.Tensor] = None,
@@ -742,7 +754,7 @@ def linear_unfolded(x, w: torch.Tensor, out: torch.Tensor, status: Optional[torc
     Returns `out`, filled; or, when the tensor-core product is cut along K (few tokens), a
     PartialProduct: each split's CTAs store their tile and are done, with no fold across CTAs inside
     the product, and the consumer adds the splits while it reads."""
-    if unfolded_products() and x.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and out.is_contiguous() \
+    if unfolded_products() and x.dtype == torch.bfloat16 and out.dtype in (torch.bfloat16, torch.float32) and out.is_contiguous() \
             and gemm_backend() == "tcgen05" and tc_usable(x, w):
         M, K = x.shape
         N = w.shape[0]
@@ -962,7 +974,8 @@ def split_plan(n_tok: int, nkv: int, upper_context: int, sms: Optional[int] = No
 
 def paged_attention_split(q, k_cache, v_cache, positions, item_of_token, table, page_size, n_pages, window, scale,
                           out, part_acc, part_ml, chunk, n_splits, nh, nkv, hd, status, mma: bool = True,
-                          fresh: int = 0, overlap_prev: bool = False, sink: bool = False, softcap: float = 0.0) -> bool:
+                          fresh: int = 0, overlap_prev: bool = False, sink: bool = False, softcap: float = 0.0,
+                          sink_values: Optional[torch.Tensor] = None) -> bool:
     """Split-key attention (one CTA per key chunk, kv head and query token, then an ordered
     combine).  Returns False, having launched nothing, when the group size is above 8, or when a soft cap on the scores
     (softcap c > 0: c * tanh(score / c)) is asked of the kernel without tensor cores, which has none.
@@ -980,10 +993,12 @@ def paged_attention_split(q, k_cache, v_cache, positions, item_of_token, table, 
     runs beside it instead of after it (and completes after it).
 
     sink: the softmax's denominator counts one more term of score 0 that has no value; it enters in the combine, so
-    the partials are left uncombined by the first kernel and the combine runs as a launch of its own (out is needed)."""
+    the partials are left uncombined by the first kernel and the combine runs as a launch of its own (out is needed).
+    sink_values (float32 [nh], unscaled; tensor-core kernel only): the extra term's score per head; it enters the partial
+    result of the chunk that holds the query's own position, so every way of combining the partials has it."""
     if nh // nkv > 8:
         return False
-    if softcap and not (mma and q.dtype == torch.bfloat16 and hd in (64, 128) and chunk >= 64):
+    if (softcap or sink_values is not None) and not (mma and q.dtype == torch.bfloat16 and hd in (64, 128) and chunk >= 64):
         return False
     if sink:
         _need(out is not None, "paged_attention_split: a sink is added by the combine, which needs out")
@@ -993,7 +1008,8 @@ def paged_attention_split(q, k_cache, v_cache, positions, item_of_token, table, 
         if ok:
             attention_split_combine(part_acc, part_ml, out, q.shape[0] * nh, hd, n_splits, sink=True)
         return ok
-    _cuda(q, k_cache, v_cache, positions, item_of_token, table, out, part_acc, part_ml, status)
+    _cuda(q, k_cache, v_cache, positions, item_of_token, table, out, part_acc, part_ml, status, sink_values)
+    _need(sink_values is None or (sink_values.dtype == torch.float32 and sink_values.numel() == nh), "sink values float32 [heads]")
     use_mma = mma and q.dtype == torch.bfloat16 and hd in (64, 128) and chunk >= 64
     T = q.shape[0]
     _need(q.shape == (T, nh * hd) and (out is None or (out.shape == (T, nh * hd) and out.dtype == q.dtype)),
@@ -1012,8 +1028,8 @@ def paged_attention_split(q, k_cache, v_cache, positions, item_of_token, table, 
         rc = _lib.kernels().imparo_attention_decode_mma_capped(
             _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(positions), _ptr(item_of_token), _ptr(table),
             table.shape[1], page_size, n_pages, int(window or 0), float(scale), _ptr(out), _ptr(part_acc), _ptr(part_ml),
-            T, nh, nkv, hd, int(chunk), int(n_splits), int(fresh), int(bool(overlap_prev)), float(softcap or 0.0), _ptr(status),
-            _stream())
+            T, nh, nkv, hd, int(chunk), int(n_splits), int(fresh), int(bool(overlap_prev)), float(softcap or 0.0),
+            _ptr(sink_values), _ptr(status), _stream())
     else:
         rc = _lib.kernels().imparo_paged_attention_split(
             _ptr(q), _ptr(k_cache), _ptr(v_cache), _code(q), _ptr(positions), _ptr(item_of_token), _ptr(table),
@@ -1027,18 +1043,22 @@ def paged_attention_split(q, k_cache, v_cache, positions, item_of_token, table, 
 
 def attention_decode_from_qkv(qkv, positions, item_of_token, q_w, k_w, inv_freq, n_rot, eps, k_cache, v_cache, table,
                               page_size, n_pages, window, scale, out, part_acc, part_ml, chunk, n_splits, nh, nkv, hd,
-                              status) -> bool:
+                              status, v_from_k: bool = False, sink_values: Optional[torch.Tensor] = None) -> bool:
     """The split-key attention of a step in which every request brings ONE token, straight from the qkv product's
     split partials: the kernel makes its queries itself (sum in split order, per-head norm, rotation) and writes the
     new key and value rows into their pages, so no q/k kernel runs before it.  Returns False, having launched
     nothing, unless qkv is a PartialProduct in bfloat16 with head size 64 or 128 and at most 8 query heads per kv
-    head.  out None: the partial results stay uncombined (linear_of_attention_partials)."""
-    if not isinstance(qkv, PartialProduct) or qkv.dtype != torch.bfloat16 or hd not in (64, 128) or nkv < 1 \
+    head.  out None: the partial results stay uncombined (linear_of_attention_partials).  v_from_k: the product is [q | k], a key
+    head before the rotation is also the value head, and the sums go into the rotation unrounded.  sink_values (float32 [nh]):
+    one more term exp(value) in each head's denominator."""
+    if not isinstance(qkv, PartialProduct) or (qkv.dtype != torch.bfloat16 and not v_from_k) or hd not in (64, 128) or nkv < 1 \
             or nh % nkv or nh // nkv > 8 or chunk < 64:
         return False
     T = qkv.shape[0]
     _cuda(qkv.parts, positions, item_of_token, q_w, k_w, inv_freq, k_cache, v_cache, table, out, part_acc, part_ml, status)
-    _need(tuple(qkv.shape) == (T, (nh + 2 * nkv) * hd), "attention_decode_from_qkv: the product's width is (heads + 2 kv heads) * head size")
+    _need(tuple(qkv.shape) == (T, (nh + (1 if v_from_k else 2) * nkv) * hd),
+          "attention_decode_from_qkv: the product's width is (heads + 2 kv heads) * head size (one kv head less where keys are values)")
+    _need(sink_values is None or (sink_values.is_cuda and sink_values.dtype == torch.float32 and sink_values.numel() == nh), "sink values float32 [heads]")
     _need(positions.dtype == torch.int32 and item_of_token.dtype == torch.int32 and positions.numel() >= T
           and item_of_token.numel() >= T, "positions / item_of_token must be int32 per token")
     _need(q_w is None or (q_w.dtype == torch.float32 and q_w.numel() == hd), "q norm weight must be float32 [head]")
@@ -1058,7 +1078,7 @@ def attention_decode_from_qkv(qkv, positions, item_of_token, q_w, k_w, inv_freq,
         _ptr(qkv.parts), qkv.splits, qkv.stride, _ptr(q_w), _ptr(k_w), _ptr(inv_freq), int(n_rot), float(eps),
         _ptr(k_cache), _ptr(v_cache), _ptr(positions), _ptr(item_of_token), _ptr(table), table.shape[1], page_size, n_pages,
         int(window or 0), float(scale), _ptr(out), _ptr(part_acc), _ptr(part_ml), T, nh, nkv, hd, int(chunk), int(n_splits),
-        _ptr(status), _stream()), "attention_decode_from_qkv")
+        int(bool(v_from_k)), _ptr(sink_values), _ptr(status), _stream()), "attention_decode_from_qkv")
     if out is not None:
         COUNTS["own"] += 1      # partial + combine
     return True
@@ -1280,6 +1300,10 @@ def linear_act(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, kind: str, b
     if (x.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and out.is_contiguous() and gemm_backend() == "tcgen05"
             and tc_usable(x, w)):
         gemm_tc(x, w, out, EPI_STORE_BF16, status, plain=kind, bias=bias)
+        return
+    if kind == "relu2" and bias is None and out.dtype == torch.bfloat16 and prefill_tc_usable(x, w, out):
+        # (an exponential per element costs more in this product's epilogue than a kernel of its own: relu2 only)
+        gemm_prefill(x, w, out, EPI_STORE_BF16, status, plain=kind)
         return
     linear(x, w, out, status=status)
     activation(out, out, kind, bias=bias)
@@ -1647,115 +1671,207 @@ def gate_group_rmsnorm(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, eps: f
 
 
 # ---- routed feed-forward (csrc/kernels/moe.cu) -------------------------------------------------------------------
-def _pick_args(top, ids, wts, n, groups, keep, always):
+def _pick_args(top, ids, wts, n, experts, groups, keep, always, group_score, correction, extra):
+    """-> the arguments the two choosing entry points share, in their order after `renormalise`."""
     stride = int(top) + int(always)
     _need(ids.dtype == torch.int32 and wts.dtype == torch.float32 and ids.numel() >= n * stride and wts.numel() >= n * stride,
           "moe: ids int32 and wts float32 [rows, top + always]")
-    return int(groups), int(keep if keep else groups), stride
+    _need(group_score in ("max", "top2"), "moe: a group's score is 'max' or 'top2'")
+    _need(correction is None or (correction.is_cuda and correction.dtype == torch.float32 and correction.numel() == experts),
+          "moe: correction float32 [experts]")
+    _need(extra is None or (extra.is_cuda and extra.dtype == torch.float32 and extra.numel() >= n), "moe: extra float32 [rows]")
+    return (int(groups), int(keep if keep else groups), int(group_score == "top2"), _ptr(correction)), stride
 
 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, top: int, ids: torch.Tensor, wts: torch.Tensor, softmax: bool = False,
               renormalise: bool = False, logits: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 0,
-              renorm_eps: float = 0.0, weight_scale: float = 1.0, always: int = 0) -> None:
+              renorm_eps: float = 0.0, weight_scale: float = 1.0, always: int = 0, group_score: str = "max",
+              correction: Optional[torch.Tensor] = None, extra: Optional[torch.Tensor] = None) -> None:
     """Router logits W_r h in 32-bit, sigmoid (or softmax) scores, the `top` largest per row: ids int32 [rows, top],
-    wts float32 [rows, top].  logits: float32 scratch [rows, experts] (made here when not given).
-    groups, keep: the experts form `groups` equal groups of neighbours, a group's score is its largest, and only the `keep`
-    best groups' experts can be chosen.  renormalise divides the chosen scores by their sum + renorm_eps; weight_scale
-    multiplies the weights.  always = a: ids and wts are [rows, top + a], the last a entries name experts number
-    experts, experts + 1, ... with weight 1 (experts every row uses, stacked behind the routed ones)."""
+    wts float32 [rows, top].  logits: float32 scratch [rows, rows of w_router] (made here when not given).
+    groups, keep: the experts form `groups` equal groups of neighbours, a group's score is its largest (group_score "max") or
+    the sum of its two largest ("top2"), and only the `keep` best groups' experts can be chosen.  correction (float32 [experts],
+    sigmoid scores): experts and groups are chosen by score + correction, weighted by the score alone.  renormalise divides the
+    chosen scores by their sum + renorm_eps; weight_scale multiplies the weights.  always = a: ids and wts are [rows, top + a],
+    the last a entries name experts number experts, experts + 1, ... with weight 1 (experts every row uses, stacked behind the
+    routed ones).  extra (float32 [rows]): w_router has one more row behind the experts', and extra[r] = sigmoid of its logit."""
     n, width = h.shape
-    E = w_router.shape[0]
+    E = w_router.shape[0] - (0 if extra is None else 1)
     if logits is None:
-        logits = torch.empty(n, E, dtype=torch.float32, device=h.device)
+        logits = torch.empty(n, w_router.shape[0], dtype=torch.float32, device=h.device)
     _cuda(h, w_router, ids, wts, logits)
-    _need(logits.dtype == torch.float32 and logits.numel() >= n * E, "moe_route: logits float32 [rows, experts]")
+    _need(logits.dtype == torch.float32 and logits.numel() >= n * w_router.shape[0], "moe_route: logits float32 [rows, router rows]")
     _need(w_router.dtype == torch.float32 and w_router.shape[1] == width, "moe_route: router float32 [experts, width]")
-    groups, keep, stride = _pick_args(top, ids, wts, n, groups, keep, always)
+    how, stride = _pick_args(top, ids, wts, n, E, groups, keep, always, group_score, correction, extra)
     _check(_lib.kernels().imparo_moe_route(_ptr(h), _code(h), _ptr(w_router), n, width, E, int(top), int(bool(softmax)),
-                                           int(bool(renormalise)), groups, keep, float(renorm_eps), float(weight_scale), stride,
-                                           _ptr(logits), _ptr(ids), _ptr(wts), _stream()), "moe_route")
+                                           int(bool(renormalise)), *how, float(renorm_eps), float(weight_scale), stride,
+                                           _ptr(logits), _ptr(ids), _ptr(wts), _ptr(extra), _stream()), "moe_route")
     COUNTS["own"] += 1
 
 
 def moe_pick(logits: torch.Tensor, experts: int, parts: int, top: int, ids: torch.Tensor, wts: torch.Tensor, softmax: bool = False,
              renormalise: bool = False, groups: int = 1, keep: int = 0, renorm_eps: float = 0.0, weight_scale: float = 1.0,
-             always: int = 0) -> None:
-    """The router's choice from logits a product has made: logits float32 [rows, parts * experts], a logit being the sum of
-    its `parts` entries `experts` apart (a 32-bit router matrix cut into bfloat16 pieces that add up to it to its last bit).
-    groups, keep, renorm_eps, weight_scale, always: as for moe_route."""
+             always: int = 0, group_score: str = "max", correction: Optional[torch.Tensor] = None,
+             extra: Optional[torch.Tensor] = None) -> None:
+    """The router's choice from logits a product has made: logits float32 [rows, parts * columns] (columns: experts, one more
+    with extra), a logit being the sum of its `parts` entries `columns` apart (a 32-bit router matrix cut into bfloat16 pieces
+    that add up to it to its last bit).  The rest as for moe_route."""
     _cuda(logits, ids, wts)
     n = logits.shape[0]
-    _need(logits.dtype == torch.float32 and logits.shape[1] == parts * experts, "moe_pick: logits float32 [rows, parts * experts]")
-    groups, keep, stride = _pick_args(top, ids, wts, n, groups, keep, always)
+    _need(logits.dtype == torch.float32 and logits.shape[1] == parts * (experts + (0 if extra is None else 1)),
+          "moe_pick: logits float32 [rows, parts * columns]")
+    how, stride = _pick_args(top, ids, wts, n, experts, groups, keep, always, group_score, correction, extra)
     _check(_lib.kernels().imparo_moe_pick(_ptr(logits), n, int(experts), int(parts), int(top), int(bool(softmax)),
-                                          int(bool(renormalise)), groups, keep, float(renorm_eps), float(weight_scale), stride,
-                                          _ptr(ids), _ptr(wts), _stream()), "moe_pick")
+                                          int(bool(renormalise)), *how, float(renorm_eps), float(weight_scale), stride,
+                                          _ptr(ids), _ptr(wts), _ptr(extra), _stream()), "moe_pick")
 
 
 MOE_GROUP_FROM = 32          # steps with at least this many (row, choice) pairs per expert on average run grouped by expert
 
 
-def moe_tiles_usable(h: torch.Tensor, w_gu: torch.Tensor) -> bool:
+def _expert_form(w_gu: torch.Tensor, act: str):
+    """(gated, activation code, features) of stacked expert matrices: a gated activation's name says that w_gu holds gate and up
+    rows, a plain one ("plain:" + one of ACTIVATIONS) that it holds up rows alone."""
+    if act.startswith("plain:"):
+        return 0, ACTIVATIONS[act[6:]], w_gu.shape[1]
+    return 1, GATED_ACTIVATIONS[act], w_gu.shape[1] // 2
+
+
+def _sum_tail(n, width, extra, accumulate, copy):
+    """Pointers of what the pairs' sum adds and leaves besides (moe_sum)."""
+    y, w = extra if extra is not None else (None, None)
+    _need(y is None or (y.is_cuda and y.dtype == torch.float32 and y.is_contiguous() and tuple(y.shape) == (n, width)
+                        and w.is_cuda and w.dtype == torch.float32 and w.numel() >= n), "moe: extra = (float32 [rows, width], float32 [rows])")
+    _need(copy is None or (copy.is_cuda and copy.dtype == torch.bfloat16 and copy.is_contiguous() and tuple(copy.shape) == (n, width)),
+          "moe: copy bfloat16 [rows, width]")
+    return _ptr(y), _ptr(w), int(bool(accumulate))
+
+
+def moe_sum(pair_out: torch.Tensor, top: int, out: torch.Tensor, extra=None, accumulate: bool = False,
+            copy: Optional[torch.Tensor] = None) -> None:
+    """out[r] = (accumulate: out[r] +) sum_k pair_out[r * top + k] (+ extra[1][r] * extra[0][r]); copy (bfloat16 [rows, width])
+    receives the rounded result.  pair_out, out, extra float32."""
+    _cuda(pair_out, out)
+    n, width = out.shape
+    _need(pair_out.dtype == torch.float32 and pair_out.numel() >= n * top * width and out.dtype == torch.float32, "moe_sum: float32")
+    tail = _sum_tail(n, width, extra, accumulate, copy)
+    _check(_lib.kernels().imparo_moe_sum(_ptr(pair_out), n, width, int(top), *tail, _ptr(out), _ptr(copy), _stream()), "moe_sum")
+
+
+def moe_tiles_usable(h: torch.Tensor, w_gu: torch.Tensor, act: str = "silu") -> bool:
     """Whether moe_experts_tiles takes these sizes: bfloat16, width and features in multiples of 8, at most 256 experts."""
-    return (h.dtype == torch.bfloat16 and h.shape[1] % 8 == 0 and (w_gu.shape[1] // 2) % 8 == 0 and w_gu.shape[0] <= 256
+    return (h.dtype == torch.bfloat16 and h.shape[1] % 8 == 0 and _expert_form(w_gu, act)[2] % 8 == 0 and w_gu.shape[0] <= 256
             and gemm_backend() == "tcgen05")
 
 
 def moe_experts_tiles(h: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, top: int,
                       weight_input: bool, xg: torch.Tensor, mid_g: torch.Tensor, out_g: torch.Tensor, scratch_i: torch.Tensor,
-                      out: torch.Tensor, status: torch.Tensor, act: str = "silu", limit: float = 0.0) -> None:
+                      out: torch.Tensor, status: torch.Tensor, act: str = "silu", limit: float = 0.0, extra=None,
+                      accumulate: bool = False, copy: Optional[torch.Tensor] = None) -> None:
     """The same result as moe_experts for steps of many rows in bfloat16: the (row, choice) pairs are sorted by expert into
     a buffer in which every expert's rows start at a multiple of 128 (xg, inputs already weighted), and both products run
-    on the persistent tensor-memory kernel in its grouped form (silu(gate) * up in the first one's epilogue).  With
+    on the persistent tensor-memory kernel in its grouped form (the activation in the first one's epilogue).  With
     m_tiles = rows * top // 128 + experts: xg bfloat16 [m_tiles * 128, width], mid_g bfloat16 [m_tiles * 128, ff], out_g
-    float32 [m_tiles * 128, width], scratch_i int32 [rows * top + m_tiles]."""
+    float32 [m_tiles * 128, width], scratch_i int32 [rows * top + m_tiles].  extra, accumulate, copy: as for moe_sum."""
     _cuda(h, w_gu, w_down, ids, wts, xg, mid_g, out_g, scratch_i, out, status)
     n, width = h.shape
-    E, ff2, _ = w_gu.shape
-    ff = ff2 // 2
+    E = w_gu.shape[0]
+    gated, code, ff = _expert_form(w_gu, act)
     m_tiles = n * top // 128 + E
-    _need(moe_tiles_usable(h, w_gu), "moe_experts_tiles: bfloat16, width and features multiples of 8, at most 256 experts")
+    _need(moe_tiles_usable(h, w_gu, act), "moe_experts_tiles: bfloat16, width and features multiples of 8, at most 256 experts")
     _need(w_gu.dtype == h.dtype and w_down.dtype == h.dtype and xg.dtype == h.dtype and mid_g.dtype == h.dtype,
           "moe_experts_tiles: one dtype for h, the experts and the sorted buffers")
+    _need(w_gu.shape[2] == width and tuple(w_down.shape) == (E, width, ff), "moe_experts_tiles: expert shapes")
     _need(xg.numel() >= m_tiles * 128 * width and mid_g.numel() >= m_tiles * 128 * ff and out_g.dtype == torch.float32
           and out_g.numel() >= m_tiles * 128 * width and scratch_i.dtype == torch.int32 and scratch_i.numel() >= n * top + m_tiles,
           "moe_experts_tiles: scratch too small")
     _need(out.dtype == torch.float32 and tuple(out.shape) == (n, width), "moe_experts_tiles: out float32 [rows, width]")
+    tail = _sum_tail(n, width, extra, accumulate, copy)
     _check(_lib.kernels().imparo_moe_tiles(_ptr(h), _ptr(w_gu), _ptr(w_down), _ptr(ids), _ptr(wts), n, width, ff, int(top), E,
-                                           int(bool(weight_input)), GATED_ACTIVATIONS[act], float(limit), _ptr(xg), _ptr(mid_g),
-                                           _ptr(out_g), _ptr(scratch_i), _ptr(out), _ptr(status), _stream()), "moe_tiles")
+                                           int(bool(weight_input)), gated, code, float(limit), _ptr(xg), _ptr(mid_g),
+                                           _ptr(out_g), _ptr(scratch_i), *tail, _ptr(out), _ptr(copy), _ptr(status), _stream()), "moe_tiles")
     COUNTS["own"] += 4
 
 
 def moe_experts(h: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, top: int,
-                weight_input: bool, mid: torch.Tensor, out: torch.Tensor, scratch=None, act: str = "silu", limit: float = 0.0) -> None:
+                weight_input: bool, mid: torch.Tensor, out: torch.Tensor, scratch=None, act: str = "silu", limit: float = 0.0,
+                extra=None, accumulate: bool = False, copy: Optional[torch.Tensor] = None, shared=None) -> None:
     """out[r] = sum_k expert_{ids[r,k]}(wts[r,k] * h[r])  (weight_input) or sum_k wts[r,k] * expert(h[r]).
-    act, limit: the experts' gated activation (gated_act's kinds).
-    w_gu [experts, 2 ff, width] = [gate; up], w_down [experts, width, ff]; mid [rows*top, ff] in h's dtype; out float32
+    act, limit: the experts' activation: gated (gated_act's kinds; w_gu [experts, 2 ff, width] = [gate; up]) or "plain:" + one of
+    ACTIVATIONS (w_gu [experts, ff, width]); w_down [experts, width, ff]; mid [rows*top, ff] in h's dtype; out float32
     [rows, width], overwritten.  scratch = (float32 [rows*top, width], int32 [rows*top + experts + 2 + 3*(rows*top//32 + experts)]):
-    when given, pairs are sorted by expert and run as tiles (steps of many rows); else each pair on its own."""
+    when given, pairs are sorted by expert and run as tiles (steps of many rows) and extra, accumulate, copy are as for moe_sum;
+    else each pair on its own, and shared = (up [s_ff, width], down [width, s_ff], mid [rows, s_ff] in h's dtype, out float32
+    [rows, width]) may add an ungated expert of any size that every row uses: its unweighted output goes to its own tensor."""
     _cuda(h, w_gu, w_down, ids, wts, mid, out)
     n, width = h.shape
-    E, ff2, _ = w_gu.shape
-    ff = ff2 // 2
+    E = w_gu.shape[0]
+    gated, code, ff = _expert_form(w_gu, act)
     _need(w_gu.dtype == h.dtype and w_down.dtype == h.dtype and mid.dtype == h.dtype, "moe_experts: one dtype for h, the experts and mid")
     _need(w_gu.shape[2] == width and tuple(w_down.shape) == (E, width, ff), "moe_experts: expert shapes")
     _need(mid.numel() >= n * top * ff and out.dtype == torch.float32 and tuple(out.shape) == (n, width), "moe_experts: mid / out sizes")
     if scratch is not None:
+        _need(shared is None, "moe_experts: a shared expert rides along pair by pair only")
         pair_out, si = scratch
         _cuda(pair_out, si)
         _need(pair_out.dtype == torch.float32 and pair_out.numel() >= n * top * width and si.dtype == torch.int32
               and si.numel() >= n * top + E + 2 + 3 * (n * top // 32 + E), "moe_experts: grouped scratch too small")
+        tail = _sum_tail(n, width, extra, accumulate, copy)
         _check(_lib.kernels().imparo_moe_grouped(_ptr(h), _ptr(w_gu), _ptr(w_down), _code(h), _ptr(ids), _ptr(wts), n, width, ff, int(top),
-                                                 E, int(bool(weight_input)), GATED_ACTIVATIONS[act], float(limit), _ptr(mid), _ptr(pair_out),
-                                                 _ptr(si), _ptr(out), _stream()),
+                                                 E, int(bool(weight_input)), gated, code, float(limit), _ptr(mid), _ptr(pair_out),
+                                                 _ptr(si), *tail, _ptr(out), _ptr(copy), _stream()),
                "moe_grouped")
         COUNTS["own"] += 3
         return
+    _need(extra is None and not accumulate and copy is None, "moe_experts: pair by pair the result is written as it is (moe_sum adds)")
+    s_up = s_down = s_mid = s_out = None
+    s_ff = 0
+    if shared is not None:
+        s_up, s_down, s_mid, s_out = shared
+        _cuda(s_up, s_down, s_mid, s_out)
+        s_ff = s_up.shape[0]
+        _need(not gated and s_up.dtype == h.dtype and s_down.dtype == h.dtype and s_mid.dtype == h.dtype and s_up.shape[1] == width
+              and tuple(s_down.shape) == (width, s_ff) and s_mid.numel() >= n * s_ff and s_out.dtype == torch.float32
+              and tuple(s_out.shape) == (n, width), "moe_experts: the shared expert's shapes")
     _check(_lib.kernels().imparo_moe_rows(_ptr(h), _ptr(w_gu), _ptr(w_down), _code(h), _ptr(ids), _ptr(wts), n, width, ff, int(top), E,
-                                          int(bool(weight_input)), GATED_ACTIVATIONS[act], float(limit), _ptr(mid), _ptr(out), _stream()),
+                                          int(bool(weight_input)), gated, code, float(limit), _ptr(mid), _ptr(out), _ptr(s_up),
+                                          _ptr(s_down), s_ff, _ptr(s_mid), _ptr(s_out), _stream()),
            "moe_rows")
     COUNTS["own"] += 1
+
+
+# ---- a layer's own token input (csrc/kernels/token_side.cu) ------------------------------------------------------------
+SIDE_GATE_ROWS = 32          # up to this many rows the gate's product, activation and side entry are one launch
+
+
+def token_side_gate(x: torch.Tensor, w: torch.Tensor, table: torch.Tensor, col0: int, ids: torch.Tensor, out: torch.Tensor,
+                    status: torch.Tensor, rows: Optional[torch.Tensor] = None, copy: Optional[torch.Tensor] = None, tmp=None) -> None:
+    """out [rows, dim] = gelu_tanh(x w^T) * table[ids[rows[r]], col0 : col0 + dim] (rows None: row r of x is token r of ids).
+    x: the float32 stream [rows, width]; w [dim, width], table [vocab, columns] and out in one dtype.  Few rows: one kernel on x
+    itself.  Many: the product from `copy` (x in the dtype of w; None: made here from x through tmp("copy")) into tmp("product")
+    (float32 [rows, dim]), then one kernel."""
+    _cuda(x, w, table, ids, out, status, rows, copy)
+    settle(x)
+    n, width = x.shape
+    dim = w.shape[0]
+    _need(x.dtype == torch.float32 and w.shape[1] == width and tuple(out.shape) == (n, dim) and out.dtype == w.dtype == table.dtype
+          and table.dim() == 2 and 0 <= col0 and col0 + dim <= table.shape[1], "token_side_gate: shapes and dtypes")
+    _need(ids.dtype == torch.int32 and (rows is None or (rows.dtype == torch.int32 and rows.numel() >= n)), "token_side_gate: int32 ids and rows")
+    _need(rows is not None or ids.numel() >= n, "token_side_gate: a token per row")
+    if n <= SIDE_GATE_ROWS or tmp is None:
+        _check(_lib.kernels().imparo_token_side_gate(_ptr(x), _ptr(w), _ptr(table), table.stride(0), int(col0), _code(w), _ptr(ids),
+                                                     _ptr(rows), n, width, dim, table.shape[0], _ptr(out), _ptr(status), _stream()),
+               "token_side_gate")
+        return
+    if w.dtype == torch.float32:
+        copy = x
+    elif copy is None:
+        copy = tmp("copy")
+        cast_rows(x, copy)
+    z = tmp("product")
+    linear(copy, w, z, status=status)
+    _check(_lib.kernels().imparo_token_side_act(_ptr(z), _ptr(table), table.stride(0), int(col0), _code(w), _ptr(ids), _ptr(rows), n,
+                                                dim, table.shape[0], _ptr(out), _ptr(status), _stream()), "token_side_act")
 
 
 # ---- a stream kept as n copies per token (csrc/kernels/hyper_connections.cu) -----------------------------------
@@ -2104,30 +2220,37 @@ def latent_norm_store(proj: torch.Tensor, q_off: int, q_rank: int, c_off: int, c
                                                    _stream()), "latent_norm_store")
 
 
-def latent_rot_store(proj: torch.Tensor, heads: int, dim: int, rot: int, rank: int, wc: torch.Tensor, eps: float,
+def latent_rot_store(proj: torch.Tensor, heads: int, dim: int, rot: int, rank: int, wc: Optional[torch.Tensor], eps: float,
                      inv_freq: Optional[torch.Tensor], n_rot: int, positions, item_of_token, q_plain: torch.Tensor,
-                     q_lat: torch.Tensor, cache: torch.Tensor, table, page_size: int, n_pages: int, status: torch.Tensor) -> None:
+                     q_lat: torch.Tensor, cache: Optional[torch.Tensor], table, page_size: int, n_pages: int, status: torch.Tensor,
+                     interleaved: bool = False, magnitude: float = 1.0, row: Optional[int] = None) -> None:
     """The latent attention's row preparation when a rotated part stands beside the latent.  proj: a 32-bit product's rows
-    [heads x (dim | rot) | rank | rot | ...].  The page row becomes [rms(latent) * wc | turned key part] (rank + rot wide);
-    q_plain [T, heads * dim] gets every head's plain query dimensions, q_lat [T, heads * (rank + rot)] the turned ones in each
-    head's last rot entries.  The turn is the half-split rotation of the first n_rot of the rot dimensions by
-    position * inv_freq (float32 [n_rot / 2])."""
+    [heads x (dim | rot) | rank | rot | ...].  The page row becomes [rms(latent) * wc | turned key part | zeros] (`row` wide,
+    default rank + rot); q_plain [T, heads * dim] gets every head's plain query dimensions, q_lat [T, heads * row] the turned ones
+    behind each head's first rank entries (and zeros behind them).  The turn is the rotation of the first n_rot of the rot
+    dimensions by position * inv_freq (float32 [n_rot / 2]), half-split pairs or interleaved ones, sines and cosines times
+    magnitude.  cache None: only the queries are made (proj [heads x (dim | rot) | ...])."""
     _cuda(wc, positions, item_of_token, q_plain, q_lat, cache, table, status)
     _need(proj.is_cuda, "kernels run on CUDA tensors only (there is no CPU path)")
     T = q_plain.shape[0]
-    _need(proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[0] == T and proj.shape[1] >= heads * (dim + rot) + rank + rot,
-          "latent_rot_store: a float32 product with dense rows [heads * (dim + rot) + rank + rot]")
-    _need(wc.dtype == torch.float32 and wc.numel() == rank, "latent_rot_store: norm weight float32 [rank]")
+    row = rank + rot if row is None else int(row)
+    needs = heads * (dim + rot) + (rank + rot if cache is not None else 0)
+    _need(row >= rank + rot, "latent_rot_store: a row holds rank + rot entries at least")
+    _need(proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[0] == T and proj.shape[1] >= needs,
+          f"latent_rot_store: a float32 product with dense rows of at least {needs}")
+    _need(cache is None or (wc is not None and wc.dtype == torch.float32 and wc.numel() == rank), "latent_rot_store: norm weight float32 [rank]")
     _need(q_plain.is_contiguous() and tuple(q_plain.shape) == (T, heads * dim) and q_lat.is_contiguous()
-          and tuple(q_lat.shape) == (T, heads * (rank + rot)) and q_plain.dtype == q_lat.dtype == cache.dtype, "latent_rot_store: outputs")
+          and tuple(q_lat.shape) == (T, heads * row) and q_plain.dtype == q_lat.dtype
+          and (cache is None or cache.dtype == q_plain.dtype), "latent_rot_store: outputs")
     _need(n_rot == 0 or (inv_freq is not None and inv_freq.is_cuda and inv_freq.dtype == torch.float32 and inv_freq.numel() == n_rot // 2
                          and n_rot % 2 == 0 and n_rot <= rot), "latent_rot_store: rotation table float32 [n_rot / 2]")
-    _need(cache.numel() >= n_pages * page_size * (rank + rot), "cache arena smaller than n_pages")
+    _need(cache is None or cache.numel() >= n_pages * page_size * row, "cache arena smaller than n_pages")
     _need(table.dtype == torch.int32 and table.dim() == 2, "block table must be int32 [items, blocks]")
-    _check(_lib.kernels().imparo_latent_rot_store(_ptr(proj), proj.stride(0), heads, dim, rot, rank, _ptr(wc), float(eps),
-                                                  _ptr(inv_freq) if n_rot else None, int(n_rot), _ptr(positions), _ptr(item_of_token),
-                                                  _ptr(q_plain), _ptr(q_lat), _ptr(cache), _code(q_plain), _ptr(table), table.shape[1],
-                                                  page_size, n_pages, T, _ptr(status), _stream()), "latent_rot_store")
+    _check(_lib.kernels().imparo_latent_rot_store(_ptr(proj), proj.stride(0), heads, dim, rot, rank, row, _ptr(wc), float(eps),
+                                                  _ptr(inv_freq) if n_rot else None, int(n_rot), int(bool(interleaved)), float(magnitude),
+                                                  _ptr(positions), _ptr(item_of_token), _ptr(q_plain), _ptr(q_lat), _ptr(cache),
+                                                  _code(q_plain), _ptr(table), table.shape[1], page_size, n_pages, T, _ptr(status),
+                                                  _stream()), "latent_rot_store")
 
 
 def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor, group: int = 1) -> None:

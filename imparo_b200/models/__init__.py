@@ -5,3 +5,4 @@ from . import negotar  # noqa: F401
 from . import keralix  # noqa: F401
 from . import zepesun  # noqa: F401
 from . import modinex  # noqa: F401
+from . import zinunex  # noqa: F401

@@ -22,8 +22,9 @@ class AttentionMixer(Part):
     (PartSpec), qk_norm (bool, default True: per-head RMS norm of q and k with a weight each; False: none, and
     no norm tensors are declared), bias (bool, default False: True declares optional q/k/v/out biases, used
     when the file carries them), names (optional dict of tensor names), v_head_dim (the value size per head, default
-    head_dim), scale (the factor on q.k, default 1/sqrt(head_dim)), sink (bool, default False: the softmax's denominator
-    counts one more term of score 0 that has no value, p_j = exp(s_j) / (1 + sum exp(s_j))), softcap (c > 0: the scaled
+    head_dim), scale (the factor on q.k, default 1/sqrt(head_dim)), sink (False; True: the softmax's denominator counts one more
+    term of score 0 that has no value, p_j = exp(s_j) / (1 + sum exp(s_j)); "learned": the term is exp(sink_h), the tensor "sink"
+    [n_heads], a number per head that is not scaled), softcap (c > 0: the scaled
     score becomes c * tanh(score / c)), unit_norm (bool: after the rotation q and k are divided by their own root mean
     square per head, eps as given, no weight), bias "required" (q/k/v biases that the file must carry, added in 32-bit
     before the rotation), v_share ({"role": "source" | "blend", "lambda": tensor name}: the source layer leaves the values
@@ -52,7 +53,7 @@ class AttentionMixer(Part):
              "o": "self_attn.out_proj.weight", "q_norm": "self_attn.q_layernorm.weight",
              "k_norm": "self_attn.k_layernorm.weight", "q_bias": "self_attn.q_proj.bias", "k_bias": "self_attn.k_proj.bias",
              "v_bias": "self_attn.v_proj.bias", "o_bias": "self_attn.out_proj.bias", "g": "self_attn.gate.weight",
-             "score_bias": "self_attn.score_bias"}
+             "score_bias": "self_attn.score_bias", "sink": "self_attn.sink"}
 
     def __init__(self, params, prefix, rt):
         super().__init__(params, prefix, rt)
@@ -63,6 +64,8 @@ class AttentionMixer(Part):
         self.hd = int(p["head_dim"])
         self.vd = int(p.get("v_head_dim") or self.hd)
         self.sink = bool(p.get("sink", False))
+        self.sink_learned = p.get("sink") == "learned"
+        self.sinks = None
         self.eps = float(p.get("eps", 0.0))
         self.window = int(p["window"]) if p.get("window") else None
         self.qk_norm = bool(p.get("qk_norm", True))
@@ -140,6 +143,8 @@ class AttentionMixer(Part):
             specs.append(WeightSpec(self.prefix + self.v_share["lambda"], ((),), role="vector", init=("uniform", 0.2, 0.8)))
         if self.sigmoid:
             specs.append(WeightSpec(n["score_bias"], ((self.nh,),), role="vector", init=("uniform", -4.0, -1.0)))
+        if self.sink_learned:
+            specs.append(WeightSpec(n["sink"], ((self.nh,),), role="vector", init=("uniform", -1.0, 2.0)))
         if self.gate:
             specs.append(WeightSpec(n["g"], ((self.nh * vd, H),)))
         if self.o_bias_required:
@@ -171,6 +176,8 @@ class AttentionMixer(Part):
             self.b_o = tensors[n["o_bias"]]
         if self.sigmoid:
             self.score_bias = tensors[n["score_bias"]]
+        if self.sink_learned:
+            self.sinks = tensors[n["sink"]].contiguous()
         self.position.bind(tensors)
 
     def cache_specs(self):
@@ -284,12 +291,12 @@ class AttentionMixer(Part):
             if batch.max_tokens_per_item >= 8 and 0 < n1 < batch.n_items:
                 done = ops.attention_prefill(q, kv.k, kv.v, batch.item_row_start[n1:], batch.item_start_pos[n1:],
                                              batch.n_items - n1, table[n1:], kv.page_size, kv.n_pages, self.window, self.scale,
-                                             out, nh, self.nkv, hd, rt.status, sink=self.sink, softcap=self.softcap)
+                                             out, nh, self.nkv, hd, rt.status, sink=self.sink, softcap=self.softcap, sink_values=self.sinks)
                 first_split = n1 if done else T
             elif batch.max_tokens_per_item >= 8:
                 done = ops.attention_prefill(q, kv.k, kv.v, batch.item_row_start, batch.item_start_pos, batch.n_items, table,
                                              kv.page_size, kv.n_pages, self.window, self.scale, out, nh, self.nkv, hd, rt.status,
-                                             sink=self.sink, softcap=self.softcap)
+                                             sink=self.sink, softcap=self.softcap, sink_values=self.sinks)
                 first_split = 0 if done else T
             else:
                 first_split = T
@@ -301,11 +308,12 @@ class AttentionMixer(Part):
                 part_ml = rt.workspace.get("attn_part_ml", (n * nh * n_splits * 2,), torch.float32, reserve=room * 2)
                 done = ops.paged_attention_split(q[:n], kv.k, kv.v, batch.positions[:n], batch.item_of_token[:n], table,
                                                  kv.page_size, kv.n_pages, self.window, self.scale, out[:n], part_acc, part_ml,
-                                                 chunk, n_splits, nh, self.nkv, hd, rt.status, sink=self.sink, softcap=self.softcap)
+                                                 chunk, n_splits, nh, self.nkv, hd, rt.status, sink=self.sink and self.sinks is None,
+                                                 softcap=self.softcap, sink_values=self.sinks)
         if not done:
             ops.attention_any(q, kv.k, kv.v, batch.positions, batch.item_of_token, table, kv.page_size, kv.n_pages, self.window,
                               self.scale, self.sink, out, nh, self.nkv, hd, vd, rt.status, softcap=self.softcap, chunk=self.chunk,
-                              score_bias=self.score_bias)
+                              score_bias=self.score_bias, sink_values=self.sinks)
         if self.prepared and self.gate:
             ops.sigmoid_gate(out, gate)
         ops.linear(out, self.w_o, residual, accumulate=accumulate, status=rt.status)

@@ -7,16 +7,25 @@ from .base import Block, make_part
 
 
 class PreNormResidualBlock(Block):
-    """params: layer (LayerSpec)."""
+    """params: layer (LayerSpec).  feed_forward may be None.  layer.params["after"] (optional): a "stream_op" part that works on
+    the stream behind both sublayers; its forward takes `rows` (which of the step's tokens the stream's rows are) and, when it
+    declares reads_copy, `copy` (the stream rounded to the activation dtype), which a feed-forward that declares leaves_copy
+    writes in the pass that adds its output."""
 
     def __init__(self, params, prefix, rt):
         super().__init__(params, prefix, rt)
         spec = params["layer"]
         self.mixer_norm = make_part("norm", spec.mixer_norm, prefix, rt)
         self.mixer = make_part("mixer", spec.mixer, prefix, rt)
-        self.ff_norm = make_part("norm", spec.feed_forward_norm, prefix, rt)
-        self.ff = make_part("feed_forward", spec.feed_forward, prefix, rt)
-        self.parts = (self.mixer_norm, self.mixer, self.ff_norm, self.ff)
+        self.ff = self.ff_norm = None
+        if spec.feed_forward is not None:
+            self.ff_norm = make_part("norm", spec.feed_forward_norm, prefix, rt)
+            self.ff = make_part("feed_forward", spec.feed_forward, prefix, rt)
+        self.after = make_part("stream_op", spec.params["after"], prefix, rt) if spec.params.get("after") else None
+        self.parts = tuple(p for p in (self.mixer_norm, self.mixer, self.ff_norm, self.ff, self.after) if p is not None)
+        import inspect
+        self._ff_accumulates = self.ff is not None and "accumulate" in inspect.signature(self.ff.forward).parameters
+        self._copies = (self.after is not None and getattr(self.after, "reads_copy", False) and getattr(self.ff, "leaves_copy", False))
         self.graph_safe = all(p.graph_safe for p in self.parts)
         self.picks_rows = True         # forward(only_rows=...) is implemented
 
@@ -49,12 +58,30 @@ class PreNormResidualBlock(Block):
                 return None
             xs = self.rt.workspace.get("stream_picked", (n, x.shape[1]), x.dtype, first="rows")
             ops.gather_rows(x, rows, xs)
-            picked_in = self.ff_norm.forward(xs, tag="normed_ff")
-            self._run(self.ff, xs, lambda: self.ff.forward(picked_in, batch, xs))
+            self._behind_mixer(xs, batch, rows)
             return xs
-        ff_in = self.ff_norm.forward(x, tag="normed_ff")
-        self._run(self.ff, x, lambda: self.ff.forward(ff_in, batch, x))
+        self._behind_mixer(x, batch, None)
         return None
+
+    def _behind_mixer(self, x, batch, rows, probe=None):
+        """The feed-forward and what comes after it.  rows: which of the step's tokens x's rows are (None: all, in order)."""
+        from ..kernels import ops
+        copy = None
+        if self.ff is not None:
+            ff_in = self.ff_norm.forward(x, tag="normed_ff")
+            if probe:
+                probe("ff_norm", ff_in)
+            kw = {"accumulate": True} if self._ff_accumulates else {}
+            if self._copies and self.after.wants_copy(x.shape[0]):
+                copy = self.rt.workspace.get("stream_copy", tuple(x.shape), self.rt.act_dtype, first="tokens" if rows is None else "rows")
+                kw["copy"] = copy
+            if probe:
+                self.ff.forward(ff_in, batch, x, **kw)
+                ops.settle(x)
+            else:
+                self._run(self.ff, x, lambda: self.ff.forward(ff_in, batch, x, **kw))
+        if self.after is not None:
+            self.after.forward(x, batch, rows=rows, **({"copy": copy} if copy is not None else {}))
 
     def _forward_probed(self, x, batch, caches, only_rows):
         """The same block with every stage evaluated and shown to the runtime's probe: the stream
@@ -77,9 +104,7 @@ class PreNormResidualBlock(Block):
             xs = self.rt.workspace.get("stream_picked", (n, x.shape[1]), x.dtype, first="rows")
             ops.gather_rows(x, rows, xs)
             x = xs
-        ff_in = self.ff_norm.forward(x, tag="normed_ff")
-        probe("ff_norm", ff_in)
-        self.ff.forward(ff_in, batch, x)
+        self._behind_mixer(x, batch, rows if only_rows is not None else None, probe)
         ops.settle(x)
         probe("stream_out", x)
         return x if only_rows is not None else None

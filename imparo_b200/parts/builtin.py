@@ -16,7 +16,7 @@ from .norm import RMSNorm
 from .position import NoPosition, RotaryInterleaved, RotaryNeox
 from .shortconv import ShortConvMixer
 from .sidebyside import SideBySideMixer
-from .streamop import StretchEntry
+from .streamop import StretchEntry, TokenSideInput
 
 register_part("mixer", "attention", AttentionMixer, replace=True)
 register_part("mixer", "short_conv", ShortConvMixer, replace=True)
@@ -42,3 +42,4 @@ register_part("mixer", "gated_delta_rule", GatedDeltaRule, replace=True)
 register_part("mixer", "matrix_memory", MatrixMemory, replace=True)
 register_part("block", "sandwich_residual", SandwichResidualBlock, replace=True)
 register_part("mixer", "gated_linear_attention", GatedLinearAttention, replace=True)
+register_part("stream_op", "token_side_input", TokenSideInput, replace=True)

@@ -9,8 +9,11 @@ latent there may be a ROTATED part: every head's query is [dim plain | rot_dim r
 of which the last rot_dim, not normed, are one key part kr that all heads share; the rotated parts of q and kr are turned
 by the position (half-split pairs) and score = scale * (q_plain . k + q_rot . kr).  The cached row is then [c | kr], and
 the latent-space query [U_k^T q_plain | q_rot], so the attention over the cached rows is unchanged; of its result only
-the first kv_rank entries (the weighted sum of the latents) go on to U_v.  The output gate is a number per output element
-or one per head.
+the first kv_rank entries (the weighted sum of the latents) go on to U_v.  The rotation may pair neighbours and may carry a
+magnitude.  The output gate is a number per output element or one per head.  A window keeps only the last positions.
+
+A layer may make no latent of its own (reads): it attends over the rows that an earlier layer of the schedule has cached
+(ScheduleEntry.cache_from), with its own queries, U_k, U_v and window.
 
 Only c (and kr) is cached (one row per position that is key and value at once, PagedKV.values_are_keys).  Because
 q . (U_k c) = (U_k^T q) . c and sum_j p_j U_v c_j = U_v sum_j p_j c_j, the queries are taken into the latent space before
@@ -30,8 +33,10 @@ class LatentAttention(Part):
     """params: hidden, heads, dim, vdim, q_rank (None: queries straight from the input, tensor "q"), kv_rank, scale, eps (of
     the latent norms), sink (bool: a learned number per head in the softmax's denominator), gate (False; True: output gate
     sigmoid(W_g h) per output element; "head": one gate per head), rot_dim (default 0: rotated dimensions per head and of
-    the shared key part; needs q_rank None), position (PartSpec of the rotation over the rot_dim part), names (optional dict
-    of tensor names after the prefix).
+    the shared key part; needs q_rank None), position (PartSpec of the rotation over the rot_dim part), window (None: all earlier
+    positions; w: the last w), reads (bool: no W_dkv; the entry must name another one's cache; needs q_rank None), pad_row (bool,
+    default False: in the bfloat16 path a cached row of more than 32 and not yet 64, or more than 64 and not yet 128, is padded
+    with zeros to 64 or 128, the sizes the tensor-core kernels take), names (optional dict of tensor names after the prefix).
 
     forward(..., accumulate=False) overwrites `residual` (then any float32 [tokens, hidden] buffer)."""
     adds_with_linear = True
@@ -50,13 +55,17 @@ class LatentAttention(Part):
         self.kv_rank = int(p["kv_rank"])
         self.rot_dim = int(p.get("rot_dim") or 0)
         self.row = self.kv_rank + self.rot_dim          # what the cache keeps per position
+        if p.get("pad_row") and rt.act_dtype == torch.bfloat16 and 32 < self.row < 128:
+            self.row = 64 if self.row <= 64 else 128
+        self.window = int(p["window"]) if p.get("window") else None
+        self.reads = bool(p.get("reads", False))
+        if self.reads and self.q_rank is not None:
+            raise ValueError("latent attention: a layer that reads another one's cache takes its queries straight from the input")
         if self.rot_dim and self.q_rank is not None:
             raise ValueError("latent attention: a rotated part needs queries straight from the input (q_rank None)")
         from .base import make_part
         from .spec import PartSpec
         self.position = make_part("position", p.get("position", PartSpec("none")), prefix, rt)
-        if self.position.interleaved or self.position.magnitude != 1.0:
-            raise ValueError("latent attention: the rotated part takes a half-split rotation without a magnitude")
         self.scale = float(p["scale"])
         self.eps = float(p["eps"])
         self.sink = bool(p.get("sink", False))
@@ -77,9 +86,10 @@ class LatentAttention(Part):
                      WeightSpec(n["uq"], ((hd, self.q_rank),))]
         else:
             specs = [WeightSpec(n["q"], ((self.heads * (self.dim + self.rot_dim), H),))]
-        specs += [WeightSpec(n["dkv"], ((self.row, H),)),
-                  WeightSpec(n["dkv_norm"], ((self.kv_rank,),), role="vector", init=("norm",)),
-                  WeightSpec(n["uk"], ((hd, self.kv_rank),)), WeightSpec(n["uv"], ((hv, self.kv_rank),)),
+        if not self.reads:
+            specs += [WeightSpec(n["dkv"], ((self.kv_rank + self.rot_dim, H),)),
+                      WeightSpec(n["dkv_norm"], ((self.kv_rank,),), role="vector", init=("norm",))]
+        specs += [WeightSpec(n["uk"], ((hd, self.kv_rank),)), WeightSpec(n["uv"], ((hv, self.kv_rank),)),
                   WeightSpec(n["o"], ((H, hv),))]
         if self.sink:
             specs.append(WeightSpec(n["sink"], ((self.heads,),), role="vector", init=("uniform", -1.0, 2.0)))
@@ -91,9 +101,9 @@ class LatentAttention(Part):
         n = self.names
         # one product for everything that reads the input: [query latent (or the queries) | key/value latent (| key part) | gate]
         first = tensors[n["dq"]] if self.q_rank is not None else tensors[n["q"]]
-        self.w_in = torch.cat([first, tensors[n["dkv"]]] + ([tensors[n["g"]]] if self.gate else []), dim=0).contiguous()
+        self.w_in = torch.cat([first] + ([] if self.reads else [tensors[n["dkv"]]]) + ([tensors[n["g"]]] if self.gate else []), dim=0).contiguous()
         self.w_o = tensors[n["o"]]
-        self.n_kv = tensors[n["dkv_norm"]]
+        self.n_kv = None if self.reads else tensors[n["dkv_norm"]]
         if self.q_rank is not None:
             self.w_uq, self.n_q = tensors[n["uq"]], tensors[n["dq_norm"]]
         self.position.bind(tensors)
@@ -103,7 +113,7 @@ class LatentAttention(Part):
         self.sinks = tensors[n["sink"]] if self.sink else None
 
     def cache_specs(self):
-        return (PagedKV(1, self.row, None, None, values_are_keys=True),)
+        return (PagedKV(1, self.row, self.window, None, values_are_keys=True),)
 
     def _partials_room(self, upper_context: int, groups: int) -> int:
         """Partial results (per head) that the split-key kernel leaves for this engine's largest step of one-token rows at
@@ -118,6 +128,8 @@ class LatentAttention(Part):
 
     def forward(self, x, batch, caches, residual, accumulate=True):
         kv = caches[0]
+        if kv.writes == self.reads:
+            raise ValueError("latent attention: a layer that makes no latent reads another entry's cache, any other owns one")
         rt, T = self.rt, x.shape[0]
         ws = rt.workspace
         H, R = self.heads, self.row
@@ -139,8 +151,9 @@ class LatentAttention(Part):
             rot = self.position.rotary() if self.rot_dim else None
             inv_freq, n_rot = rot if rot is not None else (None, 0)
             ops.latent_rot_store(proj, H, self.dim, self.rot_dim, self.kv_rank, self.n_kv, self.eps, inv_freq, n_rot,
-                                 batch.positions, batch.item_of_token, q, ql, kv.k, table, kv.page_size, kv.n_pages, rt.status)
-            gate_off = H * (self.dim + self.rot_dim) + R
+                                 batch.positions, batch.item_of_token, q, ql, None if self.reads else kv.k, table, kv.page_size,
+                                 kv.n_pages, rt.status, interleaved=self.position.interleaved, magnitude=self.position.magnitude, row=R)
+            gate_off = H * (self.dim + self.rot_dim) + (0 if self.reads else self.kv_rank + self.rot_dim)
         ops.heads_linear(q, self.w_ukT, ql, out_head=R)
         ol = ws.get("latent_ol", (T, H * R), rt.act_dtype, first="tokens")
         done = False
@@ -153,7 +166,7 @@ class LatentAttention(Part):
             if batch.max_tokens_per_item >= 8:
                 a = n1 if 0 < n1 < batch.n_items else 0
                 if ops.attention_prefill(ql, kv.k, kv.k, batch.item_row_start[a:], batch.item_start_pos[a:], batch.n_items - a,
-                                         table[a:], kv.page_size, kv.n_pages, None, self.scale, ol, H, 1, R, rt.status,
+                                         table[a:], kv.page_size, kv.n_pages, self.window, self.scale, ol, H, 1, R, rt.status,
                                          sink_values=self.sinks, max_group=128):
                     first_split = a
             done = first_split == 0
@@ -166,10 +179,10 @@ class LatentAttention(Part):
                 part_acc = ws.get("latent_part_acc", (n * H * n_splits * R,), torch.float32, reserve=room * R)
                 part_ml = ws.get("latent_part_ml", (n * H * n_splits * 2,), torch.float32, reserve=room * 2)
                 done = ops.paged_attention_split_shared(ql[:n], kv.k, kv.k, batch.positions[:n], batch.item_of_token[:n], table,
-                                                        kv.page_size, kv.n_pages, None, self.scale, ol[:n], part_acc, part_ml,
+                                                        kv.page_size, kv.n_pages, self.window, self.scale, ol[:n], part_acc, part_ml,
                                                         chunk, n_splits, H, 1, R, rt.status, sink_values=self.sinks)
         if not done:
-            ops.attention_any(ql, kv.k, kv.k, batch.positions, batch.item_of_token, table, kv.page_size, kv.n_pages, None,
+            ops.attention_any(ql, kv.k, kv.k, batch.positions, batch.item_of_token, table, kv.page_size, kv.n_pages, self.window,
                               self.scale, self.sink, ol, H, 1, R, R, rt.status, sink_values=self.sinks)
         o = ws.get("latent_o", (T, hv), rt.act_dtype, first="tokens")
         ops.heads_linear(ol, self.w_uv, o, gate=proj[:, gate_off:] if self.gate else None, x_head=R)

@@ -7,7 +7,7 @@ from typing import Dict, List, Optional, Sequence, Tuple
 import torch
 
 from .base import Part, Runtime, make_part
-from .spec import ModelSpec, PartSpec, WeightSpec
+from .spec import ModelSpec, PartSpec, WeightSpec, keeping_for, reads_as
 
 
 class Model:
@@ -28,7 +28,7 @@ class Model:
             if e.cache_from is not None:
                 mine = self.layers[e.layer].cache_specs()
                 theirs = self.layers[self.schedule[e.cache_from].layer].cache_specs()
-                if mine != theirs:
+                if not all(reads_as(a, b) for a, b in zip(mine, theirs)) or len(mine) != len(theirs):
                     raise ValueError(f"schedule entry {i} reads the cache of entry {e.cache_from}, "
                                      f"but their cache needs differ: {mine} vs {theirs}")
 
@@ -54,13 +54,17 @@ class Model:
 
     # -- cache needs -------------------------------------------------------------------
     def cache_requirements(self) -> List[Tuple[int, Tuple]]:
-        """For every schedule entry that OWNS a cache: (entry index, its cache specs)."""
+        """For every schedule entry that OWNS a cache: (entry index, its cache specs), widened to what the entries that read it
+        still see (a reader's window may be longer than its source's)."""
         out = []
         for i, e in enumerate(self.schedule):
             if e.cache_from is None:
-                specs = self.layers[e.layer].cache_specs()
+                specs = tuple(self.layers[e.layer].cache_specs())
+                for r in self.schedule:
+                    if r.cache_from == i:
+                        specs = tuple(keeping_for(a, b) for a, b in zip(specs, self.layers[r.layer].cache_specs()))
                 if specs:
-                    out.append((i, tuple(specs)))
+                    out.append((i, specs))
         return out
 
     # -- running -----------------------------------------------------------------------

@@ -2,11 +2,13 @@
 
 Router logits z = W_r h in 32-bit; scores sigmoid(z) (or a softmax over the experts); each row uses the `top` experts
 with the largest scores, weighted by those scores (optionally renormalised to sum 1, and times a factor).  The experts may
-form equal groups of neighbours of which only the groups with the best single scores can be chosen from.  An expert is a
-gated feed-forward without biases, W_down act(W_gate u, W_up u) with act(g, u) = silu(g) u, or, with a limit c,
+form equal groups of neighbours of which only the groups with the best single scores (or the best sums of their two largest)
+can be chosen from.  With a correction per expert the choice, of groups and of experts, goes by score + correction; the weights
+are the scores without it.  An expert is a gated feed-forward without biases, W_down act(W_gate u, W_up u) with act(g, u) = silu(g) u, or, with a limit c,
 g' = min(g, c), u' = clamp(u, -c, c): g' sigmoid(1.702 g') (u' + 1); the weight multiplies the expert's input u = w h
 (weight_on "input") or its output (weight_on "output").  The row's result is the sum over its experts, in the order of
-their scores.  A shared expert of the same form runs for every row and is added.
+their scores.  A shared expert of the same form runs for every row and is added, as it is or times sigmoid(W_sg h), one number
+per row.  Experts may have no gate: W_down act(W_up u) with one activation on its own.
 """
 from __future__ import annotations
 
@@ -24,15 +26,21 @@ class RoutedExperts(Part):
     group's score its largest; only the `keep` best groups' experts can be chosen; default: no groups), renorm_eps (added
     to the sum the chosen scores are divided by), weight_scale (a factor on the weights), act ("silu" | "clamped_swish")
     with limit, shared ({"ff", "limit", "names": {gate, up, down}}: an expert of the same form that every row uses with
-    weight 1; with the experts' own size and limit it is stacked behind them and runs in the same launches).
+    weight 1; with the experts' own size and limit it is stacked behind them and runs in the same launches), gated (default
+    True; False: no gate tensors, act is one of ops.ACTIVATIONS, and so is the shared expert), group_score ("max" | "top2": the sum
+    of a group's two largest choice scores), correction (bool: the tensor "correction" [experts]; sigmoid scores only); shared may
+    then name "factor": a tensor [1, hidden] whose sigmoid product with the row multiplies the shared expert's output (ungated
+    experts).
 
     forward(x, batch, residual, accumulate=False) overwrites `residual` (a float32 [rows, hidden] buffer); with
-    accumulate=True the result is added into it (through a buffer of the part's own), times `scale`."""
+    accumulate=True the result is added into it, times `scale`.  copy (ungated experts, with accumulate): an activation-dtype
+    [rows, hidden] tensor that receives the updated rows rounded, in the pass that adds."""
     takes_scale = True
     GROUP_FROM = 65           # steps with at least this many (row, expert) pairs run sorted by expert, in tiles
+    RIDE_BYTES = 128 * 1024   # a shared expert rides along pair by pair while eight of its rows fit a block's shared memory
     TILES_FROM = 256          # and from this many on (bfloat16, aligned sizes) on the tensor-memory product, tiles of 128 rows
 
-    NAMES = {"router": "router", "gate": "e{e}.gate", "up": "e{e}.up", "down": "e{e}.down"}
+    NAMES = {"router": "router", "gate": "e{e}.gate", "up": "e{e}.up", "down": "e{e}.down", "correction": "correction"}
 
     def __init__(self, params, prefix, rt):
         super().__init__(params, prefix, rt)
@@ -58,25 +66,43 @@ class RoutedExperts(Part):
         self.weight_scale = float(p.get("weight_scale", 1.0))
         self.act = p.get("act", "silu")
         self.limit = float(p.get("limit", 0.0))
-        if self.act not in ("silu", "clamped_swish"):
-            raise ValueError(f"routed experts: unknown activation '{self.act}' (silu, clamped_swish)")
+        self.gated = bool(p.get("gated", True))
+        known = ("silu", "clamped_swish") if self.gated else tuple(sorted(ops.ACTIVATIONS))
+        if self.act not in known:
+            raise ValueError(f"routed experts: unknown activation '{self.act}' ({', '.join(known)})")
+        self.form = self.act if self.gated else "plain:" + self.act        # as the expert kernels name it
+        self.group_score = p.get("group_score", "max")
+        if self.group_score not in ("max", "top2"):
+            raise ValueError(f"routed experts: a group's score is 'max' or 'top2', found '{self.group_score}'")
+        self.has_correction = bool(p.get("correction", False))
+        if self.has_correction and self.score != "sigmoid":
+            raise ValueError("routed experts: a correction belongs to sigmoid scores")
         self.shared = dict(p["shared"]) if p.get("shared") else None
         # a shared expert of the experts' own form is one more expert that every row chooses with weight 1
-        self.shared_stacked = (self.shared is not None and int(self.shared["ff"]) == self.ff and self.weight_on == "output"
+        self.shared_stacked = (self.gated and self.shared is not None and int(self.shared["ff"]) == self.ff and self.weight_on == "output"
                                and float(self.shared.get("limit", self.limit)) == self.limit)
+        self.factor_name = prefix + self.shared["factor"] if self.shared and self.shared.get("factor") else None
+        if self.factor_name is not None and self.gated:
+            raise ValueError("routed experts: a shared expert's factor goes with experts without a gate")
         self.names = {k: prefix + v for k, v in {**self.NAMES, **p.get("names", {})}.items()}
-        self.w_router = self.w_gu = self.w_down = None
+        self.w_router = self.w_gu = self.w_down = self.correction = None
         self.w_shared_gu = self.w_shared_down = None
+        # an ungated shared expert without a factor counts once
+        self.leaves_copy = not self.gated
 
     def weight_specs(self):
         n, H, F = self.names, self.hidden, self.ff
         specs = [WeightSpec(n["router"], ((self.experts, H),), role="vector", init=("normal", 0.5))]
+        if self.has_correction:
+            specs.append(WeightSpec(n["correction"], ((self.experts,),), role="vector", init=("uniform", -0.1, 0.1)))
+        gate = lambda name, f: [WeightSpec(name, ((f, H),))] if self.gated else []
         for e in range(self.experts):
-            specs += [WeightSpec(n["gate"].format(e=e), ((F, H),)), WeightSpec(n["up"].format(e=e), ((F, H),)),
-                      WeightSpec(n["down"].format(e=e), ((H, F),))]
+            specs += gate(n["gate"].format(e=e), F) + [WeightSpec(n["up"].format(e=e), ((F, H),)), WeightSpec(n["down"].format(e=e), ((H, F),))]
         if self.shared is not None:
             sn, sf = self._shared_names(), int(self.shared["ff"])
-            specs += [WeightSpec(sn["gate"], ((sf, H),)), WeightSpec(sn["up"], ((sf, H),)), WeightSpec(sn["down"], ((H, sf),))]
+            specs += gate(sn["gate"], sf) + [WeightSpec(sn["up"], ((sf, H),)), WeightSpec(sn["down"], ((H, sf),))]
+            if self.factor_name is not None:
+                specs.append(WeightSpec(self.factor_name, ((1, H),), role="vector", init=("normal", 0.5)))
         return specs
 
     def _shared_names(self):
@@ -86,6 +112,9 @@ class RoutedExperts(Part):
     def bind(self, tensors):
         n = self.names
         self.w_router = tensors[n["router"]]
+        if self.factor_name is not None:                  # one more row: the shared expert's factor comes with the logits
+            self.w_router = torch.cat([self.w_router, tensors[self.factor_name]], dim=0).contiguous()
+        self.correction = tensors[n["correction"]].contiguous() if self.has_correction else None
         # For bfloat16 rows the router's logits come from the tensor-core product: the 32-bit matrix cut into three
         # bfloat16 pieces that add up to it to its last bit, so every product is exact and the sums are 32-bit.
         self.w_router_pieces = None
@@ -99,13 +128,19 @@ class RoutedExperts(Part):
                     break
             self.router_parts = len(pieces)
             self.w_router_pieces = torch.cat(pieces, dim=0).contiguous()
-        # experts stacked: [experts, 2 ff, hidden] = [gate; up] and [experts, hidden, ff]
-        gu = [torch.cat([tensors[n["gate"].format(e=e)], tensors[n["up"].format(e=e)]], dim=0) for e in range(self.experts)]
+        # experts stacked: [experts, 2 ff, hidden] = [gate; up] (ungated: [experts, ff, hidden]) and [experts, hidden, ff]
+        if self.gated:
+            gu = [torch.cat([tensors[n["gate"].format(e=e)], tensors[n["up"].format(e=e)]], dim=0) for e in range(self.experts)]
+        else:
+            gu = [tensors[n["up"].format(e=e)] for e in range(self.experts)]
         down = [tensors[n["down"].format(e=e)] for e in range(self.experts)]
         if self.shared is not None:
             sn = self._shared_names()
-            s_gu, s_down = torch.cat([tensors[sn["gate"]], tensors[sn["up"]]], dim=0), tensors[sn["down"]]
-            if self.shared_stacked:
+            s_down = tensors[sn["down"]]
+            s_gu = torch.cat([tensors[sn["gate"]], tensors[sn["up"]]], dim=0) if self.gated else tensors[sn["up"]]
+            if not self.gated:
+                self.w_shared_gu, self.w_shared_down = s_gu.contiguous(), s_down.contiguous()
+            elif self.shared_stacked:
                 gu.append(s_gu)
                 down.append(s_down)
             else:
@@ -113,13 +148,16 @@ class RoutedExperts(Part):
         self.w_gu = torch.stack(gu).contiguous()
         self.w_down = torch.stack(down).contiguous()
 
-    def _experts(self, x, w_gu, w_down, ids, wts, top, weight_input, limit, out, tag):
-        """One pass of the expert kernels: pair by pair, sorted into small tiles, or on the tensor-memory product."""
+    def _experts(self, x, w_gu, w_down, ids, wts, top, weight_input, limit, out, tag, extra=None, accumulate=False, copy=None,
+                 shared=None):
+        """One pass of the expert kernels: pair by pair, sorted into small tiles, or on the tensor-memory product.  extra: a
+        function that makes (float32 [rows, hidden], float32 [rows]) for the sum's tail (sorted paths only); shared: what rides
+        along pair by pair (ops.moe_experts)."""
         rt, T = self.rt, x.shape[0]
         ws = rt.workspace
-        n_experts, ff = w_gu.shape[0], w_gu.shape[1] // 2
+        n_experts, ff = w_gu.shape[0], w_gu.shape[1] // (2 if self.gated else 1)
         pairs = T * top
-        if pairs >= self.TILES_FROM and ops.moe_tiles_usable(x, w_gu):
+        if pairs >= self.TILES_FROM and ops.moe_tiles_usable(x, w_gu, self.form):
             # many rows in bfloat16: sorted into tiles of 128 rows per expert, both products on the tensor-memory kernel
             rows = (pairs // 128 + n_experts) * 128
             ops.moe_experts_tiles(x, w_gu, w_down, ids, wts, top, weight_input,
@@ -127,31 +165,41 @@ class RoutedExperts(Part):
                                   ws.get(tag + "sorted_mid", (rows, ff), rt.act_dtype),
                                   ws.get(tag + "sorted_out", (rows, self.hidden), torch.float32),
                                   ws.get(tag + "tile_plan", (pairs + rows // 128,), torch.int32), out, rt.status,
-                                  act=self.act, limit=limit)
+                                  act=self.form, limit=limit, extra=extra() if extra else None, accumulate=accumulate, copy=copy)
             return
         mid = ws.get(tag + "mid", (pairs, ff), rt.act_dtype, first="tokens")
-        scratch = None
         if pairs >= self.GROUP_FROM:
             scratch = (ws.get(tag + "pair_out", (pairs, self.hidden), torch.float32, first="tokens"),
                        ws.get(tag + "plan", (pairs + n_experts + 2 + 3 * (pairs // 32 + n_experts),), torch.int32))
-        ops.moe_experts(x, w_gu, w_down, ids, wts, top, weight_input, mid, out, scratch=scratch, act=self.act, limit=limit)
+            ops.moe_experts(x, w_gu, w_down, ids, wts, top, weight_input, mid, out, scratch=scratch, act=self.form, limit=limit,
+                            extra=extra() if extra else None, accumulate=accumulate, copy=copy)
+            return
+        ops.moe_experts(x, w_gu, w_down, ids, wts, top, weight_input, mid, out, act=self.form, limit=limit, shared=shared)
 
-    def forward(self, x, batch, residual, accumulate=False, scale: float = 1.0):
+    def forward(self, x, batch, residual, accumulate=False, scale: float = 1.0, copy=None):
         rt, T = self.rt, x.shape[0]
         ws = rt.workspace
         always = 1 if self.shared_stacked else 0
         chosen = self.top + always
         ids = ws.get("moe_ids", (T, chosen), torch.int32, first="tokens")
         wts = ws.get("moe_wts", (T, chosen), torch.float32, first="tokens")
+        factor = None
+        if self.factor_name is not None:
+            factor = ws.get("moe_factor", (T,), torch.float32, first="tokens")
+        columns = self.w_router.shape[0]
         how = dict(softmax=self.score == "softmax", renormalise=self.renormalise, groups=self.groups, keep=self.keep,
-                   renorm_eps=self.renorm_eps, weight_scale=self.weight_scale, always=always)
+                   renorm_eps=self.renorm_eps, weight_scale=self.weight_scale, always=always, group_score=self.group_score,
+                   correction=self.correction, extra=factor)
         if self.w_router_pieces is not None and x.dtype == torch.bfloat16:
-            logits = ws.get("moe_logits", (T, self.router_parts * self.experts), torch.float32, first="tokens")
+            logits = ws.get("moe_logits", (T, self.router_parts * columns), torch.float32, first="tokens")
             ops.linear(x, self.w_router_pieces, logits, status=rt.status)
             ops.moe_pick(logits, self.experts, self.router_parts, self.top, ids, wts, **how)
         else:
-            ops.moe_route(x, self.w_router, self.top, ids, wts, logits=ws.get("moe_logits", (T, self.experts), torch.float32, first="tokens"),
+            ops.moe_route(x, self.w_router, self.top, ids, wts, logits=ws.get("moe_logits", (T, columns), torch.float32, first="tokens"),
                           **how)
+        if not self.gated:
+            self._forward_ungated(x, residual, ids, wts, factor, accumulate, scale, copy)
+            return
         out = residual if not accumulate else ws.get("moe_out", tuple(residual.shape), torch.float32, first="tokens")
         self._experts(x, self.w_gu, self.w_down, ids, wts, chosen, self.weight_on == "input", self.limit, out, "moe_")
         if self.w_shared_gu is not None:
@@ -167,4 +215,46 @@ class RoutedExperts(Part):
         if accumulate:
             ops.add_scaled(residual, out, scale)
         elif scale != 1.0:
+            ops.scale_rows(out, scale)
+
+    def _forward_ungated(self, x, residual, ids, wts, factor, accumulate, scale, copy):
+        """Experts without a gate.  The shared expert is a dense feed-forward beside the sorted paths and rides along in the
+        pair-by-pair launches; the pass that sums a row's pairs also adds the shared output times its factor, adds into the
+        stream and leaves its rounded copy."""
+        rt, T = self.rt, x.shape[0]
+        ws = rt.workspace
+        through = accumulate and scale != 1.0                # a scaled result goes through a buffer of the part's own
+        add = accumulate and not through
+        out = ws.get("moe_out", tuple(residual.shape), torch.float32, first="tokens") if through else residual
+        has_shared = self.w_shared_gu is not None
+        if has_shared and factor is None:
+            factor = ws.get("moe_ones", (T,), torch.float32, first="tokens")
+            factor.fill_(1.0)
+        y = mid = None
+        if has_shared:
+            s_ff = self.w_shared_gu.shape[0]
+            y = ws.get("moe_shared_out", (T, self.hidden), torch.float32, first="tokens")
+            mid = ws.get("moe_shared_mid", (T, s_ff), rt.act_dtype, first="tokens")
+
+        def dense():
+            if rt.act_dtype == torch.float32:
+                ops.linear(x, self.w_shared_gu, mid)
+                ops.activation(mid, mid, self.act)
+            else:
+                ops.linear_act(x, self.w_shared_gu, mid, self.act, status=rt.status)
+            ops.linear(mid, self.w_shared_down, y, status=rt.status)
+            return y, factor
+        if T * self.top < self.GROUP_FROM:
+            routed = ws.get("moe_routed", (T, self.hidden), torch.float32, first="tokens")
+            ride = has_shared and 8 * max(self.hidden, self.w_shared_gu.shape[0]) * x.element_size() <= self.RIDE_BYTES
+            self._experts(x, self.w_gu, self.w_down, ids, wts, self.top, self.weight_on == "input", self.limit, routed, "moe_",
+                          shared=(self.w_shared_gu, self.w_shared_down, mid, y) if ride else None)
+            extra = (y, factor) if ride else (dense() if has_shared else None)
+            ops.moe_sum(routed, 1, out, extra=extra, accumulate=add, copy=copy if add else None)
+        else:
+            self._experts(x, self.w_gu, self.w_down, ids, wts, self.top, self.weight_on == "input", self.limit, out, "moe_",
+                          extra=dense if has_shared else None, accumulate=add, copy=copy if add else None)
+        if through:
+            ops.add_scaled(residual, out, scale)
+        elif not accumulate and scale != 1.0:
             ops.scale_rows(out, scale)

@@ -33,7 +33,8 @@ class NoPosition(PositionEncoding):
 
 
 class RotaryNeox(PositionEncoding):
-    """params: head_dim, theta, n_rot (default head_dim), wavelength_scaling (optional: factor, low, high, original).
+    """params: head_dim, theta, n_rot (default head_dim), wavelength_scaling (optional: factor, low, high, original),
+    linear_scaling (optional: a factor that divides every frequency).
 
     With wavelength_scaling a pair's frequency f depends on its wavelength l = 2 pi / f: kept where l < original / high,
     f / factor where l > original / low, and between the two (1 - s) f / factor + s f with
@@ -56,6 +57,8 @@ class RotaryNeox(PositionEncoding):
             s = (original / wavelength - low) / (high - low)
             blended = (1.0 - s) * inv / factor + s * inv
             inv = torch.where(wavelength < original / high, inv, torch.where(wavelength > original / low, inv / factor, blended))
+        if params.get("linear_scaling"):
+            inv = inv / float(params["linear_scaling"])
         self.inv_freq = inv.to(torch.float32).to(rt.device)
 
     def rotary(self):

@@ -10,7 +10,7 @@ the cache an earlier entry wrote (the reference's LayerPlan.kv_source).
 """
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Any, Mapping, Optional, Tuple
 
 
@@ -111,6 +111,22 @@ class SlotState:
     (imparo-model/src/lib.rs:205-219 recurrent_layout; :1951-1972 reset at position 0).
     Always kept in 32-bit."""
     shape: Tuple[int, ...]
+
+
+def reads_as(reader, source) -> bool:
+    """Whether an entry with the cache need `reader` can read what an entry with the need `source` keeps: the same rows; how
+    far back each looks may differ."""
+    if isinstance(reader, PagedKV) and isinstance(source, PagedKV):
+        return replace(reader, window=None, chunk=None) == replace(source, window=None, chunk=None)
+    return reader == source
+
+
+def keeping_for(source, reader):
+    """The need `source` widened to what `reader` still sees of it."""
+    if source == reader or not isinstance(source, PagedKV):
+        return source
+    window = None if source.window is None or reader.window is None else max(source.window, reader.window)
+    return replace(source, window=window, chunk=source.chunk if source.chunk == reader.chunk else None)
 
 
 # ---------------------------------------------------------------------------
