@@ -1,0 +1,684 @@
+"""Zinunex on the GPU against the plain implementation (tests/plain/zinunex_plain.py), in 32-bit and bfloat16: each mechanism's
+kernel alone, the replay families (whole, last tokens one by one, portions down to two tokens, mixed batches with pages and slots
+used again), a far position found through the latent and through the rotated key part, just inside and just outside a window and
+through another layer's cache, a far key that is its own value, sinks that hold back the first tokens, long decoding, long portions,
+and greedy generation through Engine.generate, the command line and bin/trace_run."""
+import functools
+import json
+import os
+import subprocess
+import sys
+import tempfile
+
+import numpy as np
+import pytest
+
+from tests import traces
+from tests import zinunex_cases as C
+from tests.plain import zinunex_plain as P
+from tests.plain.lfm2_plain import read_safetensors
+from tests.test_zepesun_gpu import _bf16_round, _dev, _f32, all_errors
+from tests.zinunex_configs import ALL, PAGE
+
+pytestmark = pytest.mark.gpu
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+# Fractions of the largest |logit| of the compared requests.  float32 is the sharp test.  bfloat16: nine places in ten stay
+# within TOL and none leaves WORST (a wrong key, latent, window or expert moves a place by the scale itself).
+TOL = {"float32": 3e-5, "bfloat16": 3e-2}
+WORST = {"float32": 3e-5, "bfloat16": 0.15}
+_tmp = tempfile.TemporaryDirectory(prefix="imparo_b200_zinunex_")
+
+
+def rescale(path):
+    """The drawn matrices are small, and then every token looks alike to the layers.  Matrices are scaled to a standard deviation
+    of 1 / sqrt(columns) (the embedding and the side table to 1), so that tokens, positions, projections, routers and side inputs all
+    weigh in.  Corrections are spread out, so that few of a router's decisions are close calls (which 8-bit rounding may decide the
+    other way), and the routed experts' outputs are halved, so that one such decision does not swamp a place."""
+    import torch
+    from imparo_b200.weights.safetensors_io import write_safetensors
+    out = {}
+    for i, (k, v) in enumerate(sorted(read_safetensors(path).items())):
+        t = torch.as_tensor(np.asarray(v))
+        if v.ndim == 2:
+            std = 1.0 if k in ("embed", "side.embed") else v.shape[1] ** -0.5
+            if ".mlp.e" in k and k.endswith(".down"):
+                std *= 0.5
+            t = (t.float() * (std / max(float(t.float().std(unbiased=False)), 1e-9))).to(torch.bfloat16)
+        elif k.endswith(".correction"):
+            t = torch.as_tensor(np.random.default_rng(i).permutation(len(v)) * 0.4 - 0.2 * len(v), dtype=torch.float32)
+        out[k] = t
+    write_safetensors(path, out, {"format": "pt"})
+
+
+@functools.lru_cache(maxsize=None)
+def model_dir(name, seed=1):
+    from imparo_b200.weights import write_random_model
+    d = os.path.join(_tmp.name, f"{name}_{seed}")
+    write_random_model(d, ALL[name], seed=seed, dtype="bfloat16", norm_jitter=0.3)
+    rescale(os.path.join(d, "model.safetensors"))
+    return d
+
+
+@functools.lru_cache(maxsize=None)
+def weights(name, seed=1):
+    return read_safetensors(os.path.join(model_dir(name, seed), "model.safetensors"))
+
+
+def make_requests(name, lengths, seed=0):
+    rng = np.random.default_rng(seed)
+    return {f"r{i}": rng.integers(0, ALL[name]["vocab"], n).tolist() for i, n in enumerate(lengths)}
+
+
+_plain, _gaps = {}, {}
+CLOSE_CALL = 0.006         # router decisions closer than this (in choice scores) may go the other way under 8-bit rounding
+AFTER = 1                  # and the mixers carry such a place's deviation on to the next ones
+
+
+def plain_logits(name, requests, seed=1):
+    out = {}
+    for rid, toks in requests.items():
+        key = (name, seed, tuple(toks))
+        if key not in _plain:
+            gaps = []
+            _plain[key] = P.forward(ALL[name], weights(name, seed), toks, gaps=gaps)
+            _gaps[key] = np.min(np.stack(gaps), axis=0) if gaps else np.full(len(toks), np.inf)
+        out[rid] = _plain[key]
+    return out
+
+
+def close_calls(name, requests, seed=1):
+    """(request, position) places at which a router decision of the plain implementation was a close call, and the places right
+    after each: bfloat16 may decide them the other way, and another expert's output is another vector altogether."""
+    plain_logits(name, requests, seed)
+    out = set()
+    for rid, toks in requests.items():
+        for p in np.nonzero(_gaps[(name, seed, tuple(toks))] < CLOSE_CALL)[0]:
+            out.update((rid, int(p) + k) for k in range(AFTER + 1))
+    return out
+
+
+def engine_for(name, dtype, steps, parallel=4, page=None, **kw):
+    from imparo_b200.engine import Engine
+    page = page or PAGE[name]
+    max_tokens = traces.max_live_tokens(steps, max(64, page))
+    return Engine(model_dir(name), dtype=dtype, ctx=max_tokens, parallel=parallel, page_size=page,
+                  num_pages=(max_tokens + page - 1) // page, max_step_tokens=max(256, max_tokens), **kw)
+
+
+def check_trace(engine, steps, name, requests, dtype, share=0.1):
+    from tests.gpu_helpers import run_trace
+    ref = plain_logits(name, requests)
+    want = traces.expected(steps, ref)
+    got = run_trace(engine, steps)
+    assert sorted(got) == sorted(want)
+    scale = max(float(np.abs(v).max()) for v in ref.values())
+    errs = all_errors(steps, got, want)
+    if dtype == "bfloat16":
+        skip = close_calls(name, requests)
+        kept = [e for e in errs if (e[1], e[2]) not in skip]
+        assert len(kept) >= 0.4 * len(errs), "most of the places are close calls of a router"
+        errs = kept
+    bad = next((e for e in errs if not e[3] <= WORST[dtype] * scale), None)
+    assert bad is None, (f"first wrong place: step {bad[0]}, request {bad[1]}, position {bad[2]}, "
+                         f"error {bad[3]:.3e} > {WORST[dtype] * scale:.3e}")
+    over = [e for e in errs if not e[3] <= TOL[dtype] * scale]
+    assert len(over) <= share * len(errs), f"{len(over)} of {len(errs)} places beyond {TOL[dtype] * scale:.3e}; the first: {over[0]}"
+    assert engine.cache.n_requests() == 0
+    return got
+
+
+LENGTHS = {"A": [70, 45, 96, 33, 64, 51], "B": [5, 23, 140, 67, 90, 34], "C": [81, 40, 65, 97, 58], "D": [150, 47, 96, 201, 64],
+           "E": [60, 75, 40, 104, 52, 83]}
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", sorted(ALL))
+@pytest.mark.parametrize("family", ["whole", "tail", "portions", "mixed"])
+def test_family(name, dtype, family):
+    reqs = make_requests(name, LENGTHS[name])
+    steps = {"whole": traces.whole, "tail": lambda r: traces.tail_one_by_one(r, tail=44), "portions": traces.portions,
+             "mixed": lambda r: traces.mixed(r, seed=3)}[family](reqs)
+    check_trace(engine_for(name, dtype, steps), steps, name, reqs, dtype)
+    if family == "mixed":
+        assert traces.max_live_tokens(steps) < sum(traces.round_up(len(t), 64) for t in reqs.values())
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["A", "C"])
+def test_cutting_does_not_change_logits_beyond_rounding(name, dtype):
+    from tests.gpu_helpers import run_trace
+    reqs = make_requests(name, [61, 47, 75], seed=5)
+    skip = close_calls(name, reqs) if dtype == "bfloat16" else set()
+    outs = []
+    for build in (traces.whole, traces.tail_one_by_one, traces.portions, lambda r: traces.mixed(r, seed=9)):
+        steps = build(reqs)
+        got = run_trace(engine_for(name, dtype, steps), steps)
+        by_pos, at = {}, {}
+        for s in steps:
+            r = 0
+            for e in s["entries"]:
+                start = at.get(e["id"], 0)
+                for w in e["want"]:
+                    by_pos[(e["id"], start + w)] = got[s["step"]][r]
+                    r += 1
+                at[e["id"]] = start + len(e["tokens"])
+        outs.append(by_pos)
+    keys = (set(outs[1]) & set(outs[0])) - skip
+    assert len(keys) > (90 if dtype == "float32" else 30)
+    scale = max(float(np.abs(v).max()) for v in outs[0].values())
+    tol = (2e-5 if dtype == "float32" else 0.1) * scale
+    for k in keys:
+        for o in outs[1:]:
+            if k in o:
+                assert np.abs(o[k] - outs[0][k]).max() <= tol, k
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["B", "C", "D"])
+def test_long_portions(name, dtype):
+    """Prompts of several hundred tokens, whole and in portions of 71 to 300 tokens beside another request's single tokens:
+    whole tiles of the tensor-core attention, windows that pass over many pages, experts sorted into tiles."""
+    reqs = make_requests(name, [520, 333], seed=13)
+    steps = traces.whole(reqs)
+    check_trace(engine_for(name, dtype, steps), steps, name, reqs, dtype)
+    a, b = reqs["r0"], reqs["r1"]
+    steps, at_a, at_b = [], 0, 0
+    steps.append({"step": 0, "entries": [{"id": "b", "tokens": b[:300], "want": [0, 150, 299]}], "end": []})
+    at_b = 300
+    for n in (300, 129, 20, 71):
+        steps.append({"step": len(steps), "entries": [{"id": "a", "tokens": a[at_a:at_a + n], "want": [0, n // 2, n - 1]},
+                                                     {"id": "b", "tokens": [b[at_b]], "want": [0]}],
+                      "end": ["a"] if at_a + n == 520 else []})
+        at_a += n
+        at_b += 1
+    steps.append({"step": len(steps), "entries": [{"id": "b", "tokens": b[at_b:], "want": [0, len(b) - at_b - 1]}], "end": ["b"]})
+    check_trace(engine_for(name, dtype, steps), steps, name, {"a": a, "b": b}, dtype, share=0.2)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["A", "C"])
+def test_long_decoding(name, dtype):
+    """390 tokens one by one: the caches grow over many pages, the windows pass, readers follow their source's cache."""
+    reqs = make_requests(name, [400], seed=8)
+    steps = traces.tail_one_by_one(reqs, tail=390)
+    check_trace(engine_for(name, dtype, steps), steps, name, reqs, dtype)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", sorted(ALL))
+def test_first_tokens_of_a_sequence(name, dtype):
+    reqs = make_requests(name, [1, 2, 3, 6], seed=11)
+    for build in (traces.whole, lambda r: traces.tail_one_by_one(r, tail=8)):
+        steps = build(reqs)
+        check_trace(engine_for(name, dtype, steps), steps, name, reqs, dtype, share=0.5 if dtype == "bfloat16" else 0.0)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("n_requests", [9, 30, 70])
+def test_many_decoding_requests(n_requests, dtype):
+    """Batches of unequal requests that decode together, each against the plain logits of the request alone: pairs pair by pair
+    with a second block of shared rows, sorted into small tiles and on the tensor-memory tiles; side inputs on both paths."""
+    name = "C"
+    rng = np.random.default_rng(n_requests)
+    reqs = make_requests(name, [int(n) for n in rng.integers(2, 24, n_requests)], seed=n_requests)
+    steps = [{"step": 0, "entries": [{"id": k, "tokens": t[:-2], "want": []} for k, t in reqs.items() if len(t) > 2], "end": []}]
+    for i in (2, 1):
+        steps.append({"step": len(steps), "entries": [{"id": k, "tokens": [t[-i]], "want": [0]} for k, t in reqs.items()],
+                      "end": list(reqs) if i == 1 else []})
+    check_trace(engine_for(name, dtype, steps, parallel=n_requests), steps, name, reqs, dtype)
+
+
+@pytest.mark.parametrize("name", ["A", "D"])
+def test_slots_and_pages_start_clean_when_used_again(name):
+    a = make_requests(name, [50], seed=20)
+    b = {"other": make_requests(name, [37], seed=21)["r0"]}
+    steps = traces.whole(a) + [dict(s, step=s["step"] + 1) for s in traces.portions(b, sizes=(1, 2, 3))]
+    eng = engine_for(name, "float32", steps, parallel=1)       # one slot: it must be reused
+    check_trace(eng, steps, name, dict(a, **b), "float32")
+
+
+# ---- each mechanism's kernel alone ------------------------------------------------------------------------------
+
+def _latent_by_kernels(dtype, m, eps, proj, W, cuts, page, row=None, reader=None, unmap=None):
+    """The latent kernels on one request cut as `cuts`; proj: the 32-bit product [T, q | latent | key part].  row 64 or 128: on the
+    tensor-core kernels.  reader: (sizes, weights, query rows) of a layer that reads the rows this one caches (the result is the
+    reader's).  unmap: pages wholly behind this window are taken out of the table before every cut."""
+    import torch
+    from imparo_b200.kernels import ops
+    from imparo_b200.parts.base import Runtime
+    from imparo_b200.parts.position import RotaryInterleaved
+    tdt = torch.float32 if dtype == "float32" else torch.bfloat16
+    R, Cr = m["rot_dim"], m["kv_rank"]
+    tensor_cores = row is not None
+    row = row or Cr + R
+    T = len(proj)
+    n_blocks = -(-T // page)
+    n_pages = n_blocks + 3
+    table = torch.arange(n_pages - 1, n_pages - 1 - n_blocks, -1, dtype=torch.int32, device="cuda").reshape(1, -1).contiguous()
+    cache = torch.full((n_pages * page * row,), 9.0, dtype=tdt, device="cuda")
+    status = ops.new_status("cuda")
+    rt = Runtime(precision=dtype, device=torch.device("cuda"))
+    rot = RotaryInterleaved({"head_dim": R, "theta": m["rot"]["base"], "scaling": m["rot"].get("scaling")}, "", rt) if R else None
+    how = dict(interleaved=True, magnitude=rot.magnitude if R else 1.0, row=row)
+    inv_freq = rot.inv_freq if R else None
+    layers = [(m, W, proj)] + ([reader] if reader else [])
+    out_all, at = None, 0
+    for n in cuts:
+        pos, iot = _dev(np.arange(at, at + n, dtype=np.int32)), _dev(np.zeros(n, dtype=np.int32))
+        if unmap is not None:
+            table[0, :max(0, at + 1 - unmap) // page] = -1
+        for k, (lm, lW, lrows) in enumerate(layers):
+            H, D, V = lm["heads"], lm["dim"], lm["vdim"]
+            p = _f32(lrows[at:at + n])
+            q = torch.empty(n, H * D, dtype=tdt, device="cuda")
+            ql = torch.full((n, H * row), 3.0, dtype=tdt, device="cuda")
+            ops.latent_rot_store(p, H, D, R, Cr, _f32(W["dkv.norm"]) if k == 0 else None, eps, inv_freq, R, pos, iot, q, ql,
+                                 cache if k == 0 else None, table, page, n_pages, status, **how)
+            ops.heads_linear(q, _dev(lW["uk"].reshape(H, D, Cr).transpose(0, 2, 1), tdt), ql, out_head=row)
+            window = lm["mask"]["size"] if lm.get("mask") else None
+            ol = torch.empty(n, H * row, dtype=tdt, device="cuda")
+            if not tensor_cores:
+                ops.attention_any(ql, cache, cache, pos, iot, table, page, n_pages, window, lm["scale"], False, ol, H, 1, row, row, status)
+            elif n >= 8 and page in (16, 32, 64, 128):
+                assert ops.attention_prefill(ql, cache, cache, _dev(np.array([0, n], dtype=np.int32)), _dev(np.array([at], dtype=np.int32)), 1,
+                                             table, page, n_pages, window, lm["scale"], ol, H, 1, row, status, max_group=128)
+            else:
+                chunk, n_splits = ops.split_plan(n, ops.head_groups(H, 1), table.shape[1] * page)
+                part_acc = torch.empty(n * H * n_splits * row, device="cuda")
+                part_ml = torch.empty(n * H * n_splits * 2, device="cuda")
+                assert ops.paged_attention_split_shared(ql, cache, cache, pos, iot, table, page, n_pages, window, lm["scale"], ol, part_acc,
+                                                        part_ml, chunk, n_splits, H, 1, row, status)
+            o = torch.empty(n, H * V, dtype=tdt, device="cuda")
+            ops.heads_linear(ol, _dev(lW["uv"].reshape(H, V, Cr), tdt), o, x_head=row)
+        if out_all is None:
+            out_all = np.zeros((T, o.shape[1]))
+        out_all[at:at + n] = o.float().cpu().numpy()
+        at += n
+    ops.read_status(status)
+    return out_all
+
+
+def _latent_weights(rng, m, dtype):
+    H, D, V, Cr = m["heads"], m["dim"], m["vdim"], m["kv_rank"]
+    W = {"uk": rng.standard_normal((H * D, Cr)) / np.sqrt(Cr), "uv": rng.standard_normal((H * V, Cr)) / np.sqrt(Cr),
+         "dkv.norm": rng.uniform(0.5, 1.5, Cr)}
+    if dtype == "bfloat16":
+        W.update({k: _bf16_round(W[k]) for k in ("uk", "uv")})
+    return W
+
+
+def _latent_sizes(H, D, R, V, Cr, window=None, scaling=None):
+    m = {"heads": H, "dim": D, "rot_dim": R, "vdim": V, "kv_rank": Cr, "scale": 0.4}
+    if R:
+        m["rot"] = {"base": 300.0, "dims": R}
+        if scaling:
+            m["rot"]["scaling"] = scaling
+    if window:
+        m["mask"] = {"size": window}
+    return m
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("H,D,R,V,Cr,window", [(3, 16, 8, 12, 24, 9), (5, 12, 12, 20, 28, None), (6, 64, 32, 48, 128, 30), (2, 24, 4, 8, 260, 64),
+                                               (2, 16, 64, 8, 512, 17), (1, 7, 0, 5, 9, 1), (4, 8, 16, 8, 16, 70)])
+def test_latent_attention_kernels(dtype, H, D, R, V, Cr, window):
+    """The latent's norm, the rotation of neighbours with scaled frequencies and a magnitude, the cache write, queries taken into
+    the latent space, the windowed attention over the cached rows, the way back: a prompt of 45 tokens, then 30 tokens one by one
+    (pages of 4, those behind the window unmapped)."""
+    rng = np.random.default_rng(H * D + Cr)
+    m = _latent_sizes(H, D, R, V, Cr, window, C.SCALING)
+    W = _latent_weights(rng, m, dtype)
+    proj = rng.standard_normal((75, H * (D + R) + Cr + R)) * 1.5
+    want = C.latent_rows_plain(m, 1e-5, proj, W)
+    got = _latent_by_kernels(dtype, m, 1e-5, proj, W, [45] + [1] * 30, 4, unmap=window)
+    assert np.abs(got - want).max() <= (3e-5 if dtype == "float32" else 3e-2) * np.abs(want).max()
+
+
+@pytest.mark.parametrize("H,D,R,V,Cr,row,page,window", [(16, 32, 32, 16, 96, 128, 16, 40), (12, 16, 16, 24, 48, 64, 32, None), (3, 64, 8, 64, 40, 64, 16, 17),
+                                                        (40, 8, 64, 8, 64, 128, 64, 100), (5, 16, 8, 8, 60, 128, 8, 33), (4, 64, 16, 64, 60, 128, 16, 150)])
+def test_latent_attention_on_tensor_cores(H, D, R, V, Cr, row, page, window):
+    """Cached rows of 64 and 128, full or padded, in bfloat16, with and without a window: prompt portions of 150, 9 and 60 tokens
+    on the tcgen05 kernel with all heads on the one cached row, portions of 3 and single tokens on the split-key kernel with the
+    heads in groups of at most 8; pages of 8 leave everything to the latter; pages behind the window are unmapped."""
+    rng = np.random.default_rng(H * D + Cr)
+    m = _latent_sizes(H, D, R, V, Cr, window, C.SCALING)
+    W = _latent_weights(rng, m, "bfloat16")
+    T = 150 + 9 + 3 + 60 + 20
+    proj = rng.standard_normal((T, H * (D + R) + Cr + R)) * 1.5
+    want = C.latent_rows_plain(m, 1e-5, proj, W)
+    got = _latent_by_kernels("bfloat16", m, 1e-5, proj, W, [150, 9, 3, 60] + [1] * 20, page, row=row, unmap=window)
+    assert np.abs(got - want).max() <= 3e-2 * np.abs(want).max()
+
+
+@pytest.mark.parametrize("dtype,Cr,R,row", [("float32", 24, 8, None), ("bfloat16", 24, 8, None), ("bfloat16", 48, 16, 64), ("bfloat16", 60, 8, 128)])
+@pytest.mark.parametrize("own,other", [(9, 30), (30, 9), (20, 20), (12, None)])
+def test_reading_another_layers_latents(dtype, Cr, R, row, own, other):
+    """A layer with other heads, sizes, matrices and window over the rows another one has cached in the same step and in earlier
+    ones; pages that neither sees are unmapped."""
+    rng = np.random.default_rng(own * 7 + Cr)
+    m = _latent_sizes(4, 16, R, 12, Cr, own, C.SCALING)
+    reader = dict(_latent_sizes(6, 24, R, 20, Cr, other, C.SCALING), scale=0.3)
+    W, Wr = _latent_weights(rng, m, dtype), _latent_weights(rng, reader, dtype)
+    T = 100
+    proj = rng.standard_normal((T, 4 * (16 + R) + Cr + R)) * 1.5
+    queries = rng.standard_normal((T, 6 * (24 + R))) * 1.5
+    want = C.latent_rows_plain(reader, 1e-5, proj, dict(Wr, **{"dkv.norm": W["dkv.norm"]}), queries=queries)
+    got = _latent_by_kernels(dtype, m, 1e-5, proj, W, [40, 2, 13] + [1] * 45, 16, row=row, reader=(reader, Wr, queries),
+                             unmap=None if other is None else max(own, other))
+    assert np.abs(got - want).max() <= (3e-5 if dtype == "float32" else 3e-2) * np.abs(want).max()
+
+
+@pytest.mark.parametrize("through", ["latent", "rotated"])
+@pytest.mark.parametrize("dtype,Cr,R,row", [("float32", 16, 8, None), ("bfloat16", 16, 8, None), ("bfloat16", 48, 16, 64), ("bfloat16", 90, 32, 128)])
+@pytest.mark.parametrize("far,page,window", [(0, 16, None), (15, 16, 16), (16, 16, 17), (3, 4, 33), (31, 8, 64), (127, 32, 300), (128, 64, 45), (200, 16, 128)])
+def test_a_far_position_and_the_windows_edge(dtype, Cr, R, row, far, page, window, through):
+    """One position, before, at or after a page border, outweighs all others for the queries that look for it, through the latent
+    or through the rotated key part alone (where only the right turn by the distance finds it), in a prompt of 600 and in 20 single
+    tokens; with a window the query window - 1 positions behind it still finds it and the next one does not
+    (tests/zinunex_cases.py: far_latent_case)."""
+    H = 12 if row else 2
+    for prompt in (600,) if window is None else (600, far + window):         # (the edge in the prompt, and decoded)
+        m, W, proj, seen, unseen, v_far, want = C.far_latent_case(far, seed=far * 31 + page, T=620, prompt=prompt, C=Cr, R=R, H=H,
+                                                                  through=through, window=window)
+        if dtype == "bfloat16":
+            W = dict(W, uv=_bf16_round(W["uv"]))
+            want = C.latent_rows_plain(m, 1e-5, proj, W)
+        cuts = [600] + [1] * 20 if prompt == 600 else [far + window - 2, 1, 1, 1, 620 - far - window - 1]
+        got = _latent_by_kernels(dtype, m, 1e-5, proj, W, cuts, page, row=row)
+        assert np.abs(got - want).max() <= (3e-5 if dtype == "float32" else 3e-2) * np.abs(want).max()
+        for t in seen:
+            assert np.abs(got[t, :8] - v_far[0]).max() < 0.06 * np.abs(v_far[0]).max()
+        for t in unseen:
+            assert np.abs(got[t] - v_far.reshape(-1)).max() > 0.3 * np.abs(v_far).max()
+
+
+def _attention_by_kernels(dtype, m, rows, sink, cuts, page, how="any"):
+    """Head preparation (keys are values, rotation with divided frequencies), cache write and attention with a sink per head on one
+    request cut as `cuts`; rows: the 32-bit product [T, q | k].  how: "any" (the general kernel), "tc" (tcgen05 for portions, the
+    split-key kernel for single tokens), "fused" (single tokens straight from a product's split partials)."""
+    import torch
+    from imparo_b200.kernels import ops
+    tdt = torch.float32 if dtype == "float32" else torch.bfloat16
+    nh, nkv, hd = m["heads"], m["kv_heads"], m["dim"]
+    T = len(rows)
+    n_blocks = -(-T // page)
+    n_pages = n_blocks + 3
+    table = torch.arange(n_pages - 1, n_pages - 1 - n_blocks, -1, dtype=torch.int32, device="cuda").reshape(1, -1)
+    kc, vc = (torch.zeros(n_pages * page * nkv * hd, dtype=tdt, device="cuda") for _ in range(2))
+    status = ops.new_status("cuda")
+    n_rot = m["rot"]["dims"] if m.get("rot") else 0
+    factor = m["rot"]["scaling"]["factor"] if n_rot and m["rot"].get("scaling") else 1.0
+    inv = _f32([float(m["rot"]["base"]) ** (-2.0 * i / n_rot) / factor for i in range(n_rot // 2)]) if n_rot else None
+    sinks = _f32(sink)
+    out_all, at = np.zeros((T, nh * hd)), 0
+    for n in cuts:
+        pos, iot = _dev(np.arange(at, at + n, dtype=np.int32)), _dev(np.zeros(n, dtype=np.int32))
+        x = _f32(rows[at:at + n])
+        out = torch.empty(n, nh * hd, dtype=tdt, device="cuda")
+        chunk, n_splits = ops.split_plan(n, nkv, table.shape[1] * page)
+        part_acc = torch.empty(n * nh * n_splits * hd, device="cuda")
+        part_ml = torch.empty(n * nh * n_splits * 2, device="cuda")
+        if how == "fused" and n == 1:
+            third = torch.randn_like(x)
+            parts = torch.stack([x * 0.5 - third, third, x * 0.5]).contiguous()
+            prod = ops.PartialProduct(parts, 3, tuple(x.shape), torch.empty_like(x))
+            assert ops.attention_decode_from_qkv(prod, pos, iot, None, None, inv, n_rot, 0.0, kc, vc, table, page, n_pages, None, m["scale"],
+                                                 out, part_acc, part_ml, chunk, n_splits, nh, nkv, hd, status, v_from_k=True,
+                                                 sink_values=sinks)
+        else:
+            q = torch.empty(n, nh * hd, dtype=tdt, device="cuda")
+            ops.qkv_prepare_store(x, None, pos, iot, inv, n_rot, None, None, None, None, q, kc, vc, table, page, n_pages, nh, nkv, hd, hd,
+                                  status, v_from_k=True)
+            if how == "any":
+                ops.attention_any(q, kc, vc, pos, iot, table, page, n_pages, None, m["scale"], True, out, nh, nkv, hd, hd, status, sink_values=sinks)
+            elif n >= 8 and page in (16, 32, 64, 128):
+                assert ops.attention_prefill(q, kc, vc, _dev(np.array([0, n], dtype=np.int32)), _dev(np.array([at], dtype=np.int32)), 1, table, page,
+                                             n_pages, None, m["scale"], out, nh, nkv, hd, status, sink_values=sinks)
+            else:
+                assert ops.paged_attention_split(q, kc, vc, pos, iot, table, page, n_pages, None, m["scale"], out, part_acc, part_ml, chunk, n_splits,
+                                                 nh, nkv, hd, status, sink_values=sinks)
+        out_all[at:at + n] = out.float().cpu().numpy()
+        at += n
+    ops.read_status(status)
+    return out_all
+
+
+FORMS = [("float32", "any"), ("bfloat16", "any"), ("bfloat16", "tc"), ("bfloat16", "fused")]
+
+
+@pytest.mark.parametrize("dtype,how", FORMS)
+@pytest.mark.parametrize("nh,nkv,hd,n_rot", [(4, 2, 16, 16), (6, 1, 8, 4), (3, 3, 24, 10), (1, 1, 12, 0), (8, 2, 64, 64), (8, 1, 64, 20), (4, 4, 128, 128),
+                                             (6, 2, 128, 64), (10, 1, 20, 20)])
+def test_attention_with_keys_as_values_and_sinks(dtype, how, nh, nkv, hd, n_rot):
+    """Grouped heads, partial and whole rotation with divided frequencies, values that are the keys before it, a learned number per
+    head in the denominator: a prompt of 45 tokens, portions of 2 and 17, then 30 tokens one by one."""
+    if how != "any" and hd not in (64, 128):
+        pytest.skip("sizes of the general kernel")
+    rng = np.random.default_rng(hd + nh)
+    m = {"heads": nh, "kv_heads": nkv, "dim": hd, "vdim": hd, "scale": 0.35}
+    if n_rot:
+        m["rot"] = {"base": 500.0, "dims": n_rot, "scaling": {"factor": 2.5}}
+    rows, sink = rng.standard_normal((94, (nh + nkv) * hd)), rng.standard_normal(nh) * 3.0
+    want = C.attention_rows_plain(m, rows, sink)
+    got = _attention_by_kernels(dtype, m, rows, sink, [45, 2, 17] + [1] * 30, 16 if how != "any" else 4, how)
+    assert np.abs(got - want).max() <= (2e-5 if dtype == "float32" else 2.5e-2) * np.abs(want).max()
+
+
+@pytest.mark.parametrize("dtype,how", FORMS)
+@pytest.mark.parametrize("far,page,hd,n_rot", [(0, 16, 64, None), (15, 16, 64, 20), (16, 32, 128, None), (127, 64, 128, 64), (128, 16, 32, None), (63, 8, 24, 12)])
+def test_a_far_key_that_is_its_own_value(dtype, how, far, page, hd, n_rot):
+    """One large key among hundreds of small ones is what the queries that look for it return, unrotated; only the right turn by
+    their distance finds it (tests/zinunex_cases.py: far_key_case)."""
+    if how != "any" and (hd not in (64, 128) or page == 8):
+        pytest.skip("sizes of the general kernel")
+    m, rows, sink, seekers, v_far, want = C.far_key_case(far, hd, seed=far + hd, H=4, G=2, n_rot=n_rot)
+    got = _attention_by_kernels(dtype, m, rows, sink, [600] + [1] * 20, page, how)
+    assert np.abs(got - want).max() <= (3e-5 if dtype == "float32" else 3e-2) * np.abs(want).max()
+    for t in seekers:
+        assert np.abs(got[t, :hd] - v_far).max() < 0.06 * np.abs(v_far).max()
+
+
+@pytest.mark.parametrize("dtype,how", FORMS)
+@pytest.mark.parametrize("hd,H,G", [(64, 4, 2), (128, 8, 1), (16, 5, 1)])
+def test_sinks_hold_back_the_first_tokens(dtype, how, hd, H, G):
+    """Scores near zero and sinks as strong as dozens of keys: leaving the sinks out (or scaling them) shows at every place, most at
+    the first tokens (tests/zinunex_cases.py: sink_case); the first tokens in a prompt and one by one."""
+    if how != "any" and hd not in (64, 128):
+        pytest.skip("sizes of the general kernel")
+    m, rows, sink, want = C.sink_case(hd, seed=hd, H=H, G=G)
+    without = C.attention_rows_plain(m, rows, np.full(H, -50.0))
+    for cuts in ([150], [1] * 12 + [2, 136], [100] + [1] * 50):
+        got = _attention_by_kernels(dtype, m, rows, sink, cuts, 16, how)
+        err = np.abs(got - want).max(axis=1)
+        assert (err <= (2e-5 if dtype == "float32" else 2.5e-2) * np.abs(want).max()).all()
+        assert (err < 0.15 * np.abs(without - want).max(axis=1)).all()
+
+
+@pytest.mark.parametrize("E,top,groups,keep,scale", [(16, 4, 4, 2, 1.5), (6, 2, 3, 2, 1.7), (8, 2, 2, 1, 1.0), (5, 5, 1, 1, 2.0), (3, 2, 3, 3, 3.0),
+                                                     (64, 6, 8, 2, 1.0), (40, 3, 40, 5, 0.5), (1, 1, 1, 1, 2.0)])
+@pytest.mark.parametrize("shift", [0.0, -3.0])
+def test_router_with_correction(E, top, groups, keep, scale, shift):
+    """Sigmoid scores, experts and groups chosen by score + correction (also where all of those are negative), a group's score the
+    sum of its two largest, weights the bare scores times the scale; from the 32-bit kernel and from logits a product made, with
+    and without one more column whose sigmoid goes to each row."""
+    import torch
+    from imparo_b200.kernels import ops
+    rng = np.random.default_rng(E * top)
+    width, T = 48, 37
+    h, wr = _bf16_round(rng.standard_normal((T, width))), rng.standard_normal((E + 1, width)) * 0.3
+    corr = rng.uniform(-0.4, 0.4, E) + shift
+    gaps = []
+    ids_w, wts_w = P.route(h @ wr[:E].T, corr, top, groups, keep, scale, gaps)
+    sure = gaps[0] > 1e-5
+    assert sure.mean() > 0.9
+    for extra in (False, True):
+        rows = E + (1 if extra else 0)
+        ids = torch.zeros(T, top, dtype=torch.int32, device="cuda")
+        wts = torch.zeros(T, top, dtype=torch.float32, device="cuda")
+        fac = torch.zeros(T, device="cuda") if extra else None
+        how = dict(groups=groups, keep=keep, weight_scale=scale, group_score="top2", correction=_f32(corr), extra=fac)
+
+        def check():
+            assert np.array_equal(ids.cpu().numpy()[sure], ids_w[sure])
+            assert np.abs(wts.cpu().numpy() - wts_w)[sure].max() <= 1e-5 * scale
+            if extra:
+                assert np.abs(fac.cpu().numpy() - P.sigmoid(h @ wr[E])).max() <= 1e-5
+        ops.moe_route(_f32(h), _f32(wr[:rows]), top, ids, wts, **how)
+        check()
+        z = h @ wr[:rows].T
+        for parts in (1, 3):
+            ids.zero_(); wts.zero_()
+            logits = z if parts == 1 else np.concatenate([z * 0.5, z * 0.25, z * 0.25], axis=1)
+            ops.moe_pick(_f32(logits), E, parts, top, ids, wts, **how)
+            check()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("T,E,top,ff,width,shared_ff", [(1, 6, 2, 24, 64, 40), (5, 6, 2, 24, 64, 24), (19, 8, 3, 32, 128, 200), (40, 8, 3, 32, 128, 64),
+                                                        (300, 8, 2, 64, 128, 96), (70, 4, 1, 16, 52, None), (150, 12, 3, 80, 256, 80), (7, 3, 2, 13, 41, 27),
+                                                        (90, 3, 2, 13, 41, 27), (11, 4, 2, 24, 64, None), (513, 16, 1, 40, 64, 8)])
+def test_ungated_experts_with_a_shared_one(dtype, T, E, top, ff, width, shared_ff):
+    """The routed feed-forward as a part: squared-relu experts pair by pair (the shared expert in the same launches), sorted into
+    small tiles and on the tensor-memory product (the shared expert beside them), its factor per row, the pass that adds into the
+    stream and leaves the rounded copy; written, added, and added scaled."""
+    import torch
+    from imparo_b200.kernels import ops
+    from imparo_b200.parts.base import Runtime, Workspace
+    from imparo_b200.parts.moe import RoutedExperts
+    tdt = torch.float32 if dtype == "float32" else torch.bfloat16
+    rng = np.random.default_rng(T + E)
+    rnd = (lambda a: a) if dtype == "float32" else _bf16_round
+    g = (2, 1) if E % 2 == 0 and top <= E // 2 else (1, 1)
+    mlp = {"router": {"experts": E, "top": top, "scale": 2.0, "groups": {"count": g[0], "keep": g[1]}}, "expert": {"ff": ff}}
+    W = {"router": rnd(rng.standard_normal((E, width)) * 0.5), "correction": rng.uniform(-0.3, 0.3, E)}
+    for e in range(E):
+        W.update({f"e{e}.up": rnd(rng.standard_normal((ff, width)) / np.sqrt(width) * 1.5), f"e{e}.down": rnd(rng.standard_normal((width, ff)) / np.sqrt(ff))})
+    shared = None
+    if shared_ff:
+        mlp["shared"] = {"ff": shared_ff}
+        shared = {"ff": shared_ff, "factor": "shared.sg"}
+        W.update({"shared.up": rnd(rng.standard_normal((shared_ff, width)) / np.sqrt(width)), "shared.sg": rnd(rng.standard_normal((1, width)) * 0.5),
+                  "shared.down": rnd(rng.standard_normal((width, shared_ff)) / np.sqrt(shared_ff))})
+    h = rnd(rng.standard_normal((T, width)))
+    gaps = []
+    want = P.moe_ff(h, W, "", mlp, gaps)
+    sure = gaps[0] > 1e-4
+    assert sure.mean() > 0.9
+    status = ops.new_status("cuda")
+    rt = Runtime(precision=dtype, device=torch.device("cuda"), status=status, workspace=Workspace(torch.device("cuda")))
+    part = RoutedExperts({"hidden": width, "ff": ff, "experts": E, "top": top, "weight_scale": 2.0, "groups": g[0], "keep": g[1], "group_score": "top2",
+                          "correction": True, "gated": False, "act": "relu2", "shared": shared}, "", rt)
+    part.bind({w.name: _dev(W[w.name], torch.float32 if w.role == "vector" else tdt) for w in part.weight_specs()})
+    tol = (3e-5 if dtype == "float32" else 3e-2) * np.abs(want).max()
+    out = torch.zeros(T, width, device="cuda")
+    part.forward(_dev(h, tdt), None, out)
+    ops.read_status(status)
+    assert np.abs(out.cpu().numpy() - want)[sure].max() <= tol
+    start = rng.standard_normal((T, width))
+    for scale in (1.0, 0.5):
+        base = _f32(start)
+        copy = torch.zeros(T, width, dtype=torch.bfloat16, device="cuda") if dtype == "bfloat16" and scale == 1.0 else None
+        part.forward(_dev(h, tdt), None, base, accumulate=True, scale=scale, copy=copy)
+        assert np.abs(base.cpu().numpy() - start - scale * want)[sure].max() <= tol
+        if copy is not None:
+            assert torch.equal(copy, base.to(torch.bfloat16))
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("T,width,dim,index,L", [(1, 64, 12, 0, 3), (9, 52, 7, 2, 3), (33, 128, 40, 1, 2), (300, 128, 16, 3, 5), (20, 41, 1, 0, 1), (70, 41, 5, 1, 2),
+                                                 (8, 1536, 128, 1, 2), (300, 2048, 64, 0, 1)])
+def test_token_side_input(dtype, T, width, dim, index, L):
+    """The layer's token input as a part, on all rows and on picked ones, settled alone and carried out by the norm that follows."""
+    from types import SimpleNamespace
+    import torch
+    from imparo_b200.kernels import ops
+    from imparo_b200.parts.base import Runtime, Workspace
+    from imparo_b200.parts.streamop import TokenSideInput
+    tdt = torch.float32 if dtype == "float32" else torch.bfloat16
+    rnd = (lambda a: a) if dtype == "float32" else _bf16_round
+    rng = np.random.default_rng(T + width)
+    vocab = 50
+    W = {"side.embed": rnd(rng.standard_normal((vocab, L * dim))), "side.gate": rnd(rng.standard_normal((dim, width)) / np.sqrt(width)),
+         "side.proj": rnd(rng.standard_normal((width, dim)) / np.sqrt(dim)), "side.norm": rng.uniform(0.5, 1.5, width)}
+    x, ids = rng.standard_normal((T, width)) * 2.0, rng.integers(0, vocab, T).astype(np.int32)
+    want = P.token_side(x, W["side.embed"][ids, index * dim:(index + 1) * dim], W, "", 1e-5)
+    status = ops.new_status("cuda")
+    rt = Runtime(precision=dtype, device=torch.device("cuda"), status=status, workspace=Workspace(torch.device("cuda")))
+    part = TokenSideInput({"width": width, "dim": dim, "index": index, "columns": L * dim, "vocab": vocab, "eps": 1e-5, "table": "side.embed"}, "", rt)
+    part.bind({w.name: _dev(W[w.name], torch.float32 if w.role == "vector" else tdt) for w in part.weight_specs()})
+    batch = SimpleNamespace(token_ids=_dev(ids))
+    tol = (2e-5 if dtype == "float32" else 2e-2) * np.abs(want).max()
+    xd = _f32(x)
+    part.forward(xd, batch)
+    ops.settle(xd)
+    assert np.abs(xd.cpu().numpy() - want).max() <= tol
+    xd, w2 = _f32(x), rng.uniform(0.5, 1.5, width)
+    part.forward(xd, batch)
+    normed = torch.empty(T, width, dtype=tdt, device="cuda")
+    ops.rmsnorm(xd, _f32(w2), 1e-6, normed)                          # carries the pending add out
+    assert np.abs(xd.cpu().numpy() - want).max() <= tol
+    assert np.abs(normed.float().cpu().numpy() - P.unit_rms(want, 1e-6) * w2).max() <= 2 * tol
+    rows = np.sort(rng.permutation(T)[:max(1, T // 2)]).astype(np.int32)
+    xd = _f32(x[rows])
+    part.forward(xd, batch, rows=_dev(rows))
+    ops.settle(xd)
+    assert np.abs(xd.cpu().numpy() - want[rows]).max() <= tol
+    ops.read_status(status)
+
+
+# ---- generation ------------------------------------------------------------------------------------------------
+
+def plain_generate(name, prompt, n_new):
+    toks, out, margins = list(prompt), [], []
+    for _ in range(n_new):
+        row = plain_logits(name, {"g": toks})["g"][-1]
+        t = int(np.argmax(row))
+        top2 = np.partition(row, -2)[-2:]
+        out.append(t)
+        margins.append(float(top2[1] - top2[0]))
+        toks.append(t)
+    return out, margins
+
+
+@pytest.mark.parametrize("dtype,min_margin", [("float32", 1e-3), ("bfloat16", 1.0)])
+@pytest.mark.parametrize("name", ["A", "B", "C"])
+def test_greedy_generation_through_the_scheduler(name, dtype, min_margin):
+    """Three prompts through Engine.generate: continuous batching with prompt portions of at most 8 tokens beside
+    decoding requests, two state slots for three requests, pages used again."""
+    from imparo_b200.engine import Engine
+    from tests.test_generate_gpu import agree
+    prompts = list(make_requests(name, [5, 23, 40], seed=1).values())
+    page = PAGE[name]
+    eng = Engine(model_dir(name), dtype=dtype, ctx=64, parallel=2, page_size=page, num_pages=2 * (64 // page), max_step_tokens=8)
+    got = eng.generate(prompts, max_tokens=10)
+    for i, p in enumerate(prompts):
+        want, margins = plain_generate(name, p, 10)
+        agree(got[i], want, margins, min_margin)
+    assert eng.cache.n_requests() == 0
+    eng.cache.check()
+
+
+def test_command_line_and_trace_runner(tmp_path):
+    from tests.test_trace_run_gpu import replay
+    name = "A"
+    prompt = make_requests(name, [16], seed=0)["r0"]
+    want, _ = plain_generate(name, prompt, 6)
+    tf = tmp_path / "tokens.txt"
+    tf.write_text(" ".join(map(str, prompt)))
+    r = subprocess.run([sys.executable, "-m", "imparo_b200", "-m", model_dir(name), "--dtype", "float32", "--decode", "6",
+                        "-c", "64", "-t", str(tf), "--json"], cwd=ROOT, capture_output=True, text=True, timeout=600)
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert json.loads(r.stdout.strip().splitlines()[-1])["tokens"] == [want]
+    reqs = make_requests(name, [70, 33, 90, 41, 64, 52], seed=7)
+    steps = traces.mixed(reqs, seed=1)
+    max_tokens = traces.max_live_tokens(steps, 64)
+    out = tmp_path / "out"
+    replay(model_dir(name), "bfloat16", steps, out, max_tokens)
+    ref = plain_logits(name, reqs)
+    want = traces.expected(steps, ref)
+    got = {s["step"]: np.fromfile(out / f"{s['step']}.f32", dtype="<f4").reshape(-1, ALL[name]["vocab"]) for s in steps if s["step"] in want}
+    scale = max(float(np.abs(v).max()) for v in ref.values())
+    skip = close_calls(name, reqs)
+    errs = [e for e in all_errors(steps, got, want) if (e[1], e[2]) not in skip]
+    assert max(e[3] for e in errs) <= WORST["bfloat16"] * scale
+    assert sum(e[3] > TOL["bfloat16"] * scale for e in errs) <= 0.1 * len(errs)
