@@ -22,7 +22,8 @@ continuous batching; LFM2-350M sizes with 32,768-token prompts in bfloat16 and 3
 print one JSON line each; --workload sizes runs the headline's model at further prompt lengths
 and decode contexts; --workload vipotar / negotar run the Vipotar / Negotar design at two sizes that resemble a real model's layers beside
 LFM2 at equal width, depth, heads and feed-forward size (prefill of one prompt, decode at batch 8), --workload keralix the
-Keralix design beside Vipotar likewise, --workload zepesun the Zepesun design beside Negotar, --workload modinex the Modinex design beside Vipotar; the default is the headline above.
+Keralix design beside Vipotar likewise, --workload zepesun the Zepesun design beside Negotar, --workload modinex the Modinex design beside Vipotar,
+--workload zinunex the Zinunex design beside Zepesun (--only-size NAME: one of its sizes); the default is the headline above.
 """
 import argparse
 import json
@@ -733,6 +734,107 @@ def workload_modinex(args):
     return 0
 
 
+def zinunex_config(width, layers, lat_heads, lat_dim, rot_dim, lat_vdim, kv_rank, heads, kv_heads, head, window, experts, top, groups, keep,
+                   ff, side, vocab):
+    """A Zinunex config.json of the given sizes: per four layers a windowed latent attention, two attentions and a latent attention
+    that reads the first one's cache; a routed feed-forward with a shared expert of the experts' size everywhere."""
+    rot = {"base": 500000.0, "dims": rot_dim, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}
+    lat = {"heads": lat_heads, "dim": lat_dim, "rot_dim": rot_dim, "vdim": lat_vdim, "kv_rank": kv_rank, "scale": (lat_dim + rot_dim) ** -0.5,
+           "mask": {"size": window}, "rot": rot}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": head, "vdim": head, "scale": head ** -0.5,
+           "rot": {"base": 500000.0, "dims": head, "scaling": {"factor": 4.0}}}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top, "scale": 2.0, "groups": {"count": groups, "keep": keep}},
+           "expert": {"ff": ff}, "shared": {"ff": ff}}
+    kinds = []
+    for i in range(0, layers, 4):
+        kinds += [("latent_attention", lat), ("attention", att), ("attention", att), ("latent_attention", dict(lat, kv_from=i))]
+    return {"architecture": "Zinunex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "token_side": {"dim": side},
+            "layers": [{"type": t, "mixer": m, "mlp": moe} for t, m in kinds[:layers]]}
+
+
+def workload_zinunex(args):
+    """Zinunex at three sizes beside Zepesun (whose latent attention, grouped router and shared expert are the closest the engine
+    serves) at equal width, depth, latent heads and cached rows, experts and parameters per expert (two matrices of 1.5 ff features
+    beside three of ff): every Zepesun layer a latent attention with a routed feed-forward; every second pair of Zinunex layers an
+    attention of as many heads instead.  Prefill of one prompt of 512 and 2,048 tokens, decode steps of 8 requests with 2,048
+    positions each.  Rooflines: prefill against the measured bfloat16 peak with the flops the design needs (products over all tokens,
+    the experts a token uses and the shared one, attention over the keys a position sees, the latent attention in its latent space);
+    decode against the measured copy bandwidth with the bytes a step must move (every dense matrix once, the experts the step's
+    rows can reach at most and the shared ones, the cached keys and values or latent rows the rows see, the tokens' side entries)."""
+    import numpy as np
+    import torch
+    from imparo_b200.engine import Engine
+    rng = np.random.default_rng(0)
+    pk = peaks()
+    sizes = {"width1024": dict(width=1024, layers=8, lat_heads=16, lat_dim=64, rot_dim=32, lat_vdim=64, kv_rank=96, heads=16, kv_heads=4,
+                               head=64, window=512, experts=16, top=2, groups=4, keep=2, ff=1536, side=128, vocab=32768),
+             "width2048": dict(width=2048, layers=8, lat_heads=32, lat_dim=64, rot_dim=32, lat_vdim=64, kv_rank=96, heads=32, kv_heads=8,
+                               head=64, window=1024, experts=32, top=4, groups=8, keep=4, ff=1536, side=256, vocab=65536),
+             "width2048_head128": dict(width=2048, layers=8, lat_heads=16, lat_dim=128, rot_dim=32, lat_vdim=128, kv_rank=96, heads=16,
+                                       kv_heads=4, head=128, window=1024, experts=16, top=2, groups=4, keep=2, ff=3072, side=256, vocab=65536)}
+    if args.only_size:
+        sizes = {k: v for k, v in sizes.items() if k == args.only_size}
+    out = {"metric": "Zinunex beside Zepesun at equal sizes: prefill of one prompt, decode at batch 8 with 2,048 positions",
+           "unit": "tokens/s", "dtype": "bf16", "data": "synthetic (random weights, uniform-random token ids)", "sizes": {}}
+    with ClockSampler() as clocks:
+        for name, z in sizes.items():
+            row = {}
+            W, L, V, S = z["width"], z["layers"], z["vocab"], z["side"]
+            LH, LD, LR, LV, C = z["lat_heads"], z["lat_dim"], z["rot_dim"], z["lat_vdim"], z["kv_rank"]
+            H, G, D = z["heads"], z["kv_heads"], z["head"]
+            expert = 2 * W * z["ff"]
+            for model in ("zinunex", "zepesun"):
+                lat = LH * (LD + LR) * W + LH * (LD + LV) * C + W * LH * LV          # without the latent's own projection
+                if model == "zinunex":
+                    cfg = zinunex_config(**z)
+                    n_lat = sum(e["type"] == "latent_attention" for e in cfg["layers"])
+                    n_own = sum("kv_from" not in e["mixer"] for e in cfg["layers"] if e["type"] == "latent_attention")
+                    n_att, window = L - n_lat, z["window"]
+                    dense = (n_lat * lat + n_own * (C + LR) * W + n_att * ((2 * H + G) * D * W) + L * (z["experts"] + 1) * W + L * 2 * S * W)
+                    side = L * S
+                else:
+                    cfg = zepesun_config(width=W, layers=L, lat_heads=LH, lat_dim=LD, rot_dim=LR, lat_vdim=LV, kv_rank=C, heads=H, kv_heads=G,
+                                         head=D, window=z["window"], mem_heads=1, mem_dim=8, mem_vdim=8, experts=z["experts"], top=z["top"],
+                                         groups=z["groups"], keep=z["keep"], ff=z["ff"] * 2 // 3, vocab=V, positions=CTX)
+                    first, moe = cfg["layers"][0], cfg["layers"][1]["mlp"]
+                    cfg["layers"] = [dict(first, mlp=moe) for _ in range(L)]
+                    n_lat = n_own = L
+                    n_att, window, side = 0, None, 0
+                    dense = L * (lat + (C + LR + LH) * W) + L * z["experts"] * W
+
+                def flops(T):
+                    keys = sum(min(t + 1, window or T) for t in range(T))
+                    return (2.0 * T * (dense + L * (z["top"] + 1) * expert) + 2.0 * V * W + n_att * 4.0 * H * D * T * (T + 1) / 2
+                            + n_lat * 2.0 * LH * (2 * C + LR) * keys)
+
+                def step_bytes(batch, ctx):
+                    reached = min(z["experts"], batch * z["top"]) + 1
+                    # (a layer that reads another one's cached rows reads them again)
+                    per_request = n_att * ctx * 2 * G * D * 2 + n_lat * min(ctx, window or ctx) * (C + LR) * 2 + side * 2
+                    return (dense + L * reached * expert + V * W) * 2 + batch * per_request
+                params = dense + L * (z["experts"] + 1) * expert + 2 * V * W + V * side + (CTX * W if model == "zepesun" else 0)
+                engine = Engine(config=cfg, seed=0, dtype="bfloat16", ctx=CTX, parallel=8, page_size=PAGE, max_step_tokens=PROMPT,
+                                random_init={"norm_jitter": 0.0})
+                r = {"params": params, "prefill": {}}
+                for T in (512, 2048):
+                    ms = measure_prefill(engine, reps=5, warmup=3, rng=rng, prompt=T)
+                    r["prefill"][str(T)] = {"value": round(T * 1000.0 / ms, 1), "ms": round(ms, 3),
+                                            "frac": round(flops(T) / (ms * 1e-3) / (pk["bf16_tflops_burst"] * 1e12), 4)}
+                ms, launches, library, ctx = measure_decode(engine, 8, max(20, args.steps // 4), max(args.warmup, 3), rng, prompt=PROMPT)
+                nbytes = step_bytes(8, ctx)
+                r["decode_b8"] = {"value": round(8 * 1000.0 / ms, 1), "ms_per_step": round(ms, 4), "own_kernels_per_step": round(launches, 1),
+                                  "library_gemms_per_step": round(library, 1), "bytes_per_step": int(nbytes),
+                                  "frac": round(nbytes / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)}
+                row[model] = r
+                del engine
+                torch.cuda.empty_cache()
+            out["sizes"][name] = dict(row, config=z)
+    out["peaks"] = pk["source"]
+    out["clocks"] = clocks.summary()
+    print(json.dumps(out))
+    return 0
+
+
 def _preset(name):
     with open(os.path.join(ROOT, "imparo_b200", "config", "presets", name + ".json")) as f:
         return json.load(f)
@@ -951,11 +1053,12 @@ def main():
     ap.add_argument("--skip-points", action="store_true", help="skip the batch-1 and batch-64 points")
     ap.add_argument("--only-decode", action="store_true", help="time the decode steps only (for profiler captures)")
     ap.add_argument("--only-prefill", action="store_true", help="time the 2,048-token prompt only (for profiler captures)")
-    ap.add_argument("--workload", default="headline", choices=["headline", "continuous", "long", "sizes", "vipotar", "negotar", "keralix", "zepesun", "modinex"],
+    ap.add_argument("--workload", default="headline", choices=["headline", "continuous", "long", "sizes", "vipotar", "negotar", "keralix", "zepesun", "modinex", "zinunex"],
                     help="headline (default): the one JSON line described at the top of this file.  continuous: LFM2-700M sizes, requests with prompts "
                          "of 64 to 4,096 tokens through 32 slots in 512-token portions beside decode rows, temperature 0.7, 128 new "
                          "tokens each.  long: LFM2-350M sizes, 4 prompts of 32,768 tokens and 512 greedy tokens each, bfloat16 and 32-bit.  "
                          "vipotar / negotar: that design at two sizes beside LFM2 at equal sizes.  keralix: the Keralix design at two sizes beside Vipotar")
+    ap.add_argument("--only-size", default=None, help="zinunex: run one of the sizes")
     ap.add_argument("--requests", type=int, default=32, help="continuous: requests in all (the baseline's workload has 32)")
     ap.add_argument("--long-check-layers", type=int, default=4, help="long: layers of the 32-bit check against the plain implementation")
     args = ap.parse_args()
@@ -987,6 +1090,8 @@ def main():
         return workload_zepesun(args)
     if args.workload == "modinex":
         return workload_modinex(args)
+    if args.workload == "zinunex":
+        return workload_zinunex(args)
     cfg = dict(LFM2_1_2B)
     if args.layers is not None and args.layers < cfg["num_hidden_layers"]:
         cfg["layer_types"] = cfg["layer_types"][:args.layers]

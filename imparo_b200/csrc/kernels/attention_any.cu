@@ -250,6 +250,70 @@ qkv_prepare_store_kernel(const float* __restrict__ qkv, size_t in_width, const f
     }
 }
 
+// The same without biases, norm and shared values, for sizes in quads (hd, vd, half of the rotated dimensions and the row stride
+// multiples of 4, 16-byte aligned pointers): a block per token (or per stretch of its heads) that computes the position's sines and
+// cosines once; a thread moves four entries and, where they turn, their four partners.
+template <typename T>
+__device__ __forceinline__ void put4(T* p, float4 v) {
+    if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(p) = v;
+    } else {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(ANY_WARPS * 32)
+qkv_prepare_store_token_kernel(const float* __restrict__ qkv, size_t in_width, const int* __restrict__ positions,
+                               const int* __restrict__ item_of_token, const float* __restrict__ inv_freq, int n_rot,
+                               T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ table,
+                               int max_blocks, int page_size, int n_pages, int nh, int nkv, int hd, int vd, int v_from_k, int* status) {
+    __shared__ __align__(16) float sn_s[ANY_MAX_HEAD / 2], cs_s[ANY_MAX_HEAD / 2];
+    pdl_trigger();
+    const int t = blockIdx.x;
+    const int pos = positions[t];
+    const int half = inv_freq ? (n_rot >> 1) : 0;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * inv_freq[i], &sn_s[i], &cs_s[i]);
+    const int blk = pos / page_size;
+    const int page = blk < max_blocks ? table[(size_t)item_of_token[t] * max_blocks + blk] : -1;
+    const bool mapped = page >= 0 && page < n_pages;
+    const size_t cache_row = mapped ? (size_t)page * page_size + (pos % page_size) : 0;
+    __syncthreads();
+    pdl_wait();
+    if (!mapped && threadIdx.x == 0 && blockIdx.y == 0) report(status, IMPARO_ST_PAGE_RANGE, 43, t, page);   // its keys and values are skipped
+    const float* row = qkv + (size_t)t * in_width;
+    T* kd = k_cache + cache_row * ((size_t)nkv * hd);
+    T* vd_row = v_cache + cache_row * ((size_t)nkv * vd);
+    const int pairs = half / 4, per = pairs + (hd - 2 * half) / 4;            // quads of work per head
+    const int total = (nh + nkv) * per, first = blockIdx.y * blockDim.x + threadIdx.x, step = gridDim.y * blockDim.x;
+#pragma unroll 2
+    for (int i = first; i < total; i += step) {
+        const int hh = i / per, u = i - hh * per;
+        const bool is_q = hh < nh;
+        if (!is_q && !mapped) continue;
+        const float* src = row + (size_t)hh * hd;                             // (key heads follow the query heads)
+        T* dst = is_q ? q_out + ((size_t)t * nh + hh) * hd : kd + (size_t)(hh - nh) * hd;
+        T* raw = !is_q && v_from_k ? vd_row + (size_t)(hh - nh) * vd : nullptr;
+        if (u < pairs) {
+            const int d = 4 * u;
+            const float4 a = *reinterpret_cast<const float4*>(src + d), b = *reinterpret_cast<const float4*>(src + d + half);
+            const float4 c = *reinterpret_cast<const float4*>(cs_s + d), s = *reinterpret_cast<const float4*>(sn_s + d);
+            put4<T>(dst + d, make_float4(a.x * c.x - b.x * s.x, a.y * c.y - b.y * s.y, a.z * c.z - b.z * s.z, a.w * c.w - b.w * s.w));
+            put4<T>(dst + d + half, make_float4(b.x * c.x + a.x * s.x, b.y * c.y + a.y * s.y, b.z * c.z + a.z * s.z, b.w * c.w + a.w * s.w));
+            if (raw) { put4<T>(raw + d, a); put4<T>(raw + d + half, b); }
+        } else {
+            const int d = 2 * half + 4 * (u - pairs);
+            const float4 a = *reinterpret_cast<const float4*>(src + d);
+            put4<T>(dst + d, a);
+            if (raw) put4<T>(raw + d, a);
+        }
+    }
+    if (v_from_k || !mapped) return;
+    const float* vs = row + (size_t)(nh + nkv) * hd;
+    for (int i = first; i < nkv * vd / 4; i += step) put4<T>(vd_row + 4 * i, *reinterpret_cast<const float4*>(vs + 4 * i));
+}
+
 // A block owns one token's heads [blockIdx.y * heads_per_block, + heads_per_block) of the row [q heads | k heads | v heads].
 // A lane moves pairs of neighbouring elements where PAIRS (sizes and strides even, pointers aligned), else single ones.
 template <typename T, bool PAIRS>
@@ -624,6 +688,23 @@ extern "C" int imparo_qkv_prepare_store(const float* qkv, long long row_stride, 
     if (n_rot < 0 || n_rot > hd || (n_rot & 1)) return -4;
     if (v_from_k && vd != hd) return -6;
     if (row_stride < (long long)(nh + nkv) * hd + (v_from_k ? 0 : (long long)nkv * vd)) return -2;
+    const bool quads = bias == nullptr && unit_eps < 0.f && v_other == nullptr && v_save == nullptr && hd % 4 == 0 && vd % 4 == 0
+                       && (inv_freq == nullptr || n_rot % 8 == 0) && row_stride % 4 == 0
+                       && (((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) == 0;
+    if (quads && (dtype == IMPARO_DT_F32 || dtype == IMPARO_DT_BF16)) {
+        const int items = (nh + nkv) * hd / 8;
+        int stretches = n_tok >= 256 ? 1 : (items + ANY_WARPS * 32 - 1) / (ANY_WARPS * 32);
+        stretches = stretches > 8 ? 8 : stretches;
+        const dim3 grid(n_tok, stretches);
+#define IMPARO_QPS(T_) launch(qkv_prepare_store_token_kernel<T_>, grid, dim3(ANY_WARPS * 32), 0, stream, qkv, (size_t)row_stride, positions, \
+        item_of_token, inv_freq, n_rot, (T_*)q_out, (T_*)k_cache, (T_*)v_cache, table, max_blocks, page_size, n_pages, nh, nkv, hd, vd, \
+        v_from_k, status)
+        if (dtype == IMPARO_DT_F32) IMPARO_QPS(float);
+        else IMPARO_QPS(__nv_bfloat16);
+#undef IMPARO_QPS
+        IMPARO_CHECK_LAUNCH();
+        return 0;
+    }
     dim3 grid(n_tok, (nh + 2 * nkv + ANY_WARPS - 1) / ANY_WARPS);
     if (dtype == IMPARO_DT_F32)
         launch(qkv_prepare_store_kernel<float>, grid, dim3(ANY_WARPS * 32), 0, stream, qkv, (size_t)row_stride, bias, positions,

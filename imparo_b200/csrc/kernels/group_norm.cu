@@ -11,8 +11,8 @@
 //
 // Few rows: a block per row.  A group belongs to a team of `wpg` warps (one warp per group when there are at least as many groups as
 // warps); the sum over a group is a fixed tree over the team's lanes, so a row's result depends on the row alone.
-// Many rows (a prompt portion) with groups of up to 1,024 elements: a warp per (row, group) that keeps the group in registers;
-// every load of the group is in flight at once and there is no barrier.  All arithmetic is 32-bit.
+// Many rows (a prompt portion) with groups of up to 4,096 elements: one, two or four warps per (row, group) that keep the group in
+// registers; every load of the group is in flight at once.  All arithmetic is 32-bit.
 #include "common.cuh"
 
 namespace imparo {
@@ -223,67 +223,86 @@ __global__ void group_norm_add_kernel(float* __restrict__ x, const float* __rest
     }
 }
 
-// ---- many rows: a warp per (row, group), NV float4 per lane (groups of up to 128 * NV elements, multiples of 4) ---------------
+// ---- many rows: WPG warps per (row, group), NV float4 per lane (groups of up to 128 * NV * WPG elements, multiples of 4) -------
 constexpr int ROW_WARPS = 4, MANY_ROWS = 256;
 
-template <typename TOut, int NV>
+// sum over a team of WPG warps (every thread of the block calls it; scratch: a float per warp, one array per sum of the kernel)
+template <int WPG>
+__device__ __forceinline__ float rows_team_sum(float v, float* scratch) {
+    v = warp_sum(v);
+    if (WPG == 1) return v;
+    const int warp = threadIdx.x >> 5;
+    if ((threadIdx.x & 31) == 0) scratch[warp] = v;
+    __syncthreads();
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < WPG; ++i) s += scratch[warp / WPG * WPG + i];
+    return s;
+}
+
+template <typename TOut, int NV, int WPG>
 __global__ void __launch_bounds__(ROW_WARPS * 32)
 group_rmsnorm_rows_kernel(const float* __restrict__ x, const int* __restrict__ rows, const float* __restrict__ w, float eps,
                           TOut* __restrict__ out, int n_rows, int width, int groups) {
+    __shared__ float scratch[ROW_WARPS];
     pdl_trigger();
-    const int lane = threadIdx.x & 31;
-    const long long task = (long long)blockIdx.x * ROW_WARPS + (threadIdx.x >> 5);
+    const int warp = threadIdx.x >> 5, at = (threadIdx.x & 31) + 32 * (warp % WPG);
+    constexpr int STEP = 32 * WPG;
+    const long long task = (long long)blockIdx.x * (ROW_WARPS / WPG) + warp / WPG;
     const int r = (int)(task / groups), g = (int)(task - (long long)r * groups), gw = width / groups, n4 = gw / 4;
     const float4* wg = reinterpret_cast<const float4*>(w + (size_t)g * gw);
     float4 ww[NV];
 #pragma unroll
-    for (int i = 0; i < NV; ++i) if (lane + 32 * i < n4) ww[i] = __ldg(wg + lane + 32 * i);
+    for (int i = 0; i < NV; ++i) if (at + STEP * i < n4) ww[i] = __ldg(wg + at + STEP * i);
     pdl_wait();
-    if (r >= n_rows) return;
-    const float4* xr = reinterpret_cast<const float4*>(x + (size_t)(rows ? rows[r] : r) * width + (size_t)g * gw);
+    const bool live = r < n_rows;
+    const float4* xr = reinterpret_cast<const float4*>(x + (size_t)(live ? (rows ? rows[r] : r) : 0) * width + (size_t)g * gw);
     float4 v[NV];
 #pragma unroll
-    for (int i = 0; i < NV; ++i) v[i] = lane + 32 * i < n4 ? xr[lane + 32 * i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = 0; i < NV; ++i) v[i] = live && at + STEP * i < n4 ? xr[at + STEP * i] : make_float4(0.f, 0.f, 0.f, 0.f);
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
-    const float scale = 1.0f / sqrtf(warp_sum(ss) / (float)gw + eps);
+    const float scale = 1.0f / sqrtf(rows_team_sum<WPG>(ss, scratch) / (float)gw + eps);
+    if (!live) return;
     TOut* o = out + (size_t)r * width + (size_t)g * gw;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-        if (lane + 32 * i < n4) {
+        if (at + STEP * i < n4) {
             const float y[4] = {v[i].x * scale * ww[i].x, v[i].y * scale * ww[i].y, v[i].z * scale * ww[i].z, v[i].w * scale * ww[i].w};
-            Vec<TOut, 4>::put(o + 4 * (lane + 32 * i), y);
+            Vec<TOut, 4>::put(o + 4 * (at + STEP * i), y);
         }
     }
 }
 
-template <typename TOut, int NV>
+template <typename TOut, int NV, int WPG>
 __global__ void __launch_bounds__(ROW_WARPS * 32)
 group_norm_add_rows_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ ybias,
                            const float* __restrict__ wb, float eps_b, const float* __restrict__ wn, float eps_n,
                            TOut* __restrict__ out, int n_rows, int width, int groups) {
+    __shared__ float scratch[2][ROW_WARPS];
     pdl_trigger();
-    const int lane = threadIdx.x & 31;
-    const long long task = (long long)blockIdx.x * ROW_WARPS + (threadIdx.x >> 5);
+    const int warp = threadIdx.x >> 5, at = (threadIdx.x & 31) + 32 * (warp % WPG);
+    constexpr int STEP = 32 * WPG;
+    const long long task = (long long)blockIdx.x * (ROW_WARPS / WPG) + warp / WPG;
     const int r = (int)(task / groups), g = (int)(task - (long long)r * groups), gw = width / groups, n4 = gw / 4;
     const size_t col = (size_t)g * gw;
     pdl_wait();
-    if (r >= n_rows) return;
-    const size_t row = (size_t)r * width + col;
+    const bool live = r < n_rows;
+    const size_t row = (size_t)(live ? r : 0) * width + col;
     const float4* yr = reinterpret_cast<const float4*>(y + row);
     float4* xr = reinterpret_cast<float4*>(x + row);
     float4 v[NV], xv[NV];
 #pragma unroll
-    for (int i = 0; i < NV; ++i) v[i] = lane + 32 * i < n4 ? yr[lane + 32 * i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = 0; i < NV; ++i) v[i] = live && at + STEP * i < n4 ? yr[at + STEP * i] : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-    for (int i = 0; i < NV; ++i) xv[i] = lane + 32 * i < n4 ? xr[lane + 32 * i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = 0; i < NV; ++i) xv[i] = live && at + STEP * i < n4 ? xr[at + STEP * i] : make_float4(0.f, 0.f, 0.f, 0.f);
     if (ybias) {
         const float4* b = reinterpret_cast<const float4*>(ybias + col);
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
-            if (lane + 32 * i < n4) {
-                const float4 t = __ldg(b + lane + 32 * i);
+            if (at + STEP * i < n4) {
+                const float4 t = __ldg(b + at + STEP * i);
                 v[i].x += t.x; v[i].y += t.y; v[i].z += t.z; v[i].w += t.w;
             }
         }
@@ -291,27 +310,28 @@ group_norm_add_rows_kernel(float* __restrict__ x, const float* __restrict__ y, c
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
-    const float scale = 1.0f / sqrtf(warp_sum(ss) / (float)gw + eps_b);
+    const float scale = 1.0f / sqrtf(rows_team_sum<WPG>(ss, scratch[0]) / (float)gw + eps_b);
     float ss2 = 0.f;
     const float4* b4 = reinterpret_cast<const float4*>(wb + col);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-        if (lane + 32 * i < n4) {
-            const float4 t = __ldg(b4 + lane + 32 * i);
+        if (live && at + STEP * i < n4) {
+            const float4 t = __ldg(b4 + at + STEP * i);
             xv[i].x += v[i].x * scale * t.x; xv[i].y += v[i].y * scale * t.y; xv[i].z += v[i].z * scale * t.z; xv[i].w += v[i].w * scale * t.w;
-            xr[lane + 32 * i] = xv[i];
+            xr[at + STEP * i] = xv[i];
             ss2 += xv[i].x * xv[i].x + xv[i].y * xv[i].y + xv[i].z * xv[i].z + xv[i].w * xv[i].w;
         }
     }
     if (out == nullptr) return;
-    const float nscale = 1.0f / sqrtf(warp_sum(ss2) / (float)gw + eps_n);
+    const float nscale = 1.0f / sqrtf(rows_team_sum<WPG>(ss2, scratch[1]) / (float)gw + eps_n);
+    if (!live) return;
     const float4* n4w = reinterpret_cast<const float4*>(wn + col);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-        if (lane + 32 * i < n4) {
-            const float4 t = __ldg(n4w + lane + 32 * i);
+        if (at + STEP * i < n4) {
+            const float4 t = __ldg(n4w + at + STEP * i);
             const float o[4] = {xv[i].x * nscale * t.x, xv[i].y * nscale * t.y, xv[i].z * nscale * t.z, xv[i].w * nscale * t.w};
-            Vec<TOut, 4>::put(out + row + 4 * (lane + 32 * i), o);
+            Vec<TOut, 4>::put(out + row + 4 * (at + STEP * i), o);
         }
     }
 }
@@ -336,11 +356,12 @@ extern "C" int imparo_group_rmsnorm(const float* x, const int* rows, const float
     if (n_rows <= 0) return 0;
     if (groups < 1 || width < 1 || width % groups != 0) return -2;
     const bool vec = (width / groups) % 4 == 0 && (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) == 0;
-    if (vec && n_rows >= gn::MANY_ROWS && width / groups <= 1024) {
-        const dim3 grid((unsigned)(((long long)n_rows * groups + gn::ROW_WARPS - 1) / gn::ROW_WARPS)), block(gn::ROW_WARPS * 32);
-        const int nv = (width / groups + 127) / 128;
-#define IMPARO_GR(T_, N_) launch(gn::group_rmsnorm_rows_kernel<T_, N_>, grid, block, 0, stream, x, rows, w, eps, (T_*)out, n_rows, width, groups)
-#define IMPARO_GRN(T_) do { if (nv <= 1) IMPARO_GR(T_, 1); else if (nv <= 2) IMPARO_GR(T_, 2); else if (nv <= 4) IMPARO_GR(T_, 4); else IMPARO_GR(T_, 8); } while (0)
+    if (vec && n_rows >= gn::MANY_ROWS && width / groups <= 4096) {
+        const int nv = (width / groups + 127) / 128, wpg = nv <= 8 ? 1 : (nv <= 16 ? 2 : 4), per = gn::ROW_WARPS / wpg;
+        const dim3 grid((unsigned)(((long long)n_rows * groups + per - 1) / per)), block(gn::ROW_WARPS * 32);
+#define IMPARO_GR(T_, N_, W_) launch(gn::group_rmsnorm_rows_kernel<T_, N_, W_>, grid, block, 0, stream, x, rows, w, eps, (T_*)out, n_rows, width, groups)
+#define IMPARO_GRN(T_) do { if (nv <= 1) IMPARO_GR(T_, 1, 1); else if (nv <= 2) IMPARO_GR(T_, 2, 1); else if (nv <= 4) IMPARO_GR(T_, 4, 1); \
+        else if (wpg == 1) IMPARO_GR(T_, 8, 1); else if (wpg == 2) IMPARO_GR(T_, 8, 2); else IMPARO_GR(T_, 8, 4); } while (0)
         if (out_dtype == IMPARO_DT_F32) IMPARO_GRN(float);
         else if (out_dtype == IMPARO_DT_BF16) IMPARO_GRN(__nv_bfloat16);
         else return -1;
@@ -372,12 +393,13 @@ extern "C" int imparo_group_norm_add(float* x, const float* y, int parts, long l
     if (out != nullptr && wn == nullptr) return -2;
     const uintptr_t all = (uintptr_t)x | (uintptr_t)y | (uintptr_t)ybias | (uintptr_t)wb | (uintptr_t)wn | (uintptr_t)out;
     const bool vec = (width / groups) % 4 == 0 && (all & 15) == 0 && (parts == 1 || part_stride % 4 == 0);
-    if (vec && parts == 1 && n_rows >= gn::MANY_ROWS && width / groups <= 1024) {
-        const dim3 grid((unsigned)(((long long)n_rows * groups + gn::ROW_WARPS - 1) / gn::ROW_WARPS)), block(gn::ROW_WARPS * 32);
-        const int nv = (width / groups + 127) / 128;
-#define IMPARO_GR(T_, N_) launch(gn::group_norm_add_rows_kernel<T_, N_>, grid, block, 0, stream, x, y, ybias, wb, eps_b, wn, eps_n, (T_*)out, \
+    if (vec && parts == 1 && n_rows >= gn::MANY_ROWS && width / groups <= 4096) {
+        const int nv = (width / groups + 127) / 128, wpg = nv <= 8 ? 1 : (nv <= 16 ? 2 : 4), per = gn::ROW_WARPS / wpg;
+        const dim3 grid((unsigned)(((long long)n_rows * groups + per - 1) / per)), block(gn::ROW_WARPS * 32);
+#define IMPARO_GR(T_, N_, W_) launch(gn::group_norm_add_rows_kernel<T_, N_, W_>, grid, block, 0, stream, x, y, ybias, wb, eps_b, wn, eps_n, (T_*)out, \
         n_rows, width, groups)
-#define IMPARO_GRN(T_) do { if (nv <= 1) IMPARO_GR(T_, 1); else if (nv <= 2) IMPARO_GR(T_, 2); else if (nv <= 4) IMPARO_GR(T_, 4); else IMPARO_GR(T_, 8); } while (0)
+#define IMPARO_GRN(T_) do { if (nv <= 1) IMPARO_GR(T_, 1, 1); else if (nv <= 2) IMPARO_GR(T_, 2, 1); else if (nv <= 4) IMPARO_GR(T_, 4, 1); \
+        else if (wpg == 1) IMPARO_GR(T_, 8, 1); else if (wpg == 2) IMPARO_GR(T_, 8, 2); else IMPARO_GR(T_, 8, 4); } while (0)
         if (out == nullptr || out_dtype == IMPARO_DT_F32) IMPARO_GRN(float);
         else if (out_dtype == IMPARO_DT_BF16) IMPARO_GRN(__nv_bfloat16);
         else return -1;

@@ -13,8 +13,8 @@
 //      query q_lat [T, heads * row_w] (the first rank entries are U_k^T q_plain, made by heads_linear).  The turn: of the
 //      first n_rot of the rot dimensions, i pairs with i + n_rot/2 (or, interleaved, 2i with 2i + 1), angle = position *
 //      inv_freq[i] in 32-bit, sines and cosines times a magnitude.  A row may be wider than rank + rot (row_w): the rest of
-//      cached rows and latent-space queries is zero.  Two CTAs per token: one for the queries, one for the cached row; a layer
-//      that reads rows another layer has cached launches the first alone.
+//      cached rows and latent-space queries is zero.  Per token one CTA for the cached row and one (few tokens: several) for the
+//      queries; a layer that reads rows another layer has cached launches the latter alone.
 //  (2) heads_linear: out[t, h, :] = W[h] x[t, h, :] for every head h (W [heads, out, in]), optionally times
 //      sigmoid(gate[t, h, :]) (a 32-bit product's columns).  A warp per output feature of a head and tile of eight rows;
 //      32-bit sums (for steps of few rows: many rows go to the library's batched product).
@@ -72,21 +72,35 @@ __device__ __forceinline__ float turned(const float* __restrict__ v, int d, int 
 }
 
 template <typename T>
+__device__ __forceinline__ void put4(T* p, float a, float b, float c, float d) {
+    if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d);
+    } else {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+    }
+}
+
+// VEC: four entries at a time (dim, rot, rank, row_w and the row stride multiples of 4, 16-byte aligned pointers).
+// grid (tokens, q_blocks (+ 1 for the cached row))
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(128)
 latent_rot_store_kernel(const float* __restrict__ proj, size_t stride, int heads, int dim, int rot, int rank, int row_w,
                         const float* __restrict__ wc, float eps, const float* __restrict__ inv_freq, int n_rot, int interleaved,
                         float magnitude, const int* __restrict__ positions, const int* __restrict__ item_of_token,
                         T* __restrict__ q_plain, T* __restrict__ q_lat, T* __restrict__ cache, const int* __restrict__ table,
-                        int max_blocks, int page_size, int n_pages, int* status) {
+                        int max_blocks, int page_size, int n_pages, int q_blocks, int* status) {
+    constexpr int N = VEC ? 4 : 1;
     __shared__ float scratch[33];
     __shared__ float cs_s[256], sn_s[256];         // the position's cosines and sines, once for all heads (n_rot <= 512)
     pdl_trigger();
     const int t = blockIdx.x;
     const int pos = positions[t];
+    const bool is_row = (int)blockIdx.y == q_blocks;
     const int blk = pos / page_size;
     int page = -1;
-    if (blockIdx.y == 1 && blk < max_blocks) page = table[(size_t)item_of_token[t] * max_blocks + blk];
-    const int q_width = heads * (dim + rot), half = n_rot / 2;
+    if (is_row && blk < max_blocks) page = table[(size_t)item_of_token[t] * max_blocks + blk];
+    const int half = n_rot / 2, tail = row_w - rank;
     const float fpos = (float)pos;
     for (int j = threadIdx.x; j < half; j += blockDim.x) {
         float sn, cs;
@@ -97,22 +111,43 @@ latent_rot_store_kernel(const float* __restrict__ proj, size_t stride, int heads
     pdl_wait();
     __syncthreads();
     const float* row = proj + (size_t)t * stride;
-    if (blockIdx.y == 0) {
-        // queries: plain dimensions as they are, rotated ones turned
-        for (int i = threadIdx.x; i < heads * dim; i += blockDim.x) {
-            const int h = i / dim, d = i % dim;
-            q_plain[(size_t)t * heads * dim + i] = from_f32<T>(row[(size_t)h * (dim + rot) + d]);
+    auto turn_to = [&](const float* v, int d, T* dst) {          // N entries of a rotated part, zeros behind it
+        if constexpr (VEC) {
+            float o[4] = {0.f, 0.f, 0.f, 0.f};
+            if (d < rot) {
+#pragma unroll
+                for (int u = 0; u < 4; ++u) o[u] = turned(v, d + u, n_rot, interleaved, cs_s, sn_s);
+            }
+            put4<T>(dst, o[0], o[1], o[2], o[3]);
+        } else {
+            *dst = from_f32<T>(d < rot ? turned(v, d, n_rot, interleaved, cs_s, sn_s) : 0.f);
         }
-        const int tail = row_w - rank;
-        for (int i = threadIdx.x; i < heads * tail; i += blockDim.x) {
-            const int h = i / tail, d = i % tail;
-            const float v = d < rot ? turned(row + (size_t)h * (dim + rot) + dim, d, n_rot, interleaved, cs_s, sn_s) : 0.f;
-            q_lat[((size_t)t * heads + h) * row_w + rank + d] = from_f32<T>(v);
+    };
+    if (!is_row) {
+        // queries: plain dimensions as they are, rotated ones turned
+        const int first = blockIdx.y * blockDim.x + threadIdx.x, step = q_blocks * blockDim.x;
+        const int per = dim / N, per_tail = tail / N;
+#pragma unroll 4
+        for (int i = first; i < heads * per; i += step) {
+            const int h = i / per, d = (i - h * per) * N;
+            const float* src = row + (size_t)h * (dim + rot) + d;
+            T* dst = q_plain + ((size_t)t * heads + h) * dim + d;
+            if constexpr (VEC) {
+                const float4 v = *reinterpret_cast<const float4*>(src);
+                put4<T>(dst, v.x, v.y, v.z, v.w);
+            } else {
+                *dst = from_f32<T>(*src);
+            }
+        }
+#pragma unroll 2
+        for (int i = first; i < heads * per_tail; i += step) {
+            const int h = i / per_tail, d = (i - h * per_tail) * N;
+            turn_to(row + (size_t)h * (dim + rot) + dim, d, q_lat + ((size_t)t * heads + h) * row_w + rank + d);
         }
         return;
     }
     // the cached row
-    const float* c = row + q_width;
+    const float* c = row + (size_t)heads * (dim + rot);
     float ss = 0.f;
     for (int i = threadIdx.x; i < rank; i += blockDim.x) ss += c[i] * c[i];
     ss = block_sum(ss, scratch);
@@ -123,9 +158,7 @@ latent_rot_store_kernel(const float* __restrict__ proj, size_t stride, int heads
     T* dst = cache + ((size_t)page * page_size + (pos % page_size)) * row_w;
     const float scale = 1.0f / sqrtf(ss / (float)rank + eps);
     for (int i = threadIdx.x; i < rank; i += blockDim.x) dst[i] = from_f32<T>(c[i] * scale * wc[i]);
-    const float* kr = c + rank;
-    for (int d = threadIdx.x; d < row_w - rank; d += blockDim.x)
-        dst[rank + d] = from_f32<T>(d < rot ? turned(kr, d, n_rot, interleaved, cs_s, sn_s) : 0.f);
+    for (int d = threadIdx.x * N; d < tail; d += blockDim.x * N) turn_to(c + rank, d, dst + rank + d);
 }
 
 constexpr int HL_ROWS = 8;
@@ -233,16 +266,20 @@ extern "C" int imparo_latent_rot_store(const float* proj, long long stride, int 
     if (heads < 1 || dim < 1 || rot < 0 || rank < 1 || row_w < rank + rot || n_rot < 0 || n_rot > rot || n_rot > 512 || n_rot % 2
         || (n_rot > 0 && inv_freq == nullptr) || page_size < 1
         || stride < (long long)heads * (dim + rot) + (cache != nullptr ? rank + rot : 0)) return -2;
-    const dim3 grid(n_tok, cache != nullptr ? 2 : 1);
-    if (dtype == IMPARO_DT_F32)
-        launch(latent_rot_store_kernel<float>, grid, dim3(128), 0, stream, proj, (size_t)stride, heads, dim, rot, rank, row_w, wc, eps,
-               inv_freq, n_rot, interleaved, magnitude, positions, item_of_token, (float*)q_plain, (float*)q_lat, (float*)cache, table,
-               max_blocks, page_size, n_pages, status);
-    else if (dtype == IMPARO_DT_BF16)
-        launch(latent_rot_store_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, proj, (size_t)stride, heads, dim, rot, rank, row_w, wc,
-               eps, inv_freq, n_rot, interleaved, magnitude, positions, item_of_token, (__nv_bfloat16*)q_plain, (__nv_bfloat16*)q_lat,
-               (__nv_bfloat16*)cache, table, max_blocks, page_size, n_pages, status);
+    const bool vec = dim % 4 == 0 && rot % 4 == 0 && rank % 4 == 0 && row_w % 4 == 0 && stride % 4 == 0
+                     && (((uintptr_t)proj | (uintptr_t)q_plain | (uintptr_t)q_lat | (uintptr_t)cache) & 15) == 0;
+    // few tokens: the queries of one over several blocks, so that no thread walks them in a row
+    const int items = heads * (dim > row_w - rank ? dim : row_w - rank) / (vec ? 4 : 1);
+    int q_blocks = n_tok >= 256 ? 1 : (items + 127) / 128;
+    if (q_blocks > 16) q_blocks = 16;
+    const dim3 grid(n_tok, q_blocks + (cache != nullptr ? 1 : 0));
+#define IMPARO_LRS(T_, V_) launch(latent_rot_store_kernel<T_, V_>, grid, dim3(128), 0, stream, proj, (size_t)stride, heads, dim, rot, rank, \
+        row_w, wc, eps, inv_freq, n_rot, interleaved, magnitude, positions, item_of_token, (T_*)q_plain, (T_*)q_lat, (T_*)cache, table, \
+        max_blocks, page_size, n_pages, q_blocks, status)
+    if (dtype == IMPARO_DT_F32) { if (vec) IMPARO_LRS(float, true); else IMPARO_LRS(float, false); }
+    else if (dtype == IMPARO_DT_BF16) { if (vec) IMPARO_LRS(__nv_bfloat16, true); else IMPARO_LRS(__nv_bfloat16, false); }
     else return -1;
+#undef IMPARO_LRS
     IMPARO_CHECK_LAUNCH();
     return 0;
 }

@@ -5,9 +5,10 @@
 //      renormalised to sum 1.  Leaves expert ids [rows, top] and weights [rows, top].  With a correction per expert the choice
 //      (and the groups' verdict) goes by score + correction, the weights by the score alone; a logit column behind the experts'
 //      may give each row one more number, sigmoid(z) (the factor of an expert that every row uses).
-//  (2) moe_rows_*: each (row, choice) pair on its own: the expert's gate and up rows times the (optionally weighted)
-//      input, silu(gate) * up, then the expert's down rows; the choices of a row are added in order.  Weights are
-//      streamed once per pair: the form for steps of few rows.
+//  (2) moe_few_*: steps of few rows (up to 256 pairs a launch), where reading the experts' matrices is the work.  A block belongs
+//      to one of the experts the launch's pairs name and a stretch of its features; it finds its pairs itself, keeps up to eight of
+//      their rows in shared memory and reads its matrix rows once for them.  The up kernel leaves act(..) per pair, the down kernel
+//      the (weighted) output per pair, which moe_sum adds in the order of the choices.
 //  (3) moe_group_*: pairs sorted by expert (a counting sort whose order inside an expert is the row order, so the
 //      result does not depend on what else is in the step), tiles of 32 pairs x 64 outputs per CTA: bfloat16 on
 //      tensor cores (mma.sync through wmma fragments, 32-bit accumulation), 32-bit with FFMA.  The tile list is made
@@ -18,9 +19,9 @@
 // ([ff, width]) and one activation on its own (plain_act's kinds).  The weight multiplies the expert's input (weight_input = 1)
 // or its output (0).
 //
-// A shared expert without a gate, of any size, may run in the launches of (2): blocks of their own, each for up to eight rows at
-// once, so that its matrices are read once for them.  Its rows' factors and the residual stream come in where the pairs are
-// summed (moe_sum_pairs / moe_tile_sum), which can add into the stream and leave the rounded copy that the next product reads.
+// A shared expert without a gate, of any size, may run in the launches of (2) as one more expert that every row uses.  Its rows'
+// factors and the residual stream come in where the pairs are summed (moe_sum_pairs / moe_tile_sum), which can add into the stream
+// and leave the rounded copy that the next product reads.
 #include "common.cuh"
 #include <mma.h>
 
@@ -47,30 +48,6 @@ __device__ __forceinline__ float dot16(const uint4 raw, const float* __restrict_
         for (int u = 0; u < 4; ++u) a = fmaf(v[u], x[u], a);
     }
     return a;
-}
-
-template <typename T>
-__device__ __forceinline__ float warp_dot(const T* __restrict__ w, const float* __restrict__ x, int n, bool vec, int lane) {
-    float acc = 0.f;
-    if (vec) {
-        constexpr int PER = Vec16<T>::N;
-        const uint4* w4 = reinterpret_cast<const uint4*>(w);
-        const int n4 = n / PER;
-        int i = lane;
-        float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
-        for (; i + 96 < n4; i += 128) {
-            const uint4 r0 = w4[i], r1 = w4[i + 32], r2 = w4[i + 64], r3 = w4[i + 96];
-            a0 += dot16<T>(r0, x + (size_t)i * PER);
-            a1 += dot16<T>(r1, x + (size_t)(i + 32) * PER);
-            a2 += dot16<T>(r2, x + (size_t)(i + 64) * PER);
-            a3 += dot16<T>(r3, x + (size_t)(i + 96) * PER);
-        }
-        for (; i < n4; i += 32) a0 += dot16<T>(w4[i], x + (size_t)i * PER);
-        acc = (a0 + a1) + (a2 + a3);
-    } else {
-        for (int i = lane; i < n; i += 32) acc += to_f32(w[i]) * x[i];
-    }
-    return warp_sum(acc);
 }
 
 // ---- (1) router -------------------------------------------------------------------------------------------------
@@ -236,209 +213,189 @@ moe_pick_kernel(const float* __restrict__ logits, int n_rows, int experts, int c
     }
 }
 
-// ---- (2) pair by pair ---------------------------------------------------------------------------------------------
-// two rows against the same vector at once: eight loads in flight
-template <typename T>
-__device__ __forceinline__ void warp_dot2(const T* __restrict__ w0, const T* __restrict__ w1, const float* __restrict__ x, int n,
-                                          bool vec, int lane, float& r0, float& r1) {
-    if (!vec) {
-        r0 = warp_dot<T>(w0, x, n, false, lane);
-        r1 = warp_dot<T>(w1, x, n, false, lane);
-        return;
-    }
-    constexpr int PER = Vec16<T>::N;
-    const uint4* p0 = reinterpret_cast<const uint4*>(w0);
-    const uint4* p1 = reinterpret_cast<const uint4*>(w1);
-    const int n4 = n / PER;
-    int i = lane;
-    float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
-    for (; i + 96 < n4; i += 128) {
-        uint4 u[4], v[4];
-#pragma unroll
-        for (int k = 0; k < 4; ++k) { u[k] = p0[i + 32 * k]; v[k] = p1[i + 32 * k]; }
-#pragma unroll
-        for (int k = 0; k < 4; ++k) {
-            a[k] += dot16<T>(u[k], x + (size_t)(i + 32 * k) * PER);
-            b[k] += dot16<T>(v[k], x + (size_t)(i + 32 * k) * PER);
-        }
-    }
-    for (; i < n4; i += 32) {
-        a[0] += dot16<T>(p0[i], x + (size_t)i * PER);
-        b[0] += dot16<T>(p1[i], x + (size_t)i * PER);
-    }
-    r0 = warp_sum((a[0] + a[1]) + (a[2] + a[3]));
-    r1 = warp_sum((b[0] + b[1]) + (b[2] + b[3]));
-}
+// ---- (2) few rows ---------------------------------------------------------------------------------------------------
+constexpr int FEW_ROWS = 8, FEW_PAIRS = 256;          // rows a block works on at once; pairs a launch may have
 
-// ---- blocks of the shared expert: up to SHARED_ROWS rows at once ------------------------------------------------------------
-constexpr int SHARED_ROWS = 8;
-
-// acc[j][r] = W row f0 + j . x row r for the four rows of W (those below n_feat) and the block's rows; xs: [rows][n] in shared
-// memory.  A lane takes every 32nd 16 bytes of a row; the sums end with a fixed tree over the warp.
+// acc[j][r] = w[j] . x row r for four matrix rows (null: left out) and the block's rows; xs: [rows][n] in shared memory.  A lane
+// takes every 32nd 16 bytes of a row, two of them in flight; the sums end with a fixed tree over the warp.
 template <typename T>
-__device__ __forceinline__ void warp_dot_rows(const T* __restrict__ w, int f0, int n_feat, const T* xs, int rows, int n, bool vec,
-                                              int lane, float (&acc)[4][SHARED_ROWS]) {
+__device__ __forceinline__ void warp_dot_rows(const T* const (&w)[4], const T* xs, int rows, int n, bool vec, int lane,
+                                              float (&acc)[4][FEW_ROWS]) {
 #pragma unroll
     for (int j = 0; j < 4; ++j)
 #pragma unroll
-        for (int r = 0; r < SHARED_ROWS; ++r) acc[j][r] = 0.f;
+        for (int r = 0; r < FEW_ROWS; ++r) acc[j][r] = 0.f;
     if (vec) {
         constexpr int PER = Vec16<T>::N;
         const int n4 = n / PER;
-        for (int i = lane; i < n4; i += 32) {
-            uint4 wv[4];
+        auto part = [&](const uint4 (&wv)[4], int i) {
 #pragma unroll
-            for (int j = 0; j < 4; ++j)
-                wv[j] = f0 + j < n_feat ? reinterpret_cast<const uint4*>(w + (size_t)(f0 + j) * n)[i] : make_uint4(0u, 0u, 0u, 0u);
+            for (int r = 0; r < FEW_ROWS; ++r) {
+                if (r >= rows) break;
+                const uint4 xv = reinterpret_cast<const uint4*>(xs + (size_t)r * n)[i];
+                float xf[PER];
 #pragma unroll
-            for (int r = 0; r < SHARED_ROWS; ++r) {
-                if (r < rows) {
-                    const uint4 xv = reinterpret_cast<const uint4*>(xs + (size_t)r * n)[i];
-                    float xf[PER];
+                for (int u = 0; u < PER; ++u) xf[u] = to_f32(reinterpret_cast<const T*>(&xv)[u]);
 #pragma unroll
-                    for (int u = 0; u < PER; ++u) xf[u] = to_f32(reinterpret_cast<const T*>(&xv)[u]);
-#pragma unroll
-                    for (int j = 0; j < 4; ++j) acc[j][r] += dot16<T>(wv[j], xf);
-                }
+                for (int j = 0; j < 4; ++j) acc[j][r] += dot16<T>(wv[j], xf);
             }
+        };
+        auto load = [&](uint4 (&wv)[4], int i) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) wv[j] = w[j] ? __ldg(reinterpret_cast<const uint4*>(w[j]) + i) : make_uint4(0u, 0u, 0u, 0u);
+        };
+        int i = lane;
+        for (; i + 32 < n4; i += 64) {
+            uint4 a[4], b[4];
+            load(a, i);
+            load(b, i + 32);
+            part(a, i);
+            part(b, i + 32);
+        }
+        if (i < n4) {
+            uint4 a[4];
+            load(a, i);
+            part(a, i);
         }
     } else {
         for (int i = lane; i < n; i += 32)
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-                if (f0 + j >= n_feat) break;
-                const float wv = to_f32(w[(size_t)(f0 + j) * n + i]);
+                if (w[j] == nullptr) continue;
+                const float wv = to_f32(w[j][i]);
 #pragma unroll
-                for (int r = 0; r < SHARED_ROWS; ++r) if (r < rows) acc[j][r] += wv * to_f32(xs[(size_t)r * n + i]);
+                for (int r = 0; r < FEW_ROWS; ++r) if (r < rows) acc[j][r] += wv * to_f32(xs[(size_t)r * n + i]);
             }
     }
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
+    for (int r = 0; r < FEW_ROWS; ++r) {
+        if (r >= rows) break;
 #pragma unroll
-        for (int r = 0; r < SHARED_ROWS; ++r) acc[j][r] = warp_sum(acc[j][r]);
-}
-
-// One block of the shared expert: 32 features (8 warps, each 4) of the rows tile * SHARED_ROWS ..; out rows of n_feat entries.
-template <typename T, typename TOut>
-__device__ __forceinline__ void shared_block(const T* __restrict__ x, const T* __restrict__ w, int tile, int block_y, int n_rows, int n,
-                                             int n_feat, int act, void* smem, TOut* __restrict__ out) {
-    if (block_y * 32 >= n_feat) return;
-    T* xs = reinterpret_cast<T*>(smem);
-    const int r0 = tile * SHARED_ROWS, rows = min(SHARED_ROWS, n_rows - r0);
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const bool vec = n % Vec16<T>::N == 0 && (((uintptr_t)w | (uintptr_t)x) & 15) == 0;
-    if (vec) {
-        const uint4* src = reinterpret_cast<const uint4*>(x + (size_t)r0 * n);
-        for (int i = threadIdx.x; i < rows * (n / Vec16<T>::N); i += blockDim.x) reinterpret_cast<uint4*>(xs)[i] = src[i];
-    } else {
-        for (int i = threadIdx.x; i < rows * n; i += blockDim.x) xs[i] = x[(size_t)r0 * n + i];
+        for (int j = 0; j < 4; ++j) acc[j][r] = warp_sum(acc[j][r]);
     }
-    __syncthreads();
-    const int f0 = block_y * 32 + warp * 4;
-    if (f0 >= n_feat) return;
-    float acc[4][SHARED_ROWS];
-    warp_dot_rows<T>(w, f0, n_feat, xs, rows, n, vec, lane, acc);
-#pragma unroll
-    for (int j = 0; j < 4; ++j)
-#pragma unroll
-        for (int r = 0; r < SHARED_ROWS; ++r)
-            if (lane == j * SHARED_ROWS + r && r < rows && f0 + j < n_feat)
-                out[(size_t)(r0 + r) * n_feat + f0 + j] = from_f32<TOut>(act >= 0 ? plain_act(act, acc[j][r]) : acc[j][r]);
 }
 
-// What the shared expert adds to a launch of the rows kernels (w null: nothing): the up kernel reads x rows of `n` entries and
-// writes mid rows of `n_feat`, the down kernel the other way round into float32 rows.
+// What an expert-by-expert launch does besides the routed experts (w null: nothing): an ungated expert with `n_feat` matrix rows
+// of `n` entries that every row uses; in: [n_rows, n], out: [n_rows, n_feat].
 struct SharedRows {
     const void* w;
-    int n_feat, n;
+    const void* in;
     void* out;
+    int n_feat, n;
 };
 
-// grid (rows * top + shared row tiles, ceil(features / 32)); 8 warps, each 4 features
-template <typename T>
-__global__ void __launch_bounds__(256)
-moe_rows_up_kernel(const T* __restrict__ h, const T* __restrict__ w_gu, const int* __restrict__ ids, const float* __restrict__ wts,
-                   int n_rows, int width, int ff, int top, int experts, int weight_input, int gated, int act, float limit,
-                   T* __restrict__ mid, SharedRows sh) {
-    extern __shared__ __align__(16) float up_smem[];
-    pdl_trigger();
-    pdl_wait();
-    // the shared expert's blocks come first: they have the most to do
-    const int shared_tiles = sh.w ? (n_rows + SHARED_ROWS - 1) / SHARED_ROWS : 0;
-    if ((int)blockIdx.x < shared_tiles) {
-        shared_block<T, T>(h, (const T*)sh.w, blockIdx.x, blockIdx.y, n_rows, sh.n, sh.n_feat, act, up_smem, (T*)sh.out);
-        return;
-    }
-    if ((int)blockIdx.y * 32 >= ff) return;
-    const int pair = blockIdx.x - shared_tiles, r = pair / top;
-    const int e = ids[pair];
-    if (e < 0 || e >= experts) return;
-    const float wt = weight_input ? wts[pair] : 1.0f;
-    const T* hr = h + (size_t)r * width;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) up_smem[i] = to_f32(from_f32<T>(wt * to_f32(hr[i])));
+// The launch's pairs as a block of 256 threads sees them: which expert is the k-th distinct one in the pairs' order of first
+// appearance (-1: there are fewer), its pairs (in order) in list, and how many.
+__device__ __forceinline__ int few_pairs_of(const int* __restrict__ ids, int n_pairs, int experts, int k, int* list, int& count) {
+    __shared__ int id_s[FEW_PAIRS];
+    __shared__ int firsts[8];
+    __shared__ int chosen;
+    const int p = threadIdx.x, lane = p & 31, warp = p >> 5;
+    int mine = p < n_pairs ? ids[p] : -1;
+    if (mine >= experts) mine = -1;
+    id_s[p] = mine;
+    if (p == 0) chosen = -1;
     __syncthreads();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const T* base = w_gu + (size_t)e * (gated ? 2 : 1) * ff * width;
-    const bool vec = width % Vec16<T>::N == 0 && ((uintptr_t)w_gu & 15) == 0;
-    if (!gated) {
-        for (int j = 0; j < 4; j += 2) {
-            const int f = blockIdx.y * 32 + warp * 4 + j;
-            if (f >= ff) break;
-            float a0, a1;
-            warp_dot2<T>(base + (size_t)f * width, base + (size_t)min(f + 1, ff - 1) * width, up_smem, width, vec, lane, a0, a1);
-            if (lane == 0) {
-                mid[(size_t)pair * ff + f] = from_f32<T>(plain_act(act, a0));
-                if (f + 1 < ff) mid[(size_t)pair * ff + f + 1] = from_f32<T>(plain_act(act, a1));
-            }
-        }
-        return;
+    int before = 0;                                     // earlier pairs of the same expert
+    if (mine >= 0)
+        for (int q = 0; q < p; ++q) before += id_s[q] == mine;
+    const bool first = mine >= 0 && before == 0;
+    const unsigned mask = __ballot_sync(0xffffffffu, first);
+    if (lane == 0) firsts[warp] = __popc(mask);
+    __syncthreads();
+    if (first) {
+        int rank = __popc(mask & ((1u << lane) - 1u));
+        for (int w = 0; w < warp; ++w) rank += firsts[w];
+        if (rank == k) chosen = mine;
     }
-    for (int j = 0; j < 4; ++j) {
-        const int f = blockIdx.y * 32 + warp * 4 + j;
-        if (f >= ff) break;
-        float ag, au;
-        warp_dot2<T>(base + (size_t)f * width, base + (size_t)(ff + f) * width, up_smem, width, vec, lane, ag, au);
-        if (lane == 0) mid[(size_t)pair * ff + f] = from_f32<T>(gated_act(act, limit, ag, au));
-    }
+    __syncthreads();
+    const int e = chosen;
+    const bool member = e >= 0 && mine == e;
+    if (member) list[before] = p;
+    count = __syncthreads_count(member);
+    return e;
 }
 
-// grid (rows + shared row tiles, ceil(width / 32)); 8 warps, each 4 outputs; out float32 [rows, width] is overwritten
-template <typename T>
-__global__ void __launch_bounds__(256)
-moe_rows_down_kernel(const T* __restrict__ mid, const T* __restrict__ w_down, const int* __restrict__ ids,
-                     const float* __restrict__ wts, int n_rows, int width, int ff, int top, int experts, int weight_input,
-                     float* __restrict__ out, SharedRows sh, const T* __restrict__ shared_mid) {
-    extern __shared__ __align__(16) float down_smem[];
+// Blocks: grid (shared row tiles + experts at most, feature stretches), 256 threads; a warp works on four matrix rows: four
+// features, or the gate and up rows of two (gated).
+//   UP:   in = h [n_rows, n], matrices [features (2x with gated), n], out = mid [pairs, features] in T: act(..)
+//   down: in = mid [pairs, n], matrices [features, n], out = pair_out float32 [pairs, features], times the weight unless weight_input
+template <typename T, bool UP>
+__global__ void __launch_bounds__(256, 2)
+moe_few_kernel(const T* __restrict__ in, const T* __restrict__ w, const int* __restrict__ ids, const float* __restrict__ wts, int n_rows,
+               int n, int n_feat, int top, int experts, int weight_input, int gated, int act, float limit, void* __restrict__ out,
+               SharedRows sh) {
+    extern __shared__ __align__(16) uint8_t few_smem[];
+    __shared__ int list[FEW_PAIRS];
     pdl_trigger();
     pdl_wait();
-    const int shared_tiles = sh.w ? (n_rows + SHARED_ROWS - 1) / SHARED_ROWS : 0;
-    if ((int)blockIdx.x < shared_tiles) {
-        shared_block<T, float>(shared_mid, (const T*)sh.w, blockIdx.x, blockIdx.y, n_rows, sh.n, sh.n_feat, -1, down_smem, (float*)sh.out);
-        return;
-    }
-    const int r = blockIdx.x - shared_tiles;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const bool vec = ff % Vec16<T>::N == 0 && ((uintptr_t)w_down & 15) == 0;
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    for (int k = 0; k < top; ++k) {
-        const int pair = r * top + k;
-        const int e = ids[pair];
-        __syncthreads();
-        for (int i = threadIdx.x; i < ff; i += blockDim.x) down_smem[i] = to_f32(mid[(size_t)pair * ff + i]);
-        __syncthreads();
-        if (e < 0 || e >= experts) continue;
-        const float wt = weight_input ? 1.0f : wts[pair];
-        for (int j = 0; j < 4; ++j) {
-            const int o = blockIdx.y * 32 + warp * 4 + j;
-            if (o >= width) break;
-            acc[j] += wt * warp_dot<T>(w_down + ((size_t)e * width + o) * ff, down_smem, ff, vec, lane);
-        }
+    T* xs = reinterpret_cast<T*>(few_smem);
+    // the shared expert's blocks come first: they have the most to do
+    const int shared_tiles = sh.w ? (n_rows + FEW_ROWS - 1) / FEW_ROWS : 0;
+    const bool shared = (int)blockIdx.x < shared_tiles;
+    if (shared) { n = sh.n; n_feat = sh.n_feat; gated = 0; }
+    const int per_warp = gated ? 2 : 4, f_block = blockIdx.y * 8 * per_warp;
+    if (f_block >= n_feat) return;
+    int e = 0, count = n_rows;
+    if (!shared) {
+        e = few_pairs_of(ids, n_rows * top, experts, blockIdx.x - shared_tiles, list, count);
+        if (e < 0) return;
     }
-    if (lane == 0)
-        for (int j = 0; j < 4; ++j) {
-            const int o = blockIdx.y * 32 + warp * 4 + j;
-            if (o < width) out[(size_t)r * width + o] = acc[j];
+    const T* src = shared ? (const T*)sh.in : in;
+    const T* mat = shared ? (const T*)sh.w : w + (size_t)e * (gated ? 2 : 1) * n_feat * n;
+    const bool vec = n % Vec16<T>::N == 0 && (((uintptr_t)mat | (uintptr_t)src) & 15) == 0;
+    const int f0 = f_block + warp * per_warp;
+    const T* rowp[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const int f = gated ? f0 + (j >> 1) : f0 + j;
+        rowp[j] = f < n_feat ? mat + (size_t)((gated && (j & 1)) ? n_feat + f : f) * n : nullptr;
+    }
+    const int lo = shared ? blockIdx.x * FEW_ROWS : 0, hi = shared ? min(n_rows, lo + FEW_ROWS) : count;
+    for (int r0 = lo; r0 < hi; r0 += FEW_ROWS) {
+        const int rows = min(FEW_ROWS, hi - r0);
+        __syncthreads();                                   // the rows before have been read
+        for (int r = 0; r < rows; ++r) {
+            const int item = shared ? r0 + r : list[r0 + r];
+            const T* xr = src + (size_t)(UP && !shared ? item / top : item) * n;
+            const float wt = UP && weight_input && !shared ? wts[item] : 1.0f;
+            if (vec) {
+                for (int i = threadIdx.x; i < n / Vec16<T>::N; i += 256) {
+                    uint4 raw = reinterpret_cast<const uint4*>(xr)[i];
+                    if (UP && weight_input && !shared) {
+                        T* v = reinterpret_cast<T*>(&raw);
+#pragma unroll
+                        for (int u = 0; u < Vec16<T>::N; ++u) v[u] = from_f32<T>(wt * to_f32(v[u]));
+                    }
+                    reinterpret_cast<uint4*>(xs + (size_t)r * n)[i] = raw;
+                }
+            } else {
+                for (int i = threadIdx.x; i < n; i += 256) xs[(size_t)r * n + i] = from_f32<T>(wt * to_f32(xr[i]));
+            }
         }
+        __syncthreads();
+        if (f0 >= n_feat) continue;
+        float acc[4][FEW_ROWS];
+        warp_dot_rows<T>(rowp, xs, rows, n, vec, lane, acc);
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int r = 0; r < FEW_ROWS; ++r) {
+                if (lane != j * FEW_ROWS + r || r >= rows) continue;
+                const int item = shared ? r0 + r : list[r0 + r];
+                if (gated) {
+                    const int f = f0 + (j >> 1);
+                    if ((j & 1) == 0 && f < n_feat)
+                        reinterpret_cast<T*>(out)[(size_t)item * n_feat + f] = from_f32<T>(gated_act(act, limit, acc[j][r], acc[(j + 1) & 3][r]));
+                } else if (f0 + j < n_feat) {
+                    const size_t at = (size_t)item * n_feat + f0 + j;
+                    if (UP) reinterpret_cast<T*>(shared ? sh.out : out)[at] = from_f32<T>(plain_act(act, acc[j][r]));
+                    else if (shared) reinterpret_cast<float*>(sh.out)[at] = acc[j][r];
+                    else reinterpret_cast<float*>(out)[at] = (weight_input ? 1.0f : wts[item]) * acc[j][r];
+                }
+            }
+    }
 }
 
 // ---- (3) grouped by expert ----------------------------------------------------------------------------------------
@@ -853,82 +810,93 @@ extern "C" int imparo_moe_route(const void* h, int dtype, const float* w_r, int 
     return 0;
 }
 
-// The choice alone, from logits that a product has made: [n_rows, parts * columns] float32 (columns: experts, or experts + 1
-// with extra_out).  With bfloat16 rows h (exact in 32-bit) and the 32-bit router matrix cut into three bfloat16 pieces (w1 = W
+// The choice alone, from logits that a product has made: [n_rows, parts * columns] float32 (columns >= experts, or >= experts + 1
+// with extra_out; more pad the product's width).  With bfloat16 rows h (exact in 32-bit) and the 32-bit router matrix cut into three bfloat16 pieces (w1 = W
 // rounded, w2 = W - w1 rounded, w3 the rest rounded: 8 + 8 + 8 bits of mantissa, their sum is W to its last bit), the
 // tensor-core product h [w1; w2; w3]^T has exact products and 32-bit sums: the router's logits in 32-bit, at the product's speed.
-extern "C" int imparo_moe_pick(const float* logits, int n_rows, int experts, int parts, int top, int softmax_scores, int renormalise,
+extern "C" int imparo_moe_pick(const float* logits, int n_rows, int experts, int columns, int parts, int top, int softmax_scores, int renormalise,
                                int groups, int keep, int group_pair, const float* correction, float renorm_eps, float weight_scale,
                                int out_stride, int* ids, float* wts, float* extra_out, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
-    if (!pick_args_ok(experts, top, groups, keep, out_stride, softmax_scores, correction) || parts < 1 || parts > 4) return -2;
+    if (!pick_args_ok(experts, top, groups, keep, out_stride, softmax_scores, correction) || parts < 1 || parts > 4
+        || columns < experts + (extra_out != nullptr ? 1 : 0)) return -2;
     launch(moe_pick_kernel, dim3((n_rows + 3) / 4), dim3(128), pick_smem_bytes(experts, groups), stream, logits, n_rows, experts,
-           experts + (extra_out != nullptr ? 1 : 0), parts, top, softmax_scores, renormalise, groups, keep, group_pair, correction,
+           columns, parts, top, softmax_scores, renormalise, groups, keep, group_pair, correction,
            renorm_eps, weight_scale, out_stride, ids, wts, extra_out);
     IMPARO_CHECK_LAUNCH();
     return 0;
 }
 
-constexpr size_t ROWS_SMEM_MOST = 160 * 1024;
+constexpr size_t FEW_SMEM_MOST = 200 * 1024;
 
-template <typename K>
-static int rows_smem(K kern, size_t smem, size_t* allowed) {
-    if (smem <= 48 * 1024 || smem <= *allowed) return 0;
-    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ROWS_SMEM_MOST);
-    if (e != cudaSuccess) return (int)e;
-    *allowed = ROWS_SMEM_MOST;
-    return 0;
-}
-
-template <typename T>
-static int moe_rows_launch(const void* h, const void* w_gu, const void* w_down, const int* ids, const float* wts, int n_rows, int width,
-                           int ff, int top, int experts, int weight_input, int gated, int act, float limit, void* mid, float* out,
-                           const void* s_up, const void* s_down, int s_ff, void* s_mid, float* s_out, cudaStream_t stream) {
-    const bool shared = s_up != nullptr;
-    const int tiles = shared ? (n_rows + SHARED_ROWS - 1) / SHARED_ROWS : 0, rows = n_rows < SHARED_ROWS ? n_rows : SHARED_ROWS;
-    const int most_ff = shared && s_ff > ff ? s_ff : ff;
-    size_t smem1 = (size_t)width * 4, smem2 = (size_t)ff * 4;
-    if (shared) {
-        const size_t a = (size_t)rows * width * sizeof(T), b = (size_t)rows * s_ff * sizeof(T);
-        smem1 = smem1 > a ? smem1 : a;
-        smem2 = smem2 > b ? smem2 : b;
+template <typename T, bool UP>
+static int few_launch(const void* in, const void* w, const int* ids, const float* wts, int n_rows, int n, int n_feat, int top, int experts,
+                      int weight_input, int gated, int act, float limit, void* out, const SharedRows& sh, cudaStream_t stream) {
+    const int rows = FEW_ROWS, pairs = n_rows * top;
+    size_t smem = (size_t)(pairs < rows ? pairs : rows) * n * sizeof(T);
+    int stretches = (n_feat + (gated ? 15 : 31)) / (gated ? 16 : 32), tiles = 0;
+    if (sh.w) {
+        const size_t b = (size_t)(n_rows < rows ? n_rows : rows) * sh.n * sizeof(T);
+        smem = smem > b ? smem : b;
+        stretches = stretches > (sh.n_feat + 31) / 32 ? stretches : (sh.n_feat + 31) / 32;
+        tiles = (n_rows + FEW_ROWS - 1) / FEW_ROWS;
     }
-    if (smem1 > ROWS_SMEM_MOST || smem2 > ROWS_SMEM_MOST) return -25;
-    static size_t allowed1 = 0, allowed2 = 0;
-    int rc = rows_smem(moe_rows_up_kernel<T>, smem1, &allowed1);
-    if (rc == 0) rc = rows_smem(moe_rows_down_kernel<T>, smem2, &allowed2);
-    if (rc) return rc;
-    SharedRows up = {}, down = {};
-    if (shared) {
-        up = {s_up, s_ff, width, s_mid};
-        down = {s_down, width, s_ff, s_out};
+    if (smem > FEW_SMEM_MOST) return -25;
+    static size_t allowed = 48 * 1024;
+    if (smem > allowed) {
+        const cudaError_t e = cudaFuncSetAttribute(moe_few_kernel<T, UP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)FEW_SMEM_MOST);
+        if (e != cudaSuccess) return (int)e;
+        allowed = FEW_SMEM_MOST;
     }
-    launch(moe_rows_up_kernel<T>, dim3(tiles + n_rows * top, (most_ff + 31) / 32), dim3(256), smem1, stream, (const T*)h, (const T*)w_gu,
-           ids, wts, n_rows, width, ff, top, experts, weight_input, gated, act, limit, (T*)mid, up);
-    IMPARO_CHECK_LAUNCH();
-    launch(moe_rows_down_kernel<T>, dim3(tiles + n_rows, (width + 31) / 32), dim3(256), smem2, stream, (const T*)mid, (const T*)w_down,
-           ids, wts, n_rows, width, ff, top, experts, weight_input, out, down, (const T*)s_mid);
+    launch(moe_few_kernel<T, UP>, dim3(tiles + (pairs < experts ? pairs : experts), stretches), dim3(256), smem, stream, (const T*)in, (const T*)w,
+           ids, wts, n_rows, n, n_feat, top, experts, weight_input, gated, act, limit, out, sh);
     IMPARO_CHECK_LAUNCH();
     return 0;
 }
+
+extern "C" int imparo_moe_sum(const float* pair_out, int n_rows, int width, int top, const float* extra, const float* extra_w,
+                              int accumulate, float* out, void* copy, cudaStream_t stream);
 
 // gated = 1: w_gu [experts, 2 ff, width], act one of gated_act's kinds (with limit); gated = 0: w_gu [experts, ff, width], act one
-// of plain_act's.  mid: [n_rows * top, ff] in dtype; out float32 [n_rows, width].  With s_up (needs gated = 0): an expert that
-// every row uses, s_up [s_ff, width] and s_down [width, s_ff], runs in the same launches: s_mid [n_rows, s_ff] in dtype, s_out
-// float32 [n_rows, width] receives its output, unweighted.  Two launches.
+// of plain_act's.  mid: [n_rows * top, ff] in dtype; pair_out float32 [n_rows * top, width]; out float32 [n_rows, width].  With s_up
+// (needs gated = 0): an expert that every row uses, s_up [s_ff, width] and s_down [width, s_ff], runs in the same launches: s_mid
+// [n_rows, s_ff] in dtype, s_out float32 [n_rows, width] receives its output, unweighted.  extra, extra_w, accumulate, copy as for
+// imparo_moe_sum (extra may be s_out).  Three launches per 256 pairs.  -25: rows too wide for eight of them in shared memory.
 extern "C" int imparo_moe_rows(const void* h, const void* w_gu, const void* w_down, int dtype, const int* ids, const float* wts,
                                int n_rows, int width, int ff, int top, int experts, int weight_input, int gated, int act, float limit,
-                               void* mid, float* out, const void* s_up, const void* s_down, int s_ff, void* s_mid, float* s_out,
-                               cudaStream_t stream) {
+                               void* mid, float* pair_out, const void* s_up, const void* s_down, int s_ff, void* s_mid, float* s_out,
+                               const float* extra, const float* extra_w, int accumulate, float* out, void* copy, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
+    if (top < 1 || top > FEW_PAIRS || width < 1 || ff < 1) return -2;
     if (s_up != nullptr && (gated || s_down == nullptr || s_ff < 1 || s_mid == nullptr || s_out == nullptr)) return -2;
-    if (dtype == IMPARO_DT_F32)
-        return moe_rows_launch<float>(h, w_gu, w_down, ids, wts, n_rows, width, ff, top, experts, weight_input, gated, act, limit, mid, out,
-                                      s_up, s_down, s_ff, s_mid, s_out, stream);
-    if (dtype == IMPARO_DT_BF16)
-        return moe_rows_launch<__nv_bfloat16>(h, w_gu, w_down, ids, wts, n_rows, width, ff, top, experts, weight_input, gated, act, limit,
-                                              mid, out, s_up, s_down, s_ff, s_mid, s_out, stream);
-    return -1;
+    if (dtype != IMPARO_DT_F32 && dtype != IMPARO_DT_BF16) return -1;
+    const size_t elt = dtype == IMPARO_DT_F32 ? 4 : 2;
+    const int step = FEW_PAIRS / top;
+    for (int r0 = 0; r0 < n_rows; r0 += step) {
+        const int rows = n_rows - r0 < step ? n_rows - r0 : step;
+        const size_t p0 = (size_t)r0 * top;
+        const char* hr = (const char*)h + (size_t)r0 * width * elt;
+        char* mr = (char*)mid + p0 * ff * elt;
+        SharedRows up = {}, down = {};
+        if (s_up != nullptr) {
+            char* sm = (char*)s_mid + (size_t)r0 * s_ff * elt;
+            up = {s_up, hr, sm, s_ff, width};
+            down = {s_down, sm, s_out + (size_t)r0 * width, width, s_ff};
+        }
+        int rc;
+        if (dtype == IMPARO_DT_F32) {
+            rc = few_launch<float, true>(hr, w_gu, ids + p0, wts + p0, rows, width, ff, top, experts, weight_input, gated, act, limit, mr, up, stream);
+            if (rc == 0) rc = few_launch<float, false>(mr, w_down, ids + p0, wts + p0, rows, ff, width, top, experts, weight_input, 0, 0, 0.f,
+                                                       pair_out + p0 * width, down, stream);
+        } else {
+            rc = few_launch<__nv_bfloat16, true>(hr, w_gu, ids + p0, wts + p0, rows, width, ff, top, experts, weight_input, gated, act, limit, mr, up,
+                                                 stream);
+            if (rc == 0) rc = few_launch<__nv_bfloat16, false>(mr, w_down, ids + p0, wts + p0, rows, ff, width, top, experts, weight_input, 0, 0, 0.f,
+                                                               pair_out + p0 * width, down, stream);
+        }
+        if (rc) return rc;
+    }
+    return imparo_moe_sum(pair_out, n_rows, width, top, extra, extra_w, accumulate, out, copy, stream);
 }
 
 // out[r, :] = (accumulate: its old value +) sum_k pair_out[r * top + k, :] (+ extra_w[r] * extra[r, :]); copy: the result rounded

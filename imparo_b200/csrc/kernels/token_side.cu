@@ -2,15 +2,16 @@
 //   g = gelu(G x) * e,  gelu(z) = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))),
 // which a product P g and a normed add (group_norm.cu) bring back into the stream.
 //
-//  (1) token_side_gate: few rows.  A warp per entry of g and up to eight rows: the row of G is read once for them, x as it
-//      stands in 32-bit, the sums are 32-bit; activation and side entry in the same launch.
+//  (1) token_side_gate: few rows.  A block per two entries of g and up to eight rows, its warps splitting the width: the rows of G
+//      are read once for them, x as it stands in 32-bit, the sums are 32-bit in a fixed order; activation and side entry in the same
+//      launch.
 //  (2) token_side_act: many rows, from a product's 32-bit rows G x.
 #include "common.cuh"
 
 namespace imparo {
 namespace ts {
 
-constexpr int ROWS = 8, WARPS = 4;
+constexpr int ROWS = 8, WARPS = 8, FEATS = 2;
 
 // the side table's row of a step's row: rows (int32, or null) names which of the step's tokens row r of x is
 __device__ __forceinline__ int side_token(const int* __restrict__ ids, const int* __restrict__ rows, int r, int vocab, int* status) {
@@ -33,60 +34,73 @@ __global__ void __launch_bounds__(WARPS * 32)
 side_gate_kernel(const float* __restrict__ x, const T* __restrict__ w, const T* __restrict__ table, size_t table_stride, int col0,
                  const int* __restrict__ ids, const int* __restrict__ rows, int n_rows, int width, int dim, int vocab,
                  T* __restrict__ out, int* status) {
+    __shared__ float part[WARPS][FEATS * ROWS];
     pdl_trigger();
-    pdl_wait();
-    const int lane = threadIdx.x & 31, j = blockIdx.x * WARPS + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, j0 = blockIdx.x * FEATS;
     const int r0 = blockIdx.y * ROWS, R = min(ROWS, n_rows - r0);
-    if (j >= dim) return;
-    const T* wr = w + (size_t)j * width;
     const float* xr = x + (size_t)r0 * width;
-    float acc[ROWS];
+    float acc[FEATS][ROWS];
 #pragma unroll
-    for (int r = 0; r < ROWS; ++r) acc[r] = 0.f;
-    const bool vec = width % 8 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0;
+    for (int f = 0; f < FEATS; ++f)
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) acc[f][r] = 0.f;
+    pdl_wait();
+    const bool vec = width % 4 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0;
     if (vec) {
-        for (int i = lane * 8; i < width; i += 256) {
-            float wv[8];
-            if constexpr (sizeof(T) == 2) {
-                const uint4 raw = *reinterpret_cast<const uint4*>(wr + i);
+        for (int i = (warp * 32 + lane) * 4; i < width; i += WARPS * 128) {
+            float wv[FEATS][4];
 #pragma unroll
-                for (int u = 0; u < 4; ++u) {
-                    const float2 f = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&raw)[u]);
-                    wv[2 * u] = f.x;
-                    wv[2 * u + 1] = f.y;
+            for (int f = 0; f < FEATS; ++f) {
+                if (j0 + f >= dim) { wv[f][0] = wv[f][1] = wv[f][2] = wv[f][3] = 0.f; continue; }
+                const T* wr = w + (size_t)(j0 + f) * width + i;
+                if constexpr (sizeof(T) == 2) {
+                    const uint2 raw = *reinterpret_cast<const uint2*>(wr);
+                    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+                    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+                    wv[f][0] = lo.x; wv[f][1] = lo.y; wv[f][2] = hi.x; wv[f][3] = hi.y;
+                } else {
+                    const float4 v = *reinterpret_cast<const float4*>(wr);
+                    wv[f][0] = v.x; wv[f][1] = v.y; wv[f][2] = v.z; wv[f][3] = v.w;
                 }
-            } else {
-#pragma unroll
-                for (int u = 0; u < 8; ++u) wv[u] = to_f32(wr[i + u]);
             }
-            float4 a[ROWS], b[ROWS];                       // every row's entries in flight at once
+            float4 a[ROWS];                               // every row's entries in flight at once
+#pragma unroll
+            for (int r = 0; r < ROWS; ++r) if (r < R) a[r] = *reinterpret_cast<const float4*>(xr + (size_t)r * width + i);
 #pragma unroll
             for (int r = 0; r < ROWS; ++r)
                 if (r < R) {
-                    a[r] = *reinterpret_cast<const float4*>(xr + (size_t)r * width + i);
-                    b[r] = *reinterpret_cast<const float4*>(xr + (size_t)r * width + i + 4);
-                }
 #pragma unroll
-            for (int r = 0; r < ROWS; ++r)
-                if (r < R)
-                    acc[r] += (wv[0] * a[r].x + wv[1] * a[r].y) + (wv[2] * a[r].z + wv[3] * a[r].w)
-                              + ((wv[4] * b[r].x + wv[5] * b[r].y) + (wv[6] * b[r].z + wv[7] * b[r].w));
+                    for (int f = 0; f < FEATS; ++f) acc[f][r] += (wv[f][0] * a[r].x + wv[f][1] * a[r].y) + (wv[f][2] * a[r].z + wv[f][3] * a[r].w);
+                }
         }
     } else {
-        for (int i = lane; i < width; i += 32) {
-            const float wv = to_f32(wr[i]);
+        for (int i = threadIdx.x; i < width; i += WARPS * 32) {
 #pragma unroll
-            for (int r = 0; r < ROWS; ++r) if (r < R) acc[r] += wv * xr[(size_t)r * width + i];
+            for (int f = 0; f < FEATS; ++f) {
+                if (j0 + f >= dim) continue;
+                const float wv = to_f32(w[(size_t)(j0 + f) * width + i]);
+#pragma unroll
+                for (int r = 0; r < ROWS; ++r) if (r < R) acc[f][r] += wv * xr[(size_t)r * width + i];
+            }
         }
     }
 #pragma unroll
-    for (int r = 0; r < ROWS; ++r) acc[r] = warp_sum(acc[r]);
+    for (int f = 0; f < FEATS; ++f)
 #pragma unroll
-    for (int r = 0; r < ROWS; ++r) {
-        if (lane == r && r < R) {
+        for (int r = 0; r < ROWS; ++r) {
+            const float v = warp_sum(acc[f][r]);
+            if (lane == 0) part[warp][f * ROWS + r] = v;
+        }
+    __syncthreads();
+    if (threadIdx.x < FEATS * ROWS) {
+        const int f = threadIdx.x / ROWS, r = threadIdx.x % ROWS, j = j0 + f;
+        if (r < R && j < dim) {
+            float z = 0.f;
+#pragma unroll
+            for (int k = 0; k < WARPS; ++k) z += part[k][threadIdx.x];
             const int id = side_token(ids, rows, r0 + r, vocab, status);
             const float e = id < 0 ? 0.f : to_f32(table[(size_t)id * table_stride + col0 + j]);
-            out[(size_t)(r0 + r) * dim + j] = from_f32<T>(gelu_times<T>(acc[r], e));
+            out[(size_t)(r0 + r) * dim + j] = from_f32<T>(gelu_times<T>(z, e));
         }
     }
 }
@@ -120,7 +134,7 @@ extern "C" int imparo_token_side_gate(const float* x, const void* w, const void*
     if (width < 1 || dim < 1 || col0 < 0 || col0 + dim > table_stride) return -2;
     const int tiles = (n_rows + ts::ROWS - 1) / ts::ROWS;
     if (tiles > 65535) return -2;
-    const dim3 grid((dim + ts::WARPS - 1) / ts::WARPS, tiles), block(ts::WARPS * 32);
+    const dim3 grid((dim + ts::FEATS - 1) / ts::FEATS, tiles), block(ts::WARPS * 32);
     if (dtype == IMPARO_DT_F32)
         launch(ts::side_gate_kernel<float>, grid, block, 0, stream, x, (const float*)w, (const float*)table, (size_t)table_stride, col0,
                ids, rows, n_rows, width, dim, vocab, (float*)out, status);

@@ -1714,14 +1714,15 @@ def moe_pick(logits: torch.Tensor, experts: int, parts: int, top: int, ids: torc
              always: int = 0, group_score: str = "max", correction: Optional[torch.Tensor] = None,
              extra: Optional[torch.Tensor] = None) -> None:
     """The router's choice from logits a product has made: logits float32 [rows, parts * columns] (columns: experts, one more
-    with extra), a logit being the sum of its `parts` entries `columns` apart (a 32-bit router matrix cut into bfloat16 pieces
+    with extra, or any larger number), a logit being the sum of its `parts` entries `columns` apart (a 32-bit router matrix cut into bfloat16 pieces
     that add up to it to its last bit).  The rest as for moe_route."""
     _cuda(logits, ids, wts)
     n = logits.shape[0]
-    _need(logits.dtype == torch.float32 and logits.shape[1] == parts * (experts + (0 if extra is None else 1)),
+    columns = logits.shape[1] // parts
+    _need(logits.dtype == torch.float32 and logits.shape[1] == parts * columns and columns >= experts + (0 if extra is None else 1),
           "moe_pick: logits float32 [rows, parts * columns]")
     how, stride = _pick_args(top, ids, wts, n, experts, groups, keep, always, group_score, correction, extra)
-    _check(_lib.kernels().imparo_moe_pick(_ptr(logits), n, int(experts), int(parts), int(top), int(bool(softmax)),
+    _check(_lib.kernels().imparo_moe_pick(_ptr(logits), n, int(experts), columns, int(parts), int(top), int(bool(softmax)),
                                           int(bool(renormalise)), *how, float(renorm_eps), float(weight_scale), stride,
                                           _ptr(ids), _ptr(wts), _ptr(extra), _stream()), "moe_pick")
 
@@ -1795,14 +1796,17 @@ def moe_experts_tiles(h: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor,
 
 def moe_experts(h: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, top: int,
                 weight_input: bool, mid: torch.Tensor, out: torch.Tensor, scratch=None, act: str = "silu", limit: float = 0.0,
-                extra=None, accumulate: bool = False, copy: Optional[torch.Tensor] = None, shared=None) -> None:
+                extra=None, accumulate: bool = False, copy: Optional[torch.Tensor] = None, shared=None,
+                pair_out: Optional[torch.Tensor] = None) -> None:
     """out[r] = sum_k expert_{ids[r,k]}(wts[r,k] * h[r])  (weight_input) or sum_k wts[r,k] * expert(h[r]).
     act, limit: the experts' activation: gated (gated_act's kinds; w_gu [experts, 2 ff, width] = [gate; up]) or "plain:" + one of
     ACTIVATIONS (w_gu [experts, ff, width]); w_down [experts, width, ff]; mid [rows*top, ff] in h's dtype; out float32
-    [rows, width], overwritten.  scratch = (float32 [rows*top, width], int32 [rows*top + experts + 2 + 3*(rows*top//32 + experts)]):
-    when given, pairs are sorted by expert and run as tiles (steps of many rows) and extra, accumulate, copy are as for moe_sum;
-    else each pair on its own, and shared = (up [s_ff, width], down [width, s_ff], mid [rows, s_ff] in h's dtype, out float32
-    [rows, width]) may add an ungated expert of any size that every row uses: its unweighted output goes to its own tensor."""
+    [rows, width], overwritten; extra, accumulate, copy as for moe_sum.
+    scratch = (float32 [rows*top, width], int32 [rows*top + experts + 2 + 3*(rows*top//32 + experts)]): when given, pairs are sorted
+    by expert and run as tiles (steps of many rows); else a block per expert and stretch of its features finds its pairs itself (steps
+    of few rows; pair_out: float32 scratch [rows*top, width], made here when not given), and shared = (up [s_ff, width], down
+    [width, s_ff], mid [rows, s_ff] in h's dtype, y float32 [rows, width]) may add an ungated expert of any size that every row
+    uses: its unweighted output goes to y (which `extra` may name)."""
     _cuda(h, w_gu, w_down, ids, wts, mid, out)
     n, width = h.shape
     E = w_gu.shape[0]
@@ -1810,20 +1814,23 @@ def moe_experts(h: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, ids: 
     _need(w_gu.dtype == h.dtype and w_down.dtype == h.dtype and mid.dtype == h.dtype, "moe_experts: one dtype for h, the experts and mid")
     _need(w_gu.shape[2] == width and tuple(w_down.shape) == (E, width, ff), "moe_experts: expert shapes")
     _need(mid.numel() >= n * top * ff and out.dtype == torch.float32 and tuple(out.shape) == (n, width), "moe_experts: mid / out sizes")
+    tail = _sum_tail(n, width, extra, accumulate, copy)
     if scratch is not None:
-        _need(shared is None, "moe_experts: a shared expert rides along pair by pair only")
+        _need(shared is None, "moe_experts: a shared expert rides along with few rows only")
         pair_out, si = scratch
         _cuda(pair_out, si)
         _need(pair_out.dtype == torch.float32 and pair_out.numel() >= n * top * width and si.dtype == torch.int32
               and si.numel() >= n * top + E + 2 + 3 * (n * top // 32 + E), "moe_experts: grouped scratch too small")
-        tail = _sum_tail(n, width, extra, accumulate, copy)
         _check(_lib.kernels().imparo_moe_grouped(_ptr(h), _ptr(w_gu), _ptr(w_down), _code(h), _ptr(ids), _ptr(wts), n, width, ff, int(top),
                                                  E, int(bool(weight_input)), gated, code, float(limit), _ptr(mid), _ptr(pair_out),
                                                  _ptr(si), *tail, _ptr(out), _ptr(copy), _stream()),
                "moe_grouped")
         COUNTS["own"] += 3
         return
-    _need(extra is None and not accumulate and copy is None, "moe_experts: pair by pair the result is written as it is (moe_sum adds)")
+    if pair_out is None:
+        pair_out = torch.empty(n * top * width, dtype=torch.float32, device=h.device)
+    _cuda(pair_out)
+    _need(pair_out.dtype == torch.float32 and pair_out.numel() >= n * top * width, "moe_experts: pair_out float32 [rows * top, width]")
     s_up = s_down = s_mid = s_out = None
     s_ff = 0
     if shared is not None:
@@ -1834,10 +1841,10 @@ def moe_experts(h: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, ids: 
               and tuple(s_down.shape) == (width, s_ff) and s_mid.numel() >= n * s_ff and s_out.dtype == torch.float32
               and tuple(s_out.shape) == (n, width), "moe_experts: the shared expert's shapes")
     _check(_lib.kernels().imparo_moe_rows(_ptr(h), _ptr(w_gu), _ptr(w_down), _code(h), _ptr(ids), _ptr(wts), n, width, ff, int(top), E,
-                                          int(bool(weight_input)), gated, code, float(limit), _ptr(mid), _ptr(out), _ptr(s_up),
-                                          _ptr(s_down), s_ff, _ptr(s_mid), _ptr(s_out), _stream()),
+                                          int(bool(weight_input)), gated, code, float(limit), _ptr(mid), _ptr(pair_out), _ptr(s_up),
+                                          _ptr(s_down), s_ff, _ptr(s_mid), _ptr(s_out), *tail, _ptr(out), _ptr(copy), _stream()),
            "moe_rows")
-    COUNTS["own"] += 1
+    COUNTS["own"] += 2 * -(-n // (256 // top))          # (with the sum, three launches for up to 256 pairs)
 
 
 # ---- a layer's own token input (csrc/kernels/token_side.cu) ------------------------------------------------------------

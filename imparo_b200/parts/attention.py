@@ -239,7 +239,14 @@ class AttentionMixer(Part):
                 qkv = projected
             else:
                 qkv = rt.workspace.get("attn_qkv32", (T, wide), torch.float32, first="tokens")
-                ops.linear(x, self.w_qkv[:wide], qkv, status=rt.status)
+                if batch.decode_only and self._decodes_from_product():
+                    qkv = ops.linear_unfolded(x, self.w_qkv[:wide], qkv, status=rt.status)
+                    if isinstance(qkv, ops.PartialProduct):
+                        if self._decode_from_product(qkv, batch, kv, table, inv_freq, n_rot, residual, accumulate):
+                            return
+                        qkv = qkv.tensor()
+                else:
+                    ops.linear(x, self.w_qkv[:wide], qkv, status=rt.status)
             gate = qkv[:, width:] if self.gate else None
             if self.gate:
                 qkv = qkv[:, :width]
@@ -319,6 +326,40 @@ class AttentionMixer(Part):
         ops.linear(out, self.w_o, residual, accumulate=accumulate, status=rt.status)
         if self.prepared and self.b_o is not None:
             ops.add_bias(residual, self.b_o)
+
+    def _decodes_from_product(self) -> bool:
+        """Whether rows of one token can go from the q/k product's split partials straight into the split-key attention: keys that
+        are their own values, with nothing between the product and the rotation."""
+        return (self.v_from_k and not self.unit_norm and not self.bias_required and self.qk_conv is None and not self.gate
+                and not self.sigmoid and self.chunk is None and self.softcap == 0.0 and self.rt.act_dtype == torch.bfloat16
+                and self.hd in (64, 128) and self.nh // self.nkv <= 8 and (not self.sink or self.sinks is not None)
+                and ops.switches().decode_from_qkv)
+
+    def _decode_from_product(self, qkv, batch, kv, table, inv_freq, n_rot, residual, accumulate) -> bool:
+        """One kernel makes the queries, writes the new key and value rows and attends; the output product combines the key chunks'
+        partial results while it makes its operand (or a combine kernel does)."""
+        rt, T = self.rt, qkv.shape[0]
+        nh, hd = self.nh, self.hd
+        chunk, n_splits = ops.split_plan(T, self.nkv, table.shape[1] * kv.page_size)
+        if n_splits > 16 or T > 65535:       # (every chunk's CTA makes the group's queries again: for contexts of up to 16 chunks)
+            return False
+        room = self._partials_room(table.shape[1] * kv.page_size)
+        part_acc = rt.workspace.get("attn_part_acc", (T * nh * n_splits * hd,), torch.float32, reserve=room * hd)
+        part_ml = rt.workspace.get("attn_part_ml", (T * nh * n_splits * 2,), torch.float32, reserve=room * 2)
+        in_product = ops.fuse_producers() and self.b_o is None
+        out = rt.workspace.get("attn_out", (T, nh * hd), rt.act_dtype, first="tokens")
+        if not ops.attention_decode_from_qkv(qkv, batch.positions, batch.item_of_token, None, None, inv_freq, n_rot, 0.0, kv.k, kv.v, table,
+                                             kv.page_size, kv.n_pages, self.window, self.scale, None if in_product else out, part_acc,
+                                             part_ml, chunk, n_splits, nh, self.nkv, hd, rt.status, v_from_k=True, sink_values=self.sinks):
+            return False
+        if in_product:
+            if ops.linear_of_attention_partials(part_acc, part_ml, T, nh, hd, n_splits, self.w_o, residual, rt.status, accumulate=accumulate):
+                return True
+            ops.attention_split_combine(part_acc, part_ml, out, T * nh, hd, n_splits)
+        ops.linear(out, self.w_o, residual, accumulate=accumulate, status=rt.status)
+        if self.b_o is not None:
+            ops.add_bias(residual, self.b_o)
+        return True
 
     def _attend_sigmoid(self, q, batch, kv, table, out, residual, accumulate):
         """Sigmoid weights on the tensor-core kernels: prompt portions on the tcgen05 kernel, rows of one token (and portions too

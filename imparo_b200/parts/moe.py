@@ -36,8 +36,8 @@ class RoutedExperts(Part):
     accumulate=True the result is added into it, times `scale`.  copy (ungated experts, with accumulate): an activation-dtype
     [rows, hidden] tensor that receives the updated rows rounded, in the pass that adds."""
     takes_scale = True
-    GROUP_FROM = 65           # steps with at least this many (row, expert) pairs run sorted by expert, in tiles
-    RIDE_BYTES = 128 * 1024   # a shared expert rides along pair by pair while eight of its rows fit a block's shared memory
+    GROUP_FROM = 256          # steps with at least this many (row, expert) pairs run sorted by expert, in tiles
+    ROW_BYTES = 200 * 1024    # below that a block per expert keeps eight rows in shared memory, if they fit
     TILES_FROM = 256          # and from this many on (bfloat16, aligned sizes) on the tensor-memory product, tiles of 128 rows
 
     NAMES = {"router": "router", "gate": "e{e}.gate", "up": "e{e}.up", "down": "e{e}.down", "correction": "correction"}
@@ -118,6 +118,8 @@ class RoutedExperts(Part):
         # For bfloat16 rows the router's logits come from the tensor-core product: the 32-bit matrix cut into three
         # bfloat16 pieces that add up to it to its last bit, so every product is exact and the sums are 32-bit.
         self.w_router_pieces = None
+        # (each piece padded with zero rows to a multiple of eight columns, which the products' kernels like)
+        self.router_columns = -(-self.w_router.shape[0] // 8) * 8
         if self.rt.act_dtype == torch.bfloat16:
             rest, pieces = self.w_router.float(), []
             for _ in range(3):
@@ -127,7 +129,8 @@ class RoutedExperts(Part):
                 if not bool(rest.any()):          # a router stored in bfloat16 is its own first piece
                     break
             self.router_parts = len(pieces)
-            self.w_router_pieces = torch.cat(pieces, dim=0).contiguous()
+            pad = self.router_columns - self.w_router.shape[0]
+            self.w_router_pieces = torch.cat([torch.nn.functional.pad(p, (0, 0, 0, pad)) for p in pieces], dim=0).contiguous()
         # experts stacked: [experts, 2 ff, hidden] = [gate; up] (ungated: [experts, ff, hidden]) and [experts, hidden, ff]
         if self.gated:
             gu = [torch.cat([tensors[n["gate"].format(e=e)], tensors[n["up"].format(e=e)]], dim=0) for e in range(self.experts)]
@@ -148,15 +151,21 @@ class RoutedExperts(Part):
         self.w_gu = torch.stack(gu).contiguous()
         self.w_down = torch.stack(down).contiguous()
 
+    def _few(self, pairs: int, x) -> bool:
+        """Whether a step of so many pairs runs expert by expert without sorting (ops.moe_experts without scratch)."""
+        widest = max(self.hidden, self.ff, int(self.shared["ff"]) if self.shared is not None else 0)
+        return pairs < self.GROUP_FROM and 8 * widest * x.element_size() <= self.ROW_BYTES
+
     def _experts(self, x, w_gu, w_down, ids, wts, top, weight_input, limit, out, tag, extra=None, accumulate=False, copy=None,
                  shared=None):
-        """One pass of the expert kernels: pair by pair, sorted into small tiles, or on the tensor-memory product.  extra: a
-        function that makes (float32 [rows, hidden], float32 [rows]) for the sum's tail (sorted paths only); shared: what rides
-        along pair by pair (ops.moe_experts)."""
+        """One pass of the expert kernels: expert by expert, sorted into small tiles, or on the tensor-memory product.  extra: a
+        function that makes (float32 [rows, hidden], float32 [rows]) for the sum's tail; shared: what rides along with few rows
+        (ops.moe_experts)."""
         rt, T = self.rt, x.shape[0]
         ws = rt.workspace
         n_experts, ff = w_gu.shape[0], w_gu.shape[1] // (2 if self.gated else 1)
         pairs = T * top
+        how = dict(act=self.form, limit=limit, extra=extra() if extra else None, accumulate=accumulate, copy=copy)
         if pairs >= self.TILES_FROM and ops.moe_tiles_usable(x, w_gu, self.form):
             # many rows in bfloat16: sorted into tiles of 128 rows per expert, both products on the tensor-memory kernel
             rows = (pairs // 128 + n_experts) * 128
@@ -164,17 +173,15 @@ class RoutedExperts(Part):
                                   ws.get(tag + "sorted_in", (rows, self.hidden), rt.act_dtype),
                                   ws.get(tag + "sorted_mid", (rows, ff), rt.act_dtype),
                                   ws.get(tag + "sorted_out", (rows, self.hidden), torch.float32),
-                                  ws.get(tag + "tile_plan", (pairs + rows // 128,), torch.int32), out, rt.status,
-                                  act=self.form, limit=limit, extra=extra() if extra else None, accumulate=accumulate, copy=copy)
+                                  ws.get(tag + "tile_plan", (pairs + rows // 128,), torch.int32), out, rt.status, **how)
             return
         mid = ws.get(tag + "mid", (pairs, ff), rt.act_dtype, first="tokens")
-        if pairs >= self.GROUP_FROM:
-            scratch = (ws.get(tag + "pair_out", (pairs, self.hidden), torch.float32, first="tokens"),
-                       ws.get(tag + "plan", (pairs + n_experts + 2 + 3 * (pairs // 32 + n_experts),), torch.int32))
-            ops.moe_experts(x, w_gu, w_down, ids, wts, top, weight_input, mid, out, scratch=scratch, act=self.form, limit=limit,
-                            extra=extra() if extra else None, accumulate=accumulate, copy=copy)
+        pair_out = ws.get(tag + "pair_out", (pairs, self.hidden), torch.float32, reserve=self.GROUP_FROM * self.hidden)
+        if self._few(pairs, x):
+            ops.moe_experts(x, w_gu, w_down, ids, wts, top, weight_input, mid, out, shared=shared, pair_out=pair_out, **how)
             return
-        ops.moe_experts(x, w_gu, w_down, ids, wts, top, weight_input, mid, out, act=self.form, limit=limit, shared=shared)
+        scratch = (pair_out, ws.get(tag + "plan", (pairs + n_experts + 2 + 3 * (pairs // 32 + n_experts),), torch.int32))
+        ops.moe_experts(x, w_gu, w_down, ids, wts, top, weight_input, mid, out, scratch=scratch, **how)
 
     def forward(self, x, batch, residual, accumulate=False, scale: float = 1.0, copy=None):
         rt, T = self.rt, x.shape[0]
@@ -186,7 +193,7 @@ class RoutedExperts(Part):
         factor = None
         if self.factor_name is not None:
             factor = ws.get("moe_factor", (T,), torch.float32, first="tokens")
-        columns = self.w_router.shape[0]
+        columns = self.router_columns
         how = dict(softmax=self.score == "softmax", renormalise=self.renormalise, groups=self.groups, keep=self.keep,
                    renorm_eps=self.renorm_eps, weight_scale=self.weight_scale, always=always, group_score=self.group_score,
                    correction=self.correction, extra=factor)
@@ -195,8 +202,8 @@ class RoutedExperts(Part):
             ops.linear(x, self.w_router_pieces, logits, status=rt.status)
             ops.moe_pick(logits, self.experts, self.router_parts, self.top, ids, wts, **how)
         else:
-            ops.moe_route(x, self.w_router, self.top, ids, wts, logits=ws.get("moe_logits", (T, columns), torch.float32, first="tokens"),
-                          **how)
+            ops.moe_route(x, self.w_router, self.top, ids, wts, logits=ws.get("moe_logits", (T, self.w_router.shape[0]), torch.float32,
+                                                                                       first="tokens"), **how)
         if not self.gated:
             self._forward_ungated(x, residual, ids, wts, factor, accumulate, scale, copy)
             return
@@ -219,7 +226,7 @@ class RoutedExperts(Part):
 
     def _forward_ungated(self, x, residual, ids, wts, factor, accumulate, scale, copy):
         """Experts without a gate.  The shared expert is a dense feed-forward beside the sorted paths and rides along in the
-        pair-by-pair launches; the pass that sums a row's pairs also adds the shared output times its factor, adds into the
+        launches of few rows; the pass that sums a row's pairs also adds the shared output times its factor, adds into the
         stream and leaves its rounded copy."""
         rt, T = self.rt, x.shape[0]
         ws = rt.workspace
@@ -244,16 +251,12 @@ class RoutedExperts(Part):
                 ops.linear_act(x, self.w_shared_gu, mid, self.act, status=rt.status)
             ops.linear(mid, self.w_shared_down, y, status=rt.status)
             return y, factor
-        if T * self.top < self.GROUP_FROM:
-            routed = ws.get("moe_routed", (T, self.hidden), torch.float32, first="tokens")
-            ride = has_shared and 8 * max(self.hidden, self.w_shared_gu.shape[0]) * x.element_size() <= self.RIDE_BYTES
-            self._experts(x, self.w_gu, self.w_down, ids, wts, self.top, self.weight_on == "input", self.limit, routed, "moe_",
-                          shared=(self.w_shared_gu, self.w_shared_down, mid, y) if ride else None)
-            extra = (y, factor) if ride else (dense() if has_shared else None)
-            ops.moe_sum(routed, 1, out, extra=extra, accumulate=add, copy=copy if add else None)
-        else:
-            self._experts(x, self.w_gu, self.w_down, ids, wts, self.top, self.weight_on == "input", self.limit, out, "moe_",
-                          extra=dense if has_shared else None, accumulate=add, copy=copy if add else None)
+        how = dict(accumulate=add, copy=copy if add else None)
+        if has_shared and self._few(T * self.top, x):
+            how.update(extra=lambda: (y, factor), shared=(self.w_shared_gu, self.w_shared_down, mid, y))
+        elif has_shared:
+            how.update(extra=dense)
+        self._experts(x, self.w_gu, self.w_down, ids, wts, self.top, self.weight_on == "input", self.limit, out, "moe_", **how)
         if through:
             ops.add_scaled(residual, out, scale)
         elif not accumulate and scale != 1.0:
