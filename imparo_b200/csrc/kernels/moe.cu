@@ -6,9 +6,11 @@
 //      (and the groups' verdict) goes by score + correction, the weights by the score alone; a logit column behind the experts'
 //      may give each row one more number, sigmoid(z) (the factor of an expert that every row uses).
 //  (2) moe_few_*: steps of few rows (up to 256 pairs a launch), where reading the experts' matrices is the work.  A block belongs
-//      to one of the experts the launch's pairs name and a stretch of its features; it finds its pairs itself, keeps up to eight of
-//      their rows in shared memory and reads its matrix rows once for them.  The up kernel leaves act(..) per pair, the down kernel
-//      the (weighted) output per pair, which moe_sum adds in the order of the choices.
+//      to one of the experts the launch's pairs name and a stretch of its features; it finds its pairs itself and reads its matrix
+//      rows once for up to eight or sixteen of their rows: in bfloat16 straight from global memory into tensor-core fragments
+//      (mma.sync, sixteen matrix rows per block, its warps splitting the row length), else with the rows in shared memory and
+//      scalar arithmetic.  The up kernel leaves act(..) per pair, the down kernel the (weighted) output per pair, which moe_sum adds
+//      in the order of the choices.
 //  (3) moe_group_*: pairs sorted by expert (a counting sort whose order inside an expert is the row order, so the
 //      result does not depend on what else is in the step), tiles of 32 pairs x 64 outputs per CTA: bfloat16 on
 //      tensor cores (mma.sync through wmma fragments, 32-bit accumulation), 32-bit with FFMA.  The tile list is made
@@ -284,35 +286,42 @@ struct SharedRows {
     int n_feat, n;
 };
 
-// The launch's pairs as a block of 256 threads sees them: which expert is the k-th distinct one in the pairs' order of first
-// appearance (-1: there are fewer), its pairs (in order) in list, and how many.
+// The launch's pairs as a block sees them: which expert is the k-th distinct one in the pairs' order of first appearance (-1: there
+// are fewer), its pairs (in order) in list, and how many.
 __device__ __forceinline__ int few_pairs_of(const int* __restrict__ ids, int n_pairs, int experts, int k, int* list, int& count) {
     __shared__ int id_s[FEW_PAIRS];
-    __shared__ int firsts[8];
-    __shared__ int chosen;
-    const int p = threadIdx.x, lane = p & 31, warp = p >> 5;
-    int mine = p < n_pairs ? ids[p] : -1;
-    if (mine >= experts) mine = -1;
-    id_s[p] = mine;
-    if (p == 0) chosen = -1;
+    __shared__ bool first_s[FEW_PAIRS];
+    __shared__ int chosen, members;
+    if (threadIdx.x == 0) { chosen = -1; members = 0; }
+    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
+        const int id = ids[p];
+        id_s[p] = id < experts ? id : -1;
+    }
     __syncthreads();
-    int before = 0;                                     // earlier pairs of the same expert
-    if (mine >= 0)
-        for (int q = 0; q < p; ++q) before += id_s[q] == mine;
-    const bool first = mine >= 0 && before == 0;
-    const unsigned mask = __ballot_sync(0xffffffffu, first);
-    if (lane == 0) firsts[warp] = __popc(mask);
+    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
+        bool first = id_s[p] >= 0;
+        for (int q = 0; q < p; ++q) first = first && id_s[q] != id_s[p];
+        first_s[p] = first;
+    }
     __syncthreads();
-    if (first) {
-        int rank = __popc(mask & ((1u << lane) - 1u));
-        for (int w = 0; w < warp; ++w) rank += firsts[w];
-        if (rank == k) chosen = mine;
+    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
+        if (!first_s[p]) continue;
+        int rank = 0;
+        for (int q = 0; q < p; ++q) rank += first_s[q];
+        if (rank == k) chosen = id_s[p];
     }
     __syncthreads();
     const int e = chosen;
-    const bool member = e >= 0 && mine == e;
-    if (member) list[before] = p;
-    count = __syncthreads_count(member);
+    if (e < 0) return e;
+    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
+        if (id_s[p] != e) continue;
+        int before = 0;
+        for (int q = 0; q < p; ++q) before += id_s[q] == e;
+        list[before] = p;
+        atomicAdd(&members, 1);
+    }
+    __syncthreads();
+    count = members;
     return e;
 }
 
@@ -395,6 +404,130 @@ moe_few_kernel(const T* __restrict__ in, const T* __restrict__ w, const int* __r
                     else reinterpret_cast<float*>(out)[at] = (weight_input ? 1.0f : wts[item]) * acc[j][r];
                 }
             }
+    }
+}
+
+// ---- few rows in bfloat16 on tensor cores ----------------------------------------------------------------------------
+constexpr int MM_WARPS = 4, MM_ROUND = 8;              // warps of a block; 32-entry stretches a warp has in flight
+
+__device__ __forceinline__ uint4 ld_stream(const void* p) {
+    uint4 v;
+    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+    return v;
+}
+__device__ __forceinline__ void mma_16x8x16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+// As moe_few_kernel, with 16 matrix rows per block (gated: the gate and up rows of eight features) and NB tiles of eight rows at
+// once.  A warp takes every MM_WARPS-th round of 32-entry stretches of the row length.  In a stretch lane (g, t) of the warp holds
+// entries 8 t .. 8 t + 7 of matrix rows g and g + 8 and of row g of the operand, 16 bytes each: a dot product does not mind in which
+// order its terms are taken, so the four entries that an mma calls k = 2t, 2t + 1, 2t + 8, 2t + 9 are the lane's own neighbours, in
+// both operands.  The warps' partial sums are added in warp order.  n a multiple of 8, 16-byte aligned pointers.
+template <bool UP, int NB>
+__global__ void __launch_bounds__(MM_WARPS * 32, NB == 1 ? 5 : 4)
+moe_few_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* __restrict__ w, const int* __restrict__ ids,
+                   const float* __restrict__ wts, int n_rows, int n, int n_feat, int top, int experts, int weight_input, int gated, int act,
+                   float limit, void* __restrict__ out, SharedRows sh) {
+    using T = __nv_bfloat16;
+    __shared__ int list[FEW_PAIRS];
+    __shared__ __align__(16) float part[MM_WARPS][NB][128];
+    pdl_trigger();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
+    const int shared_tiles = sh.w ? (n_rows + 8 * NB - 1) / (8 * NB) : 0;
+    const bool shared = (int)blockIdx.x < shared_tiles;
+    if (shared) { n = sh.n; n_feat = sh.n_feat; gated = 0; }
+    const int f0 = blockIdx.y * (gated ? 8 : 16);
+    if (f0 >= n_feat) return;
+    int e = 0, count = n_rows;
+    if (!shared) {
+        e = few_pairs_of(ids, n_rows * top, experts, blockIdx.x - shared_tiles, list, count);
+        if (e < 0) return;
+    }
+    const T* src = shared ? (const T*)sh.in : in;
+    const T* mat = shared ? (const T*)sh.w : w + (size_t)e * (gated ? 2 : 1) * n_feat * n;
+    const int fa = f0 + g, fb = gated ? f0 + g : f0 + g + 8;
+    const T* ra = fa < n_feat ? mat + (size_t)fa * n + 8 * t : nullptr;
+    const T* rb = fb < n_feat ? mat + (size_t)(gated ? n_feat + fb : fb) * n + 8 * t : nullptr;
+    const int lo = shared ? blockIdx.x * 8 * NB : 0, hi = shared ? min(n_rows, lo + 8 * NB) : count;
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    for (int r0 = lo; r0 < hi; r0 += 8 * NB) {
+        const T* xr[NB];
+        float xw[NB];
+        float acc[NB][4];
+#pragma unroll
+        for (int b = 0; b < NB; ++b) {
+            const int r = r0 + 8 * b + g;
+            xr[b] = nullptr;
+            xw[b] = 1.f;
+            acc[b][0] = acc[b][1] = acc[b][2] = acc[b][3] = 0.f;
+            if (r < hi) {
+                const int item = shared ? r : list[r];
+                xr[b] = src + (size_t)(UP && !shared ? item / top : item) * n + 8 * t;
+                if (UP && weight_input && !shared) xw[b] = wts[item];
+            }
+        }
+        for (int k0 = warp * MM_ROUND * 32; k0 < n; k0 += MM_WARPS * MM_ROUND * 32) {
+            uint4 a[MM_ROUND], c[MM_ROUND];
+#pragma unroll
+            for (int u = 0; u < MM_ROUND; ++u) {
+                const int k = k0 + 32 * u;
+                const bool live = k + 8 * t < n;
+                a[u] = live && ra ? ld_stream(ra + k) : zero;
+                c[u] = live && rb ? ld_stream(rb + k) : zero;
+            }
+#pragma unroll
+            for (int u = 0; u < MM_ROUND; ++u) {
+                const int k = k0 + 32 * u;
+                if (k >= n) break;
+                const bool live = k + 8 * t < n;
+#pragma unroll
+                for (int b = 0; b < NB; ++b) {
+                    uint4 x = live && xr[b] ? *reinterpret_cast<const uint4*>(xr[b] + k) : zero;
+                    if (UP && weight_input && !shared) {
+                        __nv_bfloat162* v = reinterpret_cast<__nv_bfloat162*>(&x);
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) {
+                            const float2 f = __bfloat1622float2(v[i]);
+                            v[i] = __floats2bfloat162_rn(xw[b] * f.x, xw[b] * f.y);
+                        }
+                    }
+                    mma_16x8x16(acc[b], a[u].x, c[u].x, a[u].y, c[u].y, x.x, x.y);
+                    mma_16x8x16(acc[b], a[u].z, c[u].z, a[u].w, c[u].w, x.z, x.w);
+                }
+            }
+        }
+        __syncthreads();                                   // the sums before have been read
+#pragma unroll
+        for (int b = 0; b < NB; ++b)
+            *reinterpret_cast<float4*>(&part[warp][b][lane * 4]) = make_float4(acc[b][0], acc[b][1], acc[b][2], acc[b][3]);
+        __syncthreads();
+        // thread = (lane's place, which of its four sums): 0, 1: matrix row g, rows 2t and 2t + 1; 2, 3: matrix row g + 8
+        const int pl = threadIdx.x >> 2, pc = threadIdx.x & 3, pg = pl >> 2, pt = pl & 3;
+#pragma unroll
+        for (int b = 0; b < NB; ++b) {
+            const int r = r0 + 8 * b + 2 * pt + (pc & 1);
+            if (r >= hi) continue;
+            const int item = shared ? r : list[r];
+            float v = 0.f, v2 = 0.f;
+#pragma unroll
+            for (int k = 0; k < MM_WARPS; ++k) v += part[k][b][pl * 4 + pc];
+            if (gated) {
+                if (pc >= 2) continue;
+#pragma unroll
+                for (int k = 0; k < MM_WARPS; ++k) v2 += part[k][b][pl * 4 + pc + 2];
+                if (f0 + pg < n_feat) reinterpret_cast<T*>(out)[(size_t)item * n_feat + f0 + pg] = from_f32<T>(gated_act_bf16(act, limit, v, v2));
+                continue;
+            }
+            const int f = f0 + pg + (pc >> 1) * 8;
+            if (f >= n_feat) continue;
+            const size_t at = (size_t)item * n_feat + f;
+            if (UP) reinterpret_cast<T*>(shared ? sh.out : out)[at] = from_f32<T>(plain_act_bf16(act, v));
+            else if (shared) reinterpret_cast<float*>(sh.out)[at] = v;
+            else reinterpret_cast<float*>(out)[at] = (weight_input ? 1.0f : wts[item]) * v;
+        }
     }
 }
 
@@ -655,49 +788,57 @@ __global__ void __launch_bounds__(1024)
 moe_tile_plan_kernel(const int* __restrict__ ids, int n_pairs, int experts, int* __restrict__ slot_of_pair,
                      int* __restrict__ tile_group, int max_tiles) {
     extern __shared__ int tp_smem[];
-    int* warp_counts = tp_smem;                          // [32][experts]
-    int* base = tp_smem + 32 * experts;                  // [experts] pairs seen so far
-    int* start_row = base + experts;                     // [experts] first row of the expert's stretch
+    int* counts = tp_smem;                               // [32][experts] pairs per warp's stretch, then those before the stretch
+    int* total = tp_smem + 32 * experts;                 // [experts]
+    int* start_row = total + experts;                    // [experts] first row of the expert's stretch
+    __shared__ int used_tiles;
     pdl_trigger();
     pdl_wait();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    for (int e = tid; e < experts; e += blockDim.x) base[e] = 0;
-    for (int p0 = 0; p0 < n_pairs; p0 += 1024) {
-        for (int i = tid; i < 32 * experts; i += blockDim.x) warp_counts[i] = 0;
-        __syncthreads();
-        const int p = p0 + tid;
-        int e = p < n_pairs ? ids[p] : -1;
+    for (int i = tid; i < 32 * experts; i += blockDim.x) counts[i] = 0;
+    __syncthreads();
+    // every warp ranks the pairs of its own stretch, in order, without a word to the others
+    const int per = ((n_pairs + 31) / 32 + 31) / 32 * 32, p0 = warp * per, p1 = min(n_pairs, p0 + per);
+    int* mine = counts + warp * experts;
+    for (int p = p0 + lane; p - lane < p1; p += 32) {
+        int e = p < p1 ? ids[p] : -1;
         if (e >= experts) e = -1;
         const unsigned same = __match_any_sync(0xffffffffu, e);
         const int rank = __popc(same & ((1u << lane) - 1u));
-        if (e >= 0 && rank == 0) warp_counts[warp * experts + e] = __popc(same);
-        __syncthreads();
-        for (int x = tid; x < experts; x += blockDim.x) {
-            int run = base[x];
-            for (int w = 0; w < 32; ++w) {
-                const int c = warp_counts[w * experts + x];
-                warp_counts[w * experts + x] = run;
-                run += c;
-            }
-            base[x] = run;
-        }
-        __syncthreads();
-        if (p < n_pairs) slot_of_pair[p] = e >= 0 ? warp_counts[warp * experts + e] + rank : -1;
-        __syncthreads();
+        const int before = e >= 0 ? mine[e] : 0;
+        __syncwarp();
+        if (e >= 0 && rank == 0) mine[e] = before + __popc(same);
+        __syncwarp();
+        if (p < p1) slot_of_pair[p] = e >= 0 ? before + rank : -1;
     }
+    __syncthreads();
+    for (int x = tid; x < experts; x += blockDim.x) {
+        int run = 0;
+        for (int w = 0; w < 32; ++w) {
+            const int c = counts[w * experts + x];
+            counts[w * experts + x] = run;
+            run += c;
+        }
+        total[x] = run;
+    }
+    __syncthreads();
     if (tid == 0) {
         int t = 0;
         for (int e = 0; e < experts; ++e) {
             start_row[e] = t * TILE_ROWS;
-            const int n = (base[e] + TILE_ROWS - 1) / TILE_ROWS;
-            for (int i = 0; i < n && t < max_tiles; ++i) tile_group[t++] = e;
+            t += (total[e] + TILE_ROWS - 1) / TILE_ROWS;
         }
-        for (; t < max_tiles; ++t) tile_group[t] = -1;
+        used_tiles = min(t, max_tiles);
     }
     __syncthreads();
-    for (int p = tid; p < n_pairs; p += blockDim.x) {
+    for (int e = tid; e < experts; e += blockDim.x) {
+        const int first = start_row[e] / TILE_ROWS, n = (total[e] + TILE_ROWS - 1) / TILE_ROWS;
+        for (int i = 0; i < n && first + i < max_tiles; ++i) tile_group[first + i] = e;
+    }
+    for (int t = used_tiles + tid; t < max_tiles; t += blockDim.x) tile_group[t] = -1;
+    for (int p = p0 + lane; p < p1; p += 32) {
         const int e = ids[p];
-        if (e >= 0 && e < experts && slot_of_pair[p] >= 0) slot_of_pair[p] += start_row[e];
+        if (e >= 0 && e < experts && slot_of_pair[p] >= 0) slot_of_pair[p] += start_row[e] + mine[e];
     }
 }
 
@@ -833,6 +974,25 @@ template <typename T, bool UP>
 static int few_launch(const void* in, const void* w, const int* ids, const float* wts, int n_rows, int n, int n_feat, int top, int experts,
                       int weight_input, int gated, int act, float limit, void* out, const SharedRows& sh, cudaStream_t stream) {
     const int rows = FEW_ROWS, pairs = n_rows * top;
+    if constexpr (sizeof(T) == 2) {
+        uintptr_t all = (uintptr_t)in | (uintptr_t)w | (uintptr_t)sh.w | (uintptr_t)sh.in;
+        if (n % 8 == 0 && (sh.w == nullptr || sh.n % 8 == 0) && (all & 15) == 0) {
+            const int nb = n_rows > 8 ? 2 : 1, per = gated ? 8 : 16;
+            int st = (n_feat + per - 1) / per, tl = 0;
+            if (sh.w) {
+                st = st > (sh.n_feat + 15) / 16 ? st : (sh.n_feat + 15) / 16;
+                tl = (n_rows + 8 * nb - 1) / (8 * nb);
+            }
+            const dim3 grid(tl + (pairs < experts ? pairs : experts), st), block(MM_WARPS * 32);
+            if (st > 65535) return -2;
+            if (nb == 1) launch(moe_few_mma_kernel<UP, 1>, grid, block, 0, stream, (const T*)in, (const T*)w, ids, wts, n_rows, n, n_feat, top,
+                                experts, weight_input, gated, act, limit, out, sh);
+            else launch(moe_few_mma_kernel<UP, 2>, grid, block, 0, stream, (const T*)in, (const T*)w, ids, wts, n_rows, n, n_feat, top, experts,
+                        weight_input, gated, act, limit, out, sh);
+            IMPARO_CHECK_LAUNCH();
+            return 0;
+        }
+    }
     size_t smem = (size_t)(pairs < rows ? pairs : rows) * n * sizeof(T);
     int stretches = (n_feat + (gated ? 15 : 31)) / (gated ? 16 : 32), tiles = 0;
     if (sh.w) {
@@ -842,7 +1002,7 @@ static int few_launch(const void* in, const void* w, const int* ids, const float
         tiles = (n_rows + FEW_ROWS - 1) / FEW_ROWS;
     }
     if (smem > FEW_SMEM_MOST) return -25;
-    static size_t allowed = 48 * 1024;
+    static size_t allowed = 44 * 1024;                     // (a few KB beside it are the kernel's own)
     if (smem > allowed) {
         const cudaError_t e = cudaFuncSetAttribute(moe_few_kernel<T, UP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)FEW_SMEM_MOST);
         if (e != cudaSuccess) return (int)e;

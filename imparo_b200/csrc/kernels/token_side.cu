@@ -105,18 +105,31 @@ side_gate_kernel(const float* __restrict__ x, const T* __restrict__ w, const T* 
     }
 }
 
-template <typename T>
+// VEC: four entries at a time (dim, col0 and the table's rows in multiples of 4, aligned pointers)
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
 side_act_kernel(const float* __restrict__ z, const T* __restrict__ table, size_t table_stride, int col0, const int* __restrict__ ids,
                 const int* __restrict__ rows, int n_rows, int dim, int vocab, T* __restrict__ out, int* status) {
+    constexpr int N = VEC ? 4 : 1;
     pdl_trigger();
     pdl_wait();
-    const size_t total = (size_t)n_rows * dim;
+    const int per = dim / N;
+    const size_t total = (size_t)n_rows * per;
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
-        const int r = (int)(i / dim), j = (int)(i - (size_t)r * dim);
+        const int r = (int)(i / per), j = (int)(i - (size_t)r * per) * N;
         const int id = side_token(ids, rows, r, vocab, status);
-        const float e = id < 0 ? 0.f : to_f32(table[(size_t)id * table_stride + col0 + j]);
-        out[i] = from_f32<T>(gelu_times<T>(z[i], e));
+        struct alignas(sizeof(T) * N) Some { T v[N]; } e, o;
+        if (id >= 0) {
+            e = *reinterpret_cast<const Some*>(table + (size_t)id * table_stride + col0 + j);
+        } else {
+#pragma unroll
+            for (int u = 0; u < N; ++u) e.v[u] = from_f32<T>(0.f);
+        }
+        struct alignas(4 * N) Row { float v[N]; };
+        const Row zv = *reinterpret_cast<const Row*>(z + (size_t)r * dim + j);
+#pragma unroll
+        for (int u = 0; u < N; ++u) o.v[u] = from_f32<T>(gelu_times<T>(zv.v[u], to_f32(e.v[u])));
+        *reinterpret_cast<Some*>(out + (size_t)r * dim + j) = o;
     }
 }
 
@@ -151,15 +164,15 @@ extern "C" int imparo_token_side_act(const float* z, const void* table, long lon
                                      const int* rows, int n_rows, int dim, int vocab, void* out, int* status, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
     if (dim < 1 || col0 < 0 || col0 + dim > table_stride) return -2;
-    const size_t total = (size_t)n_rows * dim;
+    const bool vec = dim % 4 == 0 && col0 % 4 == 0 && table_stride % 4 == 0 && (((uintptr_t)z | (uintptr_t)table | (uintptr_t)out) & 15) == 0;
+    const size_t total = (size_t)n_rows * dim / (vec ? 4 : 1);
     const dim3 grid((unsigned)((total + 255) / 256 > 8192 ? 8192 : (total + 255) / 256));
-    if (dtype == IMPARO_DT_F32)
-        launch(ts::side_act_kernel<float>, grid, dim3(256), 0, stream, z, (const float*)table, (size_t)table_stride, col0, ids, rows,
-               n_rows, dim, vocab, (float*)out, status);
-    else if (dtype == IMPARO_DT_BF16)
-        launch(ts::side_act_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, z, (const __nv_bfloat16*)table, (size_t)table_stride, col0,
-               ids, rows, n_rows, dim, vocab, (__nv_bfloat16*)out, status);
+#define IMPARO_TSA(T_, V_) launch(ts::side_act_kernel<T_, V_>, grid, dim3(256), 0, stream, z, (const T_*)table, (size_t)table_stride, col0, \
+        ids, rows, n_rows, dim, vocab, (T_*)out, status)
+    if (dtype == IMPARO_DT_F32) { if (vec) IMPARO_TSA(float, true); else IMPARO_TSA(float, false); }
+    else if (dtype == IMPARO_DT_BF16) { if (vec) IMPARO_TSA(__nv_bfloat16, true); else IMPARO_TSA(__nv_bfloat16, false); }
     else return -1;
+#undef IMPARO_TSA
     IMPARO_CHECK_LAUNCH();
     return 0;
 }

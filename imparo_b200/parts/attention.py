@@ -240,11 +240,13 @@ class AttentionMixer(Part):
             else:
                 qkv = rt.workspace.get("attn_qkv32", (T, wide), torch.float32, first="tokens")
                 if batch.decode_only and self._decodes_from_product():
-                    qkv = ops.linear_unfolded(x, self.w_qkv[:wide], qkv, status=rt.status)
-                    if isinstance(qkv, ops.PartialProduct):
-                        if self._decode_from_product(qkv, batch, kv, table, inv_freq, n_rot, residual, accumulate):
-                            return
-                        qkv = qkv.tensor()
+                    made = ops.linear_unfolded(x, self.w_qkv[:wide], qkv, status=rt.status)
+                    if not isinstance(made, ops.PartialProduct):          # (a whole product is its own one part)
+                        made = ops.PartialProduct(qkv, 1, qkv.shape, qkv)
+                    if self._decode_from_product(made, batch, kv, table, inv_freq, n_rot, residual, accumulate):
+                        return
+                    if made.parts is not qkv:
+                        qkv = made.tensor()
                 else:
                     ops.linear(x, self.w_qkv[:wide], qkv, status=rt.status)
             gate = qkv[:, width:] if self.gate else None

@@ -37,7 +37,7 @@ class RoutedExperts(Part):
     [rows, hidden] tensor that receives the updated rows rounded, in the pass that adds."""
     takes_scale = True
     GROUP_FROM = 256          # steps with at least this many (row, expert) pairs run sorted by expert, in tiles
-    ROW_BYTES = 200 * 1024    # below that a block per expert keeps eight rows in shared memory, if they fit
+    ROW_BYTES = 200 * 1024    # below that expert by expert (off the tensor cores: if eight rows fit a block's shared memory)
     TILES_FROM = 256          # and from this many on (bfloat16, aligned sizes) on the tensor-memory product, tiles of 128 rows
 
     NAMES = {"router": "router", "gate": "e{e}.gate", "up": "e{e}.up", "down": "e{e}.down", "correction": "correction"}
@@ -153,8 +153,9 @@ class RoutedExperts(Part):
 
     def _few(self, pairs: int, x) -> bool:
         """Whether a step of so many pairs runs expert by expert without sorting (ops.moe_experts without scratch)."""
-        widest = max(self.hidden, self.ff, int(self.shared["ff"]) if self.shared is not None else 0)
-        return pairs < self.GROUP_FROM and 8 * widest * x.element_size() <= self.ROW_BYTES
+        sizes = (self.hidden, self.ff, int(self.shared["ff"]) if self.shared is not None else 8)
+        on_tensor_cores = x.dtype == torch.bfloat16 and all(n % 8 == 0 for n in sizes)
+        return pairs < self.GROUP_FROM and (on_tensor_cores or 8 * max(sizes) * x.element_size() <= self.ROW_BYTES)
 
     def _experts(self, x, w_gu, w_down, ids, wts, top, weight_input, limit, out, tag, extra=None, accumulate=False, copy=None,
                  shared=None):
