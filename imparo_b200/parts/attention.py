@@ -239,7 +239,7 @@ class AttentionMixer(Part):
                 qkv = projected
             else:
                 qkv = rt.workspace.get("attn_qkv32", (T, wide), torch.float32, first="tokens")
-                if batch.decode_only and self._decodes_from_product():
+                if batch.decode_only and self._decodes_from_product(T, table.shape[1] * kv.page_size):
                     made = ops.linear_unfolded(x, self.w_qkv[:wide], qkv, status=rt.status)
                     if not isinstance(made, ops.PartialProduct):          # (a whole product is its own one part)
                         made = ops.PartialProduct(qkv, 1, qkv.shape, qkv)
@@ -315,10 +315,19 @@ class AttentionMixer(Part):
                 room = self._partials_room(table.shape[1] * kv.page_size)
                 part_acc = rt.workspace.get("attn_part_acc", (n * nh * n_splits * hd,), torch.float32, reserve=room * hd)
                 part_ml = rt.workspace.get("attn_part_ml", (n * nh * n_splits * 2,), torch.float32, reserve=room * 2)
+                # decode rows: the output product combines the partial results while it makes its operand, unless a fixed sink,
+                # a gate or a bias comes between
+                in_product = (batch.decode_only and n_splits <= 64 and ops.fuse_producers() and self.b_o is None and not self.gate
+                              and (not self.sink or self.sinks is not None))
                 done = ops.paged_attention_split(q[:n], kv.k, kv.v, batch.positions[:n], batch.item_of_token[:n], table,
-                                                 kv.page_size, kv.n_pages, self.window, self.scale, out[:n], part_acc, part_ml,
-                                                 chunk, n_splits, nh, self.nkv, hd, rt.status, sink=self.sink and self.sinks is None,
-                                                 softcap=self.softcap, sink_values=self.sinks)
+                                                 kv.page_size, kv.n_pages, self.window, self.scale, None if in_product else out[:n],
+                                                 part_acc, part_ml, chunk, n_splits, nh, self.nkv, hd, rt.status,
+                                                 sink=self.sink and self.sinks is None, softcap=self.softcap, sink_values=self.sinks)
+                if done and in_product:
+                    if ops.linear_of_attention_partials(part_acc, part_ml, T, nh, hd, n_splits, self.w_o, residual, rt.status,
+                                                        accumulate=accumulate):
+                        return
+                    ops.attention_split_combine(part_acc, part_ml, out, T * nh, hd, n_splits)
         if not done:
             ops.attention_any(q, kv.k, kv.v, batch.positions, batch.item_of_token, table, kv.page_size, kv.n_pages, self.window,
                               self.scale, self.sink, out, nh, self.nkv, hd, vd, rt.status, softcap=self.softcap, chunk=self.chunk,
@@ -329,10 +338,12 @@ class AttentionMixer(Part):
         if self.prepared and self.b_o is not None:
             ops.add_bias(residual, self.b_o)
 
-    def _decodes_from_product(self) -> bool:
+    FROM_PRODUCT_CHUNKS = 16         # every key chunk's CTA makes the group's queries again: for contexts of up to so many chunks
+
+    def _decodes_from_product(self, T: int, positions: int) -> bool:
         """Whether rows of one token can go from the q/k product's split partials straight into the split-key attention: keys that
         are their own values, with nothing between the product and the rotation."""
-        return (self.v_from_k and not self.unit_norm and not self.bias_required and self.qk_conv is None and not self.gate
+        return (T <= 65535 and ops.split_plan(T, self.nkv, positions)[1] <= self.FROM_PRODUCT_CHUNKS and self.v_from_k and not self.unit_norm and not self.bias_required and self.qk_conv is None and not self.gate
                 and not self.sigmoid and self.chunk is None and self.softcap == 0.0 and self.rt.act_dtype == torch.bfloat16
                 and self.hd in (64, 128) and self.nh // self.nkv <= 8 and (not self.sink or self.sinks is not None)
                 and ops.switches().decode_from_qkv)
@@ -343,8 +354,6 @@ class AttentionMixer(Part):
         rt, T = self.rt, qkv.shape[0]
         nh, hd = self.nh, self.hd
         chunk, n_splits = ops.split_plan(T, self.nkv, table.shape[1] * kv.page_size)
-        if n_splits > 16 or T > 65535:       # (every chunk's CTA makes the group's queries again: for contexts of up to 16 chunks)
-            return False
         room = self._partials_room(table.shape[1] * kv.page_size)
         part_acc = rt.workspace.get("attn_part_acc", (T * nh * n_splits * hd,), torch.float32, reserve=room * hd)
         part_ml = rt.workspace.get("attn_part_ml", (T * nh * n_splits * 2,), torch.float32, reserve=room * 2)
