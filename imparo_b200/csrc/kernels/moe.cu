@@ -286,42 +286,66 @@ struct SharedRows {
     int n_feat, n;
 };
 
-// The launch's pairs as a block sees them: which expert is the k-th distinct one in the pairs' order of first appearance (-1: there
-// are fewer), its pairs (in order) in list, and how many.
+// The launch's pairs as a block sees them: the k-th of the experts they name (-1: there are fewer), its pairs (in order) in list,
+// and how many.  Up to 32 pairs every warp finds the answer by itself; with more the block first marks the experts in a bit set.
+// (All warps write the same list.)  Every thread of the block calls it.
+constexpr int FEW_EXPERTS = 2048;
 __device__ __forceinline__ int few_pairs_of(const int* __restrict__ ids, int n_pairs, int experts, int k, int* list, int& count) {
-    __shared__ int id_s[FEW_PAIRS];
-    __shared__ bool first_s[FEW_PAIRS];
-    __shared__ int chosen, members;
-    if (threadIdx.x == 0) { chosen = -1; members = 0; }
+    const int lane = threadIdx.x & 31;
+    const unsigned below = (1u << lane) - 1u;
+    if (n_pairs <= 32) {
+        int id = lane < n_pairs ? ids[lane] : -1;
+        if (id >= experts) id = -1;
+        const unsigned same = __match_any_sync(0xffffffffu, id);
+        const bool first = id >= 0 && (same & below) == 0;
+        const unsigned firsts = __ballot_sync(0xffffffffu, first);
+        const unsigned hit = __ballot_sync(0xffffffffu, first && __popc(firsts & below) == k);
+        if (hit == 0) return -1;
+        const int src = __ffs(hit) - 1;
+        const int e = __shfl_sync(0xffffffffu, id, src);
+        const unsigned members = __shfl_sync(0xffffffffu, same, src);
+        if ((members >> lane) & 1u) list[__popc(members & below)] = lane;
+        __syncwarp();
+        count = __popc(members);
+        return e;
+    }
+    __shared__ unsigned named[FEW_EXPERTS / 32];
+    for (int i = threadIdx.x; i < FEW_EXPERTS / 32; i += blockDim.x) named[i] = 0u;
+    __syncthreads();
     for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
         const int id = ids[p];
-        id_s[p] = id < experts ? id : -1;
+        if (id >= 0 && id < experts) atomicOr(&named[id >> 5], 1u << (id & 31));
     }
     __syncthreads();
-    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
-        bool first = id_s[p] >= 0;
-        for (int q = 0; q < p; ++q) first = first && id_s[q] != id_s[p];
-        first_s[p] = first;
+    // a lane looks at two words; a running count over the lanes finds the word with the k-th expert
+    unsigned w0 = named[2 * lane], w1 = named[2 * lane + 1];
+    const int mine = __popc(w0) + __popc(w1);
+    int upto = mine;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, upto, o);
+        if (lane >= o) upto += v;
     }
-    __syncthreads();
-    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
-        if (!first_s[p]) continue;
-        int rank = 0;
-        for (int q = 0; q < p; ++q) rank += first_s[q];
-        if (rank == k) chosen = id_s[p];
+    int e = -1;
+    if (k < upto && k >= upto - mine) {
+        int left = k - (upto - mine), base = 64 * lane;
+        unsigned word = w0;
+        if (left >= __popc(w0)) { left -= __popc(w0); word = w1; base += 32; }
+        for (; left > 0; --left) word &= word - 1;
+        e = base + __ffs(word) - 1;
     }
-    __syncthreads();
-    const int e = chosen;
-    if (e < 0) return e;
-    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
-        if (id_s[p] != e) continue;
-        int before = 0;
-        for (int q = 0; q < p; ++q) before += id_s[q] == e;
-        list[before] = p;
-        atomicAdd(&members, 1);
+    const unsigned hit = __ballot_sync(0xffffffffu, e >= 0);
+    if (hit == 0) return -1;
+    e = __shfl_sync(0xffffffffu, e, __ffs(hit) - 1);
+    int n = 0;
+    for (int p0 = 0; p0 < n_pairs; p0 += 32) {
+        const bool member = p0 + lane < n_pairs && ids[p0 + lane] == e;
+        const unsigned m = __ballot_sync(0xffffffffu, member);
+        if (member) list[n + __popc(m & below)] = p0 + lane;
+        n += __popc(m);
     }
-    __syncthreads();
-    count = members;
+    __syncwarp();
+    count = n;
     return e;
 }
 
@@ -408,7 +432,7 @@ moe_few_kernel(const T* __restrict__ in, const T* __restrict__ w, const int* __r
 }
 
 // ---- few rows in bfloat16 on tensor cores ----------------------------------------------------------------------------
-constexpr int MM_WARPS = 4, MM_ROUND = 8;              // warps of a block; 32-entry stretches a warp has in flight
+constexpr int MM_WARPS = 8, MM_ROUND = 4;              // warps of a block; 32-entry stretches a warp has in flight
 
 __device__ __forceinline__ uint4 ld_stream(const void* p) {
     uint4 v;
@@ -426,7 +450,7 @@ __device__ __forceinline__ void mma_16x8x16(float (&d)[4], uint32_t a0, uint32_t
 // order its terms are taken, so the four entries that an mma calls k = 2t, 2t + 1, 2t + 8, 2t + 9 are the lane's own neighbours, in
 // both operands.  The warps' partial sums are added in warp order.  n a multiple of 8, 16-byte aligned pointers.
 template <bool UP, int NB>
-__global__ void __launch_bounds__(MM_WARPS * 32, NB == 1 ? 5 : 4)
+__global__ void __launch_bounds__(MM_WARPS * 32, NB == 1 ? 4 : 2)
 moe_few_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* __restrict__ w, const int* __restrict__ ids,
                    const float* __restrict__ wts, int n_rows, int n, int n_feat, int top, int experts, int weight_input, int gated, int act,
                    float limit, void* __restrict__ out, SharedRows sh) {
@@ -470,7 +494,7 @@ moe_few_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* __
             }
         }
         for (int k0 = warp * MM_ROUND * 32; k0 < n; k0 += MM_WARPS * MM_ROUND * 32) {
-            uint4 a[MM_ROUND], c[MM_ROUND];
+            uint4 a[MM_ROUND], c[MM_ROUND], x[MM_ROUND][NB];             // all loads of a round are in flight at once
 #pragma unroll
             for (int u = 0; u < MM_ROUND; ++u) {
                 const int k = k0 + 32 * u;
@@ -479,23 +503,28 @@ moe_few_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* __
                 c[u] = live && rb ? ld_stream(rb + k) : zero;
             }
 #pragma unroll
-            for (int u = 0; u < MM_ROUND; ++u) {
-                const int k = k0 + 32 * u;
-                if (k >= n) break;
-                const bool live = k + 8 * t < n;
+            for (int u = 0; u < MM_ROUND; ++u)
 #pragma unroll
                 for (int b = 0; b < NB; ++b) {
-                    uint4 x = live && xr[b] ? *reinterpret_cast<const uint4*>(xr[b] + k) : zero;
+                    const int k = k0 + 32 * u;
+                    x[u][b] = k + 8 * t < n && xr[b] ? *reinterpret_cast<const uint4*>(xr[b] + k) : zero;
+                }
+#pragma unroll
+            for (int u = 0; u < MM_ROUND; ++u) {
+                if (k0 + 32 * u >= n) break;
+#pragma unroll
+                for (int b = 0; b < NB; ++b) {
+                    uint4 xv = x[u][b];
                     if (UP && weight_input && !shared) {
-                        __nv_bfloat162* v = reinterpret_cast<__nv_bfloat162*>(&x);
+                        __nv_bfloat162* v = reinterpret_cast<__nv_bfloat162*>(&xv);
 #pragma unroll
                         for (int i = 0; i < 4; ++i) {
                             const float2 f = __bfloat1622float2(v[i]);
                             v[i] = __floats2bfloat162_rn(xw[b] * f.x, xw[b] * f.y);
                         }
                     }
-                    mma_16x8x16(acc[b], a[u].x, c[u].x, a[u].y, c[u].y, x.x, x.y);
-                    mma_16x8x16(acc[b], a[u].z, c[u].z, a[u].w, c[u].w, x.z, x.w);
+                    mma_16x8x16(acc[b], a[u].x, c[u].x, a[u].y, c[u].y, xv.x, xv.y);
+                    mma_16x8x16(acc[b], a[u].z, c[u].z, a[u].w, c[u].w, xv.z, xv.w);
                 }
             }
         }
@@ -505,9 +534,9 @@ moe_few_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* __
             *reinterpret_cast<float4*>(&part[warp][b][lane * 4]) = make_float4(acc[b][0], acc[b][1], acc[b][2], acc[b][3]);
         __syncthreads();
         // thread = (lane's place, which of its four sums): 0, 1: matrix row g, rows 2t and 2t + 1; 2, 3: matrix row g + 8
-        const int pl = threadIdx.x >> 2, pc = threadIdx.x & 3, pg = pl >> 2, pt = pl & 3;
+        const int pl = (threadIdx.x & 127) >> 2, pc = threadIdx.x & 3, pg = pl >> 2, pt = pl & 3;
 #pragma unroll
-        for (int b = 0; b < NB; ++b) {
+        for (int b = threadIdx.x >> 7; b < NB; b += 2) {
             const int r = r0 + 8 * b + 2 * pt + (pc & 1);
             if (r >= hi) continue;
             const int item = shared ? r : list[r];
