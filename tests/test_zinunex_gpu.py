@@ -216,8 +216,8 @@ def test_first_tokens_of_a_sequence(name, dtype):
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("n_requests", [9, 30, 70])
 def test_many_decoding_requests(n_requests, dtype):
-    """Batches of unequal requests that decode together, each against the plain logits of the request alone: pairs pair by pair
-    with a second block of shared rows, sorted into small tiles and on the tensor-memory tiles; side inputs on both paths."""
+    """Batches of unequal requests that decode together, each against the plain logits of the request alone: routed experts expert by
+    expert for one and two tiles of rows and for more than 32 pairs; side inputs on both paths."""
     name = "C"
     rng = np.random.default_rng(n_requests)
     reqs = make_requests(name, [int(n) for n in rng.integers(2, 24, n_requests)], seed=n_requests)
@@ -538,7 +538,7 @@ def test_router_with_correction(E, top, groups, keep, scale, shift):
                                                         (300, 8, 2, 64, 128, 96), (70, 4, 1, 16, 52, None), (150, 12, 3, 80, 256, 80), (7, 3, 2, 13, 41, 27),
                                                         (90, 3, 2, 13, 41, 27), (11, 4, 2, 24, 64, None), (513, 16, 1, 40, 64, 8)])
 def test_ungated_experts_with_a_shared_one(dtype, T, E, top, ff, width, shared_ff):
-    """The routed feed-forward as a part: squared-relu experts pair by pair (the shared expert in the same launches), sorted into
+    """The routed feed-forward as a part: squared-relu experts expert by expert (the shared expert in the same launches), sorted into
     small tiles and on the tensor-memory product (the shared expert beside them), its factor per row, the pass that adds into the
     stream and leaves the rounded copy; written, added, and added scaled."""
     import torch
